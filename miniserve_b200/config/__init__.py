@@ -4,12 +4,13 @@ from .kovusun import KovusunConfig
 from .mugipel import MugipelConfig
 from .qwen3 import Qwen3Config
 from .rofozen import RofozenConfig
+from .vumedra import VumedraConfig
 from .registry import (Architecture, architecture_of, architectures, load_config_dict,
                        register_architecture, resolve, unregister_architecture)
 from .spec import LayerSpec, ModelSpec, PartSpec, RunEntry, TensorRule
 
 __all__ = [
-    "Architecture", "LayerSpec", "ModelSpec", "PartSpec", "RunEntry", "TensorRule", "PRESETS", "FekulixConfig", "KovusunConfig", "MugipelConfig", "Qwen3Config", "RofozenConfig",
+    "Architecture", "LayerSpec", "ModelSpec", "PartSpec", "RunEntry", "TensorRule", "PRESETS", "FekulixConfig", "KovusunConfig", "MugipelConfig", "Qwen3Config", "RofozenConfig", "VumedraConfig",
     "architecture_of", "architectures", "load_config_dict", "preset", "register_architecture",
     "resolve", "unregister_architecture",
 ]

@@ -64,7 +64,22 @@ def _kovusun(width, vocab, ff, heads, kv_heads, dim, window) -> dict:
     return dict(architecture="Kovusun", width=width, vocab=vocab, norm={"eps": 1e-5}, layers=layers)
 
 
+def _vumedra(width, vocab, ff, pattern, dim, heads, kv_heads, memory_heads, blocks) -> dict:
+    """A Vumedra config.json: ``pattern`` is a string of A (attention), M (matrix memory) and R (gated linear recurrence);
+    dense and routed feed-forwards in turn."""
+    mixers = {"A": ("attention", {"dim": dim, "heads": heads, "kv_heads": kv_heads, "q_temp": {"coef": 0.2, "every": 64},
+                                  "scale": dim ** -0.5, "vdim": dim}),
+              "M": ("mlstm", {"dim": dim, "gate_cap": 15.0, "heads": memory_heads, "vdim": 2 * dim}),
+              "R": ("rglru", {"blocks": blocks, "conv": 4, "width": width})}
+    dense = {"ff": ff, "kind": "dense"}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": 6, "top": 2}, "shared": {"ff": ff // 2}}
+    layers = [{"type": mixers[ch][0], "mixer": dict(mixers[ch][1]), "mlp": dict(moe if i % 2 else dense)} for i, ch in enumerate(pattern)]
+    return dict(architecture="Vumedra", width=width, vocab=vocab, norm={"eps": 1e-5},
+                embedding={"bigram": {"buckets": 2 * vocab + 1, "mul_prev": 31, "mul_cur": 3}}, layers=layers)
+
+
 PRESETS: dict[str, dict] = {
+    "vumedra-tiny": _vumedra(96, 503, 160, "RAMR", 32, 6, 2, 3, 6),
     "kovusun-tiny": _kovusun(96, 503, 160, 6, 2, 32, 48),
     "mugipel-tiny": _mugipel(
         96, 503, 160, "ALAL",

@@ -7,7 +7,7 @@
 //   warp 1   allocates tensor memory; one elected lane issues tcgen05.mma (M=128, N=BN, K=16, four
 //            per stage) on shared-memory descriptors and releases each stage with tcgen05.commit;
 //   warps 2-5 read the accumulator back with tcgen05.ld (each warp its own 32 lanes), apply the
-//            epilogue and store: plain (bf16 or float32 out), or SiLU(gate) * up for the stacked
+//            epilogue and store: plain (bf16 or float32 out), the square of relu, or SiLU(gate) * up for the stacked
 //            gate|up projection, which then never writes the 2 x intermediate tensor.
 // Every wait on an mbarrier is bounded: after a limit the kernel raises a status word, stops
 // waiting, frees its tensor memory and returns.
@@ -27,7 +27,7 @@ namespace ms {
 constexpr int TC_BM = 128, TC_BK = 64;
 constexpr int TC_THREADS = 192;
 
-enum TcEpilogue : int { TC_OUT_BF16 = 0, TC_OUT_F32 = 1, TC_SILU_MUL = 2, TC_QKV_ROPE = 3 };
+enum TcEpilogue : int { TC_OUT_BF16 = 0, TC_OUT_F32 = 1, TC_SILU_MUL = 2, TC_QKV_ROPE = 3, TC_RELU2 = 4 };
 
 // What the q|k|v epilogue (TC_QKV_ROPE) needs besides the product: per-head RMSNorm of q and k, rotation
 // by position and the write of q to [T, nq, 128] and of k, v into their cache pages, as the separate
@@ -268,6 +268,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             for (int j = 0; j < 32; ++j) {
               float x = __uint_as_float(acc[j]);
               if (EPI == TC_SILU_MUL) x = x / (1.0f + expf(-x)) * __uint_as_float(up[j]);
+              if (EPI == TC_RELU2) {
+                x = fmaxf(x, 0.f);
+                x *= x;
+              }
               v[j] = x;
             }
             __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)row * N_out + col0;
@@ -1361,7 +1365,7 @@ MS_EXPORT int ms_gemm_tc_bf16(void* out, const void* A, const void* W, int M, in
 // The experts' products of a routed feed-forward over rows sorted by expert (tiles of 128 rows, (expert, first row)
 // each; meta[0] tiles; offsets[e + 1] ends expert e's rows; at most max_tiles tiles).
 // gated = 1: W [E, 2 N, K] (an expert's gate rows, then its up rows), out [rows, N] bfloat16 = silu(A gate^T) * (A up^T);
-// gated = 0: W [E, N, K], out [rows, N] float32 = A W^T.
+// gated = 0: W [E, N, K], out [rows, N] float32 = A W^T; gated = 2: W [E, N, K], out [rows, N] bfloat16 = relu(A W^T)^2.
 MS_EXPORT int ms_gemm_tc_experts_bf16(void* out, const void* A, const void* W, int rows, int N, int K, int experts, int gated,
                                       const int* tiles, const int* meta, const int* offsets, int max_tiles, int* status,
                                       cudaStream_t stream) {
@@ -1371,12 +1375,13 @@ MS_EXPORT int ms_gemm_tc_experts_bf16(void* out, const void* A, const void* W, i
   MS_CHECK_ARG(((uintptr_t)A % 16 == 0) && ((uintptr_t)W % 16 == 0), "gemm_tc_experts: operands must be 16-byte aligned");
   MS_CHECK_ARG(status != nullptr && tiles != nullptr && meta != nullptr && offsets != nullptr, "gemm_tc_experts: needs a plan and a status word");
   MS_CHECK_ARG(max_tiles <= 65535, "gemm_tc_experts: %d row tiles are too many for one launch", max_tiles);
-  MS_CHECK_ARG((long long)experts * (gated ? 2 : 1) * N < (1LL << 31), "gemm_tc_experts: the weights have too many rows");
-  if (gated) {
+  MS_CHECK_ARG((long long)experts * (gated == 1 ? 2 : 1) * N < (1LL << 31), "gemm_tc_experts: the weights have too many rows");
+  if (gated == 1) {
     const TcGroups grp{tiles, meta, offsets, 2 * N};
     return launch_tc_grouped<256, 4, TC_SILU_MUL>(out, A, W, rows, N, experts, 2 * N, K, N, grp, max_tiles, status, stream);
   }
   const TcGroups grp{tiles, meta, offsets, N};
+  if (gated == 2) return launch_tc_grouped<128, 5, TC_RELU2>(out, A, W, rows, N, experts, N, K, 0, grp, max_tiles, status, stream);
   return launch_tc_grouped<128, 5, TC_OUT_F32>(out, A, W, rows, N, experts, N, K, 0, grp, max_tiles, status, stream);
 }
 

@@ -115,12 +115,21 @@ __global__ void head_gate_bf16x8_kernel(__nv_bfloat16* __restrict__ out, int ld_
 // What a q|k|v preparation may do beyond norm weights and rotation. ``bias``: float32 [nq*dk | nkv*dk | nkv*dv], added to
 // the projection's columns before anything else (null: none). ``unit_norm``: q and k are divided by their root mean
 // square over dk also where no norm weight is given (a norm without a weight). ``q_scale``: float32 [nq], a factor per
-// query head applied last (a learned temperature of the scores), or null.
+// query head applied last (a learned temperature of the scores), or null. ``temp_coef``, ``temp_every``: every query is
+// multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) at position p (temp_every 0: it is not).
 struct PrepareExtras {
   const float* bias;
   const float* q_scale;
   int unit_norm;
+  float temp_coef, temp_every;
 };
+
+// The factor on query head h at position pos.
+__device__ __forceinline__ float query_factor(const PrepareExtras& ex, int h, int pos) {
+  float f = ex.q_scale ? ex.q_scale[h] : 1.f;
+  if (ex.temp_every > 0.f) f *= 1.f + ex.temp_coef * logf(floorf(((float)pos + 1.f) / ex.temp_every) + 1.f);
+  return f;
+}
 
 // bfloat16, sizes that are multiples of 8, rows on 16 bytes: a lane holds eight consecutive channels; one warp per
 // (token, head). ADJACENT: these are four rotation pairs, so the rotation needs no exchange. Otherwise channel i
@@ -188,7 +197,7 @@ __global__ void qkv_prepare_bf16x8_kernel(
     ss = warp_sum(ss);
   }
   const float inv = normed ? 1.0f / sqrtf(ss / (float)dk + eps) : 1.f;
-  const float qs = (h < nq && ex.q_scale) ? ex.q_scale[h] : 1.f;
+  const float qs = h < nq ? query_factor(ex, h, pos) : 1.f;
   const int half = rot >> 1;
   for (int c = lane * 8; c < d_pad; c += 256) {
     float v[8];
@@ -313,7 +322,7 @@ __global__ void qkv_prepare_kernel(
     ss = warp_sum(ss);
     inv = 1.0f / sqrtf(ss / (float)dk + eps);
   }
-  const float qs = (h < nq && ex.q_scale) ? ex.q_scale[h] : 1.f;
+  const float qs = h < nq ? query_factor(ex, h, pos) : 1.f;
   const int half = rot >> 1;
   for (int j = lane; j < half; j += 32) {
     const int ia = adjacent ? 2 * j : j, ib = adjacent ? 2 * j + 1 : j + half;
@@ -417,9 +426,10 @@ MS_EXPORT int ms_qkv_prepare(void* q_out, void* k_pool, void* v_pool, const void
                              const float* q_norm_w, const float* k_norm_w, const float* cos_sin, const int* positions,
                              const int* row_of_token, const int* page_indptr, const int* page_indices, int num_tokens, int nq,
                              int nkv, int dk, int dv, int d_pad, int rot, int adjacent, float eps, int page_size, int num_pages,
-                             int* status, int dtype, cudaStream_t stream, const float* bias, const float* q_scale, int unit_norm) {
+                             int* status, int dtype, cudaStream_t stream, const float* bias, const float* q_scale, int unit_norm, float temp_coef,
+                             float temp_every) {
   if (num_tokens == 0) return 0;
-  const PrepareExtras ex{bias, q_scale, unit_norm};
+  const PrepareExtras ex{bias, q_scale, unit_norm, temp_coef, temp_every};
   MS_CHECK_ARG((k_pool == nullptr) == (v_pool == nullptr), "qkv_prepare: key and value pools come together or not at all");
   MS_CHECK_ARG(nq > 0 && nkv > 0 && dk > 0 && dv > 0 && d_pad >= dk && d_pad >= dv, "qkv_prepare: bad sizes nq=%d nkv=%d dk=%d dv=%d D=%d",
                nq, nkv, dk, dv, d_pad);

@@ -72,7 +72,7 @@ decay_scan_kernel(float* __restrict__ o_out,   // [T, H, dv]
                   const TZ* __restrict__ z, int ld_z, const float* __restrict__ z_bias, const float* __restrict__ decay_coef,
                   float z_sign, int z_is_decay, const TZ* __restrict__ beta, int ld_beta,
                   const int* __restrict__ cu_q, const int* __restrict__ q_start, const int* __restrict__ state_slot,
-                  int H, int dk, int dv, int L, int chunk, float q_scale, int vec, int dkz, const float* __restrict__ v_scale) {
+                  int H, int dk, int dv, int L, int chunk, float q_scale, int vec, int dkz, const float* __restrict__ v_scale, int dv_in) {
   // words a thread's channels take in shared memory: padded so that the 16-byte loads of a quarter warp's lanes fall on different banks
   constexpr int SCAN_SEG = SCAN_KPT == 4 ? 4 : SCAN_KPT + 4;
   extern __shared__ __align__(16) float smem[];
@@ -102,7 +102,7 @@ decay_scan_kernel(float* __restrict__ o_out,   // [T, H, dv]
     S[e] = (!fresh && active && i < dk) ? srow[i] : 0.f;
   }
   const int qk_head = h / qk_group;
-  const float coef = decay_coef[h];
+  const float coef = decay_coef ? decay_coef[h] : 0.f;  // (not read where z holds the decays themselves)
   __syncthreads();
 
   for (int c0 = t0; c0 < t1; c0 += chunk) {
@@ -153,7 +153,8 @@ decay_scan_kernel(float* __restrict__ o_out,   // [T, H, dv]
     for (int idx = tid; idx < n * cols; idx += threads) {
       const int tt = idx / cols, c = idx - tt * cols;
       const int jj = blockIdx.z * cols + c;
-      float vv = jj < dv ? Elem<TIn>::load(v + (size_t)(c0 + tt) * ld_v + (size_t)h * dv + jj) : 0.f;
+      // (dv = dv_in + 1: the column behind the values is the state's sum of keys, its value is one)
+      float vv = jj < dv_in ? Elem<TIn>::load(v + (size_t)(c0 + tt) * ld_v + (size_t)h * dv_in + jj) : (jj < dv ? 1.f : 0.f);
       if (v_scale) vv *= v_scale[(size_t)(c0 + tt) * H + h];
       vs[idx] = vv;
     }
@@ -430,7 +431,7 @@ template <typename TIn, typename TZ, bool DELTA, int SCAN_KPT>
 int launch_scan_kpt(float* o_out, float* state, const void* q, int ld_q, const void* k, int ld_k, int qk_group, const void* v, int ld_v,
                 const void* z, int ld_z, const float* z_bias, const float* decay_coef, float z_sign, int z_is_decay, const void* beta,
                 int ld_beta, const int* cu_q, const int* q_start, const int* state_slot, int num_rows, int H, int dk, int dv, float q_scale,
-                int dkz, const float* v_scale, cudaStream_t stream) {
+                int dkz, const float* v_scale, int dv_in, cudaStream_t stream) {
   constexpr int SCAN_SEG = SCAN_KPT == 4 ? 4 : SCAN_KPT + 4;
   int L = 1;
   while (L * SCAN_KPT < dk) L <<= 1;
@@ -457,7 +458,7 @@ int launch_scan_kpt(float* o_out, float* state, const void* q, int ld_q, const v
                   (dkz == 1 || ((uintptr_t)z % 16 == 0 && ld_z % z8 == 0));
   MS_LAUNCH(kernel, grid, threads, smem, stream, o_out, state, (const TIn*)q, ld_q, (const TIn*)k, ld_k, qk_group,
             (const TIn*)v, ld_v, (const TZ*)z, ld_z, z_bias, decay_coef, z_sign, z_is_decay, (const TZ*)beta, ld_beta, cu_q, q_start, state_slot,
-            H, dk, dv, L, chunk, q_scale, vec, dkz, v_scale);
+            H, dk, dv, L, chunk, q_scale, vec, dkz, v_scale, dv_in);
   return 0;
 }
 
@@ -484,20 +485,22 @@ MS_DEFINE_PDL_SWITCH(ms_recurrence_set_pdl)
 
 
 // in_dtype: of q, k, v; z_dtype: of z and beta. delta: 0 decay rule, 1 delta rule. z_is_decay: z and beta are
-// float32 and hold the decays and sigmoid(beta) themselves (ms_decay_from_logits), not their logits.
+// float32 and hold the decays and sigmoid(beta) themselves (ms_decay_from_logits), not their logits. dv_in: the value channels of a head
+// in v; dv - 1 of them: the state has one more column, whose value is one (the decayed sum of the keys).
 MS_EXPORT int ms_decay_scan(float* o_out, float* state, const void* q, int ld_q, const void* k, int ld_k, int qk_group,
                             const void* v, int ld_v, const void* z, int ld_z, const float* z_bias, const float* decay_coef,
                             float z_sign, int z_is_decay, const void* beta, int ld_beta, const int* cu_q, const int* q_start,
                             const int* state_slot, int num_rows, int H, int dk, int dv, float q_scale, int delta, int in_dtype,
-                            int z_dtype, int decay_per_head, const float* v_scale, cudaStream_t stream) {
+                            int z_dtype, int decay_per_head, const float* v_scale, int dv_in, cudaStream_t stream) {
   if (num_rows == 0) return 0;
   MS_CHECK_ARG(H > 0 && dk > 0 && dv > 0 && dk <= 32 * SCAN_MAX_KPT, "decay_scan: key size %d is outside 1..%d", dk, 32 * SCAN_MAX_KPT);
   MS_CHECK_ARG(qk_group > 0 && H % qk_group == 0, "decay_scan: %d heads are not a multiple of the group of %d", H, qk_group);
   MS_CHECK_ARG(!delta || beta != nullptr, "decay_scan: the delta rule needs beta");
+  MS_CHECK_ARG(dv_in == dv || (dv_in == dv - 1 && !delta), "decay_scan: %d value columns of which %d are read", dv, dv_in);
   MS_CHECK_ARG(!z_is_decay || z_dtype == MS_F32, "decay_scan: decays worked out beforehand are float32");
 #define MS_SCAN(TIN, TZZ, D)                                                                                                  \
   return launch_scan<TIN, TZZ, D>(num_rows, H, dk, dv, o_out, state, q, ld_q, k, ld_k, qk_group, v, ld_v, z, ld_z, z_bias, decay_coef, z_sign, z_is_decay, \
-                                  beta, ld_beta, cu_q, q_start, state_slot, num_rows, H, dk, dv, q_scale, decay_per_head ? 1 : dk, v_scale, stream)
+                                  beta, ld_beta, cu_q, q_start, state_slot, num_rows, H, dk, dv, q_scale, decay_per_head ? 1 : dk, v_scale, dv_in, stream)
   if (in_dtype == MS_F32 && z_dtype == MS_F32) {
     if (delta) MS_SCAN(float, float, true);
     MS_SCAN(float, float, false);

@@ -5,7 +5,10 @@
 //   Router outputs form `group_count` equal groups of neighbours; a group's score is its largest c; only outputs of
 //   the `group_keep` best groups can be chosen. The `top` largest c among those are the token's choices; the weight of
 //   a choice is s (without the correction) times a constant, optionally divided by the sum of the chosen s.
-//   Router outputs E .. R-1 are identity experts: their output is h itself. Expert e < E: W_down[e] (act(W_gate[e] h) * (W_up[e] h)).
+//   Router outputs E .. R-1 are identity experts: their output is h itself. Expert e < E: W_down[e] (act(W_gate[e] h) * (W_up[e] h)),
+//   or without a gate W_down[e] act(W_up[e] h) with act the square of relu.
+//   The scores may be sigmoid(z) instead. A weight that multiplies the expert's INPUT is handed on as its square where act is the
+//   square of relu: W_down relu(W_up (w h))^2 = w^2 W_down relu(W_up h)^2 for w >= 0.
 //
 // Nothing here needs the host to know how many tokens an expert got: the plan lives on the device, grids are sized
 // for the worst case and surplus CTAs leave at once, so a step can be captured into a graph. Every output row is a
@@ -27,7 +30,7 @@ __global__ void __launch_bounds__(ROUTE_THREADS)
 expert_route_kernel(int* __restrict__ idx_out, float* __restrict__ wgt_out, const T* __restrict__ x, int ld_x,
                     const float* __restrict__ router, const float* __restrict__ correction, int K, int R, int top, int group_count,
                     int group_keep, float weight_scale, int renormalize, const float* __restrict__ logit_bias,
-                    const float* __restrict__ gate_w, float* __restrict__ gate_out) {
+                    const float* __restrict__ gate_w, float* __restrict__ gate_out, int sigmoid_scores, int square_weights) {
   extern __shared__ float route_smem[];
   float* xs = route_smem;      // [K]
   float* s = xs + K;           // [R] logits, then scores
@@ -53,17 +56,21 @@ expert_route_kernel(int* __restrict__ idx_out, float* __restrict__ wgt_out, cons
   }
   __syncthreads();
   if (warp != 0) return;
-  float m = -INFINITY;
-  for (int e = lane; e < R; e += 32) m = fmaxf(m, s[e]);
-  m = warp_max(m);
-  float sum = 0.f;
-  for (int e = lane; e < R; e += 32) {
-    const float p = expf(s[e] - m);
-    s[e] = p;
-    sum += p;
+  float inv = 1.f;
+  if (sigmoid_scores) {
+    for (int e = lane; e < R; e += 32) s[e] = 1.0f / (1.0f + expf(-s[e]));
+  } else {
+    float m = -INFINITY;
+    for (int e = lane; e < R; e += 32) m = fmaxf(m, s[e]);
+    m = warp_max(m);
+    float sum = 0.f;
+    for (int e = lane; e < R; e += 32) {
+      const float p = expf(s[e] - m);
+      s[e] = p;
+      sum += p;
+    }
+    inv = 1.0f / warp_sum(sum);
   }
-  sum = warp_sum(sum);
-  const float inv = 1.0f / sum;
   for (int e = lane; e < R; e += 32) {
     const float p = s[e] * inv;
     s[e] = p;
@@ -132,7 +139,10 @@ expert_route_kernel(int* __restrict__ idx_out, float* __restrict__ wgt_out, cons
   }
   if (lane == 0) {
     const float f = renormalize ? weight_scale / total : weight_scale;
-    for (int r = 0; r < top; ++r) wgt_out[(size_t)t * top + r] *= f;
+    for (int r = 0; r < top; ++r) {
+      const float w = wgt_out[(size_t)t * top + r] * f;
+      wgt_out[(size_t)t * top + r] = square_weights ? w * w : w;
+    }
   }
 }
 
@@ -185,21 +195,29 @@ expert_plan_kernel(int* __restrict__ pos, int* __restrict__ perm, int* __restric
   }
 }
 
+// act 0: SiLU, 1: the tanh form of GELU, 2: the square of relu
 __device__ __forceinline__ float act_of(float g, int act) {
+  if (act == 2) {
+    g = fmaxf(g, 0.f);
+    return g * g;
+  }
   return act == 0 ? g / (1.0f + expf(-g)) : 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
 }
 
 // ---------------------------------------------------------------- the experts' products, float32 arithmetic
 // One CTA per (tile of sorted rows of one expert, 64 output columns). GATED: out[row, n] = act(a . Wg[e][n]) * (a . Wu[e][n])
-// with a = x[perm[row] / top] (W [E, 2N, K]: N gate rows, then N up rows), written in the run's dtype; else
-// out[row, n] = a . W[e][n] with a = A[row], written in float32. Every element adds its k = 0 .. K-1 in order.
+// with a = x[perm[row] / top] (W [E, 2N, K]: N gate rows, then N up rows), written in the run's dtype; XG_ACT: out[row, n] =
+// act(a . W[e][n]) in the run's dtype, a gathered likewise; XG_PLAIN: out[row, n] = a . W[e][n] with a = A[row], written in
+// float32. Every element adds its k = 0 .. K-1 in order.
+enum XgMode : int { XG_PLAIN = 0, XG_GATED = 1, XG_ACT = 2 };
 constexpr int XG_BM = 64, XG_BN = 64, XG_BK = 16, XG_THREADS = 256;
 
-template <typename T, bool GATED>
+template <typename T, int MODE>
 __global__ void __launch_bounds__(XG_THREADS)
 expert_gemm_kernel(void* __restrict__ out_, const T* __restrict__ A, int lda, const int* __restrict__ perm, int top,
                    const T* __restrict__ W, const int* __restrict__ tiles, const int* __restrict__ meta,
                    const int* __restrict__ offsets, int N, int K, int act) {
+  constexpr bool GATED = MODE == XG_GATED;
   __shared__ float As[XG_BK][XG_BM + 4];
   __shared__ float Bg[XG_BK][XG_BN + 4];
   __shared__ float Bu[GATED ? XG_BK : 1][XG_BN + 4];
@@ -253,6 +271,7 @@ expert_gemm_kernel(void* __restrict__ out_, const T* __restrict__ A, int lda, co
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
       if (GATED) Elem<T>::store((T*)out_ + (size_t)(row0 + r) * N + n, act_of(acc[i][j], act) * acu[i][j]);
+      else if (MODE == XG_ACT) Elem<T>::store((T*)out_ + (size_t)(row0 + r) * N + n, act_of(acc[i][j], act));
       else ((float*)out_)[(size_t)(row0 + r) * N + n] = acc[i][j];
     }
   }
@@ -279,11 +298,12 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-template <bool GATED>
+template <int MODE>
 __global__ void __launch_bounds__(XM_THREADS)
 expert_gemm_mma_kernel(void* __restrict__ out_, const __nv_bfloat16* __restrict__ A, int lda, const int* __restrict__ perm, int top,
                        const __nv_bfloat16* __restrict__ W, const int* __restrict__ tiles, const int* __restrict__ meta,
                        const int* __restrict__ offsets, int N, int K, int act) {
+  constexpr bool GATED = MODE == XG_GATED;
   __shared__ __align__(16) __nv_bfloat16 As[2][XM_BM][XM_LD];
   __shared__ __align__(16) __nv_bfloat16 Bg[2][XM_BN][XM_LD];
   __shared__ __align__(16) __nv_bfloat16 Bu[GATED ? 2 : 1][GATED ? XM_BN : 1][XM_LD];
@@ -377,6 +397,8 @@ expert_gemm_mma_kernel(void* __restrict__ out_, const __nv_bfloat16* __restrict_
           if (GATED)
             ((__nv_bfloat16*)out_)[(size_t)(row0 + r) * N + n + j] =
                 __float2bfloat16_rn(act_of(v, act) * acu[GATED ? mi : 0][GATED ? ni : 0][half * 2 + j]);
+          else if (MODE == XG_ACT)
+            ((__nv_bfloat16*)out_)[(size_t)(row0 + r) * N + n + j] = __float2bfloat16_rn(act_of(v, act));
           else
             ((float*)out_)[(size_t)(row0 + r) * N + n + j] = v;
         }
@@ -416,7 +438,8 @@ MS_DEFINE_PDL_SWITCH(ms_experts_set_pdl)
 
 MS_EXPORT int ms_expert_route(int* idx, float* wgt, const void* x, int ld_x, const float* router, const float* correction, int tokens,
                               int K, int R, int top, int group_count, int group_keep, float weight_scale, int renormalize, int dtype,
-                              cudaStream_t stream, const float* logit_bias, const float* gate_w, float* gate_out) {
+                              cudaStream_t stream, const float* logit_bias, const float* gate_w, float* gate_out, int sigmoid_scores,
+                              int square_weights) {
   if (tokens == 0) return 0;
   MS_CHECK_ARG(R >= 1 && top >= 1 && top <= R && K >= 1, "expert_route: top %d of %d router outputs", top, R);
   MS_CHECK_ARG(group_count >= 1 && R % group_count == 0 && group_keep >= 1 && group_keep <= group_count &&
@@ -427,12 +450,12 @@ MS_EXPORT int ms_expert_route(int* idx, float* wgt, const void* x, int ld_x, con
   if (dtype == MS_F32) {
     if (smem > 48 * 1024) MS_CHECK_CUDA(cudaFuncSetAttribute(expert_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     MS_LAUNCH(expert_route_kernel<float>, tokens, ROUTE_THREADS, smem, stream, idx, wgt, (const float*)x, ld_x, router, correction, K, R, top,
-              group_count, group_keep, weight_scale, renormalize, logit_bias, gate_w, gate_out);
+              group_count, group_keep, weight_scale, renormalize, logit_bias, gate_w, gate_out, sigmoid_scores, square_weights);
   } else {
     if (smem > 48 * 1024)
       MS_CHECK_CUDA(cudaFuncSetAttribute(expert_route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     MS_LAUNCH(expert_route_kernel<__nv_bfloat16>, tokens, ROUTE_THREADS, smem, stream, idx, wgt, (const __nv_bfloat16*)x, ld_x, router,
-              correction, K, R, top, group_count, group_keep, weight_scale, renormalize, logit_bias, gate_w, gate_out);
+              correction, K, R, top, group_count, group_keep, weight_scale, renormalize, logit_bias, gate_w, gate_out, sigmoid_scores, square_weights);
   }
   return 0;
 }
@@ -486,35 +509,34 @@ MS_EXPORT int ms_expert_gather(void* xs, const void* x, int ld_x, const int* per
   return 0;
 }
 
-// gated = 1: out [slots, N] in the run's dtype = act(x Wg^T) * (x Wu^T) over the sorted rows (x gathered through perm);
-// gated = 0: out [slots, N] float32 = A W^T (A [slots, K] in sorted order; perm null).
+// mode 1: out [slots, N] in the run's dtype = act(x Wg^T) * (x Wu^T) over the sorted rows (x gathered through perm); mode 2: out
+// [slots, N] in the run's dtype = act(x W^T), gathered likewise; mode 0: out [slots, N] float32 = A W^T (A [slots, K] in sorted
+// order; perm null).
 MS_EXPORT int ms_expert_gemm(void* out, const void* A, int lda, const int* perm, int top, const void* W, const int* tiles, const int* meta,
-                             const int* offsets, int max_tiles, int N, int K, int gated, int act, int dtype, cudaStream_t stream) {
+                             const int* offsets, int max_tiles, int N, int K, int mode, int act, int dtype, cudaStream_t stream) {
   if (max_tiles == 0 || N == 0) return 0;
-  MS_CHECK_ARG(K >= 1 && top >= 1 && (act == 0 || act == 1), "expert_gemm: K=%d top=%d act=%d", K, top, act);
+  MS_CHECK_ARG(K >= 1 && top >= 1 && act >= 0 && act <= 2 && mode >= 0 && mode <= 2, "expert_gemm: K=%d top=%d act=%d mode=%d", K, top, act, mode);
   const dim3 grid(max_tiles, (N + XG_BN - 1) / XG_BN);
+#define MS_XG(T, M) \
+  MS_LAUNCH((expert_gemm_kernel<T, M>), grid, XG_THREADS, 0, stream, out, (const T*)A, lda, perm, top, (const T*)W, tiles, meta, offsets, N, K, act)
+#define MS_XM(M)                                                                                                                        \
+  MS_LAUNCH(expert_gemm_mma_kernel<M>, grid, XM_THREADS, 0, stream, out, (const __nv_bfloat16*)A, lda, perm, top, (const __nv_bfloat16*)W, \
+            tiles, meta, offsets, N, K, act)
   if (dtype == MS_F32) {
-    if (gated)
-      MS_LAUNCH((expert_gemm_kernel<float, true>), grid, XG_THREADS, 0, stream, out, (const float*)A, lda, perm, top, (const float*)W, tiles,
-                meta, offsets, N, K, act);
-    else
-      MS_LAUNCH((expert_gemm_kernel<float, false>), grid, XG_THREADS, 0, stream, out, (const float*)A, lda, perm, top, (const float*)W, tiles,
-                meta, offsets, N, K, act);
-    return 0;
-  }
-  const bool aligned = K % 8 == 0 && lda % 8 == 0 && (uintptr_t)A % 16 == 0 && (uintptr_t)W % 16 == 0;
-  const __nv_bfloat16* a = (const __nv_bfloat16*)A;
-  const __nv_bfloat16* w = (const __nv_bfloat16*)W;
-  if (aligned) {
-    if (gated) MS_LAUNCH(expert_gemm_mma_kernel<true>, grid, XM_THREADS, 0, stream, out, a, lda, perm, top, w, tiles, meta, offsets, N, K, act);
-    else MS_LAUNCH(expert_gemm_mma_kernel<false>, grid, XM_THREADS, 0, stream, out, a, lda, perm, top, w, tiles, meta, offsets, N, K, act);
+    if (mode == XG_GATED) MS_XG(float, XG_GATED);
+    else if (mode == XG_ACT) MS_XG(float, XG_ACT);
+    else MS_XG(float, XG_PLAIN);
+  } else if (K % 8 == 0 && lda % 8 == 0 && (uintptr_t)A % 16 == 0 && (uintptr_t)W % 16 == 0) {
+    if (mode == XG_GATED) MS_XM(XG_GATED);
+    else if (mode == XG_ACT) MS_XM(XG_ACT);
+    else MS_XM(XG_PLAIN);
   } else {
-    if (gated)
-      MS_LAUNCH((expert_gemm_kernel<__nv_bfloat16, true>), grid, XG_THREADS, 0, stream, out, a, lda, perm, top, w, tiles, meta, offsets, N, K, act);
-    else
-      MS_LAUNCH((expert_gemm_kernel<__nv_bfloat16, false>), grid, XG_THREADS, 0, stream, out, a, lda, perm, top, w, tiles, meta, offsets, N, K,
-                act);
+    if (mode == XG_GATED) MS_XG(__nv_bfloat16, XG_GATED);
+    else if (mode == XG_ACT) MS_XG(__nv_bfloat16, XG_ACT);
+    else MS_XG(__nv_bfloat16, XG_PLAIN);
   }
+#undef MS_XG
+#undef MS_XM
   return 0;
 }
 

@@ -13,10 +13,11 @@ from dataclasses import dataclass
 import torch
 
 from . import blas, experts, native
-from .mixers import (act_mul, add_dyt, add_layernorm, add_rmsnorm_scaled, add_row_vector, axpby, channel_gate, clamped_glu,  # noqa: F401
-                     conv_silu_unit, conv_state_update, decay_scan, gate_relu_squared, gated_group_norm, gelu_tanh, head_gate,
-                     head_norm_gate, latent_prepare, latent_rope_prepare, qkv_prepare, relu_squared, rope_table_scaled, row_rmsnorm,
-                     scale_, shift_state_update, ssm_step_decay, stream_concat, sum_bias, token_shift)
+from .mixers import (act_mul, add_dyt, add_layernorm, add_normed_rmsnorm, add_rmsnorm_scaled, add_row_vector, axpby, channel_gate,  # noqa: F401
+                     clamped_glu, conv_bias, conv_silu_unit, conv_state_update, decay_scan, embed_sum, gate_relu_squared, gated_group_norm,
+                     gelu_tanh, head_gate, head_norm_gate, latent_prepare, latent_rope_prepare, mlstm_gates, mlstm_output, qkv_prepare,
+                     relu_squared, rglru_scan, rope_table_scaled, row_rmsnorm, scale_, shift_state_update, ssm_step_decay, stream_concat,
+                     sum_bias, token_shift)
 from .native import NativeError, OutOfBlocks
 
 __all__ = [
@@ -303,11 +304,11 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor | None = Non
 def linear_heads(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, stream=None) -> torch.Tensor:
     """out[t, h, :] = weight[h] x[t, h, :]: every head has a matrix of its own. x [T, H, K] and out [T, H, N] may be
     views whose rows are part of wider ones; weight [H, N, K]. float32: this package's FFMA kernel, one launch over
-    all heads; bfloat16: the vendor library's strided batched product (float32 accumulation)."""
+    all heads; bfloat16: the vendor library's strided batched product (float32 accumulation; ``out`` may be float32)."""
     t, h, kdim = x.shape
     n = weight.shape[1]
     assert weight.shape == (h, n, kdim) and weight.is_contiguous() and out.shape == (t, h, n) and x.is_cuda
-    assert x.stride(2) == 1 and out.stride(2) == 1 and x.dtype == weight.dtype == out.dtype
+    assert x.stride(2) == 1 and out.stride(2) == 1 and x.dtype == weight.dtype and out.dtype in (x.dtype, torch.float32)
     if t == 0:
         return out
     if x.dtype == torch.float32:

@@ -211,13 +211,13 @@ def gemm_bf16(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, stream: 
 
 def gemm_bf16_batched(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, stream: int) -> None:
     """out[:, b, :] = x[:, b, :] times weight[b]^T for every b: ``batch`` independent products in one call
-    (``cublasGemmStridedBatchedEx``, bfloat16 operands, float32 accumulation). x [M, B, K] and out [M, B, N] may be
+    (``cublasGemmStridedBatchedEx``, bfloat16 operands, float32 accumulation, bfloat16 or float32 out). x [M, B, K] and out [M, B, N] may be
     views whose rows are part of wider ones (last stride 1); weight [B, N, K] is contiguous. These are the
     per-head matrices of a mixer whose heads each have a small matrix of their own."""
     m, b, k = x.shape
     n = weight.shape[1]
     assert weight.shape == (b, n, k) and weight.is_contiguous() and out.shape == (m, b, n)
-    assert x.stride(2) == 1 and out.stride(2) == 1 and x.dtype == weight.dtype == out.dtype == torch.bfloat16
+    assert x.stride(2) == 1 and out.stride(2) == 1 and x.dtype == weight.dtype == torch.bfloat16 and out.dtype in (torch.bfloat16, torch.float32)
     lib = _library()
     if not hasattr(lib, "_ms_batched_declared"):
         ll = ctypes.c_longlong
@@ -234,4 +234,5 @@ def gemm_bf16_batched(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, 
     # column-major view per product: out_b^T [N, M] = weight_b (as [K, N], transposed) times x_b^T [K, M]
     _check(lib.cublasGemmStridedBatchedEx(
         handle, _OP_T, _OP_N, n, m, k, _p_one, weight.data_ptr(), _R_16BF, k, n * k, x.data_ptr(), _R_16BF, x.stride(0), x.stride(1),
-        _p_zero, out.data_ptr(), _R_16BF, out.stride(0), out.stride(1), b, _COMPUTE_32F, _GEMM_DEFAULT), "cublasGemmStridedBatchedEx")
+        _p_zero, out.data_ptr(), _R_32F if out.dtype == torch.float32 else _R_16BF, out.stride(0), out.stride(1), b, _COMPUTE_32F,
+        _GEMM_DEFAULT), "cublasGemmStridedBatchedEx")

@@ -79,18 +79,20 @@ def head_gate(out: torch.Tensor, attn: torch.Tensor, gate: torch.Tensor | None, 
 
 def qkv_prepare(q_out, k_pool, v_pool, q, k, v, q_norm_w, k_norm_w, cos_sin, rotary_dim: int, adjacent: bool, eps: float,
                 positions, row_of_token, page_indptr, page_indices, page_size: int, status, stream=None, bias=None,
-                unit_norm: bool = False, q_scale=None) -> None:
+                unit_norm: bool = False, q_scale=None, q_temp: tuple[float, float] | None = None) -> None:
     """Per-head RMS norm of q and k (float32 weights or None), rotation of the first ``rotary_dim`` channels
     (pairs (2i, 2i+1) if ``adjacent`` else (i, i + rotary_dim/2)) by the step's cos/sin table, q to
     ``q_out`` [T, nq, D] and k, v into their pages [pages, nkv, page_size, D], zero beyond their own
     sizes. ``q`` [T, nq*dk], ``k`` [T, nkv*dk], ``v`` [T, nkv*dv]: views into one projection's rows.
     ``bias``: float32 [nq*dk + nkv*dk + nkv*dv], the projections' biases in the order q, k, v, added first.
     ``unit_norm``: q and k are divided by their root mean square also without norm weights. ``q_scale``: float32 [nq],
-    a factor per query head applied last. Without pools (``k_pool``, ``k`` and ``v`` None) only the queries are
+    a factor per query head applied last. ``q_temp`` (coef, every): queries at position p are also multiplied by
+    1 + coef ln(floor((p + 1) / every) + 1). Without pools (``k_pool``, ``k`` and ``v`` None) only the queries are
     prepared (a mixer that reads another's keys and values); ``bias`` is then [nq*dk]."""
     t, nq, d = q_out.shape
     dk = q.shape[1] // nq
     _f32(q_norm_w, k_norm_w, cos_sin, bias, q_scale)
+    coef, every = q_temp or (0.0, 0.0)
     assert cos_sin is None or cos_sin.shape == (t, rotary_dim)
     assert q_scale is None or q_scale.numel() == nq
     if k_pool is None:
@@ -100,7 +102,7 @@ def qkv_prepare(q_out, k_pool, v_pool, q, k, v, q_norm_w, k_norm_w, cos_sin, rot
             _ptr(q_out), None, None, q.data_ptr(), _rows(q), 0, 0, 0, _ptr(q_norm_w), None, _ptr(cos_sin), _ptr(positions),
             _ptr(row_of_token), _ptr(page_indptr), _ptr(page_indices), t, nq, 1, dk, dk, d, rotary_dim if cos_sin is not None else 0,
             int(adjacent), float(eps), page_size, 0, _ptr(status), _dt(q.dtype), _stream(stream), _ptr(bias), _ptr(q_scale),
-            int(unit_norm)))
+            int(unit_norm), float(coef), float(every)))
         return
     nkv = k_pool.shape[1]
     dv = v.shape[1] // nkv
@@ -117,7 +119,7 @@ def qkv_prepare(q_out, k_pool, v_pool, q, k, v, q_norm_w, k_norm_w, cos_sin, rot
         _ptr(q_out), _ptr(k_pool), _ptr(v_pool), base, ld, offs[0], offs[1], offs[2], _ptr(q_norm_w), _ptr(k_norm_w),
         _ptr(cos_sin), _ptr(positions), _ptr(row_of_token), _ptr(page_indptr), _ptr(page_indices), t, nq, nkv, dk, dv, d,
         rotary_dim if cos_sin is not None else 0, int(adjacent), float(eps), page_size, k_pool.shape[0], _ptr(status),
-        _dt(q.dtype), _stream(stream), _ptr(bias), _ptr(q_scale), int(unit_norm)))
+        _dt(q.dtype), _stream(stream), _ptr(bias), _ptr(q_scale), int(unit_norm), float(coef), float(every)))
 
 
 def add_layernorm(out, residual, delta, weight, bias, eps: float, rows=None, num_rows=None, write_residual=True, delta_scale: float = 1.0,
@@ -179,24 +181,27 @@ def sum_bias(out, a, b=None, vec=None, stream=None) -> None:
 
 
 def decay_scan(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign: float, beta, ctx, heads: int, dk: int, dv: int,
-               q_scale: float, delta: bool, head_decay: bool = False, v_scale=None) -> None:
+               q_scale: float, delta: bool, head_decay: bool = False, v_scale=None, ones_column: bool = False) -> None:
     """The token-by-token recurrence of every row of the step (``csrc/recurrence.cu``), from each
     request's slot of ``state`` [slots, heads, dv, dk] float32 (zero where a row starts at position 0)
     and back into it; o_out [T, heads, dv] float32. q, k [T, groups*dk], v [T, heads*dv], z [T, heads*dk]
     and beta [T, heads] are 2-d views; z_bias [heads*dk], decay_coef [heads] float32.
     ``head_decay``: z [T, heads] float32 holds the decays themselves, one for all key channels of a head and token
-    (z_bias, decay_coef and z_sign are not used). ``v_scale`` [T, heads] float32: v counts times it, per token and head."""
+    (z_bias, decay_coef and z_sign are not used; all three may be None, None and 0). ``v_scale`` [T, heads] float32: v counts times it, per token and head.
+    ``ones_column``: v has heads * (dv - 1) columns and every head's last value is one (times v_scale): that column of the state is
+    the decayed sum of the keys, that entry of the output its product with the query (the decay rule only)."""
     t = o_out.shape[0]
+    dv_in = dv - int(ones_column)
     _f32(o_out, state, z_bias, decay_coef, v_scale)
     assert o_out.shape == (t, heads, dv) and state.shape[1:] == (heads, dv, dk)
     groups = q.shape[1] // dk
-    assert q.shape == (t, groups * dk) and k.shape == q.shape and v.shape == (t, heads * dv)
+    assert q.shape == (t, groups * dk) and k.shape == q.shape and v.shape == (t, heads * dv_in)
     assert z.shape == (t, heads if head_decay else heads * dk) and (not head_decay or (z.dtype == torch.float32 and not delta))
     assert q.dtype == k.dtype == v.dtype and (beta is None or beta.dtype == z.dtype)
     assert v_scale is None or v_scale.shape == (t, heads)
     if not delta and not ctx.decode_only and t >= SEGMENT_MIN_TOKENS and SEGMENTS > 1:
         return _decay_scan_segmented(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign, ctx, heads, dk, dv, q_scale, head_decay,
-                                     v_scale)
+                                     v_scale, dv_in)
     ready = int(head_decay)
     if not ctx.decode_only and not head_decay:
         # a prompt portion: exponentials and logarithms for all tokens at once, not inside the serial walk
@@ -211,7 +216,7 @@ def decay_scan(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign: float, beta
         _ptr(o_out), _ptr(state), _ptr(q), _rows(q), _ptr(k), _rows(k), heads // groups, _ptr(v), _rows(v), _ptr(z), _rows(z),
         _ptr(z_bias), _ptr(decay_coef), float(z_sign), ready, _ptr(beta), 0 if beta is None else _rows(beta), _ptr(ctx.cu_q),
         _ptr(ctx.q_start), _ptr(ctx.state_slot), ctx.num_rows, heads, dk, dv, float(q_scale), int(delta), _dt(q.dtype),
-        _dt(z.dtype), int(head_decay), _ptr(v_scale), ctx.stream))
+        _dt(z.dtype), int(head_decay), _ptr(v_scale), dv_in, ctx.stream))
 
 
 def conv_silu_unit(out, x, conv_state, weight, ctx, unit_heads: int, dk: int, other_heads: int, dv: int, unit_eps: float,
@@ -248,7 +253,7 @@ SEGMENT_MIN_TOKENS = 512
 
 
 def _decay_scan_segmented(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign, ctx, heads, dk, dv, q_scale, head_decay=False,
-                          v_scale=None) -> None:
+                          v_scale=None, dv_in=None) -> None:
     from types import SimpleNamespace
 
     t, dev, p, rows = o_out.shape[0], o_out.device, SEGMENTS, ctx.num_rows
@@ -277,7 +282,8 @@ def _decay_scan_segmented(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign, 
     native.recurrence_check(lib.ms_decay_scan(
         _ptr(o_out), _ptr(ends), _ptr(q), _rows(q), _ptr(k), _rows(k), heads // groups, _ptr(v), _rows(v), _ptr(decay), _rows(decay),
         _ptr(z_bias), _ptr(decay_coef), float(z_sign), 1, None, 0, _ptr(pieces.cu_q), _ptr(pieces.q_start), _ptr(pieces.state_slot),
-        pieces.num_rows, heads, dk, dv, float(q_scale), 0, _dt(q.dtype), 0, int(head_decay), _ptr(v_scale), ctx.stream))
+        pieces.num_rows, heads, dk, dv, float(q_scale), 0, _dt(q.dtype), 0, int(head_decay), _ptr(v_scale), dv if dv_in is None else dv_in,
+        ctx.stream))
     native.recurrence_check(lib.ms_segment_finish(
         _ptr(o_out), _ptr(state), _ptr(ends), _ptr(before), _ptr(cum), _ptr(decay), _rows(decay), _ptr(q), _rows(q), heads // groups,
         _ptr(seg_cu), _ptr(ctx.q_start), _ptr(ctx.state_slot), rows, t, p, heads, dk, dv, float(q_scale), _dt(q.dtype), int(head_decay),
@@ -452,3 +458,100 @@ def act_mul(out, gate_up, activation: str, stream=None) -> None:
     assert out.is_contiguous() and gate_up.is_contiguous() and gate_up.shape == (t, 2 * inter) and gate_up.dtype == out.dtype
     native.mixers_check(native.mixers().ms_act_mul(_ptr(out), _ptr(gate_up), t, inter, ACTIVATIONS[activation], _dt(out.dtype),
                                                    _stream(stream)))
+
+
+# ---------------------------------------------------------------- csrc/stream_ops.cu
+
+def embed_sum(residual, table, ctx, inv_freq=None, pair_table=None, pair=None, prev_token=None) -> None:
+    """residual[t] = table[id] (+ pair_table[row]) (+ the sinusoidal vector of the position), float32. ``pair`` = (buckets,
+    mul_prev, mul_cur): row = (previous token * mul_prev + token * mul_cur) mod buckets, row ``buckets`` at position 0; the token
+    before a portion's first one is the row's slot of ``prev_token`` (int32 [slots, 1]), which gets the portion's last token.
+    ``inv_freq`` float32 [(width + 1) // 2]: entry 2i gets sin(position * inv_freq[i]), entry 2i + 1 the cosine."""
+    t, hidden = residual.shape
+    _f32(residual, inv_freq)
+    assert table.is_contiguous() and table.shape[1] == hidden and ctx.token_ids.numel() >= t
+    assert inv_freq is None or inv_freq.numel() == (hidden + 1) // 2
+    buckets, mul_prev, mul_cur = pair or (0, 0, 0)
+    assert (pair is None) == (pair_table is None) == (prev_token is None)
+    assert pair is None or (pair_table.shape == (buckets + 1, hidden) and pair_table.dtype == table.dtype and pair_table.is_contiguous()
+                            and prev_token.dtype == torch.int32)
+    native.mixers_check(native.mixers().ms_embed_sum(
+        _ptr(residual), _ptr(table), _ptr(pair_table), buckets, mul_prev, mul_cur, _ptr(inv_freq), _ptr(ctx.token_ids), _ptr(ctx.positions),
+        _ptr(ctx.row_of_token), _ptr(ctx.cu_q), _ptr(ctx.state_slot), _ptr(prev_token), t, hidden, table.shape[0], _dt(table.dtype),
+        ctx.stream))
+
+
+def add_normed_rmsnorm(out, residual, delta, weight, eps: float, delta_weight=None, delta_eps: float = 0.0, rows=None, num_rows=None,
+                       write_residual=True, stream=None) -> None:
+    """h = residual[r] + rmsnorm(delta[r]) * delta_weight (delta as it is without ``delta_weight``), written back to ``residual``
+    when there is no gather; out[i] = rmsnorm(h) * weight; r = rows[i] (or i). Weights float32: [hidden], or one element for all
+    coordinates. float32 arithmetic."""
+    _f32(residual, weight, delta_weight)
+    hidden = residual.shape[-1]
+    n = out.shape[0] if num_rows is None else num_rows
+    assert out.is_contiguous() and out.shape[-1] == hidden
+    assert delta is None or (delta.dtype == out.dtype and delta.is_contiguous())
+    native.mixers_check(native.mixers().ms_add_normed_rmsnorm(
+        _ptr(out), _ptr(residual), _ptr(delta), _ptr(delta_weight), 1 if delta_weight is None else delta_weight.numel(), float(delta_eps),
+        _ptr(weight), weight.numel(), float(eps), _ptr(rows), n, hidden, int(write_residual and rows is None), _dt(out.dtype),
+        _stream(stream)))
+
+
+# ---------------------------------------------------------------- csrc/gated_recurrence.cu
+
+def mlstm_gates(out, raw, bias, m_state, ctx, cap: float) -> None:
+    """``out`` [3, T, H] float32 = (decay of the state, factor of the token's write, exp(-m)) of a matrix memory with exponential
+    gates and a running maximum m (``m_state`` float32 [slots, H], 0 where a row starts its sequence). ``raw`` [T, 2 H] a view: the
+    input gates' products, then the forget gates'; ``bias`` float32 [2 H]."""
+    _, t, h = out.shape
+    _f32(out, bias, m_state)
+    assert out.shape == (3, t, h) and raw.shape == (t, 2 * h) and bias.numel() == 2 * h and m_state.shape[1] == h
+    native.recurrence_check(native.recurrence().ms_mlstm_gates(
+        _ptr(out[0]), _ptr(out[1]), _ptr(out[2]), _ptr(raw), _rows(raw), _ptr(bias), _ptr(m_state), _ptr(ctx.cu_q), _ptr(ctx.q_start),
+        _ptr(ctx.state_slot), ctx.num_rows, h, float(cap), int(ctx.decode_only), _dt(raw.dtype), ctx.stream))
+
+
+def mlstm_output(out, o, floor, weight, gate, eps: float, den_eps: float, stream=None) -> None:
+    """out[t, h*dv + c] = y / sqrt(mean_c y^2 + eps) * weight[h*dv + c] * sigmoid(gate[t, h*dv + c]) with
+    y = o[t, h, c] / (max(|o[t, h, dv]|, floor[t, h]) + den_eps); ``o`` [T, H, dv + 1] float32."""
+    t, heads, dv1 = o.shape
+    dv = dv1 - 1
+    _f32(o, floor, weight)
+    assert out.shape == (t, heads * dv) and gate.shape == (t, heads * dv) and gate.dtype == out.dtype and weight.numel() == heads * dv
+    assert floor.shape == (t, heads)
+    native.recurrence_check(native.recurrence().ms_mlstm_output(
+        _ptr(out), _rows(out), _ptr(o), _ptr(floor), _ptr(weight), _ptr(gate), _rows(gate), t, heads, dv, float(eps), float(den_eps),
+        _dt(out.dtype), _stream(stream)))
+
+
+def conv_bias(u, x, conv_state, weight, bias, in_bias, ctx) -> None:
+    """u [T, C] = bias + a causal convolution over time of x + in_bias (``x`` [T, C] a view; zeros before a sequence's start, where
+    no in_bias counts either), no activation. ``weight`` float32 [taps, C], tap-major, the last one the current token's;
+    ``conv_state`` [slots, taps - 1, C] holds each request's last raw inputs and is brought up to date."""
+    t, c = u.shape
+    taps = weight.shape[0]
+    _f32(weight, bias, in_bias)
+    assert x.shape == (t, c) and x.dtype == u.dtype == conv_state.dtype and u.is_contiguous() and conv_state.is_contiguous()
+    assert weight.shape == (taps, c) and bias.numel() == c and in_bias.numel() == c and conv_state.shape[1:] == (max(taps - 1, 0), c)
+    single = int(ctx.decode_only)  # one token per row: the same launch moves the history up
+    native.recurrence_check(native.recurrence().ms_conv_bias(
+        _ptr(u), _ptr(x), _rows(x), _ptr(conv_state), _ptr(weight), _ptr(bias), _ptr(in_bias), _ptr(ctx.row_of_token), _ptr(ctx.cu_q),
+        _ptr(ctx.q_start), _ptr(ctx.state_slot), t, c, taps, single, _dt(x.dtype), ctx.stream))
+    if taps > 1 and not single:
+        conv_state_update(conv_state, x, ctx, taps)
+
+
+def rglru_scan(out, state, z, u, y, bias_r, bias_i, coef, y_bias, ctx) -> None:
+    """The gated linear recurrence of every row of the step, from each request's slot of ``state`` [slots, C] float32 (zero where a
+    row starts its sequence) and back into it: with r, g = sigmoid(z[t, b, 0 | 1] + bias) of each channel, a = exp(-coef r),
+    S = a S + sqrt(1 - a^2) g u, out[t] = S * gelu_tanh(y[t] + y_bias). ``z`` float32 [T, blocks, 2, C / blocks]; ``u`` [T, C];
+    ``y`` [T, C] a view; biases and ``coef`` float32 [C]."""
+    t, c = out.shape
+    _f32(state, z, bias_r, bias_i, coef, y_bias)
+    assert out.is_contiguous() and u.is_contiguous() and u.shape == (t, c) and y.shape == (t, c) and out.dtype == u.dtype == y.dtype
+    blocks = z.shape[1]
+    assert z.shape == (t, blocks, 2, c // blocks) and blocks * z.shape[3] == c and state.shape[1] == c
+    assert all(v.numel() == c for v in (bias_r, bias_i, coef, y_bias))
+    native.recurrence_check(native.recurrence().ms_rglru_scan(
+        _ptr(out), _ptr(state), _ptr(z), _ptr(u), _ptr(y), _rows(y), _ptr(bias_r), _ptr(bias_i), _ptr(coef), _ptr(y_bias), _ptr(ctx.cu_q),
+        _ptr(ctx.q_start), _ptr(ctx.state_slot), ctx.num_rows, t, c, c // blocks, int(ctx.decode_only), _dt(out.dtype), ctx.stream))

@@ -128,7 +128,7 @@ def mixers():
     _declare(lib, "ms_scale_f32", [_p, _f, _ll, _p])
     _declare(lib, "ms_axpby", [_p, _p, _p, _f, _f, _ll, _i, _p])
     _declare(lib, "ms_head_gate", [_p, _i, _p, _p, _i, _i, _i, _i, _i, _f, _i, _p])
-    _declare(lib, "ms_qkv_prepare", [_p] * 4 + [_i] * 4 + [_p] * 7 + [_i] * 8 + [_f, _i, _i, _p, _i, _p, _p, _p, _i])
+    _declare(lib, "ms_qkv_prepare", [_p] * 4 + [_i] * 4 + [_p] * 7 + [_i] * 8 + [_f, _i, _i, _p, _i, _p, _p, _p, _i, _f, _f])
     _declare(lib, "ms_add_rmsnorm_scaled", [_p, _p, _p, _f, _p, _f, _p, _f, _i, _i, _i, _i, _p])
     _declare(lib, "ms_stream_concat", [_p, _p, _p, _f, _p, _p, _i, _i, _i, _i, _i, _i, _p])
     _declare(lib, "ms_add_row_vector", [_p, _p, _i, _i, _p])
@@ -145,6 +145,8 @@ def mixers():
     _declare(lib, "ms_shift_state_update", [_p, _p, _p, _p, _i, _i, _i, _p])
     _declare(lib, "ms_clamped_glu", [_p, _p, _p, _i, _i, _f, _f, _f, _i, _p])
     _declare(lib, "ms_sum_bias", [_p, _p, _p, _p, _i, _i, _i, _p])
+    _declare(lib, "ms_embed_sum", [_p, _p, _p, _ll, _ll, _ll, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _p])
+    _declare(lib, "ms_add_normed_rmsnorm", [_p, _p, _p, _p, _i, _f, _p, _i, _f, _p, _i, _i, _i, _i, _p])
     return lib
 
 
@@ -155,7 +157,7 @@ def recurrence():
     _declare(lib, "ms_recurrence_set_pdl", [_i], None)
     lib.ms_recurrence_set_pdl(int(pdl_enabled()))
     _declare(lib, "ms_decay_scan", [_p, _p, _p, _i, _p, _i, _i, _p, _i, _p, _i, _p, _p, _f, _i, _p, _i, _p, _p, _p,
-                                    _i, _i, _i, _i, _f, _i, _i, _i, _i, _p, _p])
+                                    _i, _i, _i, _i, _f, _i, _i, _i, _i, _p, _i, _p])
     _declare(lib, "ms_segment_setup", [_p, _p, _p, _p, _i, _i, _p])
     _declare(lib, "ms_segment_finish", [_p, _p, _p, _p, _p, _p, _i, _p, _i, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _i, _p])
     _declare(lib, "ms_decay_from_logits", [_p, _p, _i, _p, _p, _f, _p, _i, _i, _i, _i, _i, _p])
@@ -164,6 +166,10 @@ def recurrence():
     _declare(lib, "ms_gated_group_norm", [_p, _i, _p, _p, _i, _p, _p, _i, _p, _i, _i, _i, _i, _f, _i, _p])
     _declare(lib, "ms_conv_state_update", [_p, _p, _i, _p, _p, _p, _i, _i, _i, _i, _p])
     _declare(lib, "ms_head_norm_gate", [_p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _f, _i, _i, _p])
+    _declare(lib, "ms_mlstm_gates", [_p, _p, _p, _p, _i, _p, _p, _p, _p, _p, _i, _i, _f, _i, _i, _p])
+    _declare(lib, "ms_mlstm_output", [_p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _f, _f, _i, _p])
+    _declare(lib, "ms_conv_bias", [_p, _p, _i, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _p])
+    _declare(lib, "ms_rglru_scan", [_p, _p, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p])
     return lib
 
 
@@ -173,7 +179,7 @@ def experts():
     _declare(lib, "ms_experts_last_error", [], c_char_p)
     _declare(lib, "ms_experts_set_pdl", [_i], None)
     lib.ms_experts_set_pdl(int(pdl_enabled()))
-    _declare(lib, "ms_expert_route", [_p, _p, _p, _i, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _i, _p, _p, _p, _p])
+    _declare(lib, "ms_expert_route", [_p, _p, _p, _i, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _i, _p, _p, _p, _p, _i, _i])
     _declare(lib, "ms_expert_max_tiles", [_i, _i])
     _declare(lib, "ms_expert_plan", [_p, _p, _p, _p, _p, _p, _i, _i, _p])
     _declare(lib, "ms_expert_max_tiles_of", [_i, _i, _i])

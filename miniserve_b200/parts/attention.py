@@ -46,7 +46,9 @@ class GQAttention(Part):
     scaled score of query i and key j), ``keep_first`` (the first keys of a sequence stay visible behind the window;
     the cache then keeps every page) and ``cache_window`` (how far back the cache keeps keys when that is not the
     mixer's own reach: 0 for everything, for a mixer whose cache another mixer with a longer reach reads). With
-    ``kv_source`` = ``shared`` these run on the general path too: the projection holds q (and the gate) alone."""
+    ``kv_source`` = ``shared`` these run on the general path too: the projection holds q (and the gate) alone.
+    ``query_temperature`` = (coef, every): the prepared query at position p is multiplied by
+    1 + coef ln(floor((p + 1) / every) + 1), in float32."""
     shape_static = True
     input_weight = "w_qkv"  # the attribute that holds the input product's (stacked) matrix; its first ``input_rows`` rows are real
     NAMES = dict(q="q_proj.weight", k="k_proj.weight", v="v_proj.weight", o="o_proj.weight", q_norm="q_norm.weight",
@@ -86,6 +88,10 @@ class GQAttention(Part):
         self.qkv_bias = bool(spec.get("qkv_bias", False))
         self.head_temperature = bool(spec.get("head_temperature", False))
         self.distance_bias = bool(spec.get("distance_bias", False))
+        temp = spec.get("query_temperature")
+        self.query_temperature = (float(temp[0]), float(temp[1])) if temp else None
+        if self.query_temperature and self.query_temperature[1] <= 0:
+            raise ValueError(f"query_temperature={temp}: the number of positions per step must be positive")
         self.keep_first = int(spec.get("keep_first") or 0)
         self.cache_window = spec.get("cache_window")
         if self.keep_first < 0 or (self.keep_first and not self.window):
@@ -94,7 +100,7 @@ class GQAttention(Part):
         self.adjacent = getattr(self.position, "pairing", "halves") == "adjacent"  # how the position encoding pairs channels
         self.general = bool(self.out_gate or self.value_dim != self.head_dim or self.adjacent or self.learned_sink or self.softcap
                             or self.chunk or getattr(self.position, "table_only", False) or self.unit_norm or self.qkv_bias
-                            or self.head_temperature or self.distance_bias or self.keep_first or spec.get("general"))
+                            or self.head_temperature or self.distance_bias or self.keep_first or self.query_temperature or spec.get("general"))
         self.w_sink = None
         self.extras = None
         self.w_bias = self.w_temp = None
@@ -214,7 +220,8 @@ class GQAttention(Part):
                         proj[:, at_v:at_g] if own else None, self.w_q_norm, self.w_k_norm,
                         self.position.step_table(ctx), rotary_dim, self.adjacent, self.qk_norm_eps,
                         ctx.positions, ctx.row_of_token, ctx.page_indptr[cache.group], ctx.page_indices[cache.group],
-                        cache.page_size, ctx.status, stream=ctx.stream, bias=self.w_bias, unit_norm=self.unit_norm, q_scale=self.w_temp)
+                        cache.page_size, ctx.status, stream=ctx.stream, bias=self.w_bias, unit_norm=self.unit_norm, q_scale=self.w_temp,
+                        q_temp=self.query_temperature)
         att = ctx.buffer("attn.out", (t, nq, dc), dt, dev)
         ops.attention(att, q, cache.k, cache.v, ctx, cache.group, self.scale, self.reach, self.sink, extras=self.extras)
         if raw:  # the caller takes attention's output [T, heads, D] itself (no gate, values as wide as the cache's heads)

@@ -8,13 +8,15 @@ checkpoint tensors it wants by name relative to its own prefix, receives them in
 
 Categories and what each must provide:
 
-``norm``          ``forward(residual, delta, ctx, rows=None, write_residual=True, delta_scale=1.0) -> Tensor``
+``norm``          ``forward(residual, delta, ctx, rows=None, write_residual=True, delta_scale=1.0) -> Tensor`` (a norm that can
+                  also norm its addend takes ``delta_norm``, the part whose weight and eps that one has)
 ``position``      ``kernel_table() -> (inv_freq | None, rotary_dim)``, ``step_table(ctx) -> cos/sin table | None``
 ``mixer``         ``cache_need() -> CacheNeed | tuple of them | None`` and ``forward(x, ctx, cache) -> Tensor``
                   (``cache``: the view of its need, or a tuple of views in the order of the needs)
 ``feed_forward``  ``forward(x, ctx) -> Tensor``
 ``block``         ``forward(stream, ctx, cache) -> ResidualStream`` (arranges the four above)
-``embedding``     ``forward(ctx) -> float32 residual [T, hidden]``
+``embedding``     ``forward(ctx) -> float32 residual [T, hidden]``; one that keeps state per request also ``cache_need()``, and its
+                  ``forward(ctx, cache)`` gets the view
 ``head``          ``forward(x, ctx) -> float32 logits [rows, vocab]``
 ``transition``    ``forward(stream, ctx, embedding, arg) -> ResidualStream`` (acts on the stream between two layers)
 """
@@ -173,11 +175,13 @@ class ResidualStream:
     """The residual stream between blocks: ``total`` (float32 [T, hidden]) plus an addend
     that has not been added yet (the last feed-forward output), so that the add can be
     fused into the next norm. The addend counts ``pending_scale`` times (a block that adds its
-    sublayers' output times a constant hands the constant on instead of scaling the tensor)."""
+    sublayers' output times a constant hands the constant on instead of scaling the tensor).
+    ``pending_norm``: a norm part that the addend passes before it is added (a block that norms its sublayers' outputs)."""
 
     total: torch.Tensor
     pending: torch.Tensor | None = None
     pending_scale: float = 1.0
+    pending_norm: "Part | None" = None
 
 
 def param(spec: PartSpec, key: str, typ: type | None = None) -> Any:

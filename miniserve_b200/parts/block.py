@@ -10,7 +10,9 @@ from .base import BuildEnv, FixedState, Part, ResidualStream, WeightDecl, build_
 
 
 def _norm(norm, stream: ResidualStream, ctx):
-    """A block's first norm over the stream as the block before left it (its addend and the addend's factor)."""
+    """A block's first norm over the stream as the block before left it (its addend and the addend's factor or norm)."""
+    if stream.pending_norm is not None:
+        return norm.forward(stream.total, stream.pending, ctx, delta_norm=stream.pending_norm)
     if stream.pending_scale != 1.0:
         return norm.forward(stream.total, stream.pending, ctx, delta_scale=stream.pending_scale)
     return norm.forward(stream.total, stream.pending, ctx)
@@ -51,6 +53,43 @@ class PreNormBlock(Part):
             return ResidualStream(total, a)
         x = self.norm2.forward(total, a, ctx)
         return ResidualStream(total, self.feed_forward.forward(x, ctx))
+
+
+@register_part("block", "sandwich")
+class SandwichBlock(Part):
+    """h += norm1b(mixer(norm1(h))); h += norm2b(feed_forward(norm2(h))): a norm before and after each sublayer. The norm
+    behind a sublayer, the add and the next norm run as one kernel; the block hands its last sublayer's output on as the
+    pending addend together with the norm that it passes. Parameters: ``names`` (mixer / feed_forward / norm1 / norm2 / norm1b /
+    norm2b -> tensor-name prefixes). A layer without a feed-forward has neither it nor norm2 nor norm2b."""
+    shape_static = True
+
+    def __init__(self, spec, env: BuildEnv, layer: LayerSpec | None = None):
+        super().__init__(spec, env)
+        if layer is None:
+            raise ValueError("a block is built from its LayerSpec (use build_block)")
+        names = dict(spec.get("names") or {})
+        self.has_ff = layer.feed_forward is not None
+        norms = ("norm1", "norm1b") + (("norm2", "norm2b") if self.has_ff else ())
+        self.names = {k: names[k] for k in ("mixer",) + norms + (("feed_forward",) if self.has_ff else ())}
+        self.mixer = build_part("mixer", layer.mixer, env)
+        self.feed_forward = build_part("feed_forward", layer.feed_forward, env) if self.has_ff else None
+        self.norms = {k: build_part("norm", layer.norms[k], env) for k in norms}
+
+    def sub_parts(self):
+        out = {self.names["mixer"]: self.mixer, **{self.names[k]: n for k, n in self.norms.items()}}
+        if self.has_ff:
+            out[self.names["feed_forward"]] = self.feed_forward
+        return out
+
+    def forward(self, stream: ResidualStream, ctx, cache) -> ResidualStream:
+        total = stream.total
+        x = _norm(self.norms["norm1"], stream, ctx)
+        a = self.mixer.forward(x, ctx, cache)
+        if not self.has_ff:
+            return ResidualStream(total, a, pending_norm=self.norms["norm1b"])
+        x = self.norms["norm2"].forward(total, a, ctx, delta_norm=self.norms["norm1b"])
+        return ResidualStream(total, self.feed_forward.forward(x, ctx), pending_norm=self.norms["norm2b"])
+
 
 @register_part("block", "parallel_residual")
 class ParallelResidualBlock(Part):
@@ -211,7 +250,7 @@ class ParallelDualNormBlock(Part):
 
     def forward(self, stream: ResidualStream, ctx, cache) -> ResidualStream:
         total = stream.total
-        if self.paired:
+        if self.paired and stream.pending_norm is None:
             h1, h2 = self.norm1.forward_pair(self.norm2, total, stream.pending, ctx, delta_scale=stream.pending_scale)
         else:
             h1 = _norm(self.norm1, stream, ctx)

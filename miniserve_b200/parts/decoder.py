@@ -52,7 +52,19 @@ class DecoderModel:
                                      f"({mixer.spec.kind}) wants a cache of its own")
                 owner = self.entry_caches[e.cache_of]
                 self.entry_caches.append(EntryCache(owner.owner, owner.need))
+        # an embedding that keeps something per request (the token before) comes behind the run entries
+        need = self.embedding.cache_need() if hasattr(self.embedding, "cache_need") else None
+        self.embedding_entry: int | None = None
+        if need is not None:
+            self.embedding_entry = len(self.entry_caches)
+            self.entry_caches.append(EntryCache(self.embedding_entry, need))
         self.bound = False
+
+    def embed(self, ctx, caches) -> torch.Tensor:
+        """The stream's first value, float32 [T, hidden]."""
+        if self.embedding_entry is None:
+            return self.embedding.forward(ctx)
+        return self.embedding.forward(ctx, caches[self.embedding_entry])
 
     @property
     def shape_static(self) -> bool:
@@ -139,7 +151,7 @@ class DecoderModel:
     # ------------------------------------------------------------------ forward
     def forward(self, ctx, caches) -> torch.Tensor:
         """Run the tokens of ``ctx`` through every run entry; ``caches[i]`` is the cache view
-        of run entry i. Returns float32 logits at ``ctx.logit_rows``: [wanted, vocab]."""
+        of run entry i (and one more behind them for an embedding with state). Returns float32 logits at ``ctx.logit_rows``: [wanted, vocab]."""
         if not self.bound:
             raise RuntimeError("the model has no weights yet (bind() was not called)")
         # What parts share within one pass is made anew by every pass. That holds for the activation
@@ -148,12 +160,14 @@ class DecoderModel:
         # memory that goes back to the allocator while the graph still holds their addresses.
         ctx.step_cache.clear()
         ctx.buffers.clear()
-        stream = ResidualStream(self.embedding.forward(ctx))
+        stream = ResidualStream(self.embed(ctx, caches))
         for i, entry in enumerate(self.spec.run_order):
             if entry.transition is not None:
                 stream = self.transitions[entry.transition].forward(stream, ctx, self.embedding, entry.transition_arg)
             stream = self.layers[entry.layer].forward(stream, ctx, caches[i])
         extra = {"delta_scale": stream.pending_scale} if stream.pending_scale != 1.0 else {}
+        if stream.pending_norm is not None:
+            extra["delta_norm"] = stream.pending_norm
         x = self.final_norm.forward(stream.total, stream.pending, ctx, rows=ctx.logit_rows,
                                     num_rows=ctx.num_logit_rows, write_residual=False, **extra)
         return self.head.forward(x, ctx)

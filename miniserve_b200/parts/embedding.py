@@ -5,7 +5,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from .base import Part, WeightDecl, param, register_part
+from .base import FixedState, Part, WeightDecl, param, register_part
 
 
 @register_part("embedding", "token_embedding")
@@ -31,6 +31,52 @@ class TokenEmbedding(Part):
         ops.embed_gather(residual, self.table, ctx.token_ids, stream=ctx.stream)
         return residual
 
+
+@register_part("embedding", "summed_embedding")
+class SummedEmbedding(Part):
+    """h = table[id] (+ bigram[row]) (+ sinusoid(position)), summed in float32 by one kernel.
+
+    ``bigram`` (a mapping with ``buckets``, ``mul_prev``, ``mul_cur``, ``name``; or absent): a second table of buckets + 1 rows, read
+    at row (previous token * mul_prev + token * mul_cur) mod buckets, and at its last row for a sequence's first token. The
+    previous token is state of the request (one int32 in its slot), so that a portion or a decoded token continues from it.
+    ``sinusoid`` (a base, or absent): entry 2i of the position's vector is sin(position * base^(-2i / hidden)), entry 2i + 1 the
+    cosine (frequencies worked out in float64 and rounded once; the angle and its sine and cosine are float32).
+    Parameters: ``vocab``, ``hidden``, ``name`` (the table's full name), ``bigram``, ``sinusoid``."""
+    shape_static = True
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.vocab = param(spec, "vocab", int)
+        self.hidden = param(spec, "hidden", int)
+        self.name = param(spec, "name", str)
+        b = spec.get("bigram")
+        self.pair = (int(b["buckets"]), int(b["mul_prev"]), int(b["mul_cur"])) if b else None
+        self.pair_name = str(b["name"]) if b else None
+        if self.pair and (self.pair[0] < 1 or min(self.pair[1:]) < 0):
+            raise ValueError(f"summed_embedding: a bigram table needs buckets and factors that are not negative, got {self.pair}")
+        base = spec.get("sinusoid")
+        self.inv_freq = None
+        if base is not None:
+            i = torch.arange(0, (self.hidden + 1) // 2, dtype=torch.float64)
+            self.inv_freq = (float(base) ** (-2.0 * i / self.hidden)).to(torch.float32).to(env.device)
+
+    def cache_need(self):
+        return FixedState((1,), torch.int32) if self.pair else None
+
+    def weights(self):
+        w = {self.name: WeightDecl((self.vocab, self.hidden))}
+        if self.pair:
+            w[self.pair_name] = WeightDecl((self.pair[0] + 1, self.hidden))
+        return w
+
+    def bind(self, tensors):
+        self.table = tensors[self.name].contiguous()
+        self.pair_table = tensors[self.pair_name].contiguous() if self.pair else None
+
+    def forward(self, ctx, cache=None) -> torch.Tensor:
+        residual = torch.empty((ctx.num_tokens, self.hidden), dtype=torch.float32, device=self.table.device)
+        ops.embed_sum(residual, self.table, ctx, self.inv_freq, self.pair_table, self.pair, cache.state if self.pair else None)
+        return residual
 
 
 @register_part("head", "linear_head")

@@ -1,7 +1,7 @@
 """Linear-attention mixers: a matrix state per head and request instead of keys and values of every
-past token. Both run the token-by-token recurrence of ``csrc/recurrence.cu`` (prompt portions and
-decoded tokens alike), keep the state in float32 in the request's slot, and start from zero where a
-row's first token is at position 0."""
+past token, or a vector (the gated linear recurrence at the end). The matrix states run the token-by-token recurrence of
+``csrc/recurrence.cu`` (prompt portions and decoded tokens alike). All keep the state in float32 in the request's slot, and
+start from zero where a row's first token is at position 0."""
 
 from __future__ import annotations
 
@@ -316,3 +316,153 @@ class SelectiveStateSpace(Part):
         feat = ctx.buffer("ssm.feat", (t, self.feature_width), dt, dev)
         self.features(x, ctx, cache, feat)
         return ops.linear(feat, self.w_o, stream=ctx.stream, out=ctx.buffer("ssm.proj", (t, self.hidden), dt, dev))
+
+
+@register_part("mixer", "mlstm")
+class MatrixMemory(Part):
+    """A matrix memory with exponential gates and a running maximum (the mLSTM of xLSTM): per head, with log gates
+    i = cap tanh((W_i x + b_i) / cap) and f = logsigmoid(cap tanh((W_f x + b_f) / cap)),
+
+        m_t = max(f + m_(t-1), i) from m_0 = 0,   S_t = exp(f + m_(t-1) - m_t) S_(t-1) + exp(i - m_t) k_t v_t^T,   n_t likewise with k_t
+        o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-m_t)) + den_eps),   q = W_q x dk^-0.5
+
+    then each head's o is divided by its root mean square, the heads side by side times a weight, times sigmoid(W_g x), then W_o.
+    One product makes q|k|v|g|i|f. The gates' kernel works out m, both exponentials and exp(-m) for every token (float32); the walk
+    is the decay rule of ``csrc/recurrence.cu`` with one decay per head, a factor on the write, and n as one more column of S.
+    State: S with that column [heads, dv + 1, dk] and m [heads], float32.
+    Parameters: ``hidden``, ``heads``, ``key_dim``, ``value_dim``, ``gate_cap``, ``eps``, ``den_eps`` (1e-6), ``names``
+    (q, k, v, g, o, norm, i, f, i_bias, f_bias -> tensor names)."""
+    shape_static = True
+    NAMES = dict(q="q_proj.weight", k="k_proj.weight", v="v_proj.weight", g="g_proj.weight", o="o_proj.weight", norm="norm.weight",
+                 i="i_gate.weight", f="f_gate.weight", i_bias="i_gate.bias", f_bias="f_gate.bias")
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.hidden = param(spec, "hidden", int)
+        self.heads = param(spec, "heads", int)
+        self.dk = param(spec, "key_dim", int)
+        self.dv = param(spec, "value_dim", int)
+        self.cap = param(spec, "gate_cap", float)
+        self.eps = param(spec, "eps", float)
+        self.den_eps = float(spec.get("den_eps", 1e-6))
+        self.names = {**self.NAMES, **dict(spec.get("names") or {})}
+        if self.cap <= 0:
+            raise ValueError(f"mlstm: gate_cap={self.cap} must be positive")
+        self.feature_width = self.heads * self.dv
+
+    def cache_need(self):
+        return (FixedState((self.heads, self.dv + 1, self.dk), torch.float32), FixedState((self.heads,), torch.float32))
+
+    def weights(self):
+        n, h, dk, dv, w, f32 = self.names, self.heads, self.dk, self.dv, self.hidden, dict(precision="float32")
+        return {n["q"]: WeightDecl((h * dk, w)), n["k"]: WeightDecl((h * dk, w)), n["v"]: WeightDecl((h * dv, w)), n["g"]: WeightDecl((h * dv, w)),
+                n["i"]: WeightDecl((h, w)), n["f"]: WeightDecl((h, w)), n["i_bias"]: WeightDecl((h,), **f32),
+                n["f_bias"]: WeightDecl((h,), **f32), n["norm"]: WeightDecl((h * dv,), init="ones_normal", **f32),
+                n["o"]: WeightDecl((w, h * dv))}
+
+    def stacks(self):
+        n = self.names
+        return {"qkvgif_proj.weight": tuple(n[k] for k in ("q", "k", "v", "g", "i", "f"))}
+
+    def bind(self, tensors):
+        n = self.names
+        joined = self.joined(tensors, "qkvgif_proj.weight", self.stacks()["qkvgif_proj.weight"])
+        self.w_in = _pad_rows(joined, _pad8(joined.shape[0]))
+        self.w_gate_bias = torch.cat((tensors[n["i_bias"]].float(), tensors[n["f_bias"]].float())).contiguous()
+        self.w_norm = tensors[n["norm"]].float().contiguous()
+        self.w_o = tensors[n["o"]].contiguous()
+
+    def features(self, x: torch.Tensor, ctx, cache, out: torch.Tensor) -> None:
+        t, dt, dev = x.shape[0], self.env.dtype, self.w_o.device
+        h, dk, dv = self.heads, self.dk, self.dv
+        state, running = cache
+        proj = ops.linear(x, self.w_in, stream=ctx.stream, out=ctx.buffer("mlstm.in", (t, self.w_in.shape[0]), dt, dev))
+        at_k, at_v, at_g = h * dk, 2 * h * dk, 2 * h * dk + h * dv
+        at_i = at_g + h * dv
+        gates = ctx.buffer("mlstm.gates", (3, t, h), torch.float32, dev)  # the state's decay, the write's factor, exp(-m)
+        ops.mlstm_gates(gates, proj[:, at_i:at_i + 2 * h], self.w_gate_bias, running.state, ctx, self.cap)
+        o = ctx.buffer("mlstm.o", (t, h, dv + 1), torch.float32, dev)
+        ops.decay_scan(o, state.state, proj[:, :at_k], proj[:, at_k:at_v], proj[:, at_v:at_g], gates[0], None, None, 0.0, None, ctx, h, dk,
+                       dv + 1, dk ** -0.5, delta=False, head_decay=True, v_scale=gates[1], ones_column=True)
+        ops.mlstm_output(out, o, gates[2], self.w_norm, proj[:, at_g:at_i], self.eps, self.den_eps, stream=ctx.stream)
+
+    def forward(self, x, ctx, cache):
+        t, dt, dev = x.shape[0], self.env.dtype, self.w_o.device
+        feat = ctx.buffer("mlstm.feat", (t, self.feature_width), dt, dev)
+        self.features(x, ctx, cache, feat)
+        return ops.linear(feat, self.w_o, stream=ctx.stream, out=ctx.buffer("mlstm.proj", (t, self.hidden), dt, dev))
+
+
+@register_part("mixer", "rglru")
+class GatedLinearRecurrence(Part):
+    """A recurrent block with a real-gated linear recurrent unit (Griffin): two branches of ``width`` channels,
+    y = gelu_tanh(W_y x + b_y) and u = conv(W_x x + b_x), a short causal convolution per channel with a bias and no activation;
+
+        r, g = sigmoid(R_b u_b + c_b), sigmoid(G_b u_b + d_b)     (u in ``blocks`` equal parts, a square matrix each)
+        log a = -decay_scale r softplus(lam),   S_t = a S_(t-1) + sqrt(1 - a^2) g u,   out = W_o (S y)
+
+    One product makes y|x, one batched product over the parts both gates (float32 out), one kernel the gates' activations, the
+    recurrence and the multiplication with y. The state S [width] is float32; the convolution's last taps - 1 inputs are state too.
+    Parameters: ``hidden``, ``width``, ``blocks``, ``conv`` (taps), ``decay_scale`` (8), ``names`` (y, y_bias, x, x_bias, conv, conv_bias,
+    r, r_bias, i, i_bias, lam, o -> tensor names)."""
+    shape_static = True
+    NAMES = dict(y="y_proj.weight", y_bias="y_proj.bias", x="x_proj.weight", x_bias="x_proj.bias", conv="conv.weight", conv_bias="conv.bias",
+                 r="recurrence_gate.weight", r_bias="recurrence_gate.bias", i="input_gate.weight", i_bias="input_gate.bias", lam="lam",
+                 o="o_proj.weight")
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.hidden = param(spec, "hidden", int)
+        self.width = param(spec, "width", int)
+        self.blocks = param(spec, "blocks", int)
+        self.taps = param(spec, "conv", int)
+        self.decay_scale = float(spec.get("decay_scale", 8.0))
+        self.names = {**self.NAMES, **dict(spec.get("names") or {})}
+        if self.width % self.blocks:
+            raise ValueError(f"{self.width} channels do not split into {self.blocks} equal parts")
+        if self.taps < 1:
+            raise ValueError(f"the convolution needs at least one tap, got {self.taps}")
+        self.part = self.width // self.blocks
+        self.ld = _pad8(self.width)  # columns of one branch in the input product's rows
+
+    def cache_need(self):
+        state = FixedState((self.width,), torch.float32)
+        return state if self.taps == 1 else (state, FixedState((self.taps - 1, self.width), self.env.dtype))
+
+    def weights(self):
+        n, c, b, p, f32 = self.names, self.width, self.blocks, self.part, dict(precision="float32")
+        return {n["y"]: WeightDecl((c, self.hidden)), n["y_bias"]: WeightDecl((c,), **f32), n["x"]: WeightDecl((c, self.hidden)),
+                n["x_bias"]: WeightDecl((c,), **f32), n["conv"]: WeightDecl((c, self.taps), **f32), n["conv_bias"]: WeightDecl((c,), **f32),
+                n["r"]: WeightDecl((b, p, p)), n["r_bias"]: WeightDecl((b, p), **f32), n["i"]: WeightDecl((b, p, p)),
+                n["i_bias"]: WeightDecl((b, p), **f32), n["lam"]: WeightDecl((c,), **f32), n["o"]: WeightDecl((self.hidden, c))}
+
+    def bind(self, tensors):
+        n = self.names
+        self.w_in = torch.cat([_pad_rows(tensors[n[k]], self.ld) for k in ("y", "x")], dim=0).contiguous()
+        # [blocks, 2 part, part]: a part's recurrence gate rows, then its input gate rows
+        self.w_gates = torch.cat((tensors[n["r"]], tensors[n["i"]]), dim=1).contiguous()
+        f = {k: tensors[n[k]].float() for k in ("y_bias", "x_bias", "conv", "conv_bias", "r_bias", "i_bias", "lam")}
+        self.w_conv = f["conv"].t().contiguous()  # tap-major
+        self.w_conv_bias, self.w_x_bias, self.w_y_bias = (f[k].contiguous() for k in ("conv_bias", "x_bias", "y_bias"))
+        self.w_r_bias, self.w_i_bias = f["r_bias"].reshape(-1).contiguous(), f["i_bias"].reshape(-1).contiguous()
+        lam = f["lam"].double()
+        self.coef = (self.decay_scale * (lam.clamp(min=0) + torch.log1p(torch.exp(-lam.abs())))).float().contiguous()
+        self.w_o = tensors[n["o"]].contiguous()
+
+    def features(self, x: torch.Tensor, ctx, cache, out: torch.Tensor) -> None:
+        t, dt, dev = x.shape[0], self.env.dtype, self.w_o.device
+        c, b, p = self.width, self.blocks, self.part
+        state, conv = (cache if isinstance(cache, tuple) else (cache, None))
+        proj = ops.linear(x, self.w_in, stream=ctx.stream, out=ctx.buffer("rglru.in", (t, 2 * self.ld), dt, dev))
+        u = ctx.buffer("rglru.u", (t, c), dt, dev)
+        conv_state = conv.state if conv is not None else ctx.buffer("rglru.noconv", (1, 0, c), dt, dev)
+        ops.conv_bias(u, proj[:, self.ld:self.ld + c], conv_state, self.w_conv, self.w_conv_bias, self.w_x_bias, ctx)
+        z = ctx.buffer("rglru.z", (t, b, 2 * p), torch.float32, dev)
+        ops.linear_heads(u.view(t, b, p), self.w_gates, z, stream=ctx.stream)
+        ops.rglru_scan(out, state.state, z.view(t, b, 2, p), u, proj[:, :c], self.w_r_bias, self.w_i_bias, self.coef, self.w_y_bias, ctx)
+
+    def forward(self, x, ctx, cache):
+        t, dt, dev = x.shape[0], self.env.dtype, self.w_o.device
+        feat = ctx.buffer("rglru.feat", (t, self.width), dt, dev)
+        self.features(x, ctx, cache, feat)
+        return ops.linear(feat, self.w_o, stream=ctx.stream, out=ctx.buffer("rglru.proj", (t, self.hidden), dt, dev))

@@ -199,7 +199,13 @@ class RoutedExperts(Part):
     correction the weights are then the softmax over the chosen logits alone). ``shared`` (an intermediate size): one
     more gated feed-forward of the experts' form (a ``swiglu`` part under the prefix ``shared``) that every token uses;
     its output is added times sigmoid(w_sg . x), one number per token (tensor ``shared_gate`` [1, hidden], float32,
-    computed by the router's kernel from the same input), or unweighted with ``shared_gated`` False."""
+    computed by the router's kernel from the same input), or unweighted with ``shared_gated`` False.
+
+    ``score`` = ``sigmoid``: s = sigmoid(z), output by output. ``gated`` False: experts (and the shared one, then a ``dense_mlp``
+    part) without a gate, expert_e(x) = W_down[e] act(W_up[e] x) with ``activation`` = ``relu_squared``. ``weigh`` = ``input``: a
+    weight w multiplies its expert's input, expert_e(w x), instead of the output; for an expert that is homogeneous of degree
+    two (the square of relu without a gate; w is not negative) that is w^2 expert_e(x), so the router hands on squared
+    weights and the products read x as it is."""
     shape_static = True
     NAMES = dict(router="router.weight", correction="router.correction", expert="experts.{}.", gate="gate_proj.weight",
                  up="up_proj.weight", down="down_proj.weight", router_bias="router.bias", shared="shared.", shared_gate="shared.gate")
@@ -219,8 +225,17 @@ class RoutedExperts(Part):
         self.activation = spec.get("activation", "silu")
         if self.activation not in ops.experts.ACTIVATIONS:
             raise ValueError(f"routed_experts knows the activations {sorted(ops.experts.ACTIVATIONS)}, not {self.activation!r}")
-        if spec.get("score", "softmax") != "softmax":
-            raise NotImplementedError(f"routed_experts scores by softmax, not {spec.get('score')!r}")
+        self.score = spec.get("score", "softmax")
+        if self.score not in ops.experts.SCORES:
+            raise ValueError(f"routed_experts scores by {sorted(ops.experts.SCORES)}, not {self.score!r}")
+        self.gated = bool(spec.params.get("gated", True))
+        if self.gated == (self.activation == "relu_squared"):
+            raise ValueError(f"routed_experts: the activation {self.activation!r} does not go with gated={self.gated}")
+        self.weigh = spec.get("weigh", "output")
+        if self.weigh not in ("output", "input"):
+            raise ValueError(f"routed_experts: weigh must be 'output' or 'input', got {self.weigh!r}")
+        if self.weigh == "input" and (self.gated or self.identity):
+            raise NotImplementedError("routed_experts weighs inputs of experts without a gate (the square of relu) and of no identity experts")
         self.outputs = self.experts + self.identity  # what the router chooses among
         if self.experts < 1 or not 1 <= self.top <= self.outputs:
             raise ValueError(f"routed_experts: top={self.top} of {self.experts} experts and {self.identity} identity experts")
@@ -235,7 +250,8 @@ class RoutedExperts(Part):
         self.shared = None
         if self.shared_inter:
             n = self.names
-            self.shared = SwiGLU(PartSpec("swiglu", dict(hidden=self.hidden, intermediate=self.shared_inter, activation=self.activation,
+            self.shared = DenseMLP(PartSpec("dense_mlp", dict(hidden=self.hidden, intermediate=self.shared_inter, activation=self.activation,
+                                                              names=dict(up=n["up"], down=n["down"]))), env) if not self.gated else SwiGLU(PartSpec("swiglu", dict(hidden=self.hidden, intermediate=self.shared_inter, activation=self.activation,
                                                          names=dict(gate=n["gate"], up=n["up"], down=n["down"]))), env)
         self.w_router_bias = self.w_shared_gate = None
 
@@ -255,13 +271,14 @@ class RoutedExperts(Part):
         if self.shared_gated:
             w[n["shared_gate"]] = WeightDecl((1, self.hidden), precision="float32")
         for e in range(self.experts):
-            w[self._expert(e, "gate")] = WeightDecl((self.inter, self.hidden))
+            if self.gated:
+                w[self._expert(e, "gate")] = WeightDecl((self.inter, self.hidden))
             w[self._expert(e, "up")] = WeightDecl((self.inter, self.hidden))
             w[self._expert(e, "down")] = WeightDecl((self.hidden, self.inter))
         return w
 
     def stacks(self):
-        return {"experts.gate_up": tuple(self._expert(e, k) for e in range(self.experts) for k in ("gate", "up")),
+        return {"experts.gate_up": tuple(self._expert(e, k) for e in range(self.experts) for k in (("gate", "up") if self.gated else ("up",))),
                 "experts.down": tuple(self._expert(e, "down") for e in range(self.experts))}
 
     def bind(self, tensors):
@@ -270,7 +287,8 @@ class RoutedExperts(Part):
         self.w_correction = tensors[n["correction"]].float().contiguous() if self.has_correction else None
         self.w_router_bias = tensors[n["router_bias"]].float().contiguous() if self.has_router_bias else None
         self.w_shared_gate = tensors[n["shared_gate"]].float().reshape(-1).contiguous() if self.shared_gated else None
-        self.w_gate_up = self.joined(tensors, "experts.gate_up", st["experts.gate_up"]).view(self.experts, 2 * self.inter, self.hidden)
+        self.w_gate_up = self.joined(tensors, "experts.gate_up", st["experts.gate_up"]).view(
+            self.experts, (2 if self.gated else 1) * self.inter, self.hidden)
         self.w_down = self.joined(tensors, "experts.down", st["experts.down"]).view(self.experts, self.hidden, self.inter)
 
     def route(self, x, ctx):
@@ -281,7 +299,7 @@ class RoutedExperts(Part):
         gate = ctx.buffer("moe.shared_gate", (t,), torch.float32, dev) if self.shared_gated else None
         ops.experts.expert_route(idx, wgt, x, self.w_router, self.w_correction, self.top, self.group_count, self.group_keep,
                                  self.weight_scale, self.renormalize, stream=ctx.stream, logit_bias=self.w_router_bias,
-                                 gate_w=self.w_shared_gate, gate_out=gate)
+                                 gate_w=self.w_shared_gate, gate_out=gate, score=self.score, square_weights=self.weigh == "input")
         return idx, wgt
 
     def forward(self, x, ctx) -> torch.Tensor:
@@ -291,7 +309,7 @@ class RoutedExperts(Part):
         pos = ctx.buffer("moe.pos", (slots,), i32, dev)
         perm = ctx.buffer("moe.perm", (slots,), i32, dev)
         offsets = ctx.buffer("moe.offsets", (self.experts + 1,), i32, dev)
-        # bfloat16 with SiLU: both products on the tcgen05 kernel, over the tokens' inputs gathered into sorted order
+        # bfloat16: both products on the tcgen05 kernel where it has the activation, over the tokens' inputs gathered into sorted order
         tc = ops.experts.tc_experts_ok(dt, self.hidden, self.inter, self.activation) and x.stride(0) % 8 == 0
         tile_rows = ops.experts.TC_TILE_ROWS if tc else ops.experts.TILE_ROWS
         tiles = ctx.buffer("moe.tiles", (ops.experts.expert_max_tiles(slots, self.experts, tile_rows), 2), i32, dev)
@@ -302,10 +320,12 @@ class RoutedExperts(Part):
         if tc:
             xs = ctx.buffer("moe.xs", (slots, self.hidden), dt, dev)
             ops.experts.expert_gather(xs, x, perm, meta, self.top, stream=ctx.stream)
-            ops.experts.expert_products_tc(act, xs, self.w_gate_up, tiles, meta, offsets, True, stream=ctx.stream)
+            ops.experts.expert_products_tc(act, xs, self.w_gate_up, tiles, meta, offsets, self.gated, stream=ctx.stream,
+                                           relu_squared=not self.gated)
             ops.experts.expert_products_tc(y, act, self.w_down, tiles, meta, offsets, False, stream=ctx.stream)
         else:
-            ops.experts.expert_gate_up(act, x, self.w_gate_up, perm, self.top, tiles, meta, offsets, self.activation, stream=ctx.stream)
+            first = ops.experts.expert_gate_up if self.gated else ops.experts.expert_up
+            first(act, x, self.w_gate_up, perm, self.top, tiles, meta, offsets, self.activation, stream=ctx.stream)
             ops.experts.expert_down(y, act, self.w_down, tiles, meta, offsets, stream=ctx.stream)
         out = ctx.buffer("moe.out", (t, self.hidden), dt, dev)
         shared = self.shared.forward(x, ctx) if self.shared is not None else None

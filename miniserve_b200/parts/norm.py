@@ -13,8 +13,9 @@ class RMSNorm(Part):
     """y = x * rsqrt(mean(x^2) + eps) * weight, statistics in float32, no bias and no ``1 +``
     offset (miniserve/model/qwen3.py:78-82). Parameters: ``size``, ``eps``; optional ``unit_offset`` (the
     stored weight is the scale's distance from one: y = x * rsqrt(mean(x^2) + eps) * (1 + weight); the weight
-    then stays float32 whatever the run's dtype, so that 1 + weight is not rounded) and ``name`` (the
-    tensor's name relative to the part's prefix, default ``weight``)."""
+    then stays float32 whatever the run's dtype, so that 1 + weight is not rounded), ``scalar`` (the weight is one
+    number for all coordinates, a tensor of shape [], float32) and ``name`` (the tensor's name relative to the part's
+    prefix, default ``weight``). The addend may pass a norm of its own first (``delta_norm`` of ``forward``)."""
     shape_static = True
 
     def __init__(self, spec, env):
@@ -22,29 +23,49 @@ class RMSNorm(Part):
         self.size = param(spec, "size", int)
         self.eps = param(spec, "eps", float)
         self.unit_offset = bool(spec.get("unit_offset", False))
+        self.scalar = bool(spec.get("scalar", False))
+        if self.scalar and self.unit_offset:
+            raise ValueError("a norm with one number as its weight takes it as it is (no unit_offset)")
         self.name = spec.get("name", "weight")
         self._w_f32 = None
 
     def weights(self):
+        if self.scalar:
+            return {self.name: WeightDecl((), precision="float32", init="ones_normal")}
         if self.unit_offset:
             return {self.name: WeightDecl((self.size,), precision="float32")}
         return {self.name: WeightDecl((self.size,), init="ones_normal")}
 
     def bind(self, tensors):
-        self.w_weight = tensors[self.name].contiguous()
+        w = tensors[self.name]
+        self.w_weight = (w.reshape(1) if self.scalar else w).contiguous()
         self._w_f32 = self.w_weight if self.w_weight.dtype == torch.float32 else None
 
+    @property
+    def float_weight(self) -> torch.Tensor:
+        if self._w_f32 is None:
+            self._w_f32 = self.w_weight.float()
+        return self._w_f32
+
     def forward(self, residual: torch.Tensor, delta: torch.Tensor | None, ctx, rows: torch.Tensor | None = None,
-                num_rows: int | None = None, write_residual: bool = True, delta_scale: float = 1.0, role: str = "norm.out") -> torch.Tensor:
+                num_rows: int | None = None, write_residual: bool = True, delta_scale: float = 1.0, role: str = "norm.out",
+                delta_norm: "RMSNorm | None" = None) -> torch.Tensor:
         """Normalise ``residual (+ delta_scale * delta)``; without ``rows`` the sum is stored back into
         ``residual``. With ``rows`` (int32 indices) only those rows are produced. ``role``: the name of the output's
-        buffer, for a caller that keeps two norms' outputs alive at once."""
+        buffer, for a caller that keeps two norms' outputs alive at once. ``delta_norm``: the addend is
+        ``delta_norm(delta)``, in the same launch."""
         n = residual.shape[0] if rows is None else (num_rows if num_rows is not None else rows.numel())
         out = ctx.buffer(role, (n, self.size), self.env.dtype, residual.device)
+        if self.scalar or delta_norm is not None:
+            if self.unit_offset or delta_scale != 1.0 or (delta_norm is not None and delta_norm.unit_offset):
+                raise NotImplementedError("a normed addend, or one number as the weight, goes without unit_offset and without a factor on the addend")
+            ops.add_normed_rmsnorm(out, residual, delta, self.float_weight, self.eps,
+                                   delta_weight=delta_norm.float_weight if delta_norm is not None else None,
+                                   delta_eps=delta_norm.eps if delta_norm is not None else 0.0, rows=rows, num_rows=n,
+                                   write_residual=write_residual, stream=ctx.stream)
+            return out
         if self.unit_offset or delta_scale != 1.0:
-            if self._w_f32 is None:
-                self._w_f32 = self.w_weight.float()
-            ops.add_rmsnorm_scaled(out, residual, delta, delta_scale, self._w_f32, 1.0 if self.unit_offset else 0.0, self.eps,
+            ops.add_rmsnorm_scaled(out, residual, delta, delta_scale, self.float_weight, 1.0 if self.unit_offset else 0.0, self.eps,
                                    rows=rows, num_rows=n, write_residual=write_residual, stream=ctx.stream)
             return out
         ops.add_rmsnorm(out, residual, delta, self.w_weight, self.eps, rows=rows, num_rows=n,

@@ -36,6 +36,8 @@ class StreamReentry(Part):
     def forward(self, stream: ResidualStream, ctx, embedding, arg: int) -> ResidualStream:
         if not 0 <= arg < self.passes:
             raise ValueError(f"stream_reentry: pass {arg} of {self.passes}")
+        if stream.pending_norm is not None:
+            raise NotImplementedError("stream_reentry takes the stream's addend as it is, not through a norm")
         t, dt, dev = stream.total.shape[0], self.env.dtype, self.w_in.device
         both = ctx.buffer("reentry.in", (t, 2 * self.hidden), dt, dev)
         key = ("reentry.embedded", id(self))
