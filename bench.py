@@ -414,6 +414,23 @@ def kovusun_config(width: int, ff: int, runs: int, vocab: int, heads: int, kv_he
     return {"architecture": "Kovusun", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "layers": layers}
 
 
+def vumedra_config(width: int, ff: int, runs: int, vocab: int, heads: int, kv_heads: int) -> dict:
+    """A Vumedra model at a real model's layer sizes, in turns of four layers: a gated linear recurrence as wide as the model
+    (parts of 256, 4 taps), attention (the Qwen3 model's heads of 128), a matrix memory (heads of 128 x 256, as many as make the
+    values as wide as the model), a gated linear recurrence. The feed-forward is dense in even layers, and in odd ones 16 experts
+    without a gate of 3/8 ff of which a token uses 3 beside a shared expert of 3/8 ff (the products of a token equal the dense
+    layer's)."""
+    att = {"dim": 128, "heads": heads, "kv_heads": kv_heads, "q_temp": {"coef": 0.1, "every": 1024}, "scale": 128 ** -0.5, "vdim": 128}
+    mem = {"dim": 128, "gate_cap": 15.0, "heads": width // 256, "vdim": 256}
+    lru = {"blocks": width // 256, "conv": 4, "width": width}
+    dense = {"ff": ff, "kind": "dense"}
+    moe = {"kind": "moe", "expert": {"ff": 3 * ff // 8}, "router": {"experts": 16, "top": 3}, "shared": {"ff": 3 * ff // 8}}
+    turn = (("rglru", lru), ("attention", att), ("mlstm", mem), ("rglru", lru))
+    layers = [{"type": turn[i % 4][0], "mixer": dict(turn[i % 4][1]), "mlp": dict(moe if i % 2 else dense)} for i in range(runs)]
+    return {"architecture": "Vumedra", "width": width, "vocab": vocab, "norm": {"eps": 1e-5},
+            "embedding": {"bigram": {"buckets": 100003, "mul_prev": 31, "mul_cur": 7}}, "layers": layers}
+
+
 def bytes_per_step_of_weights(model) -> int:
     """Bytes of weights a step reads: every run of a layer reads that layer's tensors (a layer that runs twice
     counts twice), plus the norm before the head, the head and the parts between layers."""
@@ -462,7 +479,7 @@ def kernel_times(run_step, repeats: int = 3) -> dict:
 
 
 def run_fekulix(args, design: str = "fekulix") -> dict:
-    """Prefill and decode of a design (Fekulix, Mugipel, Rofozen) beside Qwen3 at equal width, depth, feed-forward and vocabulary."""
+    """Prefill and decode of a design (Fekulix, Mugipel, Rofozen, Kovusun, Vumedra) beside Qwen3 at equal width, depth, feed-forward and vocabulary."""
     import torch
 
     from miniserve_b200.config import preset
@@ -470,7 +487,7 @@ def run_fekulix(args, design: str = "fekulix") -> dict:
     from miniserve_b200.engine.step import StepRow
 
     peaks = load_peaks()
-    make = {"fekulix": fekulix_config, "mugipel": mugipel_config, "rofozen": rofozen_config, "kovusun": kovusun_config}[design]
+    make = {"fekulix": fekulix_config, "mugipel": mugipel_config, "rofozen": rofozen_config, "kovusun": kovusun_config, "vumedra": vumedra_config}[design]
     out = {"impl": "ours", "config": design, "dtype": "bf16", "data": "synthetic (random-init weights, uniform token ids)",
            "batch": args.batch, "context": CONTEXT, "prefill_tokens": PREFILL_TOKENS, "peaks": peaks["source"], "sizes": {}}
     steps = min(args.steps, 64)
@@ -489,6 +506,10 @@ def run_fekulix(args, design: str = "fekulix") -> dict:
             args_of = (q["hidden_size"], q["intermediate_size"], q["num_hidden_layers"], q["vocab_size"], q["num_attention_heads"],
                        q["num_key_value_heads"])
             beside += [("mugipel", mugipel_config(*args_of)), ("rofozen", rofozen_config(*args_of))]
+        if design == "vumedra":  # the closest designs: recurrent layers and routed experts; attention with biases and a shared expert
+            args_of = (q["hidden_size"], q["intermediate_size"], q["num_hidden_layers"], q["vocab_size"], q["num_attention_heads"],
+                       q["num_key_value_heads"])
+            beside += [("rofozen", rofozen_config(*args_of)), ("kovusun", kovusun_config(*args_of))]
         for name, raw in [(design, f)] + beside:
             llm = LLM(random=raw, weights_seed=0, dtype="bfloat16", kv_pool_tokens=10 * (CONTEXT + steps + 64) + 4096, page_size=16,
                       max_running=16, chunked_prefill_size=2048, cuda_graph=not args.no_graph)
@@ -699,10 +720,10 @@ def main() -> int:
     ap.add_argument("--no-graph", action="store_true", help="run decode steps without CUDA graphs")
     ap.add_argument("--profile-range", action="store_true",
                     help="bracket the timed steps with cudaProfilerStart/Stop (for ncu --profile-from-start off)")
-    ap.add_argument("--config", choices=["0.6b", "8b", "32b", "fekulix", "mugipel", "rofozen", "kovusun"], default="0.6b",
+    ap.add_argument("--config", choices=["0.6b", "8b", "32b", "fekulix", "mugipel", "rofozen", "kovusun", "vumedra"], default="0.6b",
                     help="0.6b: the benchmark line; 8b, 32b: the larger workloads through Engine.generate (a line of their own); "
-                         "fekulix, mugipel, rofozen, kovusun: prefill and decode of that design beside Qwen3 at equal sizes (a line of its own)")
-    ap.add_argument("--kernels", action="store_true", help="with --config fekulix, mugipel, rofozen or kovusun: also device time per kernel of a prompt step and a decode step")
+                         "fekulix, mugipel, rofozen, kovusun, vumedra: prefill and decode of that design beside Qwen3 at equal sizes (a line of its own)")
+    ap.add_argument("--kernels", action="store_true", help="with --config fekulix, mugipel, rofozen, kovusun or vumedra: also device time per kernel of a prompt step and a decode step")
     ap.add_argument("--only", choices=["all", "decode", "prefill"], default="all",
                     help="measure only the decode steps or only the prefill (for profiling); the line then lacks the other parts")
     args = ap.parse_args()
@@ -715,7 +736,7 @@ def main() -> int:
         args.warmup = 3
     global PROFILE_RANGE
     PROFILE_RANGE = args.profile_range
-    if args.config in ("fekulix", "mugipel", "rofozen", "kovusun") and args.impl == "ours":
+    if args.config in ("fekulix", "mugipel", "rofozen", "kovusun", "vumedra") and args.impl == "ours":
         result = run_fekulix(args, args.config)
     elif args.config != "0.6b" and args.impl == "ours":
         result = run_workload(args)

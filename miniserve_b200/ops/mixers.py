@@ -199,7 +199,7 @@ def decay_scan(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign: float, beta
     assert z.shape == (t, heads if head_decay else heads * dk) and (not head_decay or (z.dtype == torch.float32 and not delta))
     assert q.dtype == k.dtype == v.dtype and (beta is None or beta.dtype == z.dtype)
     assert v_scale is None or v_scale.shape == (t, heads)
-    if not delta and not ctx.decode_only and t >= SEGMENT_MIN_TOKENS and SEGMENTS > 1:
+    if not delta and not ctx.decode_only and t >= SEGMENT_MIN_TOKENS and SEGMENTS > 1 and dk <= SEGMENT_MAX_DK:
         return _decay_scan_segmented(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign, ctx, heads, dk, dv, q_scale, head_decay,
                                      v_scale, dv_in)
     ready = int(head_decay)
@@ -250,6 +250,7 @@ def conv_state_update(conv_state, x, ctx, taps: int) -> None:
 # number of tokens alone (what a captured graph is keyed by), never from how the tokens are shared among rows.
 SEGMENTS = 8
 SEGMENT_MIN_TOKENS = 512
+SEGMENT_MAX_DK = 320  # (what mends the outputs holds 32 tokens' queries and a column of the state in 48 KB)
 
 
 def _decay_scan_segmented(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign, ctx, heads, dk, dv, q_scale, head_decay=False,
