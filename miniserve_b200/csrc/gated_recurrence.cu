@@ -6,7 +6,8 @@
 //   o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-m_t)) + 1e-6).
 // With m known, this is the decay rule of recurrence.cu with one decay for the head and a factor on the token's write; n is
 // one more column of S whose value is 1. So three kernels surround that walk: the gates (m is a scan of the pairs
-// (f, i) under (F1, M1) o (F2, M2) = (F1 + F2, max(M1 + F2, M2))), the walk, and the division with the norm and the gate.
+// (f, i) under (F1, M1) o (F2, M2) = (F1 + F2, max(M1 + F2, M2))), the walk (recurrence.cu, or chunk_scan.cu for prompts in
+// bfloat16), and the division with the norm and the gate.
 //
 // A gated linear recurrence per channel (the real-gated linear recurrent unit):
 //   r_t, g_t = sigmoid of two products of u_t, log a_t = -c r_t, S_t = a_t S_(t-1) + sqrt(1 - a_t^2) g_t u_t,
@@ -96,9 +97,9 @@ mlstm_gates_kernel(float* __restrict__ decay, float* __restrict__ write, float* 
 }
 
 // out[t, h * dv + c] = (o[t, h, c] / (max(|o[t, h, dv]|, floor[t, h]) + den_eps)), divided by its root mean square over c, times
-// w[h * dv + c], times sigmoid(gate[t, h * dv + c]). o [T, H, dv + 1] float32. One warp per (token, head).
+// w[h * dv + c], times sigmoid(gate[t, h * dv + c]). o [T, H, ld_o] float32, its first dv + 1 columns. One warp per (token, head).
 template <typename T>
-__global__ void mlstm_output_kernel(T* __restrict__ out, int ld_out, const float* __restrict__ o, const float* __restrict__ floor_,
+__global__ void mlstm_output_kernel(T* __restrict__ out, int ld_out, const float* __restrict__ o, int ld_o, const float* __restrict__ floor_,
                                     const float* __restrict__ w, const T* __restrict__ gate, int ld_gate, long long items, int H, int dv,
                                     float eps, float den_eps) {
   pdl_prologue();
@@ -107,7 +108,7 @@ __global__ void mlstm_output_kernel(T* __restrict__ out, int ld_out, const float
   if (item >= items) return;
   const long long t = item / H;
   const int h = (int)(item - t * H);
-  const float* src = o + item * (dv + 1);
+  const float* src = o + item * ld_o;
   const float inv_den = 1.0f / (fmaxf(fabsf(src[dv]), floor_[item]) + den_eps);
   float ss = 0.f;
   for (int c = lane; c < dv; c += 32) {
@@ -315,16 +316,16 @@ MS_EXPORT int ms_mlstm_gates(float* decay, float* write, float* floor_, const vo
   return 0;
 }
 
-MS_EXPORT int ms_mlstm_output(void* out, int ld_out, const float* o, const float* floor_, const float* w, const void* gate, int ld_gate,
+MS_EXPORT int ms_mlstm_output(void* out, int ld_out, const float* o, int ld_o, const float* floor_, const float* w, const void* gate, int ld_gate,
                               int tokens, int H, int dv, float eps, float den_eps, int dtype, cudaStream_t stream) {
   if (tokens == 0) return 0;
   const long long items = (long long)tokens * H;
   const unsigned blocks = (unsigned)((items + 7) / 8);
   if (dtype == MS_F32)
-    MS_LAUNCH(mlstm_output_kernel<float>, blocks, 256, 0, stream, (float*)out, ld_out, o, floor_, w, (const float*)gate, ld_gate, items, H, dv,
+    MS_LAUNCH(mlstm_output_kernel<float>, blocks, 256, 0, stream, (float*)out, ld_out, o, ld_o, floor_, w, (const float*)gate, ld_gate, items, H, dv,
               eps, den_eps);
   else
-    MS_LAUNCH(mlstm_output_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)out, ld_out, o, floor_, w,
+    MS_LAUNCH(mlstm_output_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)out, ld_out, o, ld_o, floor_, w,
               (const __nv_bfloat16*)gate, ld_gate, items, H, dv, eps, den_eps);
   return 0;
 }

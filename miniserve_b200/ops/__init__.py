@@ -14,7 +14,7 @@ import torch
 
 from . import blas, experts, native
 from .mixers import (act_mul, add_dyt, add_layernorm, add_normed_rmsnorm, add_rmsnorm_scaled, add_row_vector, axpby, channel_gate,  # noqa: F401
-                     clamped_glu, conv_bias, conv_silu_unit, conv_state_update, decay_scan, embed_sum, gate_relu_squared, gated_group_norm,
+                     chunk_scan, chunk_scan_ok, clamped_glu, conv_bias, conv_silu_unit, conv_state_update, decay_scan, embed_sum, gate_relu_squared, gated_group_norm,
                      gelu_tanh, head_gate, head_norm_gate, latent_prepare, latent_rope_prepare, mlstm_gates, mlstm_output, qkv_prepare,
                      relu_squared, rglru_scan, rope_table_scaled, row_rmsnorm, scale_, shift_state_update, ssm_step_decay, stream_concat,
                      sum_bias, token_shift)
@@ -320,20 +320,24 @@ def linear_heads(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, strea
     return out
 
 
-def linear_gelu_tanh(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, stream=None) -> torch.Tensor:
-    """out [M, N] = gelu_tanh(x W^T). bfloat16 with at most 16 rows where the weight-streaming kernel is
-    the choice for the plain product: one kernel with the activation in its epilogue (the product is
+def linear_act(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, activation: str, stream=None) -> torch.Tensor:
+    """out [M, N] = act(x W^T), act ``gelu_tanh`` or ``relu_squared``. bfloat16 with at most 16 rows where the weight-streaming
+    kernel is the choice for the plain product: one kernel with the activation in its epilogue (the product is
     rounded to bfloat16 first, as when it is stored in between). Otherwise the product, then the
     activation kernel in place."""
     if x.dtype == torch.bfloat16 and not _tc_decode_ok(x, weight, out) and _skinny_ok(x, weight):
         _check_dev(x, weight, out)
         m, kdim = x.shape
         assert weight.shape[1] == kdim and out.shape == (m, weight.shape[0]) and out.dtype == torch.bfloat16
-        native.kernel_check(native.kernels().ms_gemm_skinny_gelu_bf16(_ptr(out), _ptr(x), _ptr(weight), m, weight.shape[0], kdim,
-                                                                      _stream(stream)))
+        k = native.kernels()
+        fused = k.ms_gemm_skinny_gelu_bf16 if activation == "gelu_tanh" else k.ms_gemm_skinny_relu2_bf16
+        native.kernel_check(fused(_ptr(out), _ptr(x), _ptr(weight), m, weight.shape[0], kdim, _stream(stream)))
         return out
     linear(x, weight, out=out, stream=stream)
-    gelu_tanh(out, out, stream=stream)
+    if activation == "gelu_tanh":
+        gelu_tanh(out, out, stream=stream)
+    else:
+        relu_squared(out, out, stream=stream)
     return out
 
 

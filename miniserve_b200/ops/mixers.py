@@ -291,6 +291,48 @@ def _decay_scan_segmented(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign, 
         ctx.stream), launches=3)
 
 
+CHUNK_MIN_TOKENS = 64  # steps with fewer tokens stay on the token-by-token walk
+
+
+def chunk_scan_ok(q, k, v, dk: int, dv: int, ctx) -> bool:
+    """Whether ``chunk_scan`` takes these operands: bfloat16, a step that is not all single tokens, heads of whole 16 bytes."""
+    if q.dtype != torch.bfloat16 or ctx.decode_only or q.shape[0] < CHUNK_MIN_TOKENS:
+        return False
+    return (bool(native.recurrence().ms_chunk_supports(dk, dv))
+            and all(x.data_ptr() % 16 == 0 and x.stride(0) % 8 == 0 for x in (q, k, v)))
+
+
+def chunk_scan(o, state, q, k, v, decay, write, ctx, heads: int, dk: int, dv: int, q_scale: float, ones: bool) -> None:
+    """The decay rule with one decay per head (``decay`` [T, H] float32 in [0, 1]; ``write`` [T, H] float32, a factor on the token's
+    write, or None) over chunks of 64 tokens on the tensor cores (``csrc/chunk_scan.cu``), from each request's slot of ``state``
+    [slots, heads, dv (+ 1), dk] float32 and back into it. q, k [T, groups * dk], v [T, heads * dv] bfloat16 views; ``o``
+    [T, heads, dv + 1 or wider, even] float32. ``ones``: one more value column whose value is one, behind the dv columns."""
+    t, _, ld_o = o.shape
+    rows, dev = ctx.num_rows, o.device
+    extra = int(ones)
+    _f32(o, state, decay, write)
+    groups = q.shape[1] // dk
+    assert q.shape == (t, groups * dk) and k.shape == q.shape and v.shape == (t, heads * dv) and state.shape[1:] == (heads, dv + extra, dk)
+    assert decay.shape == (t, heads) and (write is None or write.shape == (t, heads)) and ld_o >= dv + extra
+    lib = native.recurrence()
+    most = int(lib.ms_chunk_max(t, rows))
+    table = ctx.step_cache.get("chunk.table") if hasattr(ctx, "step_cache") else None
+    if table is None:  # the same for every layer of the step
+        ints = torch.empty(2 * most + rows + 1, dtype=torch.int32, device=dev)
+        table = (ints[:2 * most], ints[2 * most:])
+        native.recurrence_check(lib.ms_chunk_table(_ptr(table[0]), _ptr(table[1]), _ptr(ctx.cu_q), rows, ctx.stream))
+        if hasattr(ctx, "step_cache"):
+            ctx.step_cache["chunk.table"] = table
+    shape = (most, heads, dv + extra, dk)
+    added = ctx.buffer("chunk.added", shape, torch.float32, dev)
+    before = ctx.buffer("chunk.before", (2, *shape), torch.bfloat16, dev)
+    passed = ctx.buffer("chunk.decay", (most, heads), torch.float32, dev)
+    native.recurrence_check(lib.ms_chunk_scan(
+        _ptr(o), ld_o, _ptr(state), _ptr(q), _rows(q), _ptr(k), _rows(k), heads // groups, _ptr(v), _rows(v), _ptr(decay), _ptr(write), _ptr(added),
+        _ptr(before[0]), _ptr(before[1]), _ptr(passed), _ptr(table[0]), _ptr(table[1]), _ptr(ctx.cu_q), _ptr(ctx.q_start), _ptr(ctx.state_slot), rows,
+        most, heads, dk, dv, float(q_scale), extra, ctx.stream), launches=3)
+
+
 def ssm_step_decay(out, raw, bias, coef, stream=None) -> None:
     """out [2, T, H] float32: out[0] the step sizes softplus(raw[t, h] + bias[h]), out[1] the decays
     exp(-coef[h] * step size); ``raw`` [T, H] a view, bias and coef float32 [H]."""
@@ -514,14 +556,15 @@ def mlstm_gates(out, raw, bias, m_state, ctx, cap: float) -> None:
 
 def mlstm_output(out, o, floor, weight, gate, eps: float, den_eps: float, stream=None) -> None:
     """out[t, h*dv + c] = y / sqrt(mean_c y^2 + eps) * weight[h*dv + c] * sigmoid(gate[t, h*dv + c]) with
-    y = o[t, h, c] / (max(|o[t, h, dv]|, floor[t, h]) + den_eps); ``o`` [T, H, dv + 1] float32."""
-    t, heads, dv1 = o.shape
-    dv = dv1 - 1
+    y = o[t, h, c] / (max(|o[t, h, dv]|, floor[t, h]) + den_eps); ``o`` [T, H, dv + 1 or wider] float32."""
+    t, heads, ld_o = o.shape
+    dv = out.shape[1] // heads
     _f32(o, floor, weight)
+    assert ld_o >= dv + 1
     assert out.shape == (t, heads * dv) and gate.shape == (t, heads * dv) and gate.dtype == out.dtype and weight.numel() == heads * dv
     assert floor.shape == (t, heads)
     native.recurrence_check(native.recurrence().ms_mlstm_output(
-        _ptr(out), _rows(out), _ptr(o), _ptr(floor), _ptr(weight), _ptr(gate), _rows(gate), t, heads, dv, float(eps), float(den_eps),
+        _ptr(out), _rows(out), _ptr(o), ld_o, _ptr(floor), _ptr(weight), _ptr(gate), _rows(gate), t, heads, dv, float(eps), float(den_eps),
         _dt(out.dtype), _stream(stream)))
 
 

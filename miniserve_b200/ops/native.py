@@ -100,6 +100,7 @@ def kernels():
     _declare(lib, "ms_gemm_skinny_gate_up_bf16", [_p, _p, _p, _i, _i, _i, _p])
     _declare(lib, "ms_gemm_skinny_bf16", [_p, _p, _p, _i, _i, _i, _i, _p])
     _declare(lib, "ms_gemm_skinny_gelu_bf16", [_p, _p, _p, _i, _i, _i, _p])
+    _declare(lib, "ms_gemm_skinny_relu2_bf16", [_p, _p, _p, _i, _i, _i, _p])
     _declare(lib, "ms_gemm_skinny_set_stream", [_i], None)
     _declare(lib, "ms_silu_mul", [_p, _p, _i, _i, _i, _p])
     _declare(lib, "ms_to_float", [_p, _p, _ll, _i, _p])
@@ -167,8 +168,12 @@ def recurrence():
     _declare(lib, "ms_conv_state_update", [_p, _p, _i, _p, _p, _p, _i, _i, _i, _i, _p])
     _declare(lib, "ms_head_norm_gate", [_p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _f, _i, _i, _p])
     _declare(lib, "ms_mlstm_gates", [_p, _p, _p, _p, _i, _p, _p, _p, _p, _p, _i, _i, _f, _i, _i, _p])
-    _declare(lib, "ms_mlstm_output", [_p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _f, _f, _i, _p])
+    _declare(lib, "ms_mlstm_output", [_p, _i, _p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _f, _i, _p])
     _declare(lib, "ms_conv_bias", [_p, _p, _i, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _p])
+    _declare(lib, "ms_chunk_max", [_i, _i])
+    _declare(lib, "ms_chunk_supports", [_i, _i])
+    _declare(lib, "ms_chunk_table", [_p, _p, _p, _i, _p])
+    _declare(lib, "ms_chunk_scan", [_p, _i, _p, _p, _i, _p, _i, _i, _p, _i] + [_p] * 11 + [_i] * 5 + [_f, _i, _p])
     _declare(lib, "ms_rglru_scan", [_p, _p, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p])
     return lib
 

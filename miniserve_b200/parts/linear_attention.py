@@ -328,7 +328,8 @@ class MatrixMemory(Part):
 
     then each head's o is divided by its root mean square, the heads side by side times a weight, times sigmoid(W_g x), then W_o.
     One product makes q|k|v|g|i|f. The gates' kernel works out m, both exponentials and exp(-m) for every token (float32); the walk
-    is the decay rule of ``csrc/recurrence.cu`` with one decay per head, a factor on the write, and n as one more column of S.
+    is the decay rule with one decay per head, a factor on the write, and n as one more column of S (token by token, ``csrc/recurrence.cu``;
+    prompts in bfloat16 by chunks on the tensor cores, ``csrc/chunk_scan.cu``).
     State: S with that column [heads, dv + 1, dk] and m [heads], float32.
     Parameters: ``hidden``, ``heads``, ``key_dim``, ``value_dim``, ``gate_cap``, ``eps``, ``den_eps`` (1e-6), ``names``
     (q, k, v, g, o, norm, i, f, i_bias, f_bias -> tensor names)."""
@@ -381,9 +382,14 @@ class MatrixMemory(Part):
         at_i = at_g + h * dv
         gates = ctx.buffer("mlstm.gates", (3, t, h), torch.float32, dev)  # the state's decay, the write's factor, exp(-m)
         ops.mlstm_gates(gates, proj[:, at_i:at_i + 2 * h], self.w_gate_bias, running.state, ctx, self.cap)
-        o = ctx.buffer("mlstm.o", (t, h, dv + 1), torch.float32, dev)
-        ops.decay_scan(o, state.state, proj[:, :at_k], proj[:, at_k:at_v], proj[:, at_v:at_g], gates[0], None, None, 0.0, None, ctx, h, dk,
-                       dv + 1, dk ** -0.5, delta=False, head_decay=True, v_scale=gates[1], ones_column=True)
+        q, k, v = proj[:, :at_k], proj[:, at_k:at_v], proj[:, at_v:at_g]
+        if ops.chunk_scan_ok(q, k, v, dk, dv, ctx):
+            o = ctx.buffer("mlstm.o", (t, h, dv + 4), torch.float32, dev)  # (rows that start on 16 bytes)
+            ops.chunk_scan(o, state.state, q, k, v, gates[0], gates[1], ctx, h, dk, dv, dk ** -0.5, ones=True)
+        else:
+            o = ctx.buffer("mlstm.o", (t, h, dv + 1), torch.float32, dev)
+            ops.decay_scan(o, state.state, q, k, v, gates[0], None, None, 0.0, None, ctx, h, dk, dv + 1, dk ** -0.5, delta=False,
+                           head_decay=True, v_scale=gates[1], ones_column=True)
         ops.mlstm_output(out, o, gates[2], self.w_norm, proj[:, at_g:at_i], self.eps, self.den_eps, stream=ctx.stream)
 
     def forward(self, x, ctx, cache):

@@ -166,12 +166,8 @@ class DenseMLP(Part):
 
     def forward(self, x, ctx) -> torch.Tensor:
         t, dt, dev = x.shape[0], self.env.dtype, self.w_down.device
-        if self.activation == "relu_squared":
-            act = ctx.buffer("mlp.act", (t, self.inter), dt, dev)
-            self.features(x, ctx, act)
-            return ops.linear(act, self.w_down, stream=ctx.stream, out=ctx.buffer("mlp.down", (t, self.hidden), dt, dev))
         # the activation in the product's epilogue where there is such a kernel (decode steps)
-        act = ops.linear_gelu_tanh(x, self.w_up, ctx.buffer("mlp.act", (t, self.inter), dt, dev), stream=ctx.stream)
+        act = ops.linear_act(x, self.w_up, ctx.buffer("mlp.act", (t, self.inter), dt, dev), self.activation, stream=ctx.stream)
         return ops.linear(act, self.w_down, stream=ctx.stream, out=ctx.buffer("mlp.down", (t, self.hidden), dt, dev))
 
 

@@ -9,6 +9,8 @@ summaries under ``profiles/`` were measured and captured with.
     python -m miniserve_b200.tools.kernel_bench attn_prefill --tokens 2048 --softcap 30 --chunk 1024 --learned-sink
     python -m miniserve_b200.tools.kernel_bench add_rmsnorm --m 2048 --n 1024 --offset
     python -m miniserve_b200.tools.kernel_bench pointwise --op channel_gate --tokens 2048 --heads 16 --head-dim 128
+    python -m miniserve_b200.tools.kernel_bench decay_scan --tokens 2048 --heads 4 --key-dim 128 --value-dim 256 --head-decay [--chunks]
+    python -m miniserve_b200.tools.kernel_bench recurrent --op rglru_scan --tokens 2048 --n 1024 --blocks 4
 
 Each case rotates over enough copies of its inputs to exceed the L2 cache, captures one pass over
 all copies in a CUDA graph, and reports the time per launch with the bytes or flops it implies.
@@ -90,7 +92,7 @@ def _time(calls, copies, launches):
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__.splitlines()[0])
-    ap.add_argument("kernel", choices=["attn_decode", "attn_prefill", "skinny", "add_rmsnorm", "gemm", "gate_up", "sample", "decay_scan", "pointwise", "experts"])
+    ap.add_argument("kernel", choices=["attn_decode", "attn_prefill", "skinny", "add_rmsnorm", "gemm", "gate_up", "sample", "decay_scan", "pointwise", "experts", "recurrent"])
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=2048)
     ap.add_argument("--tokens", type=int, default=2048)
@@ -118,8 +120,15 @@ def main(argv=None) -> int:
     ap.add_argument("--keep-first", type=int, default=0, help="attn_*: this many first keys stay visible behind --window")
     ap.add_argument("--window", type=int, default=0, help="attn_*: a query sees only this many keys back (0: all)")
     ap.add_argument("--op", choices=["channel_gate", "head_gate", "relu_squared", "gelu_tanh", "latent_prepare", "qkv_prepare",
-                                     "layernorm", "layernorm_pair", "token_shift", "clamped_glu", "sum_bias", "act_mul", "axpby"],
+                                     "layernorm", "layernorm_pair", "token_shift", "clamped_glu", "sum_bias", "act_mul", "axpby", "normed_add",
+                                     "embed_gather", "embed_sum", "mlstm_gates", "mlstm_output", "gated_group_norm", "conv_bias", "conv_silu",
+                                     "rglru_gates", "rglru_scan"],
                     default="channel_gate", help="pointwise: which kernel (--tokens rows; --heads x --head-dim, or --n, columns)")
+    ap.add_argument("--head-decay", action="store_true", help="decay_scan: one decay per head, worked out beforehand (float32), a column of ones")
+    ap.add_argument("--chunks", action="store_true", help="decay_scan --head-decay: by chunks on the tensor cores")
+    ap.add_argument("--blocks", type=int, default=4, help="recurrent: equal parts of the --n channels, a gate matrix each")
+    ap.add_argument("--taps", type=int, default=4, help="recurrent: taps of the convolution")
+    ap.add_argument("--plain-experts", action="store_true", help="experts: without a gate, the square of relu")
     ap.add_argument("--experts", type=int, default=14, help="experts: how many experts")
     ap.add_argument("--top", type=int, default=4, help="experts: choices per token")
     ap.add_argument("--launches", type=int, default=0, help="run this many plain launches and report nothing")
@@ -187,9 +196,10 @@ def main(argv=None) -> int:
         slots = t * top
         tc = args.gemm != "library"
         tile_rows = xo.TC_TILE_ROWS if tc else xo.TILE_ROWS
-        work = dict(flops=2.0 * slots * 3 * inter * width)
-        copies = max(2, int(L2_BYTES // (e * 3 * inter * width * 2)) + 1)
-        wg = [(torch.randn(e, 2 * inter, width, device=dev) * width ** -0.5).bfloat16() for _ in range(copies)]
+        parts = 1 if args.plain_experts else 2  # matrices ahead of the down projection
+        work = dict(flops=2.0 * slots * (parts + 1) * inter * width)
+        copies = max(2, int(L2_BYTES // (e * (parts + 1) * inter * width * 2)) + 1)
+        wg = [(torch.randn(e, parts * inter, width, device=dev) * width ** -0.5).bfloat16() for _ in range(copies)]
         wd = [(torch.randn(e, width, inter, device=dev) * inter ** -0.5).bfloat16() for _ in range(copies)]
         x = torch.randn(t, width, device=dev).bfloat16()
         idx = torch.stack([torch.randperm(e, device=dev)[:top] for _ in range(t)]).to(torch.int32).contiguous()
@@ -204,10 +214,13 @@ def main(argv=None) -> int:
         def calls(i, stream):
             if tc:
                 xo.expert_gather(xs, x, perm, meta, top, stream=stream)
-                xo.expert_products_tc(act, xs, wg[i], tiles, meta, offsets, True, stream=stream)
+                xo.expert_products_tc(act, xs, wg[i], tiles, meta, offsets, not args.plain_experts, stream=stream, relu_squared=args.plain_experts)
                 xo.expert_products_tc(y, act, wd[i], tiles, meta, offsets, False, stream=stream)
             else:
-                xo.expert_gate_up(act, x, wg[i], perm, top, tiles, meta, offsets, "silu", stream=stream)
+                if args.plain_experts:
+                    xo.expert_up(act, x, wg[i], perm, top, tiles, meta, offsets, "relu_squared", stream=stream)
+                else:
+                    xo.expert_gate_up(act, x, wg[i], perm, top, tiles, meta, offsets, "silu", stream=stream)
                 xo.expert_down(y, act, wd[i], tiles, meta, offsets, stream=stream)
     elif args.kernel == "sample":
         # --batch rows of float32 logits, each row with its own seed
@@ -280,7 +293,7 @@ def main(argv=None) -> int:
         slots = torch.zeros(2, n, **bf)
         sctx = SimpleNamespace(row_of_token=row_of, cu_q=torch.tensor([0, t], **i32), q_start=torch.zeros(1, **i32),
                                state_slot=torch.zeros(1, **i32), num_rows=1, stream=0)
-        byts = {"layernorm": t * n * 12, "layernorm_pair": t * n * 14, "token_shift": t * n * 4, "clamped_glu": t * n * 6,
+        byts = {"normed_add": t * n * 12, "layernorm": t * n * 12, "layernorm_pair": t * n * 14, "token_shift": t * n * 4, "clamped_glu": t * n * 6,
                 "sum_bias": t * n * 6, "act_mul": t * n * 6, "axpby": t * n * 6,
                 "channel_gate": 3 * t * width * 2, "head_gate": 2 * t * width * 2, "relu_squared": 2 * t * width * 2,
                 "gelu_tanh": 2 * t * width * 2, "latent_prepare": 2 * t * d * 2, "qkv_prepare": 2 * 3 * t * width * 2}[args.op]
@@ -288,7 +301,9 @@ def main(argv=None) -> int:
 
         def calls(i, stream):
             att, wide, feat = sets[i]
-            if args.op == "layernorm":
+            if args.op == "normed_add":
+                ops.add_normed_rmsnorm(ln_a, res, delta, lw[:1], 1e-5, delta_weight=lb[:1], delta_eps=1e-5, stream=stream)
+            elif args.op == "layernorm":
                 ops.add_layernorm(ln_a, res, delta, lw, lb, 1e-5, stream=stream)
             elif args.op == "layernorm_pair":
                 ops.add_layernorm(ln_a, res, delta, lw, lb, 1e-5, out2=ln_b, weight2=lb, bias2=lw, stream=stream)
@@ -318,6 +333,54 @@ def main(argv=None) -> int:
                 ops.qkv_prepare(qo, kpool, vpool, wide[:, :width], wide[:, width:2 * width], wide[:, 2 * width:3 * width], None, None, table,
                                 d, False, 1e-6, positions, row_of, kctx.page_indptr[0], kctx.page_indices[0], args.page_size, status,
                                 stream=stream)
+    elif args.kernel == "recurrent":
+        # what surrounds the recurrences and the embedding: `batch` requests of `tokens` tokens each, --n channels (the model's width)
+        rows, t, n = args.batch, args.batch * args.tokens, args.n
+        i32, f32, bf = (dict(dtype=d, device=dev) for d in (torch.int32, torch.float32, torch.bfloat16))
+        hh, dv, blocks = args.heads, args.value_dim, args.blocks
+        ctx = SimpleNamespace(cu_q=torch.arange(0, t + 1, args.tokens, **i32), q_start=torch.ones(rows, **i32), state_slot=torch.arange(rows, **i32),
+                              row_of_token=torch.arange(t, **i32) // args.tokens, positions=1 + torch.arange(t, **i32) % args.tokens,
+                              token_ids=torch.randint(0, 30000, (t,), **i32), num_rows=rows, decode_only=args.tokens == 1, stream=0)
+        ctx.row_of_token = ctx.row_of_token.to(torch.int32)
+        vec = lambda size: torch.randn(size, **f32)  # noqa: E731
+        per_set = t * n * 16 + t * hh * dv * 8
+        copies = max(2, min(64, int(L2_BYTES // per_set) + 1))
+        sets = [SimpleNamespace(y=torch.randn(t, 2 * n, **bf), z=torch.randn(t, blocks, 2, n // blocks, **f32), u=torch.randn(t, n, **bf),
+                                out=torch.empty(t, n, **bf), o=torch.randn(t, hh, dv + 4, **f32), gate=torch.randn(t, hh * dv, **bf),
+                                feat=torch.empty(t, hh * dv, **bf), raw=torch.randn(t, 2 * hh, **bf), gates=torch.empty(3, t, hh, **f32),
+                                res=torch.empty(t, n, **f32), xs=torch.randn(t, n, **f32)) for _ in range(copies)]
+        table, pairs = torch.randn(30000, n, **bf), torch.randn(50001, n, **bf)
+        freq, prev = 10000.0 ** (-2.0 * torch.arange(n // 2, **f32) / n), torch.zeros(rows, 1, **i32)
+        conv_w, conv_state, state, running = vec((args.taps, n)), torch.zeros(rows, args.taps - 1, n, **bf), torch.zeros(rows, n, **f32), torch.zeros(rows, hh, **f32)
+        w_gates = (torch.randn(blocks, 2 * n // blocks, n // blocks, device=dev) * (n // blocks) ** -0.5).bfloat16()
+        va, vb, vc, vd, wn = vec(n), vec(n), torch.rand(n, **f32), vec(n), vec(hh * dv)
+        byts = {"embed_gather": t * n * 6, "embed_sum": t * n * 8, "mlstm_gates": t * hh * 16, "mlstm_output": t * hh * dv * 8, "gated_group_norm": t * n * 8,
+                "conv_bias": t * n * 4, "conv_silu": t * n * 6, "rglru_scan": t * n * 14 + 2 * rows * n * 4}
+        work = dict(bytes=byts[args.op]) if args.op in byts else dict(flops=4.0 * t * n * n / blocks)
+
+        def calls(i, stream):
+            s = sets[i]
+            ctx.stream = stream
+            if args.op == "embed_gather":
+                ops.embed_gather(s.res, table, ctx.token_ids, stream=stream)
+            elif args.op == "embed_sum":
+                ops.embed_sum(s.res, table, ctx, freq, pairs, (50000, 31, 7), prev)
+            elif args.op == "mlstm_gates":
+                ops.mlstm_gates(s.gates, s.raw, vec_gates, running, ctx, 15.0)
+            elif args.op == "mlstm_output":
+                ops.mlstm_output(s.feat, s.o, s.gates[2], wn, s.gate, 1e-5, 1e-6, stream=stream)
+            elif args.op == "gated_group_norm":
+                ops.gated_group_norm(s.out, s.xs, None, None, s.u, va, 8, n // 8, 1e-5, stream=stream)
+            elif args.op == "conv_bias":
+                ops.conv_bias(s.out, s.y[:, n:], conv_state, conv_w, va, vb, ctx)
+            elif args.op == "conv_silu":
+                ops.conv_silu_unit(s.res, s.y[:, n:], conv_state, conv_w_rows, ctx, 0, 1, n // 128, 128, 0.0, bias=va)
+            elif args.op == "rglru_gates":
+                ops.linear_heads(s.u.view(t, blocks, n // blocks), w_gates, s.z.view(t, blocks, 2 * n // blocks), stream=stream)
+            else:
+                ops.rglru_scan(s.out, state, s.z, s.u, s.y[:, :n], va, vb, vc, vd, ctx)
+
+        vec_gates, conv_w_rows = vec(2 * hh), conv_w.t().contiguous()
     else:
         # the linear-attention recurrence: `batch` requests of `tokens` tokens each (1: a decode step), from zero state
         t, hh, dk, dv, rows = args.tokens * args.batch, args.heads, args.key_dim, args.value_dim, args.batch
@@ -335,13 +398,23 @@ def main(argv=None) -> int:
         z = torch.randn(t, hh * dk, device=dev).bfloat16()
         beta = torch.randn(t, hh, device=dev).bfloat16() if args.delta else None
         bias, coef = torch.zeros(hh * dk, device=dev), torch.full((hh,), 0.1, device=dev)
-        state, o = torch.zeros(rows + 1, hh, dv, dk, device=dev), torch.empty(t, hh, dv, device=dev)
+        if args.head_decay:
+            decay, write = torch.rand(t, hh, device=dev) ** 0.02, torch.rand(t, hh, device=dev)
+            dv1 = dv + 1
+            state, o = torch.zeros(rows + 1, hh, dv1, dk, device=dev), torch.empty(t, hh, dv + 4 if args.chunks else dv1, device=dev)
+        else:
+            state, o = torch.zeros(rows + 1, hh, dv, dk, device=dev), torch.empty(t, hh, dv, device=dev)
         item = 4 if args.delta else 2
         work = dict(bytes=t * hh * ((2 * dk + dv) * item + dk * 2 + dv * 4) + 2 * rows * hh * dk * dv * 4)
         copies = 2
 
         def calls(i, stream):
             ctx.stream = stream
+            if args.head_decay and args.chunks:
+                return ops.chunk_scan(o, state, q, k, v, decay, write, ctx, hh, dk, dv, dk ** -0.5, ones=True)
+            if args.head_decay:
+                return ops.decay_scan(o, state, q, k, v, decay, None, None, 0.0, None, ctx, hh, dk, dv + 1, dk ** -0.5, delta=False, head_decay=True,
+                                      v_scale=write, ones_column=True)
             ops.decay_scan(o, state, q, k, v, z, bias, coef, -1.0, beta, ctx, hh, dk, dv, dk ** -0.5, delta=args.delta)
     us = _time(calls, copies, args.launches)
     if us is not None:

@@ -349,7 +349,7 @@ def _memory_weights(t):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads, dim, vdim, cap", [(3, 16, 24, 12.0), (5, 12, 20, 7.5), (1, 24, 16, 3.0), (4, 64, 96, 20.0), (2, 128, 40, 15.0), (1, 8, 8, 1.0),
-                                                   (2, 36, 260, 10.0)])
+                                                   (2, 36, 260, 10.0), (2, 128, 256, 15.0), (1, 256, 136, 8.0), (3, 40, 200, 9.0)])
 def test_matrix_memory_whole_in_portions_and_decoded(dtype, heads, dim, vdim, cap):
     part, m = _memory(dtype, heads, dim, vdim, cap)
     w = _bind(part, dtype, change=_memory_weights)
@@ -372,7 +372,7 @@ def test_matrix_memory_whole_in_portions_and_decoded(dtype, heads, dim, vdim, ca
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads, dim, vdim", [(2, 16, 24), (4, 64, 64), (1, 400, 16)])
+@pytest.mark.parametrize("heads, dim, vdim", [(2, 16, 24), (4, 64, 64), (1, 400, 16), (2, 128, 256)])
 def test_matrix_memory_over_a_long_portion_and_long_decoding(dtype, heads, dim, vdim):
     """Portions of hundreds of tokens (the walk may be cut into segments), behind an earlier portion, beside a short row, and
     hundreds of tokens decoded one by one from the state they left."""
@@ -452,6 +452,46 @@ def test_matrix_memory_keeps_an_early_token_through_an_open_forget_gate(dtype):
     ref = plain.mlstm(_cpu(other), w, "", m, 1e-5, torch.float32)
     noise = (plain.mlstm(_cpu(other), w, "", m, 1e-5, dtype) - ref).abs().amax(dim=1)
     _close(part.forward(other, ctx, views), ref, dtype, 3.0, noise)
+
+
+@pytest.mark.parametrize("heads, groups, dk, dv, ones", [(2, 2, 128, 256, True), (4, 2, 64, 96, False), (3, 3, 8, 8, True), (2, 1, 256, 136, True), (1, 1, 40, 200, False)])
+def test_decay_rule_over_chunks_on_the_tensor_cores(heads, groups, dk, dv, ones):
+    """Rows from one token to several chunks, some behind an earlier state, decays from one to zero, against the recurrence in
+    64-bit: the tensor cores see what is not exact in bfloat16 as two numbers, so the error stays far below bfloat16's."""
+    from miniserve_b200 import ops
+
+    rows = [(0, 1), (5, 64), (0, 65), (300, 200), (0, 7), (9, 1), (0, 129)]
+    _, ctx = _ctx(rows, dtype=torch.bfloat16, slots=[6, 0, 3, 1, 4, 5, 2])
+    t = sum(n for _, n in rows)
+    q, k = (torch.randn(t, groups * dk, device=DEV).bfloat16() for _ in range(2))
+    v = torch.randn(t, heads * dv, device=DEV).bfloat16()
+    decay = torch.rand(t, heads, device=DEV) ** 0.05
+    decay[::17] = 0.0
+    decay[5::29] = 1.0
+    decay[70:100] = 1e-20
+    write = torch.rand(t, heads, device=DEV) * 3
+    extra = int(ones)
+    state = torch.randn(7, heads, dv + extra, dk, device=DEV)
+    held = state.clone()
+    o = torch.full((t, heads, dv + 4), float("nan"), device=DEV)
+    assert ops.chunk_scan_ok(q, k, v, dk, dv, ctx)
+    ops.chunk_scan(o, state, q, k, v, decay, write, ctx, heads, dk, dv, 0.25, ones)
+    qd, kd, vd, ad, wd = (x.double().cpu() for x in (q, k, v, decay, write))
+    vd = vd.view(t, heads, dv)
+    if ones:
+        vd = torch.cat((vd, torch.ones(t, heads, 1, dtype=torch.float64)), -1)
+    head_group = [h // (heads // groups) for h in range(heads)]
+    qh, kh = qd.view(t, groups, dk)[:, head_group], kd.view(t, groups, dk)[:, head_group]
+    at = 0
+    for (start, n), slot in zip(rows, ctx.state_slot.tolist()):
+        s = held[slot].double().cpu() if start else torch.zeros(heads, dv + extra, dk, dtype=torch.float64)
+        for i in range(at, at + n):
+            s = ad[i][:, None, None] * s + wd[i][:, None, None] * vd[i][:, :, None] * kh[i][:, None, :]
+            want = (s * qh[i][:, None, :]).sum(-1) * 0.25
+            size = (s.abs() * qh[i].abs()[:, None, :]).sum(-1) * 0.25 + 1e-3
+            assert ((o[i, :, :dv + extra].double().cpu() - want).abs() / size).max() < 6e-5, (slot, i - at)
+        assert (state[slot].double().cpu() - s).abs().max() < 3e-5 * max(1.0, s.abs().max().item())
+        at += n
 
 
 # --------------------------------------------------------------------------- gated linear recurrence
