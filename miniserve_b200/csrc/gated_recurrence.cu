@@ -123,6 +123,40 @@ __global__ void mlstm_output_kernel(T* __restrict__ out, int ld_out, const float
   }
 }
 
+// The same for bfloat16 rows on 16 bytes and value sizes that are multiples of 8: eight channels per lane and trip.
+__global__ void mlstm_output_bf16x8_kernel(__nv_bfloat16* __restrict__ out, int ld_out, const float* __restrict__ o, int ld_o,
+                                           const float* __restrict__ floor_, const float* __restrict__ w, const __nv_bfloat16* __restrict__ gate,
+                                           int ld_gate, long long items, int H, int dv, float eps, float den_eps) {
+  pdl_prologue();
+  const int lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (item >= items) return;
+  const long long t = item / H;
+  const int h = (int)(item - t * H);
+  const float* src = o + item * ld_o;
+  const float inv_den = 1.0f / (fmaxf(fabsf(src[dv]), floor_[item]) + den_eps);
+  float ss = 0.f;
+  for (int c = lane * 8; c < dv; c += 256) {
+    const float4 a = *reinterpret_cast<const float4*>(src + c), b = *reinterpret_cast<const float4*>(src + c + 4);
+    const float x[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += (x[e] * inv_den) * (x[e] * inv_den);
+  }
+  ss = warp_sum(ss);
+  const float inv = 1.0f / sqrtf(ss / (float)dv + eps);
+  for (int c = lane * 8; c < dv; c += 256) {
+    const float4 a = *reinterpret_cast<const float4*>(src + c), b = *reinterpret_cast<const float4*>(src + c + 4);
+    const float4 wa = *reinterpret_cast<const float4*>(w + (size_t)h * dv + c), wb = *reinterpret_cast<const float4*>(w + (size_t)h * dv + c + 4);
+    const float x[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w}, wv[8] = {wa.x, wa.y, wa.z, wa.w, wb.x, wb.y, wb.z, wb.w};
+    float g[8], r[8];
+    bf16x8_to_float(*reinterpret_cast<const uint4*>(gate + t * ld_gate + (size_t)h * dv + c), g);
+    // (fast exponential and division: relative error about 1e-6, far below the bfloat16 rounding of the result)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) r[e] = (((x[e] * inv_den) * inv) * wv[e]) * __fdividef(1.0f, 1.0f + __expf(-g[e]));
+    *reinterpret_cast<uint4*>(out + t * ld_out + (size_t)h * dv + c) = float_to_bf16x8(r);
+  }
+}
+
 // ---------------------------------------------------------------- a short causal convolution of a biased projection, no activation
 // u[t, c] = bias[c] + sum_j w[j, c] x'(t - (taps - 1) + j), x'(s) = x[s, c] + in_bias[c] at positions from 0 on and 0 before the
 // start. w [taps, C] (tap-major). Inputs before a portion's first token come from the request's slot (the raw x, without in_bias).
@@ -170,20 +204,97 @@ __global__ void conv_bias_kernel(T* __restrict__ u, const T* __restrict__ x, int
   }
 }
 
+// The same for prompts in bfloat16 with TAPS taps: a thread takes eight channels over a run of CONV_RUN consecutive tokens of the step,
+// its taps in registers and the last inputs in a window that moves along (and starts anew where a row does).
+constexpr int CONV_RUN = 8;
+template <int TAPS>
+__global__ void conv_bias_run_kernel(__nv_bfloat16* __restrict__ u, const __nv_bfloat16* __restrict__ x, int ld,
+                                     const __nv_bfloat16* __restrict__ conv_state, const float* __restrict__ w, const float* __restrict__ bias,
+                                     const float* __restrict__ in_bias, const int* __restrict__ row_of_token, const int* __restrict__ cu_q,
+                                     const int* __restrict__ q_start, const int* __restrict__ state_slot, int tokens, int C) {
+  pdl_prologue();
+  const int groups = C >> 3;
+  const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  const int run = (int)(idx / groups), c = (int)(idx - (long long)run * groups) * 8;
+  const int t0 = run * CONV_RUN, t1 = min(tokens, t0 + CONV_RUN);
+  if (t0 >= tokens) return;
+  float wt[TAPS][8], bs[8], ib[8];
+#pragma unroll
+  for (int e = 0; e < 8; e += 4) {
+    *reinterpret_cast<float4*>(bs + e) = *reinterpret_cast<const float4*>(bias + c + e);
+    *reinterpret_cast<float4*>(ib + e) = *reinterpret_cast<const float4*>(in_bias + c + e);
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) *reinterpret_cast<float4*>(wt[j] + e) = *reinterpret_cast<const float4*>(w + (size_t)j * C + c + e);
+  }
+  uint4 raw[CONV_RUN];  // the run's own inputs, all in flight at once
+#pragma unroll
+  for (int s = 0; s < CONV_RUN; ++s) raw[s] = *reinterpret_cast<const uint4*>(x + (size_t)min(t0 + s, t1 - 1) * ld + c);
+  float win[TAPS - 1][8];
+  int row = -1, end = t0;
+#pragma unroll
+  for (int s = 0; s < CONV_RUN; ++s) {
+    const int t = t0 + s;
+    if (t >= t1) break;
+    if (t >= end) {  // the first token of the run, or of a row: what lies before it comes from the step, the slot, or is nothing
+      row = row_of_token[t];
+      const int first = cu_q[row], start = q_start[row];
+      end = cu_q[row + 1];
+      const __nv_bfloat16* st = conv_state + (size_t)state_slot[row] * (TAPS - 1) * C + c;
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) {
+        const int at = t - first - (TAPS - 1) + j;
+        float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+        if (start + at >= 0) {
+          bf16x8_to_float(*reinterpret_cast<const uint4*>(at >= 0 ? x + (size_t)(first + at) * ld + c : st + (size_t)(TAPS - 1 + at) * C), f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) f[e] += ib[e];
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) win[j][e] = f[e];
+      }
+    }
+    float now[8], acc[8];
+    bf16x8_to_float(raw[s], now);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      now[e] += ib[e];
+      acc[e] = bs[e];
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) acc[e] = fmaf(wt[j][e], win[j][e], acc[e]);
+      acc[e] = fmaf(wt[TAPS - 1][e], now[e], acc[e]);
+#pragma unroll
+      for (int j = 0; j < TAPS - 2; ++j) win[j][e] = win[j + 1][e];
+      win[TAPS - 2][e] = now[e];
+    }
+    *reinterpret_cast<uint4*>(u + (size_t)t * C + c) = float_to_bf16x8(acc);
+  }
+}
+
 // ---------------------------------------------------------------- the gated linear recurrence
-// One token's decay and write from the two gates' products (biases not yet added).
+// One token's decay and write from the two gates' products (biases not yet added). With e = exp(log a) - 1: a = 1 + e and
+// 1 - a^2 = -e (2 + e), exact where a is near one. FAST: the gates' exponential and division with relative errors of about 1e-6.
+template <bool FAST>
+__device__ __forceinline__ float gate_of(float x) {
+  return FAST ? __fdividef(1.0f, 1.0f + __expf(-x)) : sigmoid_of(x);
+}
+template <bool FAST>
 __device__ __forceinline__ void rglru_coefs(float zr, float zi, float u, float coef, float& a, float& b) {
-  const float la = -coef * sigmoid_of(zr);
-  a = expf(la);
-  b = sqrtf(-expm1f(2.f * la)) * (sigmoid_of(zi) * u);
+  const float e = expm1f(-coef * gate_of<FAST>(zr));
+  a = 1.f + e;
+  b = sqrtf(-e * (2.f + e)) * (gate_of<FAST>(zi) * u);
+}
+// gelu_tanh(z) = z sigmoid(2 sqrt(2/pi) (z + 0.044715 z^3)), since (1 + tanh x) / 2 = sigmoid(2 x)
+template <bool FAST>
+__device__ __forceinline__ float gelu_gate(float z) {
+  return FAST ? z * gate_of<true>(1.5957691216057308f * (z + 0.044715f * z * z * z)) : gelu_tanh_of(z);
 }
 
 // z [T, blocks, 2, bs] float32: the recurrence gate's and the input gate's products of each part; u [T, C]; y [T, .] the gated
-// branch's product (y_bias added here). CTA: 32 channels (a lane each), WARPS warps, each with a run of LRUN tokens; a cluster of
-// `ctas` CTAs takes consecutive runs of the row, so a pass covers ctas * WARPS * LRUN tokens. Within a pass: every warp
-// composes its run's (a, b) pairs, the pairs of warps and CTAs are composed in order, then every warp walks its run from the
-// state it found. state [slots, C] float32.
-constexpr int LRU_WARPS = 8, LRU_RUN = 8;
+// branch's product (y_bias added here). CTA: 32 channels (a lane each), LRU_WARPS warps, each with a run of LRU_RUN tokens; a
+// cluster of `ctas` CTAs takes consecutive runs of the row, so a pass covers ctas * LRU_WARPS * LRU_RUN tokens. Within a pass: every
+// warp composes its run's (a, b) pairs, the pairs of warps and CTAs are composed in order, then every warp walks its run from
+// the state it found. state [slots, C] float32.
+constexpr int LRU_WARPS = 16, LRU_RUN = 8, LRU_MAX_CTAS = 8;
 
 template <typename T>
 __global__ void __launch_bounds__(LRU_WARPS * 32)
@@ -191,6 +302,7 @@ rglru_scan_kernel(T* __restrict__ out, float* __restrict__ state, const float* _
                   const T* __restrict__ y, int ld_y, const float* __restrict__ bias_r, const float* __restrict__ bias_i,
                   const float* __restrict__ coef, const float* __restrict__ y_bias, const int* __restrict__ cu_q,
                   const int* __restrict__ q_start, const int* __restrict__ state_slot, int C, int bs, int ctas) {
+  constexpr bool FAST = sizeof(T) == 2;
   __shared__ float wa[LRU_WARPS][32], wb[LRU_WARPS][32];
   __shared__ float ta[2][32], tb[2][32];  // this CTA's composed pair of the pass, in two buffers in turn
   pdl_prologue();
@@ -210,18 +322,28 @@ rglru_scan_kernel(T* __restrict__ out, float* __restrict__ state, const float* _
   for (int p0 = 0; p0 < len; p0 += pass, buf ^= 1) {
     const int first = p0 + (rank * LRU_WARPS + warp) * LRU_RUN;
     const int n = max(0, min(LRU_RUN, len - first));
-    float a[LRU_RUN], b[LRU_RUN];
-    float A = 1.f, B = 0.f;
+    float a[LRU_RUN], b[LRU_RUN], yv[LRU_RUN];
+    {
+      float zr[LRU_RUN], zi[LRU_RUN], uv[LRU_RUN];
 #pragma unroll
-    for (int s = 0; s < LRU_RUN; ++s) {
-      a[s] = 1.f;
-      b[s] = 0.f;
-      if (s < n) {
-        const size_t t = (size_t)(t0 + first + s);
+      for (int s = 0; s < LRU_RUN; ++s) {  // the run's loads in flight together (tokens beyond the row read its last one)
+        const size_t t = (size_t)(t0 + min(first + s, len - 1));
         const float* zt = z + t * z_row + z_at;
-        rglru_coefs(zt[0] + br, zt[bs] + bi, Elem<T>::load(u + t * C + cc), cf, a[s], b[s]);
+        zr[s] = zt[0];
+        zi[s] = zt[bs];
+        uv[s] = Elem<T>::load(u + t * C + cc);
+        yv[s] = Elem<T>::load(y + t * ld_y + cc);
+      }
+#pragma unroll
+      for (int s = 0; s < LRU_RUN; ++s) {
+        rglru_coefs<FAST>(zr[s] + br, zi[s] + bi, uv[s], cf, a[s], b[s]);
+        if (s >= n) {
+          a[s] = 1.f;
+          b[s] = 0.f;
+        }
       }
     }
+    float A = 1.f, B = 0.f;
 #pragma unroll
     for (int s = 0; s < LRU_RUN; ++s) {
       B = fmaf(a[s], B, b[s]);
@@ -248,11 +370,17 @@ rglru_scan_kernel(T* __restrict__ out, float* __restrict__ state, const float* _
         tb[buf][lane] = qb;
       }
       cluster.sync();  // (a buffer is written again two passes on, behind a barrier that every CTA reaches after its reads)
+      float xa[LRU_MAX_CTAS], xb[LRU_MAX_CTAS];
+#pragma unroll
+      for (int k = 0; k < LRU_MAX_CTAS; ++k) {
+        xa[k] = k < ctas ? cluster.map_shared_rank(&ta[buf][0], k)[lane] : 1.f;
+        xb[k] = k < ctas ? cluster.map_shared_rank(&tb[buf][0], k)[lane] : 0.f;
+      }
       float before = carry;
-      for (int k = 0; k < ctas; ++k) {
+#pragma unroll
+      for (int k = 0; k < LRU_MAX_CTAS; ++k) {
         if (k == rank) before = carry;
-        const float xa = cluster.map_shared_rank(&ta[buf][0], k)[lane], xb = cluster.map_shared_rank(&tb[buf][0], k)[lane];
-        carry = fmaf(xa, carry, xb);
+        carry = fmaf(xa[k], carry, xb[k]);
       }
       pb = fmaf(pa, before, pb);
     } else {
@@ -264,10 +392,7 @@ rglru_scan_kernel(T* __restrict__ out, float* __restrict__ state, const float* _
 #pragma unroll
     for (int s = 0; s < LRU_RUN; ++s) {
       S = fmaf(a[s], S, b[s]);
-      if (s < n && active) {
-        const size_t t = (size_t)(t0 + first + s);
-        Elem<T>::store(out + t * C + c, S * gelu_tanh_of(Elem<T>::load(y + t * ld_y + c) + yb));
-      }
+      if (s < n && active) Elem<T>::store(out + (size_t)(t0 + first + s) * C + c, S * gelu_gate<FAST>(yv[s] + yb));
     }
   }
   if (ctas > 1) cluster.sync();  // no CTA leaves while another may still read its shared memory
@@ -287,11 +412,12 @@ __global__ void rglru_step_kernel(T* __restrict__ out, float* __restrict__ state
   const int blk = c / bs;
   const float* zt = z + (size_t)r * 2 * C + (size_t)blk * 2 * bs + (c - blk * bs);
   float a, b;
-  rglru_coefs(zt[0] + bias_r[c], zt[bs] + bias_i[c], Elem<T>::load(u + idx), coef[c], a, b);
+  constexpr bool FAST = sizeof(T) == 2;
+  rglru_coefs<FAST>(zt[0] + bias_r[c], zt[bs] + bias_i[c], Elem<T>::load(u + idx), coef[c], a, b);
   float* slot = state + (size_t)state_slot[r] * C + c;
   const float S = fmaf(a, q_start[r] == 0 ? 0.f : *slot, b);
   *slot = S;
-  Elem<T>::store(out + idx, S * gelu_tanh_of(Elem<T>::load(y + (size_t)r * ld_y + c) + y_bias[c]));
+  Elem<T>::store(out + idx, S * gelu_gate<FAST>(Elem<T>::load(y + (size_t)r * ld_y + c) + y_bias[c]));
 }
 
 }  // namespace ms
@@ -299,7 +425,7 @@ __global__ void rglru_step_kernel(T* __restrict__ out, float* __restrict__ state
 using namespace ms;
 
 MS_EXPORT int ms_mlstm_gates(float* decay, float* write, float* floor_, const void* raw, int ld, const float* bias, float* m_state,
-                             const int* cu_q, const int* q_start, const int* state_slot, int num_rows, int H, float cap, int single,
+                             const int* cu_q, const int* q_start, const int* state_slot, int num_rows, int tokens, int H, float cap, int single,
                              int dtype, cudaStream_t stream) {
   if (num_rows == 0) return 0;
   MS_CHECK_ARG(H > 0 && H <= 65535 && cap > 0.f, "mlstm_gates: %d heads, cap %g", H, (double)cap);
@@ -307,10 +433,12 @@ MS_EXPORT int ms_mlstm_gates(float* decay, float* write, float* floor_, const vo
 #define MS_GATES(T, N) MS_LAUNCH((mlstm_gates_kernel<T, N>), grid, N, 0, stream, decay, write, floor_, (const T*)raw, ld, bias, m_state, cu_q, q_start, state_slot, H, cap)
   if (dtype == MS_F32) {
     if (single) MS_GATES(float, 32);
-    else MS_GATES(float, 256);
+    else if (tokens < 512) MS_GATES(float, 256);
+    else MS_GATES(float, 1024);
   } else {
     if (single) MS_GATES(__nv_bfloat16, 32);
-    else MS_GATES(__nv_bfloat16, 256);
+    else if (tokens < 512) MS_GATES(__nv_bfloat16, 256);
+    else MS_GATES(__nv_bfloat16, 1024);
   }
 #undef MS_GATES
   return 0;
@@ -324,6 +452,10 @@ MS_EXPORT int ms_mlstm_output(void* out, int ld_out, const float* o, int ld_o, c
   if (dtype == MS_F32)
     MS_LAUNCH(mlstm_output_kernel<float>, blocks, 256, 0, stream, (float*)out, ld_out, o, ld_o, floor_, w, (const float*)gate, ld_gate, items, H, dv,
               eps, den_eps);
+  else if (dv % 8 == 0 && ld_o % 4 == 0 && ld_out % 8 == 0 && ld_gate % 8 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)o % 16 == 0 &&
+           (uintptr_t)gate % 16 == 0 && (uintptr_t)w % 16 == 0)
+    MS_LAUNCH(mlstm_output_bf16x8_kernel, blocks, 256, 0, stream, (__nv_bfloat16*)out, ld_out, o, ld_o, floor_, w, (const __nv_bfloat16*)gate,
+              ld_gate, items, H, dv, eps, den_eps);
   else
     MS_LAUNCH(mlstm_output_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)out, ld_out, o, ld_o, floor_, w,
               (const __nv_bfloat16*)gate, ld_gate, items, H, dv, eps, den_eps);
@@ -336,6 +468,12 @@ MS_EXPORT int ms_conv_bias(void* u, const void* x, int ld, void* conv_state, con
   if (tokens == 0) return 0;
   MS_CHECK_ARG(taps >= 1 && C >= 1, "conv_bias: %d taps over %d channels", taps, C);
   if (dtype == MS_BF16 && C % 8 == 0 && ld % 8 == 0 && (uintptr_t)u % 16 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)conv_state % 16 == 0) {
+    if (!single && taps == 4 && (uintptr_t)w % 16 == 0 && (uintptr_t)bias % 16 == 0 && (uintptr_t)in_bias % 16 == 0) {
+      const long long threads = (long long)ceil_div(tokens, CONV_RUN) * (C / 8);
+      MS_LAUNCH(conv_bias_run_kernel<4>, (unsigned)((threads + 127) / 128), 128, 0, stream, (__nv_bfloat16*)u, (const __nv_bfloat16*)x, ld,
+                (const __nv_bfloat16*)conv_state, w, bias, in_bias, row_of_token, cu_q, q_start, state_slot, tokens, C);
+      return 0;
+    }
     const long long items = (long long)tokens * (C / 8);
     MS_LAUNCH((conv_bias_kernel<__nv_bfloat16, 8>), (unsigned)((items + 127) / 128), 128, 0, stream, (__nv_bfloat16*)u, (const __nv_bfloat16*)x,
               ld, (__nv_bfloat16*)conv_state, w, bias, in_bias, row_of_token, cu_q, q_start, state_slot, items, C, taps, single);
@@ -370,7 +508,7 @@ MS_EXPORT int ms_rglru_scan(void* out, float* state, const float* z, const void*
   }
   MS_CHECK_ARG(num_rows <= 65535, "rglru_scan: %d rows", num_rows);
   // a step of few tokens has nothing to share out between CTAs
-  const int ctas = tokens >= 8 * LRU_WARPS * LRU_RUN ? 8 : tokens >= 2 * LRU_WARPS * LRU_RUN ? 2 : 1;
+  const int ctas = tokens >= 4 * LRU_WARPS * LRU_RUN ? LRU_MAX_CTAS : tokens >= 2 * LRU_WARPS * LRU_RUN ? 2 : 1;
   const dim3 grid((unsigned)(ctas * ceil_div(C, 32)), num_rows);
   if (dtype == MS_F32)
     MS_LAUNCH_CLUSTERED(rglru_scan_kernel<float>, grid, LRU_WARPS * 32, 0, stream, ctas, (float*)out, state, z, (const float*)u,

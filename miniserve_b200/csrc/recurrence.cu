@@ -218,6 +218,67 @@ decay_scan_kernel(float* __restrict__ o_out,   // [T, H, dv]
   }
 }
 
+// ---------------------------------------------------------------- one token per row (decode steps), one decay per head
+// Reading and writing the state is all there is to do: LPC lanes take a column's key channels, four at a time, a warp 32 / LPC
+// columns at once and STEP_COLS of them in turn, their loads in flight together. grid (rows, H, column runs).
+constexpr int STEP_COLS = 4, STEP_WARPS = 4;
+template <typename TIn, int LPC>
+__global__ void __launch_bounds__(STEP_WARPS * 32)
+decay_step_kernel(float* __restrict__ o_out, float* __restrict__ state, const TIn* __restrict__ q, int ld_q, const TIn* __restrict__ k, int ld_k,
+                  int qk_group, const TIn* __restrict__ v, int ld_v, const float* __restrict__ z, int ld_z, const int* __restrict__ cu_q,
+                  const int* __restrict__ q_start, const int* __restrict__ state_slot, int H, int dk, int dv, float q_scale,
+                  const float* __restrict__ v_scale, int dv_in) {
+  pdl_prologue();
+  constexpr int CPW = 32 / LPC;  // columns a warp takes at once
+  const int r = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int l = lane % LPC, sub = lane / LPC;
+  const int t = cu_q[r];
+  const bool fresh = q_start[r] == 0;
+  const float a = z[(size_t)t * ld_z + h], w = v_scale ? v_scale[(size_t)t * H + h] : 1.f;
+  const size_t qk = (size_t)(h / qk_group) * dk;
+  const int j0 = (blockIdx.z * STEP_WARPS + warp) * CPW * STEP_COLS + sub;
+  float* col = state + ((size_t)state_slot[r] * H + h) * (size_t)dv * dk;
+  float acc[STEP_COLS] = {};
+  float vj[STEP_COLS];
+#pragma unroll
+  for (int s = 0; s < STEP_COLS; ++s) {
+    const int j = j0 + s * CPW;
+    vj[s] = w * (j < dv_in ? Elem<TIn>::load(v + (size_t)t * ld_v + (size_t)h * dv_in + j) : 1.f);
+  }
+  for (int i = l * 4; i < dk; i += LPC * 4) {
+    float4 S[STEP_COLS];
+#pragma unroll
+    for (int s = 0; s < STEP_COLS; ++s) {
+      const int j = j0 + s * CPW;
+      S[s] = fresh || j >= dv ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(col + (size_t)j * dk + i);
+    }
+    float kf[4], qf[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      kf[e] = Elem<TIn>::load(k + (size_t)t * ld_k + qk + i + e);
+      qf[e] = Elem<TIn>::load(q + (size_t)t * ld_q + qk + i + e) * q_scale;
+    }
+#pragma unroll
+    for (int s = 0; s < STEP_COLS; ++s) {
+      const int j = j0 + s * CPW;
+      S[s].x = fmaf(a, S[s].x, kf[0] * vj[s]);
+      S[s].y = fmaf(a, S[s].y, kf[1] * vj[s]);
+      S[s].z = fmaf(a, S[s].z, kf[2] * vj[s]);
+      S[s].w = fmaf(a, S[s].w, kf[3] * vj[s]);
+      acc[s] += (qf[0] * S[s].x + qf[1] * S[s].y) + (qf[2] * S[s].z + qf[3] * S[s].w);
+      if (j < dv) *reinterpret_cast<float4*>(col + (size_t)j * dk + i) = S[s];
+    }
+  }
+#pragma unroll
+  for (int s = 0; s < STEP_COLS; ++s) {
+    float x = acc[s];
+#pragma unroll
+    for (int o = LPC >> 1; o > 0; o >>= 1) x += __shfl_xor_sync(0xffffffffu, x, o);
+    const int j = j0 + s * CPW;
+    if (l == 0 && j < dv) o_out[((size_t)t * H + h) * dv + j] = x;
+  }
+}
+
 // ---------------------------------------------------------------- the decay rule over segments of a long row
 // The decay rule is linear in the state with a diagonal factor: S_t = a_t (.) S_(t-1) + k_t v_t^T. So a long row
 // is cut into P segments that are walked at the same time, each from a zero state (decay_scan_kernel over the
@@ -519,6 +580,31 @@ MS_EXPORT int ms_decay_scan(float* o_out, float* state, const void* q, int ld_q,
   }
 #undef MS_SCAN
   return ms::fail("decay_scan: unsupported dtypes (%d, %d)", in_dtype, z_dtype);
+}
+
+// The decay rule for a step of one token per row: z [T, H] float32 the decays, dk a multiple of 4.
+MS_EXPORT int ms_decay_step(float* o_out, float* state, const void* q, int ld_q, const void* k, int ld_k, int qk_group, const void* v, int ld_v,
+                            const float* z, int ld_z, const int* cu_q, const int* q_start, const int* state_slot, int num_rows, int H, int dk,
+                            int dv, float q_scale, const float* v_scale, int dv_in, int in_dtype, cudaStream_t stream) {
+  if (num_rows == 0) return 0;
+  MS_CHECK_ARG(H > 0 && dk > 0 && dk % 4 == 0 && dv > 0 && (dv_in == dv || dv_in == dv - 1) && (uintptr_t)state % 16 == 0,
+               "decay_step: heads of %d x %d (%d read)", dk, dv, dv_in);
+  MS_CHECK_ARG(qk_group > 0 && H % qk_group == 0 && H <= 65535, "decay_step: %d heads are not a multiple of the group of %d", H, qk_group);
+#define MS_STEP(TIN, LPC)                                                                                                              \
+  MS_LAUNCH((decay_step_kernel<TIN, LPC>), dim3(num_rows, H, ceil_div(dv, STEP_WARPS * (32 / LPC) * STEP_COLS)), STEP_WARPS * 32, 0, stream, o_out, \
+            state, (const TIN*)q, ld_q, (const TIN*)k, ld_k, qk_group, (const TIN*)v, ld_v, z, ld_z, cu_q, q_start, state_slot, H, dk, dv, q_scale, \
+            v_scale, dv_in)
+  if (in_dtype == MS_F32) {
+    if (dk > 64) MS_STEP(float, 32);
+    else if (dk > 32) MS_STEP(float, 16);
+    else MS_STEP(float, 8);
+  } else {
+    if (dk > 64) MS_STEP(__nv_bfloat16, 32);
+    else if (dk > 32) MS_STEP(__nv_bfloat16, 16);
+    else MS_STEP(__nv_bfloat16, 8);
+  }
+#undef MS_STEP
+  return 0;
 }
 
 MS_EXPORT int ms_decay_from_logits(float* out, const void* z, int ld_z, const float* z_bias, const float* decay_coef, float z_sign,

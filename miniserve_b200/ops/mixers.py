@@ -202,6 +202,11 @@ def decay_scan(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign: float, beta
     if not delta and not ctx.decode_only and t >= SEGMENT_MIN_TOKENS and SEGMENTS > 1 and dk <= SEGMENT_MAX_DK:
         return _decay_scan_segmented(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign, ctx, heads, dk, dv, q_scale, head_decay,
                                      v_scale, dv_in)
+    if not delta and head_decay and ctx.decode_only and dk % 4 == 0:  # one token per row: the state is read and written once, nothing else
+        native.recurrence_check(native.recurrence().ms_decay_step(
+            _ptr(o_out), _ptr(state), _ptr(q), _rows(q), _ptr(k), _rows(k), heads // groups, _ptr(v), _rows(v), _ptr(z), _rows(z), _ptr(ctx.cu_q),
+            _ptr(ctx.q_start), _ptr(ctx.state_slot), ctx.num_rows, heads, dk, dv, float(q_scale), _ptr(v_scale), dv_in, _dt(q.dtype), ctx.stream))
+        return
     ready = int(head_decay)
     if not ctx.decode_only and not head_decay:
         # a prompt portion: exponentials and logarithms for all tokens at once, not inside the serial walk
@@ -551,7 +556,7 @@ def mlstm_gates(out, raw, bias, m_state, ctx, cap: float) -> None:
     assert out.shape == (3, t, h) and raw.shape == (t, 2 * h) and bias.numel() == 2 * h and m_state.shape[1] == h
     native.recurrence_check(native.recurrence().ms_mlstm_gates(
         _ptr(out[0]), _ptr(out[1]), _ptr(out[2]), _ptr(raw), _rows(raw), _ptr(bias), _ptr(m_state), _ptr(ctx.cu_q), _ptr(ctx.q_start),
-        _ptr(ctx.state_slot), ctx.num_rows, h, float(cap), int(ctx.decode_only), _dt(raw.dtype), ctx.stream))
+        _ptr(ctx.state_slot), ctx.num_rows, t, h, float(cap), int(ctx.decode_only), _dt(raw.dtype), ctx.stream))
 
 
 def mlstm_output(out, o, floor, weight, gate, eps: float, den_eps: float, stream=None) -> None:

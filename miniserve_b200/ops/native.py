@@ -159,6 +159,7 @@ def recurrence():
     lib.ms_recurrence_set_pdl(int(pdl_enabled()))
     _declare(lib, "ms_decay_scan", [_p, _p, _p, _i, _p, _i, _i, _p, _i, _p, _i, _p, _p, _f, _i, _p, _i, _p, _p, _p,
                                     _i, _i, _i, _i, _f, _i, _i, _i, _i, _p, _i, _p])
+    _declare(lib, "ms_decay_step", [_p, _p, _p, _i, _p, _i, _i, _p, _i, _p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _p, _i, _i, _p])
     _declare(lib, "ms_segment_setup", [_p, _p, _p, _p, _i, _i, _p])
     _declare(lib, "ms_segment_finish", [_p, _p, _p, _p, _p, _p, _i, _p, _i, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _i, _p])
     _declare(lib, "ms_decay_from_logits", [_p, _p, _i, _p, _p, _f, _p, _i, _i, _i, _i, _i, _p])
@@ -167,7 +168,7 @@ def recurrence():
     _declare(lib, "ms_gated_group_norm", [_p, _i, _p, _p, _i, _p, _p, _i, _p, _i, _i, _i, _i, _f, _i, _p])
     _declare(lib, "ms_conv_state_update", [_p, _p, _i, _p, _p, _p, _i, _i, _i, _i, _p])
     _declare(lib, "ms_head_norm_gate", [_p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _f, _i, _i, _p])
-    _declare(lib, "ms_mlstm_gates", [_p, _p, _p, _p, _i, _p, _p, _p, _p, _p, _i, _i, _f, _i, _i, _p])
+    _declare(lib, "ms_mlstm_gates", [_p, _p, _p, _p, _i, _p, _p, _p, _p, _p, _i, _i, _i, _f, _i, _i, _p])
     _declare(lib, "ms_mlstm_output", [_p, _i, _p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _f, _i, _p])
     _declare(lib, "ms_conv_bias", [_p, _p, _i, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _p])
     _declare(lib, "ms_chunk_max", [_i, _i])
