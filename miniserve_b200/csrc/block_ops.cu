@@ -173,6 +173,58 @@ __global__ void token_shift_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const
   }
 }
 
+// Several mixes of one input: out[m, t] = h[t] + (prev - h[t]) * mix[m], m < mixes; planes [mixes, T, width]. prev and the state slot as above.
+template <typename T>
+__global__ void token_mixes_kernel(T* __restrict__ out, const T* __restrict__ h, T* __restrict__ state, const float* __restrict__ mix, int mixes,
+                                   const int* __restrict__ row_of_token, const int* __restrict__ cu_q, const int* __restrict__ q_start,
+                                   const int* __restrict__ state_slot, int width) {
+  pdl_prologue();
+  const int t = blockIdx.x;
+  const int row = row_of_token[t];
+  const bool first = t == cu_q[row];
+  T* slot = state + (size_t)state_slot[row] * width;
+  const T* prev = first ? (q_start[row] > 0 ? slot : nullptr) : h + (size_t)(t - 1) * width;
+  const T* newest = h + (size_t)(cu_q[row + 1] - 1) * width;
+  const size_t plane = (size_t)gridDim.x * width;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    const float x = Elem<T>::load(h + (size_t)t * width + c);
+    const float p = prev ? Elem<T>::load(prev + c) : 0.f;
+    for (int m = 0; m < mixes; ++m) Elem<T>::store(out + m * plane + (size_t)t * width + c, fmaf(p - x, mix[(size_t)m * width + c], x));
+    if (first) slot[c] = newest[c];
+  }
+}
+
+__global__ void token_mixes_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ h, __nv_bfloat16* __restrict__ state,
+                                          const float* __restrict__ mix, int mixes, const int* __restrict__ row_of_token,
+                                          const int* __restrict__ cu_q, const int* __restrict__ q_start, const int* __restrict__ state_slot,
+                                          int width) {
+  pdl_prologue();
+  const int t = blockIdx.x;
+  const int row = row_of_token[t];
+  const bool first = t == cu_q[row];
+  __nv_bfloat16* slot = state + (size_t)state_slot[row] * width;
+  const __nv_bfloat16* prev = first ? (q_start[row] > 0 ? slot : nullptr) : h + (size_t)(t - 1) * width;
+  const __nv_bfloat16* newest = h + (size_t)(cu_q[row + 1] - 1) * width;
+  const size_t plane = (size_t)gridDim.x * width;
+  for (int c = threadIdx.x * 8; c < width; c += blockDim.x * 8) {
+    float x[8], p[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    bf16x8_to_float(*reinterpret_cast<const uint4*>(h + (size_t)t * width + c), x);
+    if (prev) bf16x8_to_float(*reinterpret_cast<const uint4*>(prev + c), p);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) p[e] -= x[e];
+    for (int m = 0; m < mixes; ++m) {
+      const float* mm = mix + (size_t)m * width + c;
+      const float4 ma = *reinterpret_cast<const float4*>(mm), mb = *reinterpret_cast<const float4*>(mm + 4);
+      const float mv[8] = {ma.x, ma.y, ma.z, ma.w, mb.x, mb.y, mb.z, mb.w};
+      float y[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] = fmaf(p[e], mv[e], x[e]);
+      *reinterpret_cast<uint4*>(out + m * plane + (size_t)t * width + c) = float_to_bf16x8(y);
+    }
+    if (first) *reinterpret_cast<uint4*>(slot + c) = *reinterpret_cast<const uint4*>(newest + c);
+  }
+}
+
 // state[slot of row] = h[the row's last token of this step]
 template <typename T>
 __global__ void shift_state_update_kernel(T* __restrict__ state, const T* __restrict__ h, const int* __restrict__ cu_q,
@@ -868,6 +920,27 @@ MS_EXPORT int ms_token_shift(void* out, const void* h, void* state, const float*
   else
     MS_LAUNCH(token_shift_kernel<__nv_bfloat16>, tokens, threads, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)h,
               (__nv_bfloat16*)state, mix, row_of_token, cu_q, q_start, state_slot, width, update);
+  return 0;
+}
+
+// out [mixes, tokens, width]; mix [mixes, width] float32; the state's slots get each row's last h of this step.
+MS_EXPORT int ms_token_mixes(void* out, const void* h, void* state, const float* mix, int mixes, const int* row_of_token, const int* cu_q,
+                             const int* q_start, const int* state_slot, int tokens, int width, int dtype, cudaStream_t stream) {
+  if (tokens == 0) return 0;
+  MS_CHECK_ARG(width > 0 && mixes > 0 && out != h, "token_mixes: width=%d, %d mixes, and the output may not be the input", width, mixes);
+  const int threads = width >= 1024 ? 256 : 128;
+  if (dtype == MS_BF16 && width % 8 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)state % 16 == 0 &&
+      (uintptr_t)mix % 16 == 0) {
+    MS_LAUNCH(token_mixes_bf16x8_kernel, tokens, width >= 2048 ? 256 : 128, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)h,
+              (__nv_bfloat16*)state, mix, mixes, row_of_token, cu_q, q_start, state_slot, width);
+    return 0;
+  }
+  if (dtype == MS_F32)
+    MS_LAUNCH(token_mixes_kernel<float>, tokens, threads, 0, stream, (float*)out, (const float*)h, (float*)state, mix, mixes, row_of_token, cu_q,
+              q_start, state_slot, width);
+  else
+    MS_LAUNCH(token_mixes_kernel<__nv_bfloat16>, tokens, threads, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)h, (__nv_bfloat16*)state,
+              mix, mixes, row_of_token, cu_q, q_start, state_slot, width);
   return 0;
 }
 

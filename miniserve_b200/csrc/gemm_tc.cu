@@ -27,7 +27,10 @@ namespace ms {
 constexpr int TC_BM = 128, TC_BK = 64;
 constexpr int TC_THREADS = 192;
 
-enum TcEpilogue : int { TC_OUT_BF16 = 0, TC_OUT_F32 = 1, TC_SILU_MUL = 2, TC_QKV_ROPE = 3, TC_RELU2 = 4 };
+enum TcEpilogue : int { TC_OUT_BF16 = 0, TC_OUT_F32 = 1, TC_SILU_MUL = 2, TC_QKV_ROPE = 3, TC_RELU2 = 4, TC_CLAMPED_GLU = 5 };
+
+// Epilogues whose weight is a stack of gate rows and up rows, both factors of an output in one tile.
+__host__ __device__ constexpr bool tc_gated(int epi) { return epi == TC_SILU_MUL || epi == TC_CLAMPED_GLU; }
 
 // What the q|k|v epilogue (TC_QKV_ROPE) needs besides the product: per-head RMSNorm of q and k, rotation
 // by position and the write of q to [T, nq, 128] and of k, v into their cache pages, as the separate
@@ -123,6 +126,19 @@ struct TcSmem {
   static constexpr int stage_bytes = a_bytes + b_bytes;
 };
 
+// g sigmoid(alpha g) (u + shift) with g capped at limit and u held within +-limit (a negative limit: neither). Fast exponential and
+// division: relative error about 1e-6, far below the bfloat16 rounding of the result.
+struct ClampedGlu {
+  float limit, alpha, shift;
+};
+__device__ __forceinline__ float clamped_glu_fast(float g, float u, const ClampedGlu& p) {
+  if (p.limit >= 0.f) {
+    g = fminf(g, p.limit);
+    u = fminf(fmaxf(u, -p.limit), p.limit);
+  }
+  return __fdividef(g, 1.0f + __expf(-p.alpha * g)) * (u + p.shift);
+}
+
 // The rows of A sorted into runs, one run per weight matrix (the experts of a routed feed-forward, W [E * w_rows, K]):
 // a plan on the device lists the row tiles, (matrix, first row) each, meta[0] = how many; offsets[e + 1] ends run e.
 struct TcGroups {
@@ -130,6 +146,7 @@ struct TcGroups {
   const int* meta;
   const int* offsets;
   int w_rows;  // rows of W per matrix
+  ClampedGlu glu;
 };
 
 // grid: (ceil(N_out / (BN or BN/2 for SiLU)), ceil(M / 128)). For TC_SILU_MUL, W is [2 * inter, K]
@@ -148,7 +165,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
   __shared__ int gave_up;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  constexpr int COLS = EPI == TC_SILU_MUL ? BN / 2 : BN;  // output columns per CTA
+  constexpr int COLS = tc_gated(EPI) ? BN / 2 : BN;  // output columns per CTA
   const int n0 = blockIdx.x * COLS;
   int m0 = blockIdx.y * TC_BM, w0 = n0;  // the tile's first row of A and of W
   if (GROUPED) {
@@ -199,7 +216,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         unsigned char* b_tile = a_tile + TcSmem<BN>::a_bytes;
         mbar_expect_tx(&full_bar[s], TcSmem<BN>::stage_bytes);
         tma_load_2d(a_tile, &map_a, &full_bar[s], it * TC_BK, m0);
-        if (EPI == TC_SILU_MUL) {
+        if (tc_gated(EPI)) {
           tma_load_2d(b_tile, &map_w, &full_bar[s], it * TC_BK, w0);
           tma_load_2d(b_tile + TcSmem<BN>::b_bytes / 2, &map_w, &full_bar[s], it * TC_BK, up_row_offset + w0);
         } else {
@@ -249,7 +266,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         uint32_t acc[32];
         tmem_ld32(lane_addr + (uint32_t)c, acc);
         uint32_t up[32];
-        if (EPI == TC_SILU_MUL) tmem_ld32(lane_addr + (uint32_t)(COLS + c), up);
+        if (tc_gated(EPI)) tmem_ld32(lane_addr + (uint32_t)(COLS + c), up);
         asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
         if (row < M) {
           const int col0 = n0 + c;
@@ -268,6 +285,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             for (int j = 0; j < 32; ++j) {
               float x = __uint_as_float(acc[j]);
               if (EPI == TC_SILU_MUL) x = x / (1.0f + expf(-x)) * __uint_as_float(up[j]);
+              if (EPI == TC_CLAMPED_GLU) x = clamped_glu_fast(x, __uint_as_float(up[j]), grp.glu);
               if (EPI == TC_RELU2) {
                 x = fmaxf(x, 0.f);
                 x *= x;
@@ -359,7 +377,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __gri
   __shared__ uint32_t tmem_base_slot;
   static_assert(BN <= 256, "two accumulators of BN columns must fit 512 columns of tensor memory");
   constexpr uint32_t ACC_COLS = BN <= 64 ? 64 : BN <= 128 ? 128 : 256;  // columns of one accumulator
-  constexpr int COLS = EPI == TC_SILU_MUL ? BN / 2 : BN;                // output columns per tile
+  constexpr int COLS = tc_gated(EPI) ? BN / 2 : BN;                // output columns per tile
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int k_iters = (K + TC_BK - 1) / TC_BK;
@@ -716,7 +734,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
   __shared__ uint32_t tmem_base_slot;
   __shared__ int row_dst[2][TC_BM];  // TC_QKV_ROPE: the pool row (page, kv head, slot) each row of a k or v head goes to (-1: none)
   __shared__ uint64_t cs_full[CS_SLOTS], cs_empty[CS_SLOTS];  // TC_QKV_ROPE: a slot of the cos/sin ring has landed / has been read by all eight warps
-  constexpr int COLS = EPI == TC_SILU_MUL ? BN / 2 : BN;  // output columns per tile
+  constexpr int COLS = tc_gated(EPI) ? BN / 2 : BN;  // output columns per tile
   constexpr int STAGE_BYTES = pair_stage_bytes(BN);
   constexpr uint32_t TMEM_COLS = 2 * BN;             // two accumulators (512 or 256 columns)
   constexpr int A_BYTES = TC_BM * TC_BK * 2;
@@ -1116,7 +1134,7 @@ static int launch_tc(void* out, const void* A, const void* W, int M, int N_out, 
                      int* status, cudaStream_t stream) {
   CUtensorMap map_a, map_w;
   if (int rc = make_map(&map_a, A, M, K, TC_BM)) return rc;
-  if (int rc = make_map(&map_w, W, w_rows, K, EPI == TC_SILU_MUL ? BN / 2 : BN)) return rc;
+  if (int rc = make_map(&map_w, W, w_rows, K, tc_gated(EPI) ? BN / 2 : BN)) return rc;
   constexpr size_t smem = (size_t)STAGES * TcSmem<BN>::stage_bytes + 1024;
   auto kernel = gemm_tc_kernel<BN, STAGES, EPI>;
   static bool configured = false;
@@ -1124,7 +1142,7 @@ static int launch_tc(void* out, const void* A, const void* W, int M, int N_out, 
     MS_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = true;
   }
-  constexpr int COLS = EPI == TC_SILU_MUL ? BN / 2 : BN;
+  constexpr int COLS = tc_gated(EPI) ? BN / 2 : BN;
   dim3 grid(ceil_div(N_out, COLS), ceil_div(M, TC_BM));
   MS_LAUNCH(kernel, grid, TC_THREADS, smem, stream, map_a, map_w, out, M, N_out, K, up_row_offset, status, TcGroups{});
   return 0;
@@ -1136,7 +1154,7 @@ static int launch_tc_grouped(void* out, const void* A, const void* W, int rows, 
                              int up_row_offset, const TcGroups& grp, int max_tiles, int* status, cudaStream_t stream) {
   CUtensorMap map_a, map_w;
   if (int rc = make_map(&map_a, A, rows, K, TC_BM)) return rc;
-  if (int rc = make_map(&map_w, W, (long long)matrices * w_rows, K, EPI == TC_SILU_MUL ? BN / 2 : BN)) return rc;
+  if (int rc = make_map(&map_w, W, (long long)matrices * w_rows, K, tc_gated(EPI) ? BN / 2 : BN)) return rc;
   constexpr size_t smem = (size_t)STAGES * TcSmem<BN>::stage_bytes + 1024;
   auto kernel = gemm_tc_kernel<BN, STAGES, EPI, true>;
   static bool configured = false;
@@ -1144,7 +1162,7 @@ static int launch_tc_grouped(void* out, const void* A, const void* W, int rows, 
     MS_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = true;
   }
-  constexpr int COLS = EPI == TC_SILU_MUL ? BN / 2 : BN;
+  constexpr int COLS = tc_gated(EPI) ? BN / 2 : BN;
   dim3 grid(ceil_div(N_out, COLS), max_tiles);
   MS_LAUNCH(kernel, grid, TC_THREADS, smem, stream, map_a, map_w, out, rows, N_out, K, up_row_offset, status, grp);
   return 0;
@@ -1155,7 +1173,7 @@ static int launch_tc_persistent(void* out, const void* A, const void* W, int M, 
                                 int* status, cudaStream_t stream) {
   CUtensorMap map_a, map_w;
   if (int rc = make_map(&map_a, A, M, K, TC_BM)) return rc;
-  if (int rc = make_map(&map_w, W, w_rows, K, EPI == TC_SILU_MUL ? BN / 2 : BN)) return rc;
+  if (int rc = make_map(&map_w, W, w_rows, K, tc_gated(EPI) ? BN / 2 : BN)) return rc;
   constexpr size_t smem = (size_t)STAGES * TcSmem<BN>::stage_bytes + 1024;
   static_assert(smem <= 227 * 1024, "the ring does not fit shared memory");
   auto kernel = gemm_tc_persistent_kernel<BN, STAGES, EPI>;
@@ -1168,7 +1186,7 @@ static int launch_tc_persistent(void* out, const void* A, const void* W, int M, 
     MS_CHECK_CUDA(cudaDeviceGetAttribute(&sm_count, cudaDevAttrMultiProcessorCount, dev));
     configured = true;
   }
-  constexpr int COLS = EPI == TC_SILU_MUL ? BN / 2 : BN;
+  constexpr int COLS = tc_gated(EPI) ? BN / 2 : BN;
   const long long tiles = (long long)ceil_div(N_out, COLS) * ceil_div(M, TC_BM);
   MS_CHECK_ARG(tiles < (1LL << 30), "gemm_tc: too many tiles (%lld)", tiles);
   const unsigned grid = (unsigned)(tiles < sm_count ? tiles : sm_count);
@@ -1200,7 +1218,7 @@ static int launch_tc_pair(void* out, const void* A, const void* W, int M, int N_
     MS_CHECK_CUDA(cudaDeviceGetAttribute(&sm_count, cudaDevAttrMultiProcessorCount, dev));
     configured = true;
   }
-  constexpr int COLS = EPI == TC_SILU_MUL ? BN / 2 : BN;
+  constexpr int COLS = tc_gated(EPI) ? BN / 2 : BN;
   const long long tiles = (long long)ceil_div(N_out, COLS) * ceil_div(M, 2 * TC_BM);
   MS_CHECK_ARG(tiles < (1LL << 30), "gemm_tc: too many tiles (%lld)", tiles);
   const long long pairs = tiles < sm_count / 2 ? tiles : sm_count / 2;
@@ -1365,22 +1383,27 @@ MS_EXPORT int ms_gemm_tc_bf16(void* out, const void* A, const void* W, int M, in
 // The experts' products of a routed feed-forward over rows sorted by expert (tiles of 128 rows, (expert, first row)
 // each; meta[0] tiles; offsets[e + 1] ends expert e's rows; at most max_tiles tiles).
 // gated = 1: W [E, 2 N, K] (an expert's gate rows, then its up rows), out [rows, N] bfloat16 = silu(A gate^T) * (A up^T);
-// gated = 0: W [E, N, K], out [rows, N] float32 = A W^T; gated = 2: W [E, N, K], out [rows, N] bfloat16 = relu(A W^T)^2.
+// gated = 0: W [E, N, K], out [rows, N] float32 = A W^T; gated = 2: W [E, N, K], out [rows, N] bfloat16 = relu(A W^T)^2;
+// gated = 3: W as for 1, the gate clamped and shifted (ClampedGlu).
 MS_EXPORT int ms_gemm_tc_experts_bf16(void* out, const void* A, const void* W, int rows, int N, int K, int experts, int gated,
-                                      const int* tiles, const int* meta, const int* offsets, int max_tiles, int* status,
-                                      cudaStream_t stream) {
+                                      const int* tiles, const int* meta, const int* offsets, int max_tiles, float limit,
+                                      float alpha, float shift, int* status, cudaStream_t stream) {
   if (rows == 0 || N == 0 || max_tiles == 0) return 0;
   MS_CHECK_ARG(rows > 0 && N > 0 && K > 0 && experts > 0, "gemm_tc_experts: bad sizes rows=%d N=%d K=%d experts=%d", rows, N, K, experts);
   MS_CHECK_ARG(K % 8 == 0, "gemm_tc_experts: K=%d must be a multiple of 8 (rows must be 16-byte multiples for TMA)", K);
   MS_CHECK_ARG(((uintptr_t)A % 16 == 0) && ((uintptr_t)W % 16 == 0), "gemm_tc_experts: operands must be 16-byte aligned");
   MS_CHECK_ARG(status != nullptr && tiles != nullptr && meta != nullptr && offsets != nullptr, "gemm_tc_experts: needs a plan and a status word");
   MS_CHECK_ARG(max_tiles <= 65535, "gemm_tc_experts: %d row tiles are too many for one launch", max_tiles);
-  MS_CHECK_ARG((long long)experts * (gated == 1 ? 2 : 1) * N < (1LL << 31), "gemm_tc_experts: the weights have too many rows");
+  MS_CHECK_ARG((long long)experts * (gated == 1 || gated == 3 ? 2 : 1) * N < (1LL << 31), "gemm_tc_experts: the weights have too many rows");
+  if (gated == 3) {
+    const TcGroups grp{tiles, meta, offsets, 2 * N, {limit, alpha, shift}};
+    return launch_tc_grouped<256, 4, TC_CLAMPED_GLU>(out, A, W, rows, N, experts, 2 * N, K, N, grp, max_tiles, status, stream);
+  }
   if (gated == 1) {
-    const TcGroups grp{tiles, meta, offsets, 2 * N};
+    const TcGroups grp{tiles, meta, offsets, 2 * N, {}};
     return launch_tc_grouped<256, 4, TC_SILU_MUL>(out, A, W, rows, N, experts, 2 * N, K, N, grp, max_tiles, status, stream);
   }
-  const TcGroups grp{tiles, meta, offsets, N};
+  const TcGroups grp{tiles, meta, offsets, N, {}};
   if (gated == 2) return launch_tc_grouped<128, 5, TC_RELU2>(out, A, W, rows, N, experts, N, K, 0, grp, max_tiles, status, stream);
   return launch_tc_grouped<128, 5, TC_OUT_F32>(out, A, W, rows, N, experts, N, K, 0, grp, max_tiles, status, stream);
 }

@@ -116,12 +116,16 @@ __global__ void head_gate_bf16x8_kernel(__nv_bfloat16* __restrict__ out, int ld_
 // the projection's columns before anything else (null: none). ``unit_norm``: q and k are divided by their root mean
 // square over dk also where no norm weight is given (a norm without a weight). ``q_scale``: float32 [nq], a factor per
 // query head applied last (a learned temperature of the scores), or null. ``temp_coef``, ``temp_every``: every query is
-// multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) at position p (temp_every 0: it is not).
+// multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) at position p (temp_every 0: it is not). ``v_other`` [T, nkv*dv]
+// (rows ld_other apart, the run's dtype) with ``v_share`` (one float32): values become (1 - share) v + share v_other.
 struct PrepareExtras {
   const float* bias;
   const float* q_scale;
   int unit_norm;
   float temp_coef, temp_every;
+  const void* v_other;
+  int ld_other;
+  const float* v_share;
 };
 
 // The factor on query head h at position pos.
@@ -206,6 +210,13 @@ __global__ void qkv_prepare_bf16x8_kernel(
       if (bias) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) v[e] += bias[c + e];
+      }
+      if (is_v && ex.v_other) {
+        const float share = *ex.v_share;
+        float o[8];
+        bf16x8_to_float(*reinterpret_cast<const uint4*>((const __nv_bfloat16*)ex.v_other + (size_t)t * ex.ld_other + (size_t)(h - nq - nkv) * dv + c), o);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = fmaf(share, o[e], (1.f - share) * v[e]);
       }
     } else {
 #pragma unroll
@@ -308,7 +319,16 @@ __global__ void qkv_prepare_kernel(
     if (bias) bias += (size_t)nq * dk + (is_v ? (size_t)nkv * dk + (size_t)kvh * dv : (size_t)kvh * dk);
   }
   if (is_v) {
-    for (int c = lane; c < d_pad; c += 32) Elem<T>::store(dst + c, c < dv ? Elem<T>::load(src + c) + (bias ? bias[c] : 0.f) : 0.f);
+    const T* other = ex.v_other ? (const T*)ex.v_other + (size_t)t * ex.ld_other + (size_t)(h - nq - nkv) * dv : nullptr;
+    const float share = other ? *ex.v_share : 0.f;
+    for (int c = lane; c < d_pad; c += 32) {
+      float x = 0.f;
+      if (c < dv) {
+        x = Elem<T>::load(src + c) + (bias ? bias[c] : 0.f);
+        if (other) x = fmaf(share, Elem<T>::load(other + c), (1.f - share) * x);
+      }
+      Elem<T>::store(dst + c, x);
+    }
     return;
   }
   float inv = 1.f;
@@ -427,9 +447,10 @@ MS_EXPORT int ms_qkv_prepare(void* q_out, void* k_pool, void* v_pool, const void
                              const int* row_of_token, const int* page_indptr, const int* page_indices, int num_tokens, int nq,
                              int nkv, int dk, int dv, int d_pad, int rot, int adjacent, float eps, int page_size, int num_pages,
                              int* status, int dtype, cudaStream_t stream, const float* bias, const float* q_scale, int unit_norm, float temp_coef,
-                             float temp_every) {
+                             float temp_every, const void* v_other, int ld_other, const float* v_share) {
   if (num_tokens == 0) return 0;
-  const PrepareExtras ex{bias, q_scale, unit_norm, temp_coef, temp_every};
+  const PrepareExtras ex{bias, q_scale, unit_norm, temp_coef, temp_every, v_other, ld_other, v_share};
+  MS_CHECK_ARG(!v_other || (v_share && v_pool), "qkv_prepare: values to mix in come with their share, and where there are values");
   MS_CHECK_ARG((k_pool == nullptr) == (v_pool == nullptr), "qkv_prepare: key and value pools come together or not at all");
   MS_CHECK_ARG(nq > 0 && nkv > 0 && dk > 0 && dv > 0 && d_pad >= dk && d_pad >= dv, "qkv_prepare: bad sizes nq=%d nkv=%d dk=%d dv=%d D=%d",
                nq, nkv, dk, dv, d_pad);
@@ -443,7 +464,7 @@ MS_EXPORT int ms_qkv_prepare(void* q_out, void* k_pool, void* v_pool, const void
   const unsigned blocks = (unsigned)((items + warps - 1) / warps);
   if (dtype == MS_BF16 && (adjacent || rot % 16 == 0) && dk % 8 == 0 && dv % 8 == 0 && d_pad % 8 == 0 && ld % 8 == 0 && q_off % 8 == 0 &&
       k_off % 8 == 0 && v_off % 8 == 0 && (uintptr_t)proj % 16 == 0 && (uintptr_t)q_out % 16 == 0 && (uintptr_t)k_pool % 16 == 0 &&
-      (uintptr_t)v_pool % 16 == 0) {
+      (uintptr_t)v_pool % 16 == 0 && (uintptr_t)v_other % 16 == 0 && ld_other % 8 == 0) {
     if (adjacent || rot == 0)
       MS_LAUNCH(qkv_prepare_bf16x8_kernel<true>, blocks, warps * 32, 0, stream, (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_pool,
                 (__nv_bfloat16*)v_pool, (const __nv_bfloat16*)proj, ld, q_off, k_off, v_off, q_norm_w, k_norm_w, cos_sin, positions,
@@ -488,5 +509,37 @@ MS_EXPORT int ms_act_mul(void* out, const void* gate_up, int tokens, int inter, 
   const unsigned blocks = (unsigned)((total + 255) / 256);
   if (dtype == MS_F32) MS_LAUNCH(act_mul_kernel<float>, blocks, 256, 0, stream, (float*)out, (const float*)gate_up, inter, total, act);
   else MS_LAUNCH(act_mul_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, inter, total, act);
+  return 0;
+}
+
+// x = cap * tanh(x / cap), or tanh(x) with cap 0; in place, float32 arithmetic.
+namespace ms {
+template <typename T>
+__global__ void tanh_inplace_kernel(T* __restrict__ x, float cap, long long n) {
+  pdl_prologue();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const float v = Elem<T>::load(x + i);
+  Elem<T>::store(x + i, cap > 0.f ? cap * tanhf(v / cap) : tanhf(v));
+}
+__global__ void tanh_inplace_f32x4_kernel(float4* __restrict__ x, float cap, long long n4) {
+  pdl_prologue();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n4) return;
+  float4 v = x[i];
+  if (cap > 0.f) v = make_float4(cap * tanhf(v.x / cap), cap * tanhf(v.y / cap), cap * tanhf(v.z / cap), cap * tanhf(v.w / cap));
+  else v = make_float4(tanhf(v.x), tanhf(v.y), tanhf(v.z), tanhf(v.w));
+  x[i] = v;
+}
+}  // namespace ms
+
+MS_EXPORT int ms_tanh_inplace(void* x, float cap, long long n, int dtype, cudaStream_t stream) {
+  if (n == 0) return 0;
+  MS_CHECK_ARG(cap >= 0.f, "tanh_inplace: a cap of %f", (double)cap);
+  const unsigned blocks = (unsigned)((n + 255) / 256);
+  if (dtype == MS_F32 && n % 4 == 0 && (uintptr_t)x % 16 == 0)
+    MS_LAUNCH(tanh_inplace_f32x4_kernel, (unsigned)((n / 4 + 255) / 256), 256, 0, stream, (float4*)x, cap, n / 4);
+  else if (dtype == MS_F32) MS_LAUNCH(tanh_inplace_kernel<float>, blocks, 256, 0, stream, (float*)x, cap, n);
+  else MS_LAUNCH(tanh_inplace_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)x, cap, n);
   return 0;
 }

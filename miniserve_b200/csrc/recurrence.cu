@@ -6,6 +6,7 @@
 //
 //   decay rule:  S <- diag(d_t) S + k_t v_t^T;                         o_t = S^T q_t
 //   delta rule:  S <- diag(d_t) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
+//   bonus rule:  o_t = (S + diag(b) k_t v_t^T)^T q_t;  S <- diag(d_t) S + k_t v_t^T     (b [dk] per head; the read-out comes first)
 //
 // The columns of S never meet: column j of S and element j of v, u and o make a recurrence of their
 // own. So a CTA takes (request, head, a run of columns), a column is held by L threads of a warp
@@ -63,7 +64,9 @@ __device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
   f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
 }
 
-template <typename TIn, typename TZ, bool DELTA, int SCAN_KPT>
+enum ScanRule : int { RULE_DECAY = 0, RULE_DELTA = 1, RULE_BONUS = 2 };
+
+template <typename TIn, typename TZ, int RULE, int SCAN_KPT>
 __global__ void __launch_bounds__(SCAN_THREADS)
 decay_scan_kernel(float* __restrict__ o_out,   // [T, H, dv]
                   float* __restrict__ state,   // [slots, H, dv, dk]
@@ -72,7 +75,9 @@ decay_scan_kernel(float* __restrict__ o_out,   // [T, H, dv]
                   const TZ* __restrict__ z, int ld_z, const float* __restrict__ z_bias, const float* __restrict__ decay_coef,
                   float z_sign, int z_is_decay, const TZ* __restrict__ beta, int ld_beta,
                   const int* __restrict__ cu_q, const int* __restrict__ q_start, const int* __restrict__ state_slot,
-                  int H, int dk, int dv, int L, int chunk, float q_scale, int vec, int dkz, const float* __restrict__ v_scale, int dv_in) {
+                  int H, int dk, int dv, int L, int chunk, float q_scale, int vec, int dkz, const float* __restrict__ v_scale, int dv_in,
+                  const float* __restrict__ bonus) {
+  constexpr bool DELTA = RULE == RULE_DELTA;
   // words a thread's channels take in shared memory: padded so that the 16-byte loads of a quarter warp's lanes fall on different banks
   constexpr int SCAN_SEG = SCAN_KPT == 4 ? 4 : SCAN_KPT + 4;
   extern __shared__ __align__(16) float smem[];
@@ -100,6 +105,11 @@ decay_scan_kernel(float* __restrict__ o_out,   // [T, H, dv]
   for (int e = 0; e < SCAN_KPT; ++e) {
     const int i = l * SCAN_KPT + e;
     S[e] = (!fresh && active && i < dk) ? srow[i] : 0.f;
+  }
+  float B[RULE == RULE_BONUS ? SCAN_KPT : 1];
+  if (RULE == RULE_BONUS) {
+#pragma unroll
+    for (int e = 0; e < SCAN_KPT; ++e) B[RULE == RULE_BONUS ? e : 0] = l * SCAN_KPT + e < dk ? bonus[(size_t)h * dk + l * SCAN_KPT + e] : 0.f;
   }
   const int qk_head = h / qk_group;
   const float coef = decay_coef ? decay_coef[h] : 0.f;  // (not read where z holds the decays themselves)
@@ -196,6 +206,13 @@ decay_scan_kernel(float* __restrict__ o_out,   // [T, H, dv]
           S[e] = fmaf(kt[e], u, S[e]);
           a4[e & 3] = fmaf(qt[e], S[e], a4[e & 3]);
         }
+      } else if (RULE == RULE_BONUS) {
+#pragma unroll
+        for (int e = 0; e < SCAN_KPT; ++e) {
+          const float kv = kt[e] * vj;
+          a4[e & 3] = fmaf(qt[e], fmaf(B[RULE == RULE_BONUS ? e : 0], kv, S[e]), a4[e & 3]);
+          S[e] = fmaf(dt[e], S[e], kv);
+        }
       } else {
 #pragma unroll
         for (int e = 0; e < SCAN_KPT; ++e) {
@@ -287,7 +304,8 @@ decay_step_kernel(float* __restrict__ o_out, float* __restrict__ state, const TI
 //     o_t = o_t(from zero) + S0^T (q_t (.) c_t),     S0(next segment) = c_last (.) S0 + S_end(from zero),
 // which is what the three kernels below add: the running products, the states before every segment (a
 // short walk over the P segments of a row; it also leaves the row's final state in the request's slot), and
-// the missing part of every output. All of it in float32.
+// the missing part of every output. All of it in float32. (The bonus rule reads the state before the token's own decay: its
+// missing part has c of the token before in the place of c_t.)
 
 // seg_cu[r * P + s]: first token of segment s of row r (segments of ceil(len / P) tokens; the last ones may be empty)
 __global__ void segment_setup_kernel(int* __restrict__ seg_cu, int* __restrict__ seg_zero, int* __restrict__ seg_slot,
@@ -355,7 +373,7 @@ template <typename TIn>
 __global__ void __launch_bounds__(FIX_THREADS)
 segment_fixup_kernel(float* __restrict__ o, const TIn* __restrict__ q, int ld_q, int qk_group, const float* __restrict__ c,
                      const float* __restrict__ before, const int* __restrict__ seg_cu, const int* __restrict__ q_start, int P,
-                     int H, int dk, int dv, int cols, float q_scale, int dkz) {
+                     int H, int dk, int dv, int cols, float q_scale, int dkz, int before_decay) {
   extern __shared__ float fix_smem[];
   pdl_prologue();
   const int sg = blockIdx.x, h = blockIdx.y;
@@ -369,7 +387,10 @@ segment_fixup_kernel(float* __restrict__ o, const TIn* __restrict__ q, int ld_q,
   for (int idx = threadIdx.x; idx < n * dk; idx += FIX_THREADS) {
     const int tt = idx / dk, i = idx - tt * dk;
     const size_t tok = (size_t)(t0 + tt);
-    qc[idx] = Elem<TIn>::load(q + tok * ld_q + (size_t)qk_head * dk + i) * q_scale * c[tok * H * dkz + (size_t)h * dkz + (dkz == 1 ? 0 : i)];
+    float passed = 1.f;
+    if (!before_decay) passed = c[tok * H * dkz + (size_t)h * dkz + (dkz == 1 ? 0 : i)];
+    else if ((int)tok > seg_cu[sg]) passed = c[(tok - 1) * H * dkz + (size_t)h * dkz + (dkz == 1 ? 0 : i)];
+    qc[idx] = Elem<TIn>::load(q + tok * ld_q + (size_t)qk_head * dk + i) * q_scale * passed;
   }
   for (int j0 = 0; j0 < dv; j0 += cols) {
     const int ncols = min(cols, dv - j0);
@@ -465,11 +486,11 @@ __global__ void conv_state_update_kernel(T* __restrict__ conv_state, const T* __
 }
 
 // out[t, h * dv + c] = scale * o[t, h, c] / sqrt(mean_c o^2 + eps) * w[c] * act(gate[t, h * dv + c]),
-// act = SiLU (0) or sigmoid (1). One warp per (token, head).
+// act = SiLU (0) or sigmoid (1); w [dv], or [H, dv] (w_stride dv: every head has its own). One warp per (token, head).
 template <typename T>
 __global__ void head_norm_gate_kernel(T* __restrict__ out, int ld_out, const float* __restrict__ o, const float* __restrict__ w,
                                       const T* __restrict__ gate, int ld_gate, int num_tokens, int H, int dv, float eps,
-                                      float scale, int gate_kind) {
+                                      float scale, int gate_kind, int w_stride) {
   pdl_prologue();
   const int lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -484,15 +505,15 @@ __global__ void head_norm_gate_kernel(T* __restrict__ out, int ld_out, const flo
     const float g = Elem<T>::load(gate + (size_t)t * ld_gate + (size_t)h * dv + c);
     const float sg = 1.0f / (1.0f + expf(-g));
     const float a = gate_kind == 0 ? g * sg : sg;
-    Elem<T>::store(out + (size_t)t * ld_out + (size_t)h * dv + c, scale * ((src[c] * inv) * w[c]) * a);
+    Elem<T>::store(out + (size_t)t * ld_out + (size_t)h * dv + c, scale * ((src[c] * inv) * w[(size_t)h * w_stride + c]) * a);
   }
 }
 
-template <typename TIn, typename TZ, bool DELTA, int SCAN_KPT>
+template <typename TIn, typename TZ, int RULE, int SCAN_KPT>
 int launch_scan_kpt(float* o_out, float* state, const void* q, int ld_q, const void* k, int ld_k, int qk_group, const void* v, int ld_v,
                 const void* z, int ld_z, const float* z_bias, const float* decay_coef, float z_sign, int z_is_decay, const void* beta,
                 int ld_beta, const int* cu_q, const int* q_start, const int* state_slot, int num_rows, int H, int dk, int dv, float q_scale,
-                int dkz, const float* v_scale, int dv_in, cudaStream_t stream) {
+                int dkz, const float* v_scale, int dv_in, const float* bonus, cudaStream_t stream) {
   constexpr int SCAN_SEG = SCAN_KPT == 4 ? 4 : SCAN_KPT + 4;
   int L = 1;
   while (L * SCAN_KPT < dk) L <<= 1;
@@ -511,7 +532,7 @@ int launch_scan_kpt(float* o_out, float* state, const void* q, int ld_q, const v
   // one CTA's staging hides behind the others' walks
   if ((long long)num_rows * H * ((dv + cols - 1) / cols) >= 8LL * sm_count && chunk > 8) chunk = 8;
   const size_t smem = (size_t)chunk * per_token;
-  auto kernel = decay_scan_kernel<TIn, TZ, DELTA, SCAN_KPT>;
+  auto kernel = decay_scan_kernel<TIn, TZ, RULE, SCAN_KPT>;
   const dim3 grid(num_rows, H, (dv + cols - 1) / cols);
   // 16-byte loads while staging: every row of q, k and z starts on 16 bytes and heads are whole groups of eight
   const int in8 = 16 / (int)sizeof(TIn), z8 = 16 / (int)sizeof(TZ);
@@ -519,7 +540,7 @@ int launch_scan_kpt(float* o_out, float* state, const void* q, int ld_q, const v
                   (dkz == 1 || ((uintptr_t)z % 16 == 0 && ld_z % z8 == 0));
   MS_LAUNCH(kernel, grid, threads, smem, stream, o_out, state, (const TIn*)q, ld_q, (const TIn*)k, ld_k, qk_group,
             (const TIn*)v, ld_v, (const TZ*)z, ld_z, z_bias, decay_coef, z_sign, z_is_decay, (const TZ*)beta, ld_beta, cu_q, q_start, state_slot,
-            H, dk, dv, L, chunk, q_scale, vec, dkz, v_scale, dv_in);
+            H, dk, dv, L, chunk, q_scale, vec, dkz, v_scale, dv_in, bonus);
   return 0;
 }
 
@@ -528,13 +549,13 @@ int launch_scan_kpt(float* o_out, float* state, const void* q, int ld_q, const v
 // the price of more instructions per state entry and a longer exchange within the lane group; a launch
 // that fills the GPU anyway (a batch of decoding rows, rows cut into segments) keeps 16 channels a thread.
 // The order of a sum over key channels follows the choice, so results differ between launches by rounding.
-template <typename TIn, typename TZ, bool DELTA, typename... Args>
+template <typename TIn, typename TZ, int RULE, typename... Args>
 int launch_scan(int num_rows, int H, int dk, int dv, Args... args) {
   const long long threads16 = (long long)num_rows * H * dv * ((dk + 15) / 16);  // at 16 channels a thread
   const int sm_count = scan_sm_count();
-  if (dk <= 32 * 4 && threads16 * 4 <= 128LL * sm_count) return launch_scan_kpt<TIn, TZ, DELTA, 4>(args...);
-  if (dk <= 32 * 8 && threads16 * 2 <= 128LL * sm_count) return launch_scan_kpt<TIn, TZ, DELTA, 8>(args...);
-  return launch_scan_kpt<TIn, TZ, DELTA, 16>(args...);
+  if (dk <= 32 * 4 && threads16 * 4 <= 128LL * sm_count) return launch_scan_kpt<TIn, TZ, RULE, 4>(args...);
+  if (dk <= 32 * 8 && threads16 * 2 <= 128LL * sm_count) return launch_scan_kpt<TIn, TZ, RULE, 8>(args...);
+  return launch_scan_kpt<TIn, TZ, RULE, 16>(args...);
 }
 
 }  // namespace ms
@@ -545,38 +566,42 @@ MS_DEFINE_LAST_ERROR(ms_recurrence_last_error)
 MS_DEFINE_PDL_SWITCH(ms_recurrence_set_pdl)
 
 
-// in_dtype: of q, k, v; z_dtype: of z and beta. delta: 0 decay rule, 1 delta rule. z_is_decay: z and beta are
+// in_dtype: of q, k, v; z_dtype: of z and beta. rule: 0 decay rule, 1 delta rule, 2 bonus rule (bonus [H, dk] float32; decays per channel). z_is_decay: z and beta are
 // float32 and hold the decays and sigmoid(beta) themselves (ms_decay_from_logits), not their logits. dv_in: the value channels of a head
 // in v; dv - 1 of them: the state has one more column, whose value is one (the decayed sum of the keys).
 MS_EXPORT int ms_decay_scan(float* o_out, float* state, const void* q, int ld_q, const void* k, int ld_k, int qk_group,
                             const void* v, int ld_v, const void* z, int ld_z, const float* z_bias, const float* decay_coef,
                             float z_sign, int z_is_decay, const void* beta, int ld_beta, const int* cu_q, const int* q_start,
-                            const int* state_slot, int num_rows, int H, int dk, int dv, float q_scale, int delta, int in_dtype,
-                            int z_dtype, int decay_per_head, const float* v_scale, int dv_in, cudaStream_t stream) {
+                            const int* state_slot, int num_rows, int H, int dk, int dv, float q_scale, int rule, int in_dtype,
+                            int z_dtype, int decay_per_head, const float* v_scale, int dv_in, const float* bonus, cudaStream_t stream) {
   if (num_rows == 0) return 0;
   MS_CHECK_ARG(H > 0 && dk > 0 && dv > 0 && dk <= 32 * SCAN_MAX_KPT, "decay_scan: key size %d is outside 1..%d", dk, 32 * SCAN_MAX_KPT);
   MS_CHECK_ARG(qk_group > 0 && H % qk_group == 0, "decay_scan: %d heads are not a multiple of the group of %d", H, qk_group);
-  MS_CHECK_ARG(!delta || beta != nullptr, "decay_scan: the delta rule needs beta");
-  MS_CHECK_ARG(dv_in == dv || (dv_in == dv - 1 && !delta), "decay_scan: %d value columns of which %d are read", dv, dv_in);
+  MS_CHECK_ARG(rule != RULE_DELTA || beta != nullptr, "decay_scan: the delta rule needs beta");
+  MS_CHECK_ARG(rule >= 0 && rule <= 2 && (rule == RULE_BONUS) == (bonus != nullptr) && !(rule == RULE_BONUS && decay_per_head),
+               "decay_scan: rule %d with%s a bonus", rule, bonus ? "" : "out");
+  MS_CHECK_ARG(dv_in == dv || (dv_in == dv - 1 && rule == RULE_DECAY), "decay_scan: %d value columns of which %d are read", dv, dv_in);
   MS_CHECK_ARG(!z_is_decay || z_dtype == MS_F32, "decay_scan: decays worked out beforehand are float32");
 #define MS_SCAN(TIN, TZZ, D)                                                                                                  \
   return launch_scan<TIN, TZZ, D>(num_rows, H, dk, dv, o_out, state, q, ld_q, k, ld_k, qk_group, v, ld_v, z, ld_z, z_bias, decay_coef, z_sign, z_is_decay, \
-                                  beta, ld_beta, cu_q, q_start, state_slot, num_rows, H, dk, dv, q_scale, decay_per_head ? 1 : dk, v_scale, dv_in, stream)
+                                  beta, ld_beta, cu_q, q_start, state_slot, num_rows, H, dk, dv, q_scale, decay_per_head ? 1 : dk, v_scale, dv_in, bonus, stream)
   if (in_dtype == MS_F32 && z_dtype == MS_F32) {
-    if (delta) MS_SCAN(float, float, true);
-    MS_SCAN(float, float, false);
+    if (rule == RULE_DELTA) MS_SCAN(float, float, RULE_DELTA);
+    if (rule == RULE_BONUS) MS_SCAN(float, float, RULE_BONUS);
+    MS_SCAN(float, float, RULE_DECAY);
   }
   if (in_dtype == MS_F32 && z_dtype == MS_BF16) {
-    if (delta) MS_SCAN(float, __nv_bfloat16, true);
-    MS_SCAN(float, __nv_bfloat16, false);
+    if (rule == RULE_DELTA) MS_SCAN(float, __nv_bfloat16, RULE_DELTA);
+    if (rule == RULE_DECAY) MS_SCAN(float, __nv_bfloat16, RULE_DECAY);
   }
   if (in_dtype == MS_BF16 && z_dtype == MS_F32) {
-    if (delta) MS_SCAN(__nv_bfloat16, float, true);
-    MS_SCAN(__nv_bfloat16, float, false);
+    if (rule == RULE_DELTA) MS_SCAN(__nv_bfloat16, float, RULE_DELTA);
+    if (rule == RULE_BONUS) MS_SCAN(__nv_bfloat16, float, RULE_BONUS);
+    MS_SCAN(__nv_bfloat16, float, RULE_DECAY);
   }
   if (in_dtype == MS_BF16 && z_dtype == MS_BF16) {
-    if (delta) MS_SCAN(__nv_bfloat16, __nv_bfloat16, true);
-    MS_SCAN(__nv_bfloat16, __nv_bfloat16, false);
+    if (rule == RULE_DELTA) MS_SCAN(__nv_bfloat16, __nv_bfloat16, RULE_DELTA);
+    if (rule == RULE_DECAY) MS_SCAN(__nv_bfloat16, __nv_bfloat16, RULE_DECAY);
   }
 #undef MS_SCAN
   return ms::fail("decay_scan: unsupported dtypes (%d, %d)", in_dtype, z_dtype);
@@ -633,7 +658,7 @@ MS_EXPORT int ms_segment_setup(int* seg_cu, int* seg_zero, int* seg_slot, const 
 MS_EXPORT int ms_segment_finish(float* o, float* state, const float* ends, float* before, float* c, const float* decay, int ld_decay,
                                 const void* q, int ld_q, int qk_group, const int* seg_cu, const int* q_start, const int* state_slot,
                                 int num_rows, int num_tokens, int P, int H, int dk, int dv, float q_scale, int in_dtype,
-                                int decay_per_head, cudaStream_t stream) {
+                                int decay_per_head, int before_decay, cudaStream_t stream) {
   if (num_rows == 0) return 0;
   const int dkz = decay_per_head ? 1 : dk;
   const int segments = num_rows * P, width = H * dkz;
@@ -655,10 +680,10 @@ MS_EXPORT int ms_segment_finish(float* o, float* state, const float* ends, float
   const dim3 grid(segments, H, (longest + FIX_RUN - 1) / FIX_RUN);
   if (in_dtype == MS_F32)
     MS_LAUNCH(segment_fixup_kernel<float>, grid, FIX_THREADS, smem, stream, o, (const float*)q, ld_q, qk_group, c, before, seg_cu, q_start,
-              P, H, dk, dv, cols, q_scale, dkz);
+              P, H, dk, dv, cols, q_scale, dkz, before_decay);
   else
     MS_LAUNCH(segment_fixup_kernel<__nv_bfloat16>, grid, FIX_THREADS, smem, stream, o, (const __nv_bfloat16*)q, ld_q, qk_group, c, before,
-              seg_cu, q_start, P, H, dk, dv, cols, q_scale, dkz);
+              seg_cu, q_start, P, H, dk, dv, cols, q_scale, dkz, before_decay);
   return 0;
 }
 
@@ -697,7 +722,7 @@ MS_EXPORT int ms_conv_state_update(void* conv_state, const void* proj, int ld, c
 }
 
 MS_EXPORT int ms_head_norm_gate(void* out, int ld_out, const float* o, const float* w, const void* gate, int ld_gate,
-                                int num_tokens, int H, int dv, float eps, float scale, int gate_kind, int dtype,
+                                int num_tokens, int H, int dv, float eps, float scale, int gate_kind, int w_stride, int dtype,
                                 cudaStream_t stream) {
   if (num_tokens == 0) return 0;
   const long long items = (long long)num_tokens * H;
@@ -705,10 +730,10 @@ MS_EXPORT int ms_head_norm_gate(void* out, int ld_out, const float* o, const flo
   const unsigned blocks = (unsigned)((items + warps - 1) / warps);
   if (dtype == MS_F32)
     MS_LAUNCH(head_norm_gate_kernel<float>, blocks, warps * 32, 0, stream, (float*)out, ld_out, o, w, (const float*)gate, ld_gate,
-              num_tokens, H, dv, eps, scale, gate_kind);
+              num_tokens, H, dv, eps, scale, gate_kind, w_stride);
   else
     MS_LAUNCH(head_norm_gate_kernel<__nv_bfloat16>, blocks, warps * 32, 0, stream, (__nv_bfloat16*)out, ld_out, o, w,
-              (const __nv_bfloat16*)gate, ld_gate, num_tokens, H, dv, eps, scale, gate_kind);
+              (const __nv_bfloat16*)gate, ld_gate, num_tokens, H, dv, eps, scale, gate_kind, w_stride);
   return 0;
 }
 

@@ -2,7 +2,7 @@
 // (token, choice) pairs by expert, the experts' products over those sorted rows, and the weighted sum.
 //
 //   z = W_r h (float32), s = softmax(z) over all router outputs; choice score c = s + correction.
-//   Router outputs form `group_count` equal groups of neighbours; a group's score is its largest c; only outputs of
+//   Router outputs form `group_count` equal groups of neighbours; a group's score is the sum of its `group_best` largest c; only outputs of
 //   the `group_keep` best groups can be chosen. The `top` largest c among those are the token's choices; the weight of
 //   a choice is s (without the correction) times a constant, optionally divided by the sum of the chosen s.
 //   Router outputs E .. R-1 are identity experts: their output is h itself. Expert e < E: W_down[e] (act(W_gate[e] h) * (W_up[e] h)),
@@ -30,7 +30,8 @@ __global__ void __launch_bounds__(ROUTE_THREADS)
 expert_route_kernel(int* __restrict__ idx_out, float* __restrict__ wgt_out, const T* __restrict__ x, int ld_x,
                     const float* __restrict__ router, const float* __restrict__ correction, int K, int R, int top, int group_count,
                     int group_keep, float weight_scale, int renormalize, const float* __restrict__ logit_bias,
-                    const float* __restrict__ gate_w, float* __restrict__ gate_out, int sigmoid_scores, int square_weights) {
+                    const float* __restrict__ gate_w, float* __restrict__ gate_out, int sigmoid_scores, int square_weights, int group_best,
+                    float renorm_eps) {
   extern __shared__ float route_smem[];
   float* xs = route_smem;      // [K]
   float* s = xs + K;           // [R] logits, then scores
@@ -80,9 +81,24 @@ expert_route_kernel(int* __restrict__ idx_out, float* __restrict__ wgt_out, cons
   if (group_count > 1) {
     const int per = R / group_count;
     for (int g = lane; g < group_count; g += 32) {
-      float best = -INFINITY;
-      for (int j = 0; j < per; ++j) best = fmaxf(best, choice[g * per + j]);
-      gs[g] = best;
+      // the group_best largest, one after the other: the next one is the largest of those behind (value, then index) the last
+      float sum = 0.f, last = INFINITY;
+      int last_j = -1;
+      for (int b = 0; b < group_best; ++b) {
+        float best = -INFINITY;
+        int best_j = -1;
+        for (int j = 0; j < per; ++j) {
+          const float c = choice[g * per + j];
+          if ((c < last || (c == last && j > last_j)) && (best_j < 0 || c > best)) {
+            best = c;
+            best_j = j;
+          }
+        }
+        sum += best;
+        last = best;
+        last_j = best_j;
+      }
+      gs[g] = sum;
       kept[g] = 0.f;
     }
     __syncwarp();
@@ -138,7 +154,7 @@ expert_route_kernel(int* __restrict__ idx_out, float* __restrict__ wgt_out, cons
     __syncwarp();
   }
   if (lane == 0) {
-    const float f = renormalize ? weight_scale / total : weight_scale;
+    const float f = renormalize ? weight_scale / (total + renorm_eps) : weight_scale;
     for (int r = 0; r < top; ++r) {
       const float w = wgt_out[(size_t)t * top + r] * f;
       wgt_out[(size_t)t * top + r] = square_weights ? w * w : w;
@@ -195,13 +211,29 @@ expert_plan_kernel(int* __restrict__ pos, int* __restrict__ perm, int* __restric
   }
 }
 
-// act 0: SiLU, 1: the tanh form of GELU, 2: the square of relu
+// act 0: SiLU, 1: the tanh form of GELU, 2: the square of relu; 3 (with a gate only): g sigmoid(alpha g) (u + shift) with g capped at
+// limit and u held within +-limit (a negative limit: neither)
+struct ExpertAct {
+  int act;
+  float limit, alpha, shift;
+};
 __device__ __forceinline__ float act_of(float g, int act) {
   if (act == 2) {
     g = fmaxf(g, 0.f);
     return g * g;
   }
   return act == 0 ? g / (1.0f + expf(-g)) : 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+}
+
+__device__ __forceinline__ float gated_of(float g, float u, const ExpertAct& a) {
+  if (a.act == 3) {
+    if (a.limit >= 0.f) {
+      g = fminf(g, a.limit);
+      u = fminf(fmaxf(u, -a.limit), a.limit);
+    }
+    return g / (1.0f + expf(-a.alpha * g)) * (u + a.shift);
+  }
+  return act_of(g, a.act) * u;
 }
 
 // ---------------------------------------------------------------- the experts' products, float32 arithmetic
@@ -216,7 +248,7 @@ template <typename T, int MODE>
 __global__ void __launch_bounds__(XG_THREADS)
 expert_gemm_kernel(void* __restrict__ out_, const T* __restrict__ A, int lda, const int* __restrict__ perm, int top,
                    const T* __restrict__ W, const int* __restrict__ tiles, const int* __restrict__ meta,
-                   const int* __restrict__ offsets, int N, int K, int act) {
+                   const int* __restrict__ offsets, int N, int K, const ExpertAct act) {
   constexpr bool GATED = MODE == XG_GATED;
   __shared__ float As[XG_BK][XG_BM + 4];
   __shared__ float Bg[XG_BK][XG_BN + 4];
@@ -270,8 +302,8 @@ expert_gemm_kernel(void* __restrict__ out_, const T* __restrict__ A, int lda, co
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
-      if (GATED) Elem<T>::store((T*)out_ + (size_t)(row0 + r) * N + n, act_of(acc[i][j], act) * acu[i][j]);
-      else if (MODE == XG_ACT) Elem<T>::store((T*)out_ + (size_t)(row0 + r) * N + n, act_of(acc[i][j], act));
+      if (GATED) Elem<T>::store((T*)out_ + (size_t)(row0 + r) * N + n, gated_of(acc[i][j], acu[i][j], act));
+      else if (MODE == XG_ACT) Elem<T>::store((T*)out_ + (size_t)(row0 + r) * N + n, act_of(acc[i][j], act.act));
       else ((float*)out_)[(size_t)(row0 + r) * N + n] = acc[i][j];
     }
   }
@@ -302,7 +334,7 @@ template <int MODE>
 __global__ void __launch_bounds__(XM_THREADS)
 expert_gemm_mma_kernel(void* __restrict__ out_, const __nv_bfloat16* __restrict__ A, int lda, const int* __restrict__ perm, int top,
                        const __nv_bfloat16* __restrict__ W, const int* __restrict__ tiles, const int* __restrict__ meta,
-                       const int* __restrict__ offsets, int N, int K, int act) {
+                       const int* __restrict__ offsets, int N, int K, const ExpertAct act) {
   constexpr bool GATED = MODE == XG_GATED;
   __shared__ __align__(16) __nv_bfloat16 As[2][XM_BM][XM_LD];
   __shared__ __align__(16) __nv_bfloat16 Bg[2][XM_BN][XM_LD];
@@ -396,9 +428,9 @@ expert_gemm_mma_kernel(void* __restrict__ out_, const __nv_bfloat16* __restrict_
           const float v = acc[mi][ni][half * 2 + j];
           if (GATED)
             ((__nv_bfloat16*)out_)[(size_t)(row0 + r) * N + n + j] =
-                __float2bfloat16_rn(act_of(v, act) * acu[GATED ? mi : 0][GATED ? ni : 0][half * 2 + j]);
+                __float2bfloat16_rn(gated_of(v, acu[GATED ? mi : 0][GATED ? ni : 0][half * 2 + j], act));
           else if (MODE == XG_ACT)
-            ((__nv_bfloat16*)out_)[(size_t)(row0 + r) * N + n + j] = __float2bfloat16_rn(act_of(v, act));
+            ((__nv_bfloat16*)out_)[(size_t)(row0 + r) * N + n + j] = __float2bfloat16_rn(act_of(v, act.act));
           else
             ((float*)out_)[(size_t)(row0 + r) * N + n + j] = v;
         }
@@ -439,23 +471,26 @@ MS_DEFINE_PDL_SWITCH(ms_experts_set_pdl)
 MS_EXPORT int ms_expert_route(int* idx, float* wgt, const void* x, int ld_x, const float* router, const float* correction, int tokens,
                               int K, int R, int top, int group_count, int group_keep, float weight_scale, int renormalize, int dtype,
                               cudaStream_t stream, const float* logit_bias, const float* gate_w, float* gate_out, int sigmoid_scores,
-                              int square_weights) {
+                              int square_weights, int group_best, float renorm_eps) {
   if (tokens == 0) return 0;
   MS_CHECK_ARG(R >= 1 && top >= 1 && top <= R && K >= 1, "expert_route: top %d of %d router outputs", top, R);
   MS_CHECK_ARG(group_count >= 1 && R % group_count == 0 && group_keep >= 1 && group_keep <= group_count &&
                    group_keep * (R / group_count) >= top,
                "expert_route: %d router outputs in %d groups of which %d are kept cannot give %d choices", R, group_count, group_keep, top);
+  MS_CHECK_ARG(group_best >= 1 && (group_count == 1 || group_best <= R / group_count), "expert_route: a group of %d has no %d largest",
+               R / group_count, group_best);
   const size_t smem = ((size_t)K + 2 * (size_t)R + 2 * (size_t)group_count) * sizeof(float);
   MS_CHECK_ARG(smem <= 200 * 1024, "expert_route: %d inputs and %d outputs need %zu bytes of shared memory", K, R, smem);
   if (dtype == MS_F32) {
     if (smem > 48 * 1024) MS_CHECK_CUDA(cudaFuncSetAttribute(expert_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     MS_LAUNCH(expert_route_kernel<float>, tokens, ROUTE_THREADS, smem, stream, idx, wgt, (const float*)x, ld_x, router, correction, K, R, top,
-              group_count, group_keep, weight_scale, renormalize, logit_bias, gate_w, gate_out, sigmoid_scores, square_weights);
+              group_count, group_keep, weight_scale, renormalize, logit_bias, gate_w, gate_out, sigmoid_scores, square_weights, group_best, renorm_eps);
   } else {
     if (smem > 48 * 1024)
       MS_CHECK_CUDA(cudaFuncSetAttribute(expert_route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     MS_LAUNCH(expert_route_kernel<__nv_bfloat16>, tokens, ROUTE_THREADS, smem, stream, idx, wgt, (const __nv_bfloat16*)x, ld_x, router,
-              correction, K, R, top, group_count, group_keep, weight_scale, renormalize, logit_bias, gate_w, gate_out, sigmoid_scores, square_weights);
+              correction, K, R, top, group_count, group_keep, weight_scale, renormalize, logit_bias, gate_w, gate_out, sigmoid_scores, square_weights,
+              group_best, renorm_eps);
   }
   return 0;
 }
@@ -513,9 +548,12 @@ MS_EXPORT int ms_expert_gather(void* xs, const void* x, int ld_x, const int* per
 // [slots, N] in the run's dtype = act(x W^T), gathered likewise; mode 0: out [slots, N] float32 = A W^T (A [slots, K] in sorted
 // order; perm null).
 MS_EXPORT int ms_expert_gemm(void* out, const void* A, int lda, const int* perm, int top, const void* W, const int* tiles, const int* meta,
-                             const int* offsets, int max_tiles, int N, int K, int mode, int act, int dtype, cudaStream_t stream) {
+                             const int* offsets, int max_tiles, int N, int K, int mode, int act_kind, float limit, float alpha, float shift,
+                             int dtype, cudaStream_t stream) {
   if (max_tiles == 0 || N == 0) return 0;
-  MS_CHECK_ARG(K >= 1 && top >= 1 && act >= 0 && act <= 2 && mode >= 0 && mode <= 2, "expert_gemm: K=%d top=%d act=%d mode=%d", K, top, act, mode);
+  MS_CHECK_ARG(K >= 1 && top >= 1 && act_kind >= 0 && act_kind <= 3 && mode >= 0 && mode <= 2 && (act_kind != 3 || mode == XG_GATED),
+               "expert_gemm: K=%d top=%d act=%d mode=%d", K, top, act_kind, mode);
+  const ExpertAct act{act_kind, limit, alpha, shift};
   const dim3 grid(max_tiles, (N + XG_BN - 1) / XG_BN);
 #define MS_XG(T, M) \
   MS_LAUNCH((expert_gemm_kernel<T, M>), grid, XG_THREADS, 0, stream, out, (const T*)A, lda, perm, top, (const T*)W, tiles, meta, offsets, N, K, act)

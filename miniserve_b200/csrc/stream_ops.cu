@@ -1,11 +1,13 @@
 // Kernels at the two ends of the residual stream's layers that go beyond one table and one norm:
 //
-//   * an embedding that is a sum: the token's row, a row of a second table chosen by a hash of the previous and the
+//   * an embedding that is a sum: the token's row (times a constant), a row of a second table chosen by a hash of the previous and the
 //     current token (a bigram table; a sequence's first token takes the table's last row), and a sinusoidal vector of
 //     the position. The token before a portion's first one comes from the request's state slot (int32), which the CTA of
 //     that first token, the only one that reads it, leaves holding the portion's last token;
 //   * RMS norm of the stream after an addend that is normed itself: h = residual + norm_b(delta), out = norm(h). Either
-//     norm's weight is a vector or one number for all coordinates.
+//     norm's weight is a vector or one number for all coordinates;
+//   * several residual streams (hyper-connections): a sublayer's output y changes all streams at once, x_t <- sum_s mix[s, t] x_s +
+//     out[t] y, and the next sublayer reads the norm of sum_s in[s] x_s: both in one pass over the streams.
 //
 // Angles, statistics, norms and the sums are float32; each output is rounded once.
 #include "common.cuh"
@@ -44,7 +46,7 @@ template <typename T>
 __global__ void embed_sum_kernel(float* __restrict__ residual, const T* __restrict__ table, PairTable pt, const float* __restrict__ inv_freq,
                                  const int* __restrict__ ids, const int* __restrict__ positions, const int* __restrict__ row_of_token,
                                  const int* __restrict__ cu_q, const int* __restrict__ state_slot, int* __restrict__ prev_token,
-                                 int hidden, int vocab) {
+                                 int hidden, int vocab, float scale) {
   pdl_prologue();
   const int t = blockIdx.x;
   int id = ids[t];
@@ -58,11 +60,11 @@ __global__ void embed_sum_kernel(float* __restrict__ residual, const T* __restri
     float sn = 0.f, cs = 0.f;
     if (inv_freq) sincosf(pos * inv_freq[i], &sn, &cs);
     const int c = 2 * i;
-    float a = Elem<T>::load(src + c);
+    float a = Elem<T>::load(src + c) * scale;
     if (pair) a += Elem<T>::load(pair + c);
     dst[c] = a + sn;
     if (c + 1 < hidden) {
-      float b = Elem<T>::load(src + c + 1);
+      float b = Elem<T>::load(src + c + 1) * scale;
       if (pair) b += Elem<T>::load(pair + c + 1);
       dst[c + 1] = b + cs;
     }
@@ -73,7 +75,7 @@ __global__ void embed_sum_kernel(float* __restrict__ residual, const T* __restri
 __global__ void embed_sum_bf16x8_kernel(float* __restrict__ residual, const __nv_bfloat16* __restrict__ table, PairTable pt,
                                         const float* __restrict__ inv_freq, const int* __restrict__ ids, const int* __restrict__ positions,
                                         const int* __restrict__ row_of_token, const int* __restrict__ cu_q,
-                                        const int* __restrict__ state_slot, int* __restrict__ prev_token, int hidden, int vocab) {
+                                        const int* __restrict__ state_slot, int* __restrict__ prev_token, int hidden, int vocab, float scale) {
   pdl_prologue();
   const int t = blockIdx.x;
   int id = ids[t];
@@ -86,6 +88,8 @@ __global__ void embed_sum_bf16x8_kernel(float* __restrict__ residual, const __nv
   for (int c = threadIdx.x; c < hidden >> 3; c += blockDim.x) {
     float v[8];
     bf16x8_to_float(src[c], v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] *= scale;
     if (pair) {
       float p[8];
       bf16x8_to_float(pair[c], p);
@@ -217,14 +221,136 @@ add_normed_rmsnorm_bf16x8_kernel(__nv_bfloat16* __restrict__ out, float* __restr
   *reinterpret_cast<uint4*>(out + (size_t)i * hidden + c) = float_to_bf16x8(y);
 }
 
+// ---------------------------------------------------------------- several residual streams
+// What a sublayer's output does to the streams: mix [S, S] (from, to) and out [S], float32 (null: nothing, the streams stay); and what
+// the next sublayer reads: into [S] (null: the sum of the streams).
+struct StreamLinks {
+  const float* mix;
+  const float* out;
+  const float* into;
+};
+
+constexpr int HC_MAX_STREAMS = 16;
+
+// src [T, src_streams, hidden] (one stream: all streams are equal to it), dst [T, S, hidden] (may be src). With y: the new streams go to
+// dst unless rows are gathered. out[i] = rmsnorm(sum_s into[s] x_s) * w over the new streams. One CTA per row.
+template <typename T, int THREADS>
+__global__ void __launch_bounds__(THREADS)
+stream_norm_kernel(T* __restrict__ out, float* dst, const float* src, int src_streams, int S, const T* __restrict__ y, StreamLinks links,
+                   const float* __restrict__ w, float eps, const int* __restrict__ rows, int hidden, int write) {
+  extern __shared__ float row_u[];  // hidden floats
+  __shared__ float red[32];
+  pdl_prologue();
+  const int i = blockIdx.x;
+  const int r = rows ? rows[i] : i;
+  const float* xs = src + (size_t)r * src_streams * hidden;
+  float* xd = dst + (size_t)r * S * hidden;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < hidden; c += THREADS) {
+    float x[HC_MAX_STREAMS];
+    for (int s = 0; s < S; ++s) x[s] = xs[(size_t)(src_streams == 1 ? 0 : s) * hidden + c];
+    float u = 0.f;
+    if (y) {
+      const float d = Elem<T>::load(y + (size_t)r * hidden + c);
+      for (int t = 0; t < S; ++t) {
+        float n = links.out[t] * d;
+        for (int s = 0; s < S; ++s) n = fmaf(links.mix[s * S + t], x[s], n);
+        if (write) xd[(size_t)t * hidden + c] = n;
+        u = fmaf(links.into ? links.into[t] : 1.f, n, u);
+      }
+    } else {
+      for (int s = 0; s < S; ++s) u = fmaf(links.into ? links.into[s] : 1.f, x[s], u);
+    }
+    row_u[c] = u;
+    ss += u * u;
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)hidden + eps);
+  for (int c = threadIdx.x; c < hidden; c += THREADS) Elem<T>::store(out + (size_t)i * hidden + c, (row_u[c] * inv) * w[c]);
+}
+
+// bfloat16 rows that are a multiple of 8 wide and at most 8 * THREADS, up to four streams: eight elements of every stream per thread, in
+// registers from the read to the norm
+template <int THREADS, int S>
+__global__ void __launch_bounds__(THREADS)
+stream_norm_bf16x8_kernel(__nv_bfloat16* __restrict__ out, float* dst, const float* src, int src_streams, const __nv_bfloat16* __restrict__ y,
+                          StreamLinks links, const float* __restrict__ w, float eps, const int* __restrict__ rows, int hidden, int write) {
+  __shared__ float red[32];
+  // (weights: none of an earlier kernel's output)
+  float mix[S][S], into[S], outw[S];
+#pragma unroll
+  for (int s = 0; s < S; ++s) {
+    into[s] = links.into ? links.into[s] : 1.f;
+    outw[s] = y ? links.out[s] : 0.f;
+#pragma unroll
+    for (int t = 0; t < S; ++t) mix[s][t] = y ? links.mix[s * S + t] : 0.f;
+  }
+  pdl_prologue();
+  const int i = blockIdx.x;
+  const int r = rows ? rows[i] : i;
+  const int c = threadIdx.x * 8;
+  const bool mine = c < hidden;
+  float x[S][8], u[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  if (mine) {
+    const float* xs = src + (size_t)r * src_streams * hidden + c;
+    float d[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int s = 0; s < S; ++s) {
+      if (s > 0 && src_streams == 1) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[s][e] = x[0][e];
+      } else {
+        const float4 a = *reinterpret_cast<const float4*>(xs + (size_t)s * hidden), b = *reinterpret_cast<const float4*>(xs + (size_t)s * hidden + 4);
+        x[s][0] = a.x; x[s][1] = a.y; x[s][2] = a.z; x[s][3] = a.w; x[s][4] = b.x; x[s][5] = b.y; x[s][6] = b.z; x[s][7] = b.w;
+      }
+    }
+    if (y) {
+      bf16x8_to_float(*reinterpret_cast<const uint4*>(y + (size_t)r * hidden + c), d);
+      float* xd = dst + (size_t)r * S * hidden + c;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        float n[S];
+#pragma unroll
+        for (int t = 0; t < S; ++t) {
+          n[t] = outw[t] * d[e];
+#pragma unroll
+          for (int s = 0; s < S; ++s) n[t] = fmaf(mix[s][t], x[s][e], n[t]);
+        }
+#pragma unroll
+        for (int t = 0; t < S; ++t) x[t][e] = n[t];
+      }
+      if (write) {
+#pragma unroll
+        for (int t = 0; t < S; ++t) {
+          *reinterpret_cast<float4*>(xd + (size_t)t * hidden) = make_float4(x[t][0], x[t][1], x[t][2], x[t][3]);
+          *reinterpret_cast<float4*>(xd + (size_t)t * hidden + 4) = make_float4(x[t][4], x[t][5], x[t][6], x[t][7]);
+        }
+      }
+    }
+#pragma unroll
+    for (int s = 0; s < S; ++s)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) u[e] = fmaf(into[s], x[s][e], u[e]);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < 8; ++e) ss += u[e] * u[e];
+  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)hidden + eps);
+  if (!mine) return;
+  const float4 wa = *reinterpret_cast<const float4*>(w + c), wb = *reinterpret_cast<const float4*>(w + c + 4);
+  const float wv[8] = {wa.x, wa.y, wa.z, wa.w, wb.x, wb.y, wb.z, wb.w};
+#pragma unroll
+  for (int e = 0; e < 8; ++e) u[e] = (u[e] * inv) * wv[e];
+  *reinterpret_cast<uint4*>(out + (size_t)i * hidden + c) = float_to_bf16x8(u);
+}
+
 }  // namespace ms
 
 using namespace ms;
 
-// residual [T, hidden] float32. pair_table null: no second table (the arguments about rows and slots are not read then).
+// residual [T, hidden] float32; the table's rows count times `scale`. pair_table null: no second table (the arguments about rows and slots are not read then).
 MS_EXPORT int ms_embed_sum(float* residual, const void* table, const void* pair_table, long long buckets, long long mul_prev,
                            long long mul_cur, const float* inv_freq, const int* ids, const int* positions, const int* row_of_token,
-                           const int* cu_q, const int* state_slot, int* prev_token, int tokens, int hidden, int vocab, int dtype,
+                           const int* cu_q, const int* state_slot, int* prev_token, int tokens, int hidden, int vocab, float scale, int dtype,
                            cudaStream_t stream) {
   if (tokens == 0) return 0;
   MS_CHECK_ARG(hidden > 0 && vocab > 0, "embed_sum: hidden=%d vocab=%d", hidden, vocab);
@@ -232,14 +358,14 @@ MS_EXPORT int ms_embed_sum(float* residual, const void* table, const void* pair_
   const PairTable pt{pair_table, buckets, mul_prev, mul_cur};
   if (dtype == MS_F32) {
     MS_LAUNCH(embed_sum_kernel<float>, tokens, hidden >= 1024 ? 256 : 128, 0, stream, residual, (const float*)table, pt, inv_freq, ids, positions,
-              row_of_token, cu_q, state_slot, prev_token, hidden, vocab);
+              row_of_token, cu_q, state_slot, prev_token, hidden, vocab, scale);
   } else if (hidden % 8 == 0 && ((uintptr_t)table % 16 == 0) && ((uintptr_t)pair_table % 16 == 0) && ((uintptr_t)inv_freq % 16 == 0) &&
              ((uintptr_t)residual % 16 == 0)) {
     MS_LAUNCH(embed_sum_bf16x8_kernel, tokens, hidden >= 1024 ? 128 : 64, 0, stream, residual, (const __nv_bfloat16*)table, pt, inv_freq, ids,
-              positions, row_of_token, cu_q, state_slot, prev_token, hidden, vocab);
+              positions, row_of_token, cu_q, state_slot, prev_token, hidden, vocab, scale);
   } else {
     MS_LAUNCH(embed_sum_kernel<__nv_bfloat16>, tokens, hidden >= 1024 ? 256 : 128, 0, stream, residual, (const __nv_bfloat16*)table, pt,
-              inv_freq, ids, positions, row_of_token, cu_q, state_slot, prev_token, hidden, vocab);
+              inv_freq, ids, positions, row_of_token, cu_q, state_slot, prev_token, hidden, vocab, scale);
   }
   return 0;
 }
@@ -270,5 +396,45 @@ MS_EXPORT int ms_add_normed_rmsnorm(void* out, float* residual, const void* delt
   else
     MS_LAUNCH((add_normed_rmsnorm_kernel<__nv_bfloat16, 256>), n, 256, smem, stream, (__nv_bfloat16*)out, residual,
               (const __nv_bfloat16*)delta, nb, nn, rows, hidden, write_residual);
+  return 0;
+}
+
+// dst [T, S, hidden] float32, src [T, src_streams, hidden] (src_streams 1 or S; dst may be src where it is S). y null: the streams stay as
+// they are and nothing is written to dst. rows: only those rows' norms, without writing the streams.
+MS_EXPORT int ms_stream_norm(void* out, float* dst, const float* src, int src_streams, int streams, const void* y, const float* mix,
+                             const float* out_w, const float* into, const float* w, float eps, const int* rows, int n, int hidden, int write,
+                             int dtype, cudaStream_t stream) {
+  if (n == 0) return 0;
+  MS_CHECK_ARG(hidden > 0 && streams >= 1 && streams <= HC_MAX_STREAMS && (src_streams == 1 || src_streams == streams),
+               "stream_norm: %d streams (%d stored) of %d; at most %d are taken", streams, src_streams, hidden, HC_MAX_STREAMS);
+  MS_CHECK_ARG(!y || (mix && out_w), "stream_norm: a sublayer's output needs the weights that it enters the streams with");
+  MS_CHECK_ARG(!(y && write) || (dst && (dst != src || src_streams == streams)), "stream_norm: nowhere to write %d streams", streams);
+  const StreamLinks links{mix, out_w, into};
+  if (dtype == MS_BF16 && hidden % 8 == 0 && hidden <= 8192 && streams <= 4 && (uintptr_t)out % 16 == 0 && (uintptr_t)src % 16 == 0 &&
+      (uintptr_t)dst % 16 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)w % 16 == 0) {
+    __nv_bfloat16* o = (__nv_bfloat16*)out;
+    const __nv_bfloat16* d = (const __nv_bfloat16*)y;
+#define MS_STREAM_NORM(TH)                                                                                                               \
+  do {                                                                                                                                   \
+    if (streams == 1) MS_LAUNCH((stream_norm_bf16x8_kernel<TH, 1>), n, TH, 0, stream, o, dst, src, src_streams, d, links, w, eps, rows, hidden, write);      \
+    else if (streams == 2) MS_LAUNCH((stream_norm_bf16x8_kernel<TH, 2>), n, TH, 0, stream, o, dst, src, src_streams, d, links, w, eps, rows, hidden, write); \
+    else if (streams == 3) MS_LAUNCH((stream_norm_bf16x8_kernel<TH, 3>), n, TH, 0, stream, o, dst, src, src_streams, d, links, w, eps, rows, hidden, write); \
+    else MS_LAUNCH((stream_norm_bf16x8_kernel<TH, 4>), n, TH, 0, stream, o, dst, src, src_streams, d, links, w, eps, rows, hidden, write); \
+  } while (0)
+    if (hidden <= 1024) MS_STREAM_NORM(128);
+    else if (hidden <= 2048) MS_STREAM_NORM(256);
+    else if (hidden <= 4096) MS_STREAM_NORM(512);
+    else MS_STREAM_NORM(1024);
+#undef MS_STREAM_NORM
+    return 0;
+  }
+  const size_t smem = (size_t)hidden * sizeof(float);
+  MS_CHECK_ARG(smem <= 48 * 1024, "stream_norm: rows of %d do not fit shared memory", hidden);
+  if (dtype == MS_F32)
+    MS_LAUNCH((stream_norm_kernel<float, 256>), n, 256, smem, stream, (float*)out, dst, src, src_streams, streams, (const float*)y, links, w, eps,
+              rows, hidden, write);
+  else
+    MS_LAUNCH((stream_norm_kernel<__nv_bfloat16, 256>), n, 256, smem, stream, (__nv_bfloat16*)out, dst, src, src_streams, streams,
+              (const __nv_bfloat16*)y, links, w, eps, rows, hidden, write);
   return 0;
 }

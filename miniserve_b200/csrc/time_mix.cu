@@ -1,0 +1,637 @@
+// Time mixing with a decay per key channel and token and a bonus for the token's own write (RWKV-style):
+//
+//   o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t,   S_t = diag(d_t) S_(t-1) + k_t v_t^T,   d_t = exp(-exp(z_t + w0))
+//
+// per head, S [dk, dv] kept as [dv, dk] in float32; z is the output of a low-rank product, z = W2 low. Three forms:
+//   * one token per row (decode steps): one CTA per (row, head) works out z and the decays, reads and writes the state once, and
+//     goes on to the head's norm and gate;
+//   * prompts in bfloat16, by chunks of 64 tokens on the tensor cores (below);
+//   * everything else: decays by channel_decay_kernel, then the token-by-token walk of recurrence.cu (the bonus rule).
+//
+// Chunks. With P(a..b)[c] the product of channel c's decays over tokens a..b (1 where a > b),
+//   o_i = sum_(j < i) (sum_c r_i k_j P(j+1..i-1)) v_j + (sum_c r_i u k_i) v_i + S_before^T (r_i P(first..i-1)),
+//   S_after = P(first..last) S_before + sum_j (k_j P(j+1..last)) v_j^T.
+// A decay may be as small as zero, so nothing is divided by a product of decays: a chunk is cut into blocks of 16 tokens. Between
+// two blocks the product splits at the later block's first token, and r (times the product from there) meets k (times the product up
+// to there) in a matrix product; inside a block the 120 pairs are summed channel by channel with a running product. What goes to the
+// tensor cores and is not exact in bfloat16 (r and k times products, the weights, the state) goes as two bfloat16 numbers. Launches:
+//   states (what every chunk adds), carry (the states before every chunk, and the row's last one), outputs.
+#include "chunk_mma.cuh"
+
+namespace ms {
+
+__device__ __forceinline__ float channel_decay_of(float z) { return expf(-expf(z)); }
+
+// out[t, c] = exp(-exp(z[t, c] + w0[c])), float32
+template <typename T>
+__global__ void channel_decay_kernel(float* __restrict__ out, const T* __restrict__ z, int ld_z, const float* __restrict__ w0, long long items,
+                                     int width) {
+  pdl_prologue();
+  const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= items) return;
+  const long long t = idx / width;
+  const int c = (int)(idx - t * width);
+  out[idx] = channel_decay_of(Elem<T>::load(z + t * ld_z + c) + w0[c]);
+}
+
+// ---------------------------------------------------------------- one token per row
+constexpr int TS_THREADS = 256, TS_WARPS = TS_THREADS / 32, TS_COLS = 4;
+
+// a 2-d operand: rows ld apart
+template <typename T>
+struct Rows {
+  const T* p;
+  int ld;
+};
+
+// grid (H, rows). LPC lanes take a column's key channels, four at a time; a warp 32 / LPC columns at once, TS_COLS of them in turn with
+// their loads in flight together. out [T, H * dv] = o / sqrt(mean o^2 + eps) * norm_w * silu(gate).
+template <typename T, int LPC>
+__global__ void __launch_bounds__(TS_THREADS)
+time_step_kernel(T* __restrict__ out, float* __restrict__ state, Rows<T> r, Rows<T> k, Rows<T> v, Rows<T> gate, Rows<T> low,
+                 const T* __restrict__ w2, int rank, const float* __restrict__ w0, const float* __restrict__ u,
+                 const float* __restrict__ norm_w, float eps, const int* __restrict__ cu_q, const int* __restrict__ q_start,
+                 const int* __restrict__ state_slot, int H, int dk, int dv) {
+  extern __shared__ __align__(16) float ts_smem[];
+  __shared__ float red[32];
+  float* rs = ts_smem;       // [dk]
+  float* ks = rs + dk;       // [dk]
+  float* ds = ks + dk;       // [dk]
+  float* uk = ds + dk;       // [dk] bonus times key
+  float* os = uk + dk;       // [dv]
+  float* ls = os + dv;       // [rank]
+  pdl_prologue();
+  const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int t = cu_q[row];
+  const bool fresh = q_start[row] == 0;
+  for (int c = tid; c < rank; c += TS_THREADS) ls[c] = Elem<T>::load(low.p + (size_t)t * low.ld + c);
+  for (int c = tid; c < dk; c += TS_THREADS) {
+    const size_t at = (size_t)h * dk + c;
+    const float kk = Elem<T>::load(k.p + (size_t)t * k.ld + at);
+    rs[c] = Elem<T>::load(r.p + (size_t)t * r.ld + at);
+    ks[c] = kk;
+    uk[c] = u[at] * kk;
+  }
+  __syncthreads();
+  // z of the head's channels: eight lanes a channel
+  {
+    const int l = tid & 7;
+    for (int c0 = 0; c0 < dk; c0 += TS_THREADS / 8) {
+      const int c = c0 + (tid >> 3);
+      float acc = 0.f;
+      if (c < dk) {
+        const T* w = w2 + ((size_t)h * dk + c) * rank;
+        for (int i = l; i < rank; i += 8) acc = fmaf(ls[i], Elem<T>::load(w + i), acc);
+      }
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+      if (l == 0 && c < dk) ds[c] = channel_decay_of(acc + w0[(size_t)h * dk + c]);
+    }
+  }
+  __syncthreads();
+  constexpr int CPW = 32 / LPC;
+  const int l = lane % LPC, sub = lane / LPC;
+  float* head = state + ((size_t)state_slot[row] * H + h) * (size_t)dv * dk;
+  for (int j0 = warp * CPW + sub; j0 - sub < dv; j0 += TS_WARPS * CPW * TS_COLS) {
+    float acc[TS_COLS] = {}, vj[TS_COLS];
+#pragma unroll
+    for (int s = 0; s < TS_COLS; ++s) {
+      const int j = j0 + s * TS_WARPS * CPW;
+      vj[s] = j < dv ? Elem<T>::load(v.p + (size_t)t * v.ld + (size_t)h * dv + j) : 0.f;
+    }
+    for (int i = l * 4; i < dk; i += LPC * 4) {
+      float4 S[TS_COLS];
+#pragma unroll
+      for (int s = 0; s < TS_COLS; ++s) {
+        const int j = j0 + s * TS_WARPS * CPW;
+        S[s] = fresh || j >= dv ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(head + (size_t)j * dk + i);
+      }
+      const float4 r4 = *reinterpret_cast<const float4*>(rs + i), k4 = *reinterpret_cast<const float4*>(ks + i);
+      const float4 d4 = *reinterpret_cast<const float4*>(ds + i), u4 = *reinterpret_cast<const float4*>(uk + i);
+#pragma unroll
+      for (int s = 0; s < TS_COLS; ++s) {
+        const int j = j0 + s * TS_WARPS * CPW;
+        acc[s] += (r4.x * fmaf(u4.x, vj[s], S[s].x) + r4.y * fmaf(u4.y, vj[s], S[s].y)) +
+                  (r4.z * fmaf(u4.z, vj[s], S[s].z) + r4.w * fmaf(u4.w, vj[s], S[s].w));
+        S[s] = make_float4(fmaf(d4.x, S[s].x, k4.x * vj[s]), fmaf(d4.y, S[s].y, k4.y * vj[s]), fmaf(d4.z, S[s].z, k4.z * vj[s]),
+                           fmaf(d4.w, S[s].w, k4.w * vj[s]));
+        if (j < dv) *reinterpret_cast<float4*>(head + (size_t)j * dk + i) = S[s];
+      }
+    }
+#pragma unroll
+    for (int s = 0; s < TS_COLS; ++s) {
+      float x = acc[s];
+#pragma unroll
+      for (int o = LPC >> 1; o > 0; o >>= 1) x += __shfl_xor_sync(0xffffffffu, x, o);
+      const int j = j0 + s * TS_WARPS * CPW;
+      if (l == 0 && j < dv) os[j] = x;
+    }
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < dv; c += TS_THREADS) ss += os[c] * os[c];
+  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)dv + eps);
+  for (int c = tid; c < dv; c += TS_THREADS) {
+    const size_t at = (size_t)h * dv + c;
+    const float g = Elem<T>::load(gate.p + (size_t)t * gate.ld + at);
+    Elem<T>::store(out + (size_t)t * H * dv + at, ((os[c] * inv) * norm_w[at]) * (g / (1.0f + expf(-g))));
+  }
+}
+
+// ---------------------------------------------------------------- chunks: what every chunk adds to the state
+constexpr int TC_DV = 64;  // value columns per CTA
+constexpr int TC_BLK = 16, TC_BLOCKS = CS_TOK / TC_BLK;
+
+struct ChunkPlace {
+  const int2* tab;       // (row, first flat token) of a chunk
+  const int* row_first;  // a row's first chunk; [num_rows]: how many chunks there are
+  const int* cu_q;
+  const int* q_start;
+  const int* state_slot;
+  int num_rows;
+};
+
+// The decays of a block's 16 tokens for one channel (tokens from n on: 1).
+__device__ __forceinline__ void block_decays(float (&d)[TC_BLK], const float* __restrict__ z, int ld_z, const float* __restrict__ w0, int t0, int n,
+                                             int blk, int ch, bool in) {
+#pragma unroll
+  for (int i = 0; i < TC_BLK; ++i) {
+    const int tt = blk * TC_BLK + i;
+    d[i] = in && tt < n ? z[(size_t)(t0 + tt) * ld_z + ch] : 0.f;
+  }
+  const float w = in ? w0[ch] : 0.f;
+#pragma unroll
+  for (int i = 0; i < TC_BLK; ++i) d[i] = in && blk * TC_BLK + i < n ? channel_decay_of(d[i] + w) : 1.f;
+}
+
+template <int DKT>
+struct TmStatesSmem {
+  __nv_bfloat16 v[CS_TOK][TC_DV + 8], khi[CS_TOK][DKT + 8], klo[CS_TOK][DKT + 8];
+  float whole[TC_BLOCKS][DKT];
+};
+
+// added [chunks, H, dv, dk] float32, passed [chunks, H, dk]: the product of the chunk's decays. grid (chunks, H, dv tiles).
+template <int DKT>
+__global__ void __launch_bounds__(CS_THREADS)
+tm_states_kernel(float* __restrict__ added, float* __restrict__ passed, const __nv_bfloat16* __restrict__ k, int ld_k,
+                 const __nv_bfloat16* __restrict__ v, int ld_v, const float* __restrict__ z, int ld_z, const float* __restrict__ w0,
+                 const ChunkPlace pl, int H, int dk, int dv) {
+  extern __shared__ __align__(16) unsigned char cs_raw[];
+  TmStatesSmem<DKT>& sm = *reinterpret_cast<TmStatesSmem<DKT>*>(cs_raw);
+  pdl_prologue();
+  const int chunk = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * TC_DV;
+  if (chunk >= pl.row_first[pl.num_rows]) return;
+  const int2 at = pl.tab[chunk];
+  const int t0 = at.y, n = min(CS_TOK, pl.cu_q[at.x + 1] - t0);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  for (int idx = tid; idx < CS_TOK * (TC_DV / 8); idx += CS_THREADS) {
+    const int tt = idx / (TC_DV / 8), c = (idx - tt * (TC_DV / 8)) * 8;
+    const bool in = tt < n && v0 + c < dv;
+    cs_cp16(&sm.v[tt][c], in ? (const void*)(v + (size_t)(t0 + tt) * ld_v + (size_t)h * dv + v0 + c) : (const void*)v, in);
+  }
+  cs_commit();
+  constexpr int TRIPS = DKT / 64;
+  const int blk = tid >> 6;
+  float suf[TRIPS][TC_BLK];
+#pragma unroll
+  for (int tr = 0; tr < TRIPS; ++tr) {
+    const int c = tr * 64 + (tid & 63);
+    float d[TC_BLK];
+    block_decays(d, z, ld_z, w0, t0, n, blk, h * dk + c, c < dk);
+    suf[tr][TC_BLK - 1] = 1.f;
+#pragma unroll
+    for (int i = TC_BLK - 2; i >= 0; --i) suf[tr][i] = suf[tr][i + 1] * d[i + 1];
+    sm.whole[blk][c] = suf[tr][0] * d[0];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int tr = 0; tr < TRIPS; ++tr) {
+    const int c = tr * 64 + (tid & 63);
+    float behind = 1.f;
+#pragma unroll
+    for (int b = 1; b < TC_BLOCKS; ++b)
+      if (b > blk) behind *= sm.whole[b][c];
+#pragma unroll
+    for (int i = 0; i < TC_BLK; ++i) {
+      const int tt = blk * TC_BLK + i;
+      float x = 0.f;
+      if (tt < n && c < dk) x = __bfloat162float(k[(size_t)(t0 + tt) * ld_k + (size_t)h * dk + c]) * (suf[tr][i] * behind);
+      cs_split(x, sm.khi[tt][c], sm.klo[tt][c]);
+    }
+    if (blk == 0 && c < dk && blockIdx.z == 0) passed[((size_t)chunk * H + h) * dk + c] = sm.whole[0][c] * behind;
+  }
+  cs_wait<0>();
+  __syncthreads();
+  constexpr int NC = DKT / 2;  // key columns per warp
+  const int wm = (warp >> 1) * 16, wn = (warp & 1) * NC;  // 4 x 2 warps of 16 value rows x NC key columns
+  float acc[NC / 8][4] = {};
+  const int i8 = lane & 7, mat = lane >> 3;
+#pragma unroll
+  for (int kk = 0; kk < CS_TOK; kk += 16) {
+    uint32_t a[4];
+    cs_ldsm_t(a, &sm.v[kk + i8 + (mat >= 2 ? 8 : 0)][wm + (mat & 1 ? 8 : 0)]);
+#pragma unroll
+    for (int nj = 0; nj < NC / 16; ++nj) {
+      uint32_t bh[4], bl[4];
+      const int row = kk + i8 + (mat & 1 ? 8 : 0), col = wn + nj * 16 + (mat >= 2 ? 8 : 0);
+      cs_ldsm_t(bh, &sm.khi[row][col]);
+      cs_ldsm_t(bl, &sm.klo[row][col]);
+      cs_mma(acc[2 * nj], a, bh[0], bh[1]);
+      cs_mma(acc[2 * nj], a, bl[0], bl[1]);
+      cs_mma(acc[2 * nj + 1], a, bh[2], bh[3]);
+      cs_mma(acc[2 * nj + 1], a, bl[2], bl[3]);
+    }
+  }
+  float* out = added + ((size_t)chunk * H + h) * (size_t)dv * dk;
+  const int g = lane >> 2, tg = (lane & 3) * 2;
+#pragma unroll
+  for (int ni = 0; ni < NC / 8; ++ni)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int row = v0 + wm + g + half * 8, col = wn + ni * 8 + tg;  // (dk is even: a pair is inside or outside)
+      if (row < dv && col < dk) *reinterpret_cast<float2*>(out + (size_t)row * dk + col) = make_float2(acc[ni][2 * half], acc[ni][2 * half + 1]);
+    }
+}
+
+// ---------------------------------------------------------------- chunks: the states before every chunk
+// before_hi / before_lo [chunks, H, dv, dk]: the state before every chunk as two bfloat16; the row's slot of state [slots, H, dv, dk] gets
+// the state behind its last chunk. Four elements per thread; grid (elements of a row's state, rows).
+__global__ void __launch_bounds__(CS_THREADS)
+tm_carry_kernel(float* __restrict__ state, __nv_bfloat16* __restrict__ before_hi, __nv_bfloat16* __restrict__ before_lo,
+                const float* __restrict__ added, const float* __restrict__ passed, const ChunkPlace pl, int H, int dk, int dv) {
+  pdl_prologue();
+  const int total4 = H * dv * dk / 4;
+  const int i4 = blockIdx.x * CS_THREADS + threadIdx.x, r = blockIdx.y;
+  if (i4 >= total4) return;
+  const int h = i4 / (dv * dk / 4), c = i4 * 4 % dk;
+  const int c0 = pl.row_first[r], c1 = pl.row_first[r + 1];
+  if (c1 <= c0) return;
+  float4* slot = reinterpret_cast<float4*>(state) + (size_t)pl.state_slot[r] * total4 + i4;
+  float4 S = pl.q_start[r] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : *slot;
+#pragma unroll 4
+  for (int ch = c0; ch < c1; ++ch) {
+    const size_t at = (size_t)ch * total4 + i4;
+    const float4 d = reinterpret_cast<const float4*>(added)[at];
+    const float4 a = *reinterpret_cast<const float4*>(passed + ((size_t)ch * H + h) * dk + c);
+    __align__(8) __nv_bfloat16 hi[4];
+    __align__(8) __nv_bfloat16 lo[4];
+    cs_split(S.x, hi[0], lo[0]);
+    cs_split(S.y, hi[1], lo[1]);
+    cs_split(S.z, hi[2], lo[2]);
+    cs_split(S.w, hi[3], lo[3]);
+    reinterpret_cast<uint2*>(before_hi)[at] = *reinterpret_cast<const uint2*>(hi);
+    reinterpret_cast<uint2*>(before_lo)[at] = *reinterpret_cast<const uint2*>(lo);
+    S = make_float4(fmaf(a.x, S.x, d.x), fmaf(a.y, S.y, d.y), fmaf(a.z, S.z, d.z), fmaf(a.w, S.w, d.w));
+  }
+  *slot = S;
+}
+
+// ---------------------------------------------------------------- chunks: the outputs
+template <int DKT>
+struct TmOutputsSmem {
+  static constexpr int LDK = DKT + 8, LDP = CS_TOK + 8;
+  float d[CS_TOK][DKT + 4];                         // decays
+  float whole[TC_BLOCKS][DKT];                      // a block's product
+  float dsum[2][TC_BLOCKS][TC_BLK][TC_BLK + 1];     // [channel half][block][j][i]: sums of the pairs inside a block
+  union {
+    struct {
+      __nv_bfloat16 r[CS_TOK][LDK], k[CS_TOK][LDK];
+    };
+    struct {
+      __nv_bfloat16 shi[TC_DV][LDK], slo[TC_DV][LDK];  // the state before the chunk, once r and k have been read
+    };
+  };
+  __nv_bfloat16 rhi[CS_TOK][LDK], rlo[CS_TOK][LDK];  // r times the product from its block's (then: the chunk's) first token on
+  union {
+    struct {
+      __nv_bfloat16 hi[96][LDK], lo[96][LDK];  // k times the product up to block 1 (rows 0..15), 2 (16..47), 3 (48..95)
+    } kb;
+    struct {
+      __nv_bfloat16 hi[CS_TOK][LDP], lo[CS_TOK][LDP];  // the weights of v
+    } p;
+  };
+  __nv_bfloat16 v[CS_TOK][TC_DV + 8];
+};
+
+// o [T, H, dv] float32. grid (chunks, H, dv tiles).
+template <int DKT>
+__global__ void __launch_bounds__(CS_THREADS, DKT <= 64 ? 2 : 1)
+tm_outputs_kernel(float* __restrict__ o, const __nv_bfloat16* __restrict__ r, int ld_r, const __nv_bfloat16* __restrict__ k, int ld_k,
+                  const __nv_bfloat16* __restrict__ v, int ld_v, const float* __restrict__ z, int ld_z, const float* __restrict__ w0,
+                  const float* __restrict__ u, const __nv_bfloat16* __restrict__ before_hi, const __nv_bfloat16* __restrict__ before_lo,
+                  const ChunkPlace pl, int H, int dk, int dv) {
+  extern __shared__ __align__(16) unsigned char cs_raw[];
+  TmOutputsSmem<DKT>& sm = *reinterpret_cast<TmOutputsSmem<DKT>*>(cs_raw);
+  pdl_prologue();
+  const int chunk = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * TC_DV;
+  if (chunk >= pl.row_first[pl.num_rows]) return;
+  const int2 at = pl.tab[chunk];
+  const int t0 = at.y, n = min(CS_TOK, pl.cu_q[at.x + 1] - t0);
+  const bool has_state = !(pl.q_start[at.x] == 0 && chunk == pl.row_first[at.x]);  // else nothing came before
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int i8 = lane & 7, mat = lane >> 3, g = lane >> 2, tg = (lane & 3) * 2;
+  for (int idx = tid; idx < CS_TOK * (DKT / 8); idx += CS_THREADS) {
+    const int tt = idx / (DKT / 8), c = (idx - tt * (DKT / 8)) * 8;
+    const bool in = tt < n && c < dk;
+    const size_t tok = (size_t)(t0 + tt);
+    cs_cp16(&sm.r[tt][c], in ? (const void*)(r + tok * ld_r + (size_t)h * dk + c) : (const void*)r, in);
+    cs_cp16(&sm.k[tt][c], in ? (const void*)(k + tok * ld_k + (size_t)h * dk + c) : (const void*)k, in);
+  }
+  cs_commit();
+  for (int idx = tid; idx < CS_TOK * (TC_DV / 8); idx += CS_THREADS) {
+    const int tt = idx / (TC_DV / 8), c = (idx - tt * (TC_DV / 8)) * 8;
+    const bool in = tt < n && v0 + c < dv;
+    cs_cp16(&sm.v[tt][c], in ? (const void*)(v + (size_t)(t0 + tt) * ld_v + (size_t)h * dv + v0 + c) : (const void*)v, in);
+  }
+  cs_commit();
+
+  // decays, and the products within a block, one thread per (block, channel)
+  constexpr int TRIPS = DKT / 64;
+  const int blk = tid >> 6;
+  float pre[TRIPS][TC_BLK];
+#pragma unroll
+  for (int tr = 0; tr < TRIPS; ++tr) {
+    const int c = tr * 64 + (tid & 63);
+    float d[TC_BLK];
+    block_decays(d, z, ld_z, w0, t0, n, blk, h * dk + c, c < dk);
+    float run = 1.f;
+#pragma unroll
+    for (int i = 0; i < TC_BLK; ++i) {
+      pre[tr][i] = run;  // up to the token before
+      run *= d[i];
+      sm.d[blk * TC_BLK + i][c] = d[i];
+    }
+    sm.whole[blk][c] = run;
+  }
+  cs_wait<1>();  // r and k
+  __syncthreads();
+#pragma unroll
+  for (int tr = 0; tr < TRIPS; ++tr) {
+    const int c = tr * 64 + (tid & 63);
+    const float w1 = sm.whole[1][c], w2 = sm.whole[2][c];
+    float suf = 1.f;
+#pragma unroll
+    for (int i = TC_BLK - 1; i >= 0; --i) {
+      const int tt = blk * TC_BLK + i;
+      pre[tr][i] *= __bfloat162float(sm.r[tt][c]);
+      cs_split(pre[tr][i], sm.rhi[tt][c], sm.rlo[tt][c]);
+      const float x = __bfloat162float(sm.k[tt][c]) * suf;
+      suf *= sm.d[tt][c];
+      if (blk == 0) {
+        cs_split(x, sm.kb.hi[i][c], sm.kb.lo[i][c]);
+        cs_split(x * w1, sm.kb.hi[16 + i][c], sm.kb.lo[16 + i][c]);
+        cs_split(x * (w1 * w2), sm.kb.hi[48 + i][c], sm.kb.lo[48 + i][c]);
+      } else if (blk == 1) {
+        cs_split(x, sm.kb.hi[32 + i][c], sm.kb.lo[32 + i][c]);
+        cs_split(x * w2, sm.kb.hi[64 + i][c], sm.kb.lo[64 + i][c]);
+      } else if (blk == 2) {
+        cs_split(x, sm.kb.hi[80 + i][c], sm.kb.lo[80 + i][c]);
+      }
+    }
+  }
+  __syncthreads();
+
+  const int bi = warp >> 1, half_w = warp & 1, wm = bi * TC_BLK;
+  // pairs of blocks: weights of the tokens of block jt < bi for those of block bi
+  float s[2][2][4] = {};  // [this warp's tiles: jt = half_w, half_w + 2][n8][..]
+  {
+    const int base = bi == 1 ? 0 : bi == 2 ? 16 : 48;
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      const int jt = half_w + 2 * q;
+      if (jt >= bi) continue;
+#pragma unroll
+      for (int kk = 0; kk < DKT; kk += 16) {
+        uint32_t ah[4], al[4], bh[4], bl[4];
+        const int ra = wm + i8 + (mat & 1 ? 8 : 0), ca = kk + (mat >= 2 ? 8 : 0);
+        cs_ldsm(ah, &sm.rhi[ra][ca]);
+        cs_ldsm(al, &sm.rlo[ra][ca]);
+        const int rb = base + jt * TC_BLK + i8 + (mat >= 2 ? 8 : 0), cb = kk + (mat & 1 ? 8 : 0);
+        cs_ldsm(bh, &sm.kb.hi[rb][cb]);
+        cs_ldsm(bl, &sm.kb.lo[rb][cb]);
+        cs_mma(s[q][0], ah, bh[0], bh[1]);
+        cs_mma(s[q][0], ah, bl[0], bl[1]);
+        cs_mma(s[q][0], al, bh[0], bh[1]);
+        cs_mma(s[q][1], ah, bh[2], bh[3]);
+        cs_mma(s[q][1], ah, bl[2], bl[3]);
+        cs_mma(s[q][1], al, bh[2], bh[3]);
+      }
+    }
+  }
+  // pairs inside a block: lane (j, quarter of the channels), all i at once
+  {
+    const int j = lane & 15;
+    constexpr int QC = DKT / 4;
+    const int cbeg = (half_w * 2 + (lane >> 4)) * QC;
+    float acc[TC_BLK] = {};
+    for (int c = cbeg; c < cbeg + QC; c += 4) {
+      float x[4], uk[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        x[e] = __bfloat162float(sm.k[wm + j][c + e]);
+        uk[e] = c + e < dk ? u[(size_t)h * dk + c + e] * x[e] : 0.f;
+      }
+#pragma unroll
+      for (int i = 0; i < TC_BLK; ++i) {
+        const __nv_bfloat162* rp = reinterpret_cast<const __nv_bfloat162*>(&sm.r[wm + i][c]);
+        const float2 r0 = __bfloat1622float2(rp[0]), r1 = __bfloat1622float2(rp[1]);
+        const float4 d4 = *reinterpret_cast<const float4*>(&sm.d[wm + i][c]);
+        if (i > j) {
+          acc[i] += (r0.x * x[0] + r0.y * x[1]) + (r1.x * x[2] + r1.y * x[3]);
+          x[0] *= d4.x;
+          x[1] *= d4.y;
+          x[2] *= d4.z;
+          x[3] *= d4.w;
+        } else if (i == j) {
+          acc[i] += (r0.x * uk[0] + r0.y * uk[1]) + (r1.x * uk[2] + r1.y * uk[3]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < TC_BLK; ++i) acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 16);
+    if (lane < 16) {
+#pragma unroll
+      for (int i = 0; i < TC_BLK; ++i) sm.dsum[half_w][bi][j][i] = acc[i];
+    }
+  }
+  __syncthreads();  // r, k and kb have been read, the sums are there
+  if (has_state) {
+    const size_t st = ((size_t)chunk * H + h) * (size_t)dv * dk;
+    for (int idx = tid; idx < TC_DV * (DKT / 8); idx += CS_THREADS) {
+      const int row = idx / (DKT / 8), c = (idx - row * (DKT / 8)) * 8;
+      const bool in = v0 + row < dv && c < dk;
+      const size_t src = in ? st + (size_t)(v0 + row) * dk + c : 0;
+      cs_cp16(&sm.shi[row][c], before_hi + src, in);
+      cs_cp16(&sm.slo[row][c], before_lo + src, in);
+    }
+  }
+  cs_commit();
+#pragma unroll
+  for (int q = 0; q < 2; ++q) {
+    const int jt = half_w + 2 * q;
+    if (jt >= bi) continue;
+#pragma unroll
+    for (int nj = 0; nj < 2; ++nj)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int i = wm + g + half * 8, j = jt * TC_BLK + nj * 8 + tg;
+        __align__(4) __nv_bfloat16 hi[2];
+        __align__(4) __nv_bfloat16 lo[2];
+        cs_split(s[q][nj][2 * half], hi[0], lo[0]);
+        cs_split(s[q][nj][2 * half + 1], hi[1], lo[1]);
+        *reinterpret_cast<uint32_t*>(&sm.p.hi[i][j]) = *reinterpret_cast<const uint32_t*>(hi);
+        *reinterpret_cast<uint32_t*>(&sm.p.lo[i][j]) = *reinterpret_cast<const uint32_t*>(lo);
+      }
+  }
+  for (int idx = tid; idx < TC_BLOCKS * TC_BLK * TC_BLK; idx += CS_THREADS) {
+    const int b = idx >> 8, i = (idx >> 4) & 15, j = idx & 15;
+    const float x = j <= i ? sm.dsum[0][b][j][i] + sm.dsum[1][b][j][i] : 0.f;
+    cs_split(x, sm.p.hi[b * TC_BLK + i][b * TC_BLK + j], sm.p.lo[b * TC_BLK + i][b * TC_BLK + j]);
+  }
+  if (has_state) {  // r times the product from the chunk's first token on
+#pragma unroll
+    for (int tr = 0; tr < TRIPS; ++tr) {
+      const int c = tr * 64 + (tid & 63);
+      float ahead = 1.f;
+#pragma unroll
+      for (int b = 0; b < TC_BLOCKS - 1; ++b)
+        if (b < blk) ahead *= sm.whole[b][c];
+#pragma unroll
+      for (int i = 0; i < TC_BLK; ++i) cs_split(pre[tr][i] * ahead, sm.rhi[blk * TC_BLK + i][c], sm.rlo[blk * TC_BLK + i][c]);
+    }
+  }
+  cs_wait<0>();
+  __syncthreads();
+
+  // 4 x 2 warps of 16 tokens x 32 value columns
+  const int wn = half_w * 32;
+  float acc[4][4] = {};
+  if (has_state) {
+#pragma unroll
+    for (int kk = 0; kk < DKT; kk += 16) {
+      uint32_t ah[4], al[4];
+      const int ra = wm + i8 + (mat & 1 ? 8 : 0), ca = kk + (mat >= 2 ? 8 : 0);
+      cs_ldsm(ah, &sm.rhi[ra][ca]);
+      cs_ldsm(al, &sm.rlo[ra][ca]);
+#pragma unroll
+      for (int nj = 0; nj < 2; ++nj) {
+        uint32_t bh[4], bl[4];
+        const int rb = wn + nj * 16 + i8 + (mat >= 2 ? 8 : 0), cb = kk + (mat & 1 ? 8 : 0);
+        cs_ldsm(bh, &sm.shi[rb][cb]);
+        cs_ldsm(bl, &sm.slo[rb][cb]);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          cs_mma(acc[2 * nj + e], ah, bh[2 * e], bh[2 * e + 1]);
+          cs_mma(acc[2 * nj + e], ah, bl[2 * e], bl[2 * e + 1]);
+          cs_mma(acc[2 * nj + e], al, bh[2 * e], bh[2 * e + 1]);
+        }
+      }
+    }
+  }
+  for (int kk = 0; kk <= wm; kk += 16) {  // (later tokens have no weight)
+    uint32_t ah[4], al[4];
+    const int ra = wm + i8 + (mat & 1 ? 8 : 0), ca = kk + (mat >= 2 ? 8 : 0);
+    cs_ldsm(ah, &sm.p.hi[ra][ca]);
+    cs_ldsm(al, &sm.p.lo[ra][ca]);
+#pragma unroll
+    for (int nj = 0; nj < 2; ++nj) {
+      uint32_t b[4];
+      cs_ldsm_t(b, &sm.v[kk + i8 + (mat & 1 ? 8 : 0)][wn + nj * 16 + (mat >= 2 ? 8 : 0)]);
+      cs_mma(acc[2 * nj], ah, b[0], b[1]);
+      cs_mma(acc[2 * nj], al, b[0], b[1]);
+      cs_mma(acc[2 * nj + 1], ah, b[2], b[3]);
+      cs_mma(acc[2 * nj + 1], al, b[2], b[3]);
+    }
+  }
+#pragma unroll
+  for (int ni = 0; ni < 4; ++ni)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int i = wm + g + half * 8, col = v0 + wn + ni * 8 + tg;
+      if (i < n && col < dv) *reinterpret_cast<float2*>(o + ((size_t)(t0 + i) * H + h) * dv + col) = make_float2(acc[ni][2 * half], acc[ni][2 * half + 1]);
+    }
+}
+
+template <int DKT>
+static int launch_chunks(float* o, float* state, const __nv_bfloat16* r, int ld_r, const __nv_bfloat16* k, int ld_k, const __nv_bfloat16* v, int ld_v,
+                         const float* z, int ld_z, const float* w0, const float* u, float* added, __nv_bfloat16* before_hi,
+                         __nv_bfloat16* before_lo, float* passed, const ChunkPlace& pl, int max_chunks, int H, int dk, int dv, cudaStream_t stream) {
+  static bool configured = false;
+  if (!configured) {
+    MS_CHECK_CUDA(cudaFuncSetAttribute(tm_states_kernel<DKT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(TmStatesSmem<DKT>)));
+    MS_CHECK_CUDA(cudaFuncSetAttribute(tm_outputs_kernel<DKT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(TmOutputsSmem<DKT>)));
+    configured = true;
+  }
+  const int v_tiles = ceil_div(dv, TC_DV);
+  MS_LAUNCH(tm_states_kernel<DKT>, dim3(max_chunks, H, v_tiles), CS_THREADS, sizeof(TmStatesSmem<DKT>), stream, added, passed, k, ld_k, v, ld_v, z, ld_z,
+            w0, pl, H, dk, dv);
+  MS_LAUNCH(tm_carry_kernel, dim3(ceil_div(H * dv * dk / 4, CS_THREADS), pl.num_rows), CS_THREADS, 0, stream, state, before_hi, before_lo, added, passed,
+            pl, H, dk, dv);
+  MS_LAUNCH(tm_outputs_kernel<DKT>, dim3(max_chunks, H, v_tiles), CS_THREADS, sizeof(TmOutputsSmem<DKT>), stream, o, r, ld_r, k, ld_k, v, ld_v, z, ld_z,
+            w0, u, before_hi, before_lo, pl, H, dk, dv);
+  return 0;
+}
+
+}  // namespace ms
+
+using namespace ms;
+
+MS_EXPORT int ms_channel_decay(float* out, const void* z, int ld_z, const float* w0, int tokens, int width, int dtype, cudaStream_t stream) {
+  if (tokens == 0) return 0;
+  const long long items = (long long)tokens * width;
+  const unsigned blocks = (unsigned)((items + 255) / 256);
+  if (dtype == MS_F32) MS_LAUNCH(channel_decay_kernel<float>, blocks, 256, 0, stream, out, (const float*)z, ld_z, w0, items, width);
+  else MS_LAUNCH(channel_decay_kernel<__nv_bfloat16>, blocks, 256, 0, stream, out, (const __nv_bfloat16*)z, ld_z, w0, items, width);
+  return 0;
+}
+
+// One token per row; dk a multiple of 4. r, k, v, gate and low are rows of one run dtype; w2 [H * dk, rank] in that dtype.
+MS_EXPORT int ms_time_step(void* out, float* state, const void* r, const void* k, const void* v, const void* gate, int ld, const void* low,
+                           int ld_low, const void* w2, int rank, const float* w0, const float* u, const float* norm_w, float eps,
+                           const int* cu_q, const int* q_start, const int* state_slot, int num_rows, int H, int dk, int dv, int dtype,
+                           cudaStream_t stream) {
+  if (num_rows == 0) return 0;
+  const size_t smem = ((size_t)4 * dk + dv + rank) * sizeof(float);
+  MS_CHECK_ARG(H > 0 && dk > 0 && dk % 4 == 0 && dv > 0 && rank > 0 && (uintptr_t)state % 16 == 0 && num_rows <= 65535 && smem <= 48 * 1024,
+               "time_step: %d rows, heads of %d x %d, rank %d", num_rows, dk, dv, rank);
+#define MS_STEP(T, LPC)                                                                                                                        \
+  MS_LAUNCH((time_step_kernel<T, LPC>), dim3(H, num_rows), TS_THREADS, smem, stream, (T*)out, state, Rows<T>{(const T*)r, ld},                \
+            Rows<T>{(const T*)k, ld}, Rows<T>{(const T*)v, ld}, Rows<T>{(const T*)gate, ld}, Rows<T>{(const T*)low, ld_low}, (const T*)w2, rank, w0, u, \
+            norm_w, eps, cu_q, q_start, state_slot, H, dk, dv)
+  if (dtype == MS_F32) {
+    if (dk > 64) MS_STEP(float, 32);
+    else if (dk > 32) MS_STEP(float, 16);
+    else MS_STEP(float, 8);
+  } else {
+    if (dk > 64) MS_STEP(__nv_bfloat16, 32);
+    else if (dk > 32) MS_STEP(__nv_bfloat16, 16);
+    else MS_STEP(__nv_bfloat16, 8);
+  }
+#undef MS_STEP
+  return 0;
+}
+
+// 1 if the chunk kernels take these sizes.
+MS_EXPORT int ms_time_chunk_supports(int dk, int dv) { return dk >= 8 && dk <= 128 && dk % 8 == 0 && dv >= 8 && dv % 8 == 0; }
+
+// o [T, H, dv] float32; state [slots, H, dv, dk] float32; r, k [T, H * dk], v [T, H * dv] bfloat16 rows, z [T, H * dk] float32 rows. Scratch
+// [max_chunks, H, dv, dk]: added float32, before_hi and before_lo bfloat16; passed float32 [max_chunks, H, dk].
+MS_EXPORT int ms_time_chunks(float* o, float* state, const void* r, int ld_r, const void* k, int ld_k, const void* v, int ld_v, const float* z, int ld_z,
+                             const float* w0, const float* u, float* added, void* before_hi, void* before_lo, float* passed, const int* tab,
+                             const int* row_first, const int* cu_q, const int* q_start, const int* state_slot, int num_rows, int max_chunks, int H,
+                             int dk, int dv, cudaStream_t stream) {
+  if (num_rows == 0 || max_chunks == 0) return 0;
+  MS_CHECK_ARG(ms_time_chunk_supports(dk, dv) && H > 0 && H <= 65535 && num_rows <= 65535 && (long long)H * dv * dk < (1LL << 31),
+               "time_chunks: %d heads of %d x %d, %d rows", H, dk, dv, num_rows);
+  MS_CHECK_ARG(ld_r % 8 == 0 && ld_k % 8 == 0 && ld_v % 8 == 0 && (uintptr_t)r % 16 == 0 && (uintptr_t)k % 16 == 0 && (uintptr_t)v % 16 == 0 &&
+                   (uintptr_t)o % 8 == 0 && (uintptr_t)state % 16 == 0 && (uintptr_t)added % 16 == 0 && (uintptr_t)before_hi % 16 == 0 &&
+                   (uintptr_t)before_lo % 16 == 0 && (uintptr_t)passed % 16 == 0,
+               "time_chunks: operands must be aligned");
+  const ChunkPlace pl{reinterpret_cast<const int2*>(tab), row_first, cu_q, q_start, state_slot, num_rows};
+  const __nv_bfloat16 *rb = (const __nv_bfloat16*)r, *kb = (const __nv_bfloat16*)k, *vb = (const __nv_bfloat16*)v;
+  if (dk <= 64)
+    return launch_chunks<64>(o, state, rb, ld_r, kb, ld_k, vb, ld_v, z, ld_z, w0, u, added, (__nv_bfloat16*)before_hi, (__nv_bfloat16*)before_lo, passed,
+                             pl, max_chunks, H, dk, dv, stream);
+  return launch_chunks<128>(o, state, rb, ld_r, kb, ld_k, vb, ld_v, z, ld_z, w0, u, added, (__nv_bfloat16*)before_hi, (__nv_bfloat16*)before_lo, passed,
+                            pl, max_chunks, H, dk, dv, stream);
+}

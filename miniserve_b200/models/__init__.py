@@ -1,2 +1,2 @@
 """Architectures this package ships. Importing the package registers them."""
-from . import fekulix, kovusun, mugipel, qwen3, rofozen, vumedra  # noqa: F401
+from . import fekulix, kovusun, mugipel, qwen3, rofozen, tunadra, vumedra  # noqa: F401

@@ -13,11 +13,11 @@ from dataclasses import dataclass
 import torch
 
 from . import blas, experts, native
-from .mixers import (act_mul, add_dyt, add_layernorm, add_normed_rmsnorm, add_rmsnorm_scaled, add_row_vector, axpby, channel_gate,  # noqa: F401
+from .mixers import (act_mul, add_dyt, add_layernorm, add_normed_rmsnorm, add_rmsnorm_scaled, add_row_vector, axpby, channel_decay, channel_gate,  # noqa: F401
                      chunk_scan, chunk_scan_ok, clamped_glu, conv_bias, conv_silu_unit, conv_state_update, decay_scan, embed_sum, gate_relu_squared, gated_group_norm,
                      gelu_tanh, head_gate, head_norm_gate, latent_prepare, latent_rope_prepare, mlstm_gates, mlstm_output, qkv_prepare,
                      relu_squared, rglru_scan, rope_table_scaled, row_rmsnorm, scale_, shift_state_update, ssm_step_decay, stream_concat,
-                     sum_bias, token_shift)
+                     stream_norm, sum_bias, tanh_, time_chunks, time_chunks_ok, time_step, time_step_ok, token_mixes, token_shift)
 from .native import NativeError, OutOfBlocks
 
 __all__ = [

@@ -65,7 +65,7 @@ PREBUILT_HEAD_DIMS = (16, 32, 48, 64, 80, 128, 256)
 # kernels of mixers, norms and feed-forwards that Qwen3 does not have (Dynamic Tanh, tanh-GELU, the general q|k|v step, gates,
 # the linear-attention recurrences): compiled when a model first needs one of them
 MIXERS = Module("mixers", ("mixer_pointwise.cu", "block_ops.cu", "stream_ops.cu"))
-RECURRENCE = Module("recurrence", ("recurrence.cu", "gated_recurrence.cu", "chunk_scan.cu"))
+RECURRENCE = Module("recurrence", ("recurrence.cu", "gated_recurrence.cu", "chunk_scan.cu", "time_mix.cu"))
 EXPERTS = Module("experts", ("routed_experts.cu",))  # a routed feed-forward: router, plan, the experts' products, the weighted sum
 GEMM_TC = Module("gemm_tc", ("gemm_tc.cu",))
 ATTN_TC = Module("attn_tc", ("attention_tc.cu",))

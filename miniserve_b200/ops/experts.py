@@ -10,7 +10,8 @@ import torch
 from . import native
 from .mixers import _dt, _f32, _ptr, _rows, _stream
 
-ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu_squared": 2}
+ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu_squared": 2, "clamped_glu": 3}
+NO_CLAMPS = (-1.0, 1.0, 0.0)  # (limit, alpha, shift) of a clamped GLU; other activations do not read them
 SCORES = {"softmax": 0, "sigmoid": 1}
 TILE_ROWS = 64       # sorted rows per tile of the float32 and mma.sync products
 TC_TILE_ROWS = 128   # of the products on the tcgen05 tensor cores
@@ -19,19 +20,19 @@ TC_EXPERTS = os.environ.get("MINISERVE_TC_EXPERTS", "1") != "0"  # bfloat16 expe
 
 def tc_experts_ok(dtype, hidden: int, inter: int, activation: str) -> bool:
     """Whether the experts' products of this shape run on the tcgen05 kernel (``csrc/gemm_tc.cu``, the grouped form):
-    bfloat16, an activation that the kernel has as an epilogue (SiLU times the up half, or the square of relu without a gate), rows that
-    are multiples of 16 bytes."""
-    return TC_EXPERTS and dtype == torch.bfloat16 and activation in ("silu", "relu_squared") and hidden % 8 == 0 and inter % 8 == 0
+    bfloat16, an activation that the kernel has as an epilogue (SiLU times the up half, the clamped GLU, or the square of relu without a
+    gate), rows that are multiples of 16 bytes."""
+    return TC_EXPERTS and dtype == torch.bfloat16 and activation in ("silu", "relu_squared", "clamped_glu") and hidden % 8 == 0 and inter % 8 == 0
 
 
 def expert_route(idx, wgt, x, router, correction, top: int, group_count: int, group_keep: int, weight_scale: float,
                  renormalize: bool, stream=None, logit_bias=None, gate_w=None, gate_out=None, score: str = "softmax",
-                 square_weights: bool = False) -> None:
+                 square_weights: bool = False, group_best: int = 1, renorm_eps: float = 0.0) -> None:
     """idx [T, top] int32 and wgt [T, top] float32: each token's chosen router outputs and their weights.
     Logits ``x router^T`` in float32 (``router`` [R, K] float32), scores their softmax, choice scores the scores plus
     ``correction`` [R] (float32, or None); the R outputs form ``group_count`` equal groups of neighbours of which the
-    ``group_keep`` with the largest choice score in them can be chosen from; weights are the chosen scores (without
-    the correction) times ``weight_scale``, divided by their sum if ``renormalize`` (which makes them the softmax over
+    ``group_keep`` with the largest sum of their ``group_best`` largest choice scores can be chosen from; weights are the chosen scores (without
+    the correction) times ``weight_scale``, divided by their sum (+ ``renorm_eps``) if ``renormalize`` (which makes them the softmax over
     the chosen logits alone). Ties go to the lower index. ``logit_bias`` [R] float32 is added to the logits themselves.
     ``gate_w`` [K] float32 with ``gate_out`` [T] float32: gate_out[t] = sigmoid(x[t] . gate_w), from the same staged input.
     ``score`` = ``sigmoid``: the scores are the logits' sigmoids. ``square_weights``: the final weights are squared."""
@@ -45,7 +46,7 @@ def expert_route(idx, wgt, x, router, correction, top: int, group_count: int, gr
     native.experts_check(native.experts().ms_expert_route(
         _ptr(idx), _ptr(wgt), _ptr(x), _rows(x), _ptr(router), _ptr(correction), t, k, r, top, group_count, group_keep,
         float(weight_scale), int(renormalize), _dt(x.dtype), _stream(stream), _ptr(logit_bias), _ptr(gate_w), _ptr(gate_out),
-        SCORES[score], int(square_weights)))
+        SCORES[score], int(square_weights), int(group_best), float(renorm_eps)))
 
 
 def expert_max_tiles(slots: int, experts: int, tile_rows: int = TILE_ROWS) -> int:
@@ -74,9 +75,9 @@ def expert_gather(xs, x, perm, meta, top: int, stream=None) -> None:
                                                            _stream(stream)))
 
 
-def expert_products_tc(out, a, w, tiles, meta, offsets, gated: bool, stream=None, relu_squared: bool = False) -> None:
+def expert_products_tc(out, a, w, tiles, meta, offsets, gated: bool, stream=None, relu_squared: bool = False, clamps=None) -> None:
     """The experts' products over sorted rows on the tcgen05 tensor cores (tiles of ``TC_TILE_ROWS`` rows).
-    ``gated``: out [S, I] bfloat16 = silu(a W_gate[e]^T) * (a W_up[e]^T) with ``w`` [E, 2 I, K]; else out [S, N] float32 =
+    ``gated``: out [S, I] bfloat16 = silu(a W_gate[e]^T) * (a W_up[e]^T) (or with ``clamps`` = (limit, alpha, shift) the clamped GLU of the two) with ``w`` [E, 2 I, K]; else out [S, N] float32 =
     a W[e]^T with ``w`` [E, N, K] (``relu_squared``: bfloat16, the square of its relu). ``a`` [S, K] bfloat16 in sorted order."""
     from . import device_status
 
@@ -86,14 +87,16 @@ def expert_products_tc(out, a, w, tiles, meta, offsets, gated: bool, stream=None
     assert a.dtype == w.dtype == torch.bfloat16 and w_rows == (2 * n if gated else n)
     assert out.dtype == (torch.bfloat16 if gated or relu_squared else torch.float32) and not (gated and relu_squared)
     lib = native.gemm_tc()
-    native.kernel_check(lib.ms_gemm_tc_experts_bf16(_ptr(out), _ptr(a), _ptr(w), slots, n, k, e, 2 if relu_squared else int(gated), _ptr(tiles), _ptr(meta),
-                                                    _ptr(offsets), expert_max_tiles(slots, e, TC_TILE_ROWS),
+    mode = 2 if relu_squared else (3 if clamps is not None else 1) if gated else 0
+    native.kernel_check(lib.ms_gemm_tc_experts_bf16(_ptr(out), _ptr(a), _ptr(w), slots, n, k, e, mode, _ptr(tiles), _ptr(meta),
+                                                    _ptr(offsets), expert_max_tiles(slots, e, TC_TILE_ROWS), *map(float, clamps or NO_CLAMPS),
                                                     _ptr(device_status(a.device)), _stream(stream)),
                         lib=lib, errfn="ms_gemm_tc_last_error")
 
 
-def expert_gate_up(out, x, w_gate_up, perm, top: int, tiles, meta, offsets, activation: str, stream=None) -> None:
-    """out [T * top, I] (the run's dtype), row r = act(W_gate[e] h) * (W_up[e] h) with h = x[perm[r] // top] and e the
+def expert_gate_up(out, x, w_gate_up, perm, top: int, tiles, meta, offsets, activation: str, stream=None, clamps=None) -> None:
+    """out [T * top, I] (the run's dtype), row r = act(W_gate[e] h) * (W_up[e] h) (``clamped_glu``: the clamped GLU of the two with
+    ``clamps`` = (limit, alpha, shift)) with h = x[perm[r] // top] and e the
     expert whose sorted rows hold r; ``w_gate_up`` [E, 2 I, K]: an expert's gate rows, then its up rows."""
     slots, inter = out.shape
     e, two_i, k = w_gate_up.shape
@@ -101,7 +104,7 @@ def expert_gate_up(out, x, w_gate_up, perm, top: int, tiles, meta, offsets, acti
     assert out.dtype == x.dtype == w_gate_up.dtype
     native.experts_check(native.experts().ms_expert_gemm(
         _ptr(out), _ptr(x), _rows(x), _ptr(perm), top, _ptr(w_gate_up), _ptr(tiles), _ptr(meta), _ptr(offsets),
-        expert_max_tiles(slots, e), inter, k, 1, ACTIVATIONS[activation], _dt(x.dtype), _stream(stream)))
+        expert_max_tiles(slots, e), inter, k, 1, ACTIVATIONS[activation], *map(float, clamps or NO_CLAMPS), _dt(x.dtype), _stream(stream)))
 
 
 def expert_up(out, x, w_up, perm, top: int, tiles, meta, offsets, activation: str, stream=None) -> None:
@@ -111,7 +114,7 @@ def expert_up(out, x, w_up, perm, top: int, tiles, meta, offsets, activation: st
     assert i == inter and x.shape[1] == k and out.is_contiguous() and w_up.is_contiguous() and out.dtype == x.dtype == w_up.dtype
     native.experts_check(native.experts().ms_expert_gemm(
         _ptr(out), _ptr(x), _rows(x), _ptr(perm), top, _ptr(w_up), _ptr(tiles), _ptr(meta), _ptr(offsets),
-        expert_max_tiles(slots, e), inter, k, 2, ACTIVATIONS[activation], _dt(x.dtype), _stream(stream)))
+        expert_max_tiles(slots, e), inter, k, 2, ACTIVATIONS[activation], *NO_CLAMPS, _dt(x.dtype), _stream(stream)))
 
 
 def expert_down(out, act, w_down, tiles, meta, offsets, stream=None) -> None:
@@ -122,7 +125,7 @@ def expert_down(out, act, w_down, tiles, meta, offsets, stream=None) -> None:
     assert h == hidden and act.shape == (slots, inter) and act.is_contiguous() and w_down.is_contiguous() and act.dtype == w_down.dtype
     native.experts_check(native.experts().ms_expert_gemm(
         _ptr(out), _ptr(act), inter, None, 1, _ptr(w_down), _ptr(tiles), _ptr(meta), _ptr(offsets),
-        expert_max_tiles(slots, e), hidden, inter, 0, 0, _dt(act.dtype), _stream(stream)))
+        expert_max_tiles(slots, e), hidden, inter, 0, 0, *NO_CLAMPS, _dt(act.dtype), _stream(stream)))
 
 
 def expert_combine(out, y, x, idx, wgt, pos, experts: int, stream=None, shared=None, shared_gate=None) -> None:

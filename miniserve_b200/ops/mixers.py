@@ -79,7 +79,7 @@ def head_gate(out: torch.Tensor, attn: torch.Tensor, gate: torch.Tensor | None, 
 
 def qkv_prepare(q_out, k_pool, v_pool, q, k, v, q_norm_w, k_norm_w, cos_sin, rotary_dim: int, adjacent: bool, eps: float,
                 positions, row_of_token, page_indptr, page_indices, page_size: int, status, stream=None, bias=None,
-                unit_norm: bool = False, q_scale=None, q_temp: tuple[float, float] | None = None) -> None:
+                unit_norm: bool = False, q_scale=None, q_temp: tuple[float, float] | None = None, v_other=None, v_share=None) -> None:
     """Per-head RMS norm of q and k (float32 weights or None), rotation of the first ``rotary_dim`` channels
     (pairs (2i, 2i+1) if ``adjacent`` else (i, i + rotary_dim/2)) by the step's cos/sin table, q to
     ``q_out`` [T, nq, D] and k, v into their pages [pages, nkv, page_size, D], zero beyond their own
@@ -87,7 +87,8 @@ def qkv_prepare(q_out, k_pool, v_pool, q, k, v, q_norm_w, k_norm_w, cos_sin, rot
     ``bias``: float32 [nq*dk + nkv*dk + nkv*dv], the projections' biases in the order q, k, v, added first.
     ``unit_norm``: q and k are divided by their root mean square also without norm weights. ``q_scale``: float32 [nq],
     a factor per query head applied last. ``q_temp`` (coef, every): queries at position p are also multiplied by
-    1 + coef ln(floor((p + 1) / every) + 1). Without pools (``k_pool``, ``k`` and ``v`` None) only the queries are
+    1 + coef ln(floor((p + 1) / every) + 1). ``v_other`` [T, nkv*dv] (a view whose rows may be part of wider ones) with ``v_share``
+    (float32, one number): the values become (1 - share) v + share v_other before they are cached. Without pools (``k_pool``, ``k`` and ``v`` None) only the queries are
     prepared (a mixer that reads another's keys and values); ``bias`` is then [nq*dk]."""
     t, nq, d = q_out.shape
     dk = q.shape[1] // nq
@@ -102,7 +103,7 @@ def qkv_prepare(q_out, k_pool, v_pool, q, k, v, q_norm_w, k_norm_w, cos_sin, rot
             _ptr(q_out), None, None, q.data_ptr(), _rows(q), 0, 0, 0, _ptr(q_norm_w), None, _ptr(cos_sin), _ptr(positions),
             _ptr(row_of_token), _ptr(page_indptr), _ptr(page_indices), t, nq, 1, dk, dk, d, rotary_dim if cos_sin is not None else 0,
             int(adjacent), float(eps), page_size, 0, _ptr(status), _dt(q.dtype), _stream(stream), _ptr(bias), _ptr(q_scale),
-            int(unit_norm), float(coef), float(every)))
+            int(unit_norm), float(coef), float(every), None, 0, None))
         return
     nkv = k_pool.shape[1]
     dv = v.shape[1] // nkv
@@ -110,6 +111,8 @@ def qkv_prepare(q_out, k_pool, v_pool, q, k, v, q_norm_w, k_norm_w, cos_sin, rot
     assert k_pool.shape == v_pool.shape and k_pool.shape[2] == page_size and k_pool.shape[3] == d
     assert q.dtype == k.dtype == v.dtype == q_out.dtype == k_pool.dtype
     assert bias is None or bias.numel() == (nq + nkv) * dk + nkv * dv
+    assert (v_other is None) == (v_share is None)
+    assert v_other is None or (v_other.shape == v.shape and v_other.dtype == v.dtype and v_share.dtype == torch.float32 and v_share.numel() == 1)
     ld = _rows(q)
     assert _rows(k) == ld and _rows(v) == ld, "q, k and v must be columns of the same rows"
     item = q.element_size()
@@ -119,7 +122,8 @@ def qkv_prepare(q_out, k_pool, v_pool, q, k, v, q_norm_w, k_norm_w, cos_sin, rot
         _ptr(q_out), _ptr(k_pool), _ptr(v_pool), base, ld, offs[0], offs[1], offs[2], _ptr(q_norm_w), _ptr(k_norm_w),
         _ptr(cos_sin), _ptr(positions), _ptr(row_of_token), _ptr(page_indptr), _ptr(page_indices), t, nq, nkv, dk, dv, d,
         rotary_dim if cos_sin is not None else 0, int(adjacent), float(eps), page_size, k_pool.shape[0], _ptr(status),
-        _dt(q.dtype), _stream(stream), _ptr(bias), _ptr(q_scale), int(unit_norm), float(coef), float(every)))
+        _dt(q.dtype), _stream(stream), _ptr(bias), _ptr(q_scale), int(unit_norm), float(coef), float(every),
+        _ptr(v_other), 0 if v_other is None else _rows(v_other), _ptr(v_share)))
 
 
 def add_layernorm(out, residual, delta, weight, bias, eps: float, rows=None, num_rows=None, write_residual=True, delta_scale: float = 1.0,
@@ -152,6 +156,25 @@ def token_shift(out, h, state, mix, ctx, update: bool = True) -> None:
         t, width, int(update), _dt(h.dtype), ctx.stream))
 
 
+def token_mixes(out, h, state, mix, ctx) -> None:
+    """out[m, t] = h[t] + (h[t - 1] - h[t]) * mix[m] for every row of ``mix`` (float32 [mixes, width]); ``out`` [mixes, T, width]. The
+    token before a row's first one is as in ``token_shift``; the same launch leaves each row's last h of this step in its slot."""
+    t, width = h.shape
+    mixes = mix.shape[0]
+    _f32(mix)
+    assert out.shape == (mixes, t, width) and out.dtype == h.dtype == state.dtype and out.is_contiguous() and h.is_contiguous()
+    assert state.is_contiguous() and state.shape[1] == width and mix.shape[1] == width
+    native.mixers_check(native.mixers().ms_token_mixes(
+        _ptr(out), _ptr(h), _ptr(state), _ptr(mix), mixes, _ptr(ctx.row_of_token), _ptr(ctx.cu_q), _ptr(ctx.q_start), _ptr(ctx.state_slot),
+        t, width, _dt(h.dtype), ctx.stream))
+
+
+def tanh_(x: torch.Tensor, cap: float = 0.0, stream=None) -> None:
+    """x = cap tanh(x / cap), or tanh(x) without a cap, in place; float32 arithmetic."""
+    assert x.is_cuda and x.is_contiguous()
+    native.mixers_check(native.mixers().ms_tanh_inplace(_ptr(x), float(cap), x.numel(), _dt(x.dtype), _stream(stream)))
+
+
 def shift_state_update(state, h, ctx) -> None:
     """state[slot of row] = h[the row's last token of this step], for every row of the step."""
     assert h.is_contiguous() and state.is_contiguous() and state.dtype == h.dtype and state.shape[1] == h.shape[1]
@@ -181,7 +204,7 @@ def sum_bias(out, a, b=None, vec=None, stream=None) -> None:
 
 
 def decay_scan(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign: float, beta, ctx, heads: int, dk: int, dv: int,
-               q_scale: float, delta: bool, head_decay: bool = False, v_scale=None, ones_column: bool = False) -> None:
+               q_scale: float, delta: bool, head_decay: bool = False, v_scale=None, ones_column: bool = False, bonus=None) -> None:
     """The token-by-token recurrence of every row of the step (``csrc/recurrence.cu``), from each
     request's slot of ``state`` [slots, heads, dv, dk] float32 (zero where a row starts at position 0)
     and back into it; o_out [T, heads, dv] float32. q, k [T, groups*dk], v [T, heads*dv], z [T, heads*dk]
@@ -189,10 +212,13 @@ def decay_scan(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign: float, beta
     ``head_decay``: z [T, heads] float32 holds the decays themselves, one for all key channels of a head and token
     (z_bias, decay_coef and z_sign are not used; all three may be None, None and 0). ``v_scale`` [T, heads] float32: v counts times it, per token and head.
     ``ones_column``: v has heads * (dv - 1) columns and every head's last value is one (times v_scale): that column of the state is
-    the decayed sum of the keys, that entry of the output its product with the query (the decay rule only)."""
+    the decayed sum of the keys, that entry of the output its product with the query (the decay rule only).
+    ``bonus`` [heads * dk] float32: the read-out sees the state before the token's own write, and that write times ``bonus`` per key channel;
+    z [T, heads*dk] float32 then holds the decays themselves."""
     t = o_out.shape[0]
     dv_in = dv - int(ones_column)
-    _f32(o_out, state, z_bias, decay_coef, v_scale)
+    _f32(o_out, state, z_bias, decay_coef, v_scale, bonus)
+    assert bonus is None or (bonus.numel() == heads * dk and z.dtype == torch.float32 and not delta and not head_decay and not ones_column)
     assert o_out.shape == (t, heads, dv) and state.shape[1:] == (heads, dv, dk)
     groups = q.shape[1] // dk
     assert q.shape == (t, groups * dk) and k.shape == q.shape and v.shape == (t, heads * dv_in)
@@ -201,14 +227,14 @@ def decay_scan(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign: float, beta
     assert v_scale is None or v_scale.shape == (t, heads)
     if not delta and not ctx.decode_only and t >= SEGMENT_MIN_TOKENS and SEGMENTS > 1 and dk <= SEGMENT_MAX_DK:
         return _decay_scan_segmented(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign, ctx, heads, dk, dv, q_scale, head_decay,
-                                     v_scale, dv_in)
+                                     v_scale, dv_in, bonus)
     if not delta and head_decay and ctx.decode_only and dk % 4 == 0:  # one token per row: the state is read and written once, nothing else
         native.recurrence_check(native.recurrence().ms_decay_step(
             _ptr(o_out), _ptr(state), _ptr(q), _rows(q), _ptr(k), _rows(k), heads // groups, _ptr(v), _rows(v), _ptr(z), _rows(z), _ptr(ctx.cu_q),
             _ptr(ctx.q_start), _ptr(ctx.state_slot), ctx.num_rows, heads, dk, dv, float(q_scale), _ptr(v_scale), dv_in, _dt(q.dtype), ctx.stream))
         return
-    ready = int(head_decay)
-    if not ctx.decode_only and not head_decay:
+    ready = int(head_decay or bonus is not None)
+    if not ctx.decode_only and not ready:
         # a prompt portion: exponentials and logarithms for all tokens at once, not inside the serial walk
         # (a decode step, one token a row, works them out while it stages the token)
         width = heads * dk + (heads if beta is not None else 0)
@@ -220,8 +246,8 @@ def decay_scan(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign: float, beta
     native.recurrence_check(native.recurrence().ms_decay_scan(
         _ptr(o_out), _ptr(state), _ptr(q), _rows(q), _ptr(k), _rows(k), heads // groups, _ptr(v), _rows(v), _ptr(z), _rows(z),
         _ptr(z_bias), _ptr(decay_coef), float(z_sign), ready, _ptr(beta), 0 if beta is None else _rows(beta), _ptr(ctx.cu_q),
-        _ptr(ctx.q_start), _ptr(ctx.state_slot), ctx.num_rows, heads, dk, dv, float(q_scale), int(delta), _dt(q.dtype),
-        _dt(z.dtype), int(head_decay), _ptr(v_scale), dv_in, ctx.stream))
+        _ptr(ctx.q_start), _ptr(ctx.state_slot), ctx.num_rows, heads, dk, dv, float(q_scale), 2 if bonus is not None else int(delta), _dt(q.dtype),
+        _dt(z.dtype), int(head_decay), _ptr(v_scale), dv_in, _ptr(bonus), ctx.stream))
 
 
 def conv_silu_unit(out, x, conv_state, weight, ctx, unit_heads: int, dk: int, other_heads: int, dv: int, unit_eps: float,
@@ -259,7 +285,7 @@ SEGMENT_MAX_DK = 320  # (what mends the outputs holds 32 tokens' queries and a c
 
 
 def _decay_scan_segmented(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign, ctx, heads, dk, dv, q_scale, head_decay=False,
-                          v_scale=None, dv_in=None) -> None:
+                          v_scale=None, dv_in=None, bonus=None) -> None:
     from types import SimpleNamespace
 
     t, dev, p, rows = o_out.shape[0], o_out.device, SEGMENTS, ctx.num_rows
@@ -274,7 +300,7 @@ def _decay_scan_segmented(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign, 
             ctx.step_cache[key] = seg
     seg_cu, seg_zero, seg_slot = seg
     dkz = 1 if head_decay else dk
-    if head_decay:
+    if head_decay or bonus is not None:
         decay = z
     else:
         decay = ctx.buffer("scan.decay", (t, heads * dk), torch.float32, dev)
@@ -288,12 +314,12 @@ def _decay_scan_segmented(o_out, state, q, k, v, z, z_bias, decay_coef, z_sign, 
     native.recurrence_check(lib.ms_decay_scan(
         _ptr(o_out), _ptr(ends), _ptr(q), _rows(q), _ptr(k), _rows(k), heads // groups, _ptr(v), _rows(v), _ptr(decay), _rows(decay),
         _ptr(z_bias), _ptr(decay_coef), float(z_sign), 1, None, 0, _ptr(pieces.cu_q), _ptr(pieces.q_start), _ptr(pieces.state_slot),
-        pieces.num_rows, heads, dk, dv, float(q_scale), 0, _dt(q.dtype), 0, int(head_decay), _ptr(v_scale), dv if dv_in is None else dv_in,
-        ctx.stream))
+        pieces.num_rows, heads, dk, dv, float(q_scale), 0 if bonus is None else 2, _dt(q.dtype), 0, int(head_decay), _ptr(v_scale),
+        dv if dv_in is None else dv_in, _ptr(bonus), ctx.stream))
     native.recurrence_check(lib.ms_segment_finish(
         _ptr(o_out), _ptr(state), _ptr(ends), _ptr(before), _ptr(cum), _ptr(decay), _rows(decay), _ptr(q), _rows(q), heads // groups,
         _ptr(seg_cu), _ptr(ctx.q_start), _ptr(ctx.state_slot), rows, t, p, heads, dk, dv, float(q_scale), _dt(q.dtype), int(head_decay),
-        ctx.stream), launches=3)
+        int(bonus is not None), ctx.stream), launches=3)
 
 
 CHUNK_MIN_TOKENS = 64  # steps with fewer tokens stay on the token-by-token walk
@@ -305,6 +331,20 @@ def chunk_scan_ok(q, k, v, dk: int, dv: int, ctx) -> bool:
         return False
     return (bool(native.recurrence().ms_chunk_supports(dk, dv))
             and all(x.data_ptr() % 16 == 0 and x.stride(0) % 8 == 0 for x in (q, k, v)))
+
+
+def _chunk_table(tokens: int, ctx, dev):
+    """(the most chunks of a step of this shape, (row and first token of every chunk, every row's first chunk)), made once per step."""
+    lib, rows = native.recurrence(), ctx.num_rows
+    most = int(lib.ms_chunk_max(tokens, rows))
+    table = ctx.step_cache.get("chunk.table") if hasattr(ctx, "step_cache") else None
+    if table is None:  # the same for every layer of the step
+        ints = torch.empty(2 * most + rows + 1, dtype=torch.int32, device=dev)
+        table = (ints[:2 * most], ints[2 * most:])
+        native.recurrence_check(lib.ms_chunk_table(_ptr(table[0]), _ptr(table[1]), _ptr(ctx.cu_q), rows, ctx.stream))
+        if hasattr(ctx, "step_cache"):
+            ctx.step_cache["chunk.table"] = table
+    return most, table
 
 
 def chunk_scan(o, state, q, k, v, decay, write, ctx, heads: int, dk: int, dv: int, q_scale: float, ones: bool) -> None:
@@ -320,14 +360,7 @@ def chunk_scan(o, state, q, k, v, decay, write, ctx, heads: int, dk: int, dv: in
     assert q.shape == (t, groups * dk) and k.shape == q.shape and v.shape == (t, heads * dv) and state.shape[1:] == (heads, dv + extra, dk)
     assert decay.shape == (t, heads) and (write is None or write.shape == (t, heads)) and ld_o >= dv + extra
     lib = native.recurrence()
-    most = int(lib.ms_chunk_max(t, rows))
-    table = ctx.step_cache.get("chunk.table") if hasattr(ctx, "step_cache") else None
-    if table is None:  # the same for every layer of the step
-        ints = torch.empty(2 * most + rows + 1, dtype=torch.int32, device=dev)
-        table = (ints[:2 * most], ints[2 * most:])
-        native.recurrence_check(lib.ms_chunk_table(_ptr(table[0]), _ptr(table[1]), _ptr(ctx.cu_q), rows, ctx.stream))
-        if hasattr(ctx, "step_cache"):
-            ctx.step_cache["chunk.table"] = table
+    most, table = _chunk_table(t, ctx, dev)
     shape = (most, heads, dv + extra, dk)
     added = ctx.buffer("chunk.added", shape, torch.float32, dev)
     before = ctx.buffer("chunk.before", (2, *shape), torch.bfloat16, dev)
@@ -367,13 +400,13 @@ GATE_KINDS = {"silu": 0, "sigmoid": 1}
 
 def head_norm_gate(out, o, weight, gate, eps: float, scale: float, gate_kind: str, stream=None) -> None:
     """out[t, h*dv + c] = scale * o[t, h, c] / sqrt(mean_c o^2 + eps) * weight[c] * act(gate[t, h*dv + c]);
-    ``o`` [T, heads, dv] float32, ``out`` and ``gate`` 2-d views, act SiLU or sigmoid."""
+    ``o`` [T, heads, dv] float32, ``out`` and ``gate`` 2-d views, act SiLU or sigmoid; ``weight`` [dv], or [heads * dv]: one per head."""
     t, heads, dv = o.shape
     _f32(o, weight)
-    assert out.shape == (t, heads * dv) and gate.shape == (t, heads * dv) and gate.dtype == out.dtype and weight.numel() == dv
+    assert out.shape == (t, heads * dv) and gate.shape == (t, heads * dv) and gate.dtype == out.dtype and weight.numel() in (dv, heads * dv)
     native.recurrence_check(native.recurrence().ms_head_norm_gate(
         _ptr(out), _rows(out), _ptr(o), _ptr(weight), _ptr(gate), _rows(gate), t, heads, dv, float(eps), float(scale),
-        GATE_KINDS[gate_kind], _dt(out.dtype), _stream(stream)))
+        GATE_KINDS[gate_kind], dv if weight.numel() == heads * dv else 0, _dt(out.dtype), _stream(stream)))
 
 
 # ---------------------------------------------------------------- csrc/block_ops.cu
@@ -510,8 +543,8 @@ def act_mul(out, gate_up, activation: str, stream=None) -> None:
 
 # ---------------------------------------------------------------- csrc/stream_ops.cu
 
-def embed_sum(residual, table, ctx, inv_freq=None, pair_table=None, pair=None, prev_token=None) -> None:
-    """residual[t] = table[id] (+ pair_table[row]) (+ the sinusoidal vector of the position), float32. ``pair`` = (buckets,
+def embed_sum(residual, table, ctx, inv_freq=None, pair_table=None, pair=None, prev_token=None, scale: float = 1.0) -> None:
+    """residual[t] = scale * table[id] (+ pair_table[row]) (+ the sinusoidal vector of the position), float32. ``pair`` = (buckets,
     mul_prev, mul_cur): row = (previous token * mul_prev + token * mul_cur) mod buckets, row ``buckets`` at position 0; the token
     before a portion's first one is the row's slot of ``prev_token`` (int32 [slots, 1]), which gets the portion's last token.
     ``inv_freq`` float32 [(width + 1) // 2]: entry 2i gets sin(position * inv_freq[i]), entry 2i + 1 the cosine."""
@@ -525,8 +558,8 @@ def embed_sum(residual, table, ctx, inv_freq=None, pair_table=None, pair=None, p
                             and prev_token.dtype == torch.int32)
     native.mixers_check(native.mixers().ms_embed_sum(
         _ptr(residual), _ptr(table), _ptr(pair_table), buckets, mul_prev, mul_cur, _ptr(inv_freq), _ptr(ctx.token_ids), _ptr(ctx.positions),
-        _ptr(ctx.row_of_token), _ptr(ctx.cu_q), _ptr(ctx.state_slot), _ptr(prev_token), t, hidden, table.shape[0], _dt(table.dtype),
-        ctx.stream))
+        _ptr(ctx.row_of_token), _ptr(ctx.cu_q), _ptr(ctx.state_slot), _ptr(prev_token), t, hidden, table.shape[0], float(scale),
+        _dt(table.dtype), ctx.stream))
 
 
 def add_normed_rmsnorm(out, residual, delta, weight, eps: float, delta_weight=None, delta_eps: float = 0.0, rows=None, num_rows=None,
@@ -543,6 +576,24 @@ def add_normed_rmsnorm(out, residual, delta, weight, eps: float, delta_weight=No
         _ptr(out), _ptr(residual), _ptr(delta), _ptr(delta_weight), 1 if delta_weight is None else delta_weight.numel(), float(delta_eps),
         _ptr(weight), weight.numel(), float(eps), _ptr(rows), n, hidden, int(write_residual and rows is None), _dt(out.dtype),
         _stream(stream)))
+
+
+def stream_norm(out, streams, y, mix, out_w, into, weight, eps: float, source=None, rows=None, num_rows=None, write: bool = True,
+                stream=None) -> None:
+    """Several residual streams: x_t = sum_s mix[s, t] x_s + out_w[t] y (as they are without ``y``), written to ``streams`` [T, S, W]
+    float32 unless rows are gathered; out[i] = rmsnorm(sum_s into[s] x_s) * weight (``into`` None: the sum). ``source``: where the old
+    streams are, when not in ``streams`` itself: [T, W], one stream that all are equal to. mix [S, S] (from, to), out_w and into
+    [S], weight [W] float32."""
+    t, s, w = streams.shape
+    _f32(streams, mix, out_w, into, weight, source)
+    n = out.shape[0] if num_rows is None else num_rows
+    assert out.is_contiguous() and out.shape[-1] == w and weight.numel() == w
+    assert y is None or (y.dtype == out.dtype and y.is_contiguous() and y.shape == (t, w) and mix.shape == (s, s) and out_w.numel() == s)
+    assert into is None or into.numel() == s
+    assert source is None or source.shape == (t, w)
+    native.mixers_check(native.mixers().ms_stream_norm(
+        _ptr(out), _ptr(streams), _ptr(streams if source is None else source), s if source is None else 1, s, _ptr(y), _ptr(mix), _ptr(out_w),
+        _ptr(into), _ptr(weight), float(eps), _ptr(rows), n, w, int(write and rows is None), _dt(out.dtype), _stream(stream)))
 
 
 # ---------------------------------------------------------------- csrc/gated_recurrence.cu
@@ -604,3 +655,68 @@ def rglru_scan(out, state, z, u, y, bias_r, bias_i, coef, y_bias, ctx) -> None:
     native.recurrence_check(native.recurrence().ms_rglru_scan(
         _ptr(out), _ptr(state), _ptr(z), _ptr(u), _ptr(y), _rows(y), _ptr(bias_r), _ptr(bias_i), _ptr(coef), _ptr(y_bias), _ptr(ctx.cu_q),
         _ptr(ctx.q_start), _ptr(ctx.state_slot), ctx.num_rows, t, c, c // blocks, int(ctx.decode_only), _dt(out.dtype), ctx.stream))
+
+
+# ---------------------------------------------------------------- csrc/time_mix.cu
+
+TIME_CHUNKS = True  # prompts in bfloat16 by chunks on the tensor cores (tests compare with the token-by-token walk)
+
+
+def channel_decay(out, z, w0, stream=None) -> None:
+    """out [T, C] float32 = exp(-exp(z + w0)); ``z`` [T, C] a view, ``w0`` [C] float32."""
+    t, c = z.shape
+    _f32(out, w0)
+    assert out.shape == (t, c) and w0.numel() == c
+    native.recurrence_check(native.recurrence().ms_channel_decay(_ptr(out), _ptr(z), _rows(z), _ptr(w0), t, c, _dt(z.dtype), _stream(stream)))
+
+
+def time_step_ok(dk: int, dv: int, rank: int) -> bool:
+    """Whether ``time_step`` takes these sizes."""
+    return dk % 4 == 0 and (4 * dk + dv + rank) * 4 <= 48 * 1024
+
+
+def time_step(out, state, r, k, v, gate, low, w2, w0, bonus, norm_w, eps: float, ctx, heads: int) -> None:
+    """A step of one token per row of time mixing with a bonus, from the low-rank input of the decays to the gated, normed heads:
+    d = exp(-exp(w2 low + w0)), o = (S + diag(bonus) k v^T)^T r, S = diag(d) S + k v^T per head with S the request's slot of ``state``
+    [slots, heads, dv, dk] float32 (zero where a row starts its sequence); out [T, heads * dv] = o over its root mean square per head,
+    times norm_w, times silu(gate). r, k [T, heads * dk], v, gate [T, heads * dv]: columns of the same rows; low [T, rank] a view;
+    w2 [heads * dk, rank] in the run's dtype; w0, bonus, norm_w float32."""
+    t = out.shape[0]
+    _f32(state, w0, bonus, norm_w)
+    dv, dk = state.shape[2], state.shape[3]
+    ld, rank = _rows(r), w2.shape[1]
+    assert ctx.decode_only and out.is_contiguous() and out.shape == (t, heads * dv) and state.shape[1] == heads
+    assert r.shape == k.shape == (t, heads * dk) and v.shape == gate.shape == (t, heads * dv) and _rows(k) == _rows(v) == _rows(gate) == ld
+    assert low.shape == (t, rank) and w2.shape == (heads * dk, rank) and w2.is_contiguous()
+    assert r.dtype == k.dtype == v.dtype == gate.dtype == low.dtype == w2.dtype == out.dtype
+    assert w0.numel() == heads * dk and bonus.numel() == heads * dk and norm_w.numel() == heads * dv
+    native.recurrence_check(native.recurrence().ms_time_step(
+        _ptr(out), _ptr(state), _ptr(r), _ptr(k), _ptr(v), _ptr(gate), ld, _ptr(low), _rows(low), _ptr(w2), rank, _ptr(w0), _ptr(bonus),
+        _ptr(norm_w), float(eps), _ptr(ctx.cu_q), _ptr(ctx.q_start), _ptr(ctx.state_slot), ctx.num_rows, heads, dk, dv, _dt(out.dtype), ctx.stream))
+
+
+def time_chunks_ok(r, k, v, dk: int, dv: int, ctx) -> bool:
+    """Whether ``time_chunks`` takes these operands: bfloat16, a step that is not all single tokens, heads of whole 16 bytes."""
+    if not TIME_CHUNKS or r.dtype != torch.bfloat16 or ctx.decode_only or r.shape[0] < CHUNK_MIN_TOKENS:
+        return False
+    return (bool(native.recurrence().ms_time_chunk_supports(dk, dv))
+            and all(x.data_ptr() % 16 == 0 and x.stride(0) % 8 == 0 for x in (r, k, v)))
+
+
+def time_chunks(o, state, r, k, v, z, w0, bonus, ctx, heads: int, dk: int, dv: int) -> None:
+    """The bonus rule with decays exp(-exp(z + w0)) per key channel over chunks of 64 tokens on the tensor cores (``csrc/time_mix.cu``),
+    from each request's slot of ``state`` [slots, heads, dv, dk] float32 and back into it. r, k [T, heads * dk], v [T, heads * dv]
+    bfloat16 views, z [T, heads * dk] float32; o [T, heads, dv] float32."""
+    t, dev = o.shape[0], o.device
+    _f32(o, state, w0, bonus)
+    assert o.shape == (t, heads, dv) and state.shape[1:] == (heads, dv, dk) and z.dtype == torch.float32
+    assert r.shape == k.shape == z.shape == (t, heads * dk) and v.shape == (t, heads * dv) and w0.numel() == bonus.numel() == heads * dk
+    most, table = _chunk_table(t, ctx, dev)
+    shape = (most, heads, dv, dk)
+    added = ctx.buffer("chunk.added", shape, torch.float32, dev)
+    before = ctx.buffer("chunk.before", (2, *shape), torch.bfloat16, dev)
+    passed = ctx.buffer("chunk.passed", (most, heads, dk), torch.float32, dev)
+    native.recurrence_check(native.recurrence().ms_time_chunks(
+        _ptr(o), _ptr(state), _ptr(r), _rows(r), _ptr(k), _rows(k), _ptr(v), _rows(v), _ptr(z), _rows(z), _ptr(w0), _ptr(bonus), _ptr(added),
+        _ptr(before[0]), _ptr(before[1]), _ptr(passed), _ptr(table[0]), _ptr(table[1]), _ptr(ctx.cu_q), _ptr(ctx.q_start), _ptr(ctx.state_slot),
+        ctx.num_rows, most, heads, dk, dv, ctx.stream), launches=3)

@@ -129,7 +129,10 @@ def mixers():
     _declare(lib, "ms_scale_f32", [_p, _f, _ll, _p])
     _declare(lib, "ms_axpby", [_p, _p, _p, _f, _f, _ll, _i, _p])
     _declare(lib, "ms_head_gate", [_p, _i, _p, _p, _i, _i, _i, _i, _i, _f, _i, _p])
-    _declare(lib, "ms_qkv_prepare", [_p] * 4 + [_i] * 4 + [_p] * 7 + [_i] * 8 + [_f, _i, _i, _p, _i, _p, _p, _p, _i, _f, _f])
+    _declare(lib, "ms_qkv_prepare", [_p] * 4 + [_i] * 4 + [_p] * 7 + [_i] * 8 + [_f, _i, _i, _p, _i, _p, _p, _p, _i, _f, _f, _p, _i, _p])
+    _declare(lib, "ms_tanh_inplace", [_p, _f, _ll, _i, _p])
+    _declare(lib, "ms_token_mixes", [_p, _p, _p, _p, _i, _p, _p, _p, _p, _i, _i, _i, _p])
+    _declare(lib, "ms_stream_norm", [_p, _p, _p, _i, _i, _p, _p, _p, _p, _p, _f, _p, _i, _i, _i, _i, _p])
     _declare(lib, "ms_add_rmsnorm_scaled", [_p, _p, _p, _f, _p, _f, _p, _f, _i, _i, _i, _i, _p])
     _declare(lib, "ms_stream_concat", [_p, _p, _p, _f, _p, _p, _i, _i, _i, _i, _i, _i, _p])
     _declare(lib, "ms_add_row_vector", [_p, _p, _i, _i, _p])
@@ -146,7 +149,7 @@ def mixers():
     _declare(lib, "ms_shift_state_update", [_p, _p, _p, _p, _i, _i, _i, _p])
     _declare(lib, "ms_clamped_glu", [_p, _p, _p, _i, _i, _f, _f, _f, _i, _p])
     _declare(lib, "ms_sum_bias", [_p, _p, _p, _p, _i, _i, _i, _p])
-    _declare(lib, "ms_embed_sum", [_p, _p, _p, _ll, _ll, _ll, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _p])
+    _declare(lib, "ms_embed_sum", [_p, _p, _p, _ll, _ll, _ll, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _f, _i, _p])
     _declare(lib, "ms_add_normed_rmsnorm", [_p, _p, _p, _p, _i, _f, _p, _i, _f, _p, _i, _i, _i, _i, _p])
     return lib
 
@@ -158,16 +161,16 @@ def recurrence():
     _declare(lib, "ms_recurrence_set_pdl", [_i], None)
     lib.ms_recurrence_set_pdl(int(pdl_enabled()))
     _declare(lib, "ms_decay_scan", [_p, _p, _p, _i, _p, _i, _i, _p, _i, _p, _i, _p, _p, _f, _i, _p, _i, _p, _p, _p,
-                                    _i, _i, _i, _i, _f, _i, _i, _i, _i, _p, _i, _p])
+                                    _i, _i, _i, _i, _f, _i, _i, _i, _i, _p, _i, _p, _p])
     _declare(lib, "ms_decay_step", [_p, _p, _p, _i, _p, _i, _i, _p, _i, _p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _p, _i, _i, _p])
     _declare(lib, "ms_segment_setup", [_p, _p, _p, _p, _i, _i, _p])
-    _declare(lib, "ms_segment_finish", [_p, _p, _p, _p, _p, _p, _i, _p, _i, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _i, _p])
+    _declare(lib, "ms_segment_finish", [_p, _p, _p, _p, _p, _p, _i, _p, _i, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _p])
     _declare(lib, "ms_decay_from_logits", [_p, _p, _i, _p, _p, _f, _p, _i, _i, _i, _i, _i, _p])
     _declare(lib, "ms_conv_silu_unit", [_p, _p, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _f, _i, _p, _p])
     _declare(lib, "ms_ssm_step_decay", [_p, _p, _i, _p, _p, _i, _i, _i, _p])
     _declare(lib, "ms_gated_group_norm", [_p, _i, _p, _p, _i, _p, _p, _i, _p, _i, _i, _i, _i, _f, _i, _p])
     _declare(lib, "ms_conv_state_update", [_p, _p, _i, _p, _p, _p, _i, _i, _i, _i, _p])
-    _declare(lib, "ms_head_norm_gate", [_p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _f, _i, _i, _p])
+    _declare(lib, "ms_head_norm_gate", [_p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _f, _i, _i, _i, _p])
     _declare(lib, "ms_mlstm_gates", [_p, _p, _p, _p, _i, _p, _p, _p, _p, _p, _i, _i, _i, _f, _i, _i, _p])
     _declare(lib, "ms_mlstm_output", [_p, _i, _p, _i, _p, _p, _p, _i, _i, _i, _i, _f, _f, _i, _p])
     _declare(lib, "ms_conv_bias", [_p, _p, _i, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _p])
@@ -175,6 +178,10 @@ def recurrence():
     _declare(lib, "ms_chunk_supports", [_i, _i])
     _declare(lib, "ms_chunk_table", [_p, _p, _p, _i, _p])
     _declare(lib, "ms_chunk_scan", [_p, _i, _p, _p, _i, _p, _i, _i, _p, _i] + [_p] * 11 + [_i] * 5 + [_f, _i, _p])
+    _declare(lib, "ms_channel_decay", [_p, _p, _i, _p, _i, _i, _i, _p])
+    _declare(lib, "ms_time_step", [_p, _p, _p, _p, _p, _p, _i, _p, _i, _p, _i, _p, _p, _p, _f, _p, _p, _p, _i, _i, _i, _i, _i, _p])
+    _declare(lib, "ms_time_chunk_supports", [_i, _i])
+    _declare(lib, "ms_time_chunks", [_p, _p] + [_p, _i] * 4 + [_p] * 11 + [_i] * 5 + [_p])
     _declare(lib, "ms_rglru_scan", [_p, _p, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p])
     return lib
 
@@ -185,13 +192,13 @@ def experts():
     _declare(lib, "ms_experts_last_error", [], c_char_p)
     _declare(lib, "ms_experts_set_pdl", [_i], None)
     lib.ms_experts_set_pdl(int(pdl_enabled()))
-    _declare(lib, "ms_expert_route", [_p, _p, _p, _i, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _i, _p, _p, _p, _p, _i, _i])
+    _declare(lib, "ms_expert_route", [_p, _p, _p, _i, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _i, _p, _p, _p, _p, _i, _i, _i, _f])
     _declare(lib, "ms_expert_max_tiles", [_i, _i])
     _declare(lib, "ms_expert_plan", [_p, _p, _p, _p, _p, _p, _i, _i, _p])
     _declare(lib, "ms_expert_max_tiles_of", [_i, _i, _i])
     _declare(lib, "ms_expert_plan_of", [_p, _p, _p, _p, _p, _p, _i, _i, _i, _p])
     _declare(lib, "ms_expert_gather", [_p, _p, _i, _p, _p, _i, _i, _i, _p])
-    _declare(lib, "ms_expert_gemm", [_p, _p, _i, _p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p])
+    _declare(lib, "ms_expert_gemm", [_p, _p, _i, _p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _f, _f, _f, _i, _p])
     _declare(lib, "ms_expert_combine", [_p, _p, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _p, _p, _p])
     return lib
 
@@ -215,7 +222,7 @@ def gemm_tc():
     _declare(lib, "ms_gemm_tc_set_pdl", [_i], None)
     _declare(lib, "ms_gemm_tc_bf16", [_p, _p, _p, _i, _i, _i, _i, _p, _p])
     _declare(lib, "ms_gemm_tc_decode_bf16", [_p, _p, _p, _i, _i, _i, _p, _p])
-    _declare(lib, "ms_gemm_tc_experts_bf16", [_p, _p, _p, _i, _i, _i, _i, _i, _p, _p, _p, _i, _p, _p])
+    _declare(lib, "ms_gemm_tc_experts_bf16", [_p, _p, _p, _i, _i, _i, _i, _i, _p, _p, _p, _i, _f, _f, _f, _p, _p])
     _declare(lib, "ms_gemm_tc_set_config", [_i], None)
     _declare(lib, "ms_gemm_tc_prefers", [_i, _i, _i, _i])
     _declare(lib, "ms_gemm_tc_qkv_bf16", [_p, _p, _p, _i, _i, _i, _i] + [_p] * 9 + [_i, _f, _p, _p])

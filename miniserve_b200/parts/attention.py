@@ -48,12 +48,15 @@ class GQAttention(Part):
     mixer's own reach: 0 for everything, for a mixer whose cache another mixer with a longer reach reads). With
     ``kv_source`` = ``shared`` these run on the general path too: the projection holds q (and the gate) alone.
     ``query_temperature`` = (coef, every): the prepared query at position p is multiplied by
-    1 + coef ln(floor((p + 1) / every) + 1), in float32."""
+    1 + coef ln(floor((p + 1) / every) + 1), in float32.
+    ``value_mix``: the layers with this flag share values: a layer's values become (1 - share) v + share v_first before they are cached,
+    with ``share`` a learned number (tensor ``v_share``) and v_first the same token's values in the first such layer of the pass (which
+    keeps its own; what it declares is not used)."""
     shape_static = True
     input_weight = "w_qkv"  # the attribute that holds the input product's (stacked) matrix; its first ``input_rows`` rows are real
     NAMES = dict(q="q_proj.weight", k="k_proj.weight", v="v_proj.weight", o="o_proj.weight", q_norm="q_norm.weight",
                  k_norm="k_norm.weight", gate="g_proj.weight", sink="sink", q_bias="q_proj.bias", k_bias="k_proj.bias",
-                 v_bias="v_proj.bias", temp="temperature", r1="distance.r1", r2="distance.r2")
+                 v_bias="v_proj.bias", temp="temperature", r1="distance.r1", r2="distance.r2", v_share="v_share")
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
@@ -94,13 +97,17 @@ class GQAttention(Part):
             raise ValueError(f"query_temperature={temp}: the number of positions per step must be positive")
         self.keep_first = int(spec.get("keep_first") or 0)
         self.cache_window = spec.get("cache_window")
+        self.value_mix = bool(spec.get("value_mix", False))
+        if self.value_mix and self.kv_source != "own":
+            raise ValueError("value_mix changes the values a layer caches: it needs a cache of its own")
         if self.keep_first < 0 or (self.keep_first and not self.window):
             raise ValueError(f"keep_first={self.keep_first} needs a window that it reaches behind")
         self.names = {**self.NAMES, **dict(spec.get("names") or {})}
         self.adjacent = getattr(self.position, "pairing", "halves") == "adjacent"  # how the position encoding pairs channels
         self.general = bool(self.out_gate or self.value_dim != self.head_dim or self.adjacent or self.learned_sink or self.softcap
                             or self.chunk or getattr(self.position, "table_only", False) or self.unit_norm or self.qkv_bias
-                            or self.head_temperature or self.distance_bias or self.keep_first or self.query_temperature or spec.get("general"))
+                            or self.head_temperature or self.distance_bias or self.keep_first or self.query_temperature or self.value_mix
+                            or spec.get("general"))
         self.w_sink = None
         self.extras = None
         self.w_bias = self.w_temp = None
@@ -149,6 +156,8 @@ class GQAttention(Part):
                 w[n["v_bias"]] = WeightDecl((self.kv_heads * self.value_dim,), precision="float32")
         if self.head_temperature:
             w[n["temp"]] = WeightDecl((self.heads,), precision="float32", init="ones_normal")
+        if self.value_mix:
+            w[n["v_share"]] = WeightDecl((), precision="float32")
         if self.distance_bias:
             w[n["r1"]] = WeightDecl((self.heads,), precision="float32")
             w[n["r2"]] = WeightDecl((self.heads,), precision="float32", init="ones_normal")
@@ -188,6 +197,7 @@ class GQAttention(Part):
             parts = (n["q_bias"], n["k_bias"], n["v_bias"]) if self.owns_cache else (n["q_bias"],)
             self.w_bias = torch.cat([tensors[p].float().reshape(-1) for p in parts]).contiguous()
         self.w_temp = tensors[n["temp"]].float().contiguous() if self.head_temperature else None
+        self.w_v_share = tensors[n["v_share"]].float().reshape(1).contiguous() if self.value_mix else None
         r1 = tensors[n["r1"]].float().contiguous() if self.distance_bias else None
         r2 = tensors[n["r2"]].float().contiguous() if self.distance_bias else None
         if self.learned_sink or self.softcap or self.chunk or self.distance_bias or self.keep_first:
@@ -209,10 +219,16 @@ class GQAttention(Part):
         t = x.shape[0]
         dt, dev = self.env.dtype, x.device
         nq, nkv, dk, dv, dc = self.heads, self.kv_heads, self.head_dim, self.value_dim, self.cache_dim
+        v_first = ctx.step_cache.get("attn.v_first") if self.value_mix else None
+        leads = self.value_mix and v_first is None  # the first of the layers that share values: later ones read its projection's rows
         if proj is None:
-            proj = ops.linear(x, self.w_qkv, stream=ctx.stream, out=ctx.buffer("attn.qkv", (t, self.w_qkv.shape[0]), dt, dev))
+            proj = ops.linear(x, self.w_qkv, stream=ctx.stream, out=ctx.buffer("attn.qkv_first" if leads else "attn.qkv", (t, self.w_qkv.shape[0]), dt, dev))
+        elif leads:
+            raise NotImplementedError("value_mix: the first layer's projection has to outlive it, so it is not a caller's")
         at_k = nq * dk
         at_v, at_g = ((nq + nkv) * dk, (nq + nkv) * dk + nkv * dv) if self.owns_cache else (at_k, at_k)
+        if leads:
+            ctx.step_cache["attn.v_first"] = proj[:, at_v:at_g]
         q = ctx.buffer("attn.q", (t, nq, dc), dt, dev)
         _, rotary_dim = self.position.kernel_table()
         own = self.owns_cache  # else the keys and values are another entry's, as its cache holds them
@@ -221,7 +237,7 @@ class GQAttention(Part):
                         self.position.step_table(ctx), rotary_dim, self.adjacent, self.qk_norm_eps,
                         ctx.positions, ctx.row_of_token, ctx.page_indptr[cache.group], ctx.page_indices[cache.group],
                         cache.page_size, ctx.status, stream=ctx.stream, bias=self.w_bias, unit_norm=self.unit_norm, q_scale=self.w_temp,
-                        q_temp=self.query_temperature)
+                        q_temp=self.query_temperature, v_other=v_first, v_share=self.w_v_share if v_first is not None else None)
         att = ctx.buffer("attn.out", (t, nq, dc), dt, dev)
         ops.attention(att, q, cache.k, cache.v, ctx, cache.group, self.scale, self.reach, self.sink, extras=self.extras)
         if raw:  # the caller takes attention's output [T, heads, D] itself (no gate, values as wide as the cache's heads)

@@ -176,12 +176,16 @@ class ResidualStream:
     that has not been added yet (the last feed-forward output), so that the add can be
     fused into the next norm. The addend counts ``pending_scale`` times (a block that adds its
     sublayers' output times a constant hands the constant on instead of scaling the tensor).
-    ``pending_norm``: a norm part that the addend passes before it is added (a block that norms its sublayers' outputs)."""
+    ``pending_norm``: a norm part that the addend passes before it is added (a block that norms its sublayers' outputs).
+    ``links``: there are several streams (``stream_count``), ``total`` is [T, streams, hidden], or [T, hidden] for streams that are all
+    equal; the part that says how the pending sublayer output enters them and how they mix (None: nothing is pending)."""
 
     total: torch.Tensor
     pending: torch.Tensor | None = None
     pending_scale: float = 1.0
     pending_norm: "Part | None" = None
+    links: "Part | None" = None
+    stream_count: int = 1
 
 
 def param(spec: PartSpec, key: str, typ: type | None = None) -> Any:

@@ -91,6 +91,61 @@ class SandwichBlock(Part):
         return ResidualStream(total, self.feed_forward.forward(x, ctx), pending_norm=self.norms["norm2b"])
 
 
+class StreamLinks(Part):
+    """How one sublayer is linked to several residual streams x_1 .. x_S (hyper-connections): it reads sum_s in[s] x_s, and its output y
+    changes all streams at once, x_t <- sum_s mix[s, t] x_s + out[t] y. Tensors ``in`` [S], ``out`` [S] and ``mix`` [S, S] (from, to),
+    float32. Parameters: ``streams``."""
+    shape_static = True
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.streams = int(spec["streams"])
+
+    def weights(self):
+        s, f32 = self.streams, dict(precision="float32", init="ones_normal")
+        return {"in": WeightDecl((s,), **f32), "out": WeightDecl((s,), **f32), "mix": WeightDecl((s, s), precision="float32")}
+
+    def bind(self, tensors):
+        self.w_in, self.w_out, self.w_mix = (tensors[k].float().contiguous() for k in ("in", "out", "mix"))
+
+
+@register_part("block", "linked_streams")
+class LinkedStreamsBlock(Part):
+    """Pre-norm sublayers over several residual streams: u = sum_s in[s] x_s, y = sublayer(norm(u)), then the streams take y and
+    mix (``StreamLinks``; one set for the mixer, one for the feed-forward). The update of the streams by one sublayer and the norm ahead of
+    the next run as one kernel, so a block hands its last output on as pending together with its links. Parameters: ``names`` (mixer /
+    feed_forward / norm1 / norm2 / links1 / links2 -> tensor-name prefixes), ``streams``. A layer without a feed-forward has neither it nor
+    norm2 nor links2."""
+    shape_static = True
+
+    def __init__(self, spec, env: BuildEnv, layer: LayerSpec | None = None):
+        super().__init__(spec, env)
+        if layer is None:
+            raise ValueError("a block is built from its LayerSpec (use build_block)")
+        names = dict(spec.get("names") or {})
+        self.streams = int(spec["streams"])
+        self.has_ff = layer.feed_forward is not None
+        self.names = {k: names[k] for k in ("mixer", "norm1", "links1") + (("feed_forward", "norm2", "links2") if self.has_ff else ())}
+        self.mixer = build_part("mixer", layer.mixer, env)
+        self.norm1 = build_part("norm", layer.norms["norm1"], env)
+        links = PartSpec("stream_links", dict(streams=self.streams))
+        self.links1 = StreamLinks(links, env)
+        self.feed_forward = build_part("feed_forward", layer.feed_forward, env) if self.has_ff else None
+        self.norm2 = build_part("norm", layer.norms["norm2"], env) if self.has_ff else None
+        self.links2 = StreamLinks(links, env) if self.has_ff else None
+
+    def sub_parts(self):
+        return {name: getattr(self, k) for k, name in self.names.items()}
+
+    def forward(self, stream: ResidualStream, ctx, cache) -> ResidualStream:
+        x = self.norm1.forward_streams(stream, ctx, self.links1.w_in, self.streams)
+        stream = ResidualStream(stream.total, self.mixer.forward(x, ctx, cache), links=self.links1, stream_count=self.streams)
+        if not self.has_ff:
+            return stream
+        x = self.norm2.forward_streams(stream, ctx, self.links2.w_in, self.streams)
+        return ResidualStream(stream.total, self.feed_forward.forward(x, ctx), links=self.links2, stream_count=self.streams)
+
+
 @register_part("block", "parallel_residual")
 class ParallelResidualBlock(Part):
     """h = norm1(x); x += residual_mult * (mixer(h) + feed_forward(h)): one norm, both sublayers read its output.

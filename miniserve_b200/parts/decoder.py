@@ -165,6 +165,9 @@ class DecoderModel:
             if entry.transition is not None:
                 stream = self.transitions[entry.transition].forward(stream, ctx, self.embedding, entry.transition_arg)
             stream = self.layers[entry.layer].forward(stream, ctx, caches[i])
+        if stream.links is not None:  # several streams: the head reads their sum
+            x = self.final_norm.forward_streams(stream, ctx, None, stream.stream_count, rows=ctx.logit_rows, num_rows=ctx.num_logit_rows, write=False)
+            return self.head.forward(x, ctx)
         extra = {"delta_scale": stream.pending_scale} if stream.pending_scale != 1.0 else {}
         if stream.pending_norm is not None:
             extra["delta_norm"] = stream.pending_norm

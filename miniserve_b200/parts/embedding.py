@@ -34,14 +34,14 @@ class TokenEmbedding(Part):
 
 @register_part("embedding", "summed_embedding")
 class SummedEmbedding(Part):
-    """h = table[id] (+ bigram[row]) (+ sinusoid(position)), summed in float32 by one kernel.
+    """h = scale * table[id] (+ bigram[row]) (+ sinusoid(position)), summed in float32 by one kernel.
 
     ``bigram`` (a mapping with ``buckets``, ``mul_prev``, ``mul_cur``, ``name``; or absent): a second table of buckets + 1 rows, read
     at row (previous token * mul_prev + token * mul_cur) mod buckets, and at its last row for a sequence's first token. The
     previous token is state of the request (one int32 in its slot), so that a portion or a decoded token continues from it.
     ``sinusoid`` (a base, or absent): entry 2i of the position's vector is sin(position * base^(-2i / hidden)), entry 2i + 1 the
     cosine (frequencies worked out in float64 and rounded once; the angle and its sine and cosine are float32).
-    Parameters: ``vocab``, ``hidden``, ``name`` (the table's full name), ``bigram``, ``sinusoid``."""
+    Parameters: ``vocab``, ``hidden``, ``name`` (the table's full name), ``bigram``, ``sinusoid``, ``scale`` (1)."""
     shape_static = True
 
     def __init__(self, spec, env):
@@ -49,6 +49,7 @@ class SummedEmbedding(Part):
         self.vocab = param(spec, "vocab", int)
         self.hidden = param(spec, "hidden", int)
         self.name = param(spec, "name", str)
+        self.scale = float(spec.params.get("scale", 1.0))
         b = spec.get("bigram")
         self.pair = (int(b["buckets"]), int(b["mul_prev"]), int(b["mul_cur"])) if b else None
         self.pair_name = str(b["name"]) if b else None
@@ -75,7 +76,8 @@ class SummedEmbedding(Part):
 
     def forward(self, ctx, cache=None) -> torch.Tensor:
         residual = torch.empty((ctx.num_tokens, self.hidden), dtype=torch.float32, device=self.table.device)
-        ops.embed_sum(residual, self.table, ctx, self.inv_freq, self.pair_table, self.pair, cache.state if self.pair else None)
+        ops.embed_sum(residual, self.table, ctx, self.inv_freq, self.pair_table, self.pair, cache.state if self.pair else None,
+                      scale=self.scale)
         return residual
 
 
@@ -84,7 +86,8 @@ class LinearHead(Part):
     """logits = x @ W^T, no bias (miniserve/model/qwen3.py:186); with ``tied`` the matrix is the
     embedding table itself and no tensor of its own is read (miniserve/model/weights.py:116-119,
     135-136). Logits are returned in float32. Parameters: ``vocab``, ``hidden``, ``tied``,
-    ``name``, ``tied_to``, optional ``scale`` (the float32 logits are multiplied by it)."""
+    ``name``, ``tied_to``, optional ``scale`` (the float32 logits are multiplied by it)
+    and ``softcap`` (then logits become softcap * tanh(logits / softcap))."""
     shape_static = True
 
     def __init__(self, spec, env):
@@ -95,6 +98,9 @@ class LinearHead(Part):
         self.name = param(spec, "name", str)
         self.tied_to = spec.get("tied_to")
         self.scale = float(spec.get("scale") or 1.0)
+        self.softcap = float(spec.get("softcap") or 0.0)
+        if self.softcap < 0:
+            raise ValueError(f"a head's softcap={self.softcap} must not be negative")
         if self.tied and not self.tied_to:
             raise ValueError("a tied head needs 'tied_to', the name of the embedding tensor")
 
@@ -111,4 +117,6 @@ class LinearHead(Part):
             ops.linear(x, self.weight, out=logits, stream=ctx.stream)
             if self.scale != 1.0:
                 ops.scale_(logits, self.scale, stream=ctx.stream)
+            if self.softcap:
+                ops.tanh_(logits, self.softcap, stream=ctx.stream)
         return logits

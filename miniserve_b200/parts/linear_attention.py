@@ -318,6 +318,89 @@ class SelectiveStateSpace(Part):
         return ops.linear(feat, self.w_o, stream=ctx.stream, out=ctx.buffer("ssm.proj", (t, self.hidden), dt, dev))
 
 
+@register_part("mixer", "time_mix")
+class TimeMix(Part):
+    """Time mixing with a decay per key channel and a bonus for the token's own write (RWKV-style). Each of r, k, v, g and w reads its
+    own mix of the token's input and the one before, x + (x_before - x) mu (zeros before the first token; the last input of a
+    portion is state):
+
+        d_t = exp(-exp(W_w2 tanh(W_w1 mix_w) + w0)),   o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t,   S_t = diag(d_t) S_(t-1) + k_t v_t^T
+
+    per head, S [dim, dim]; each head's o is divided by its root mean square, the heads side by side times a weight, times silu(W_g mix_g),
+    then W_o. One launch makes the five mixes, one batched product r|k|v|g, two small ones the decays' logits (the second in float32);
+    a decode step goes from the low-rank input to the gated heads in one kernel, prompts in bfloat16 run by chunks on the tensor cores,
+    the rest token by token (``csrc/time_mix.cu``, ``csrc/recurrence.cu``). S is float32.
+    Parameters: ``hidden``, ``heads``, ``head_dim``, ``decay_rank``, ``eps``, ``names`` (r, k, v, g, o, norm, w1, w2, w0, u and mu: the
+    prefix of mu.r .. mu.w)."""
+    shape_static = True
+    INPUTS = ("r", "k", "v", "g", "w")
+    NAMES = dict(r="r_proj.weight", k="k_proj.weight", v="v_proj.weight", g="g_proj.weight", o="o_proj.weight", norm="norm.weight",
+                 w1="w_proj.0.weight", w2="w_proj.1.weight", w0="w_proj.bias", u="bonus", mu="mix.")
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.hidden = param(spec, "hidden", int)
+        self.heads = param(spec, "heads", int)
+        self.dim = param(spec, "head_dim", int)
+        self.rank = param(spec, "decay_rank", int)
+        self.eps = param(spec, "eps", float)
+        self.names = {**self.NAMES, **dict(spec.get("names") or {})}
+        self.feature_width = self.heads * self.dim
+
+    def cache_need(self):
+        return (FixedState((self.heads, self.dim, self.dim), torch.float32), FixedState((self.hidden,), self.env.dtype))
+
+    def weights(self):
+        n, c, w, f32 = self.names, self.feature_width, self.hidden, dict(precision="float32")
+        out = {n["mu"] + x: WeightDecl((w,), **f32) for x in self.INPUTS}
+        out.update({n[x]: WeightDecl((c, w)) for x in "rkvg"})
+        out.update({n["w1"]: WeightDecl((self.rank, w)), n["w2"]: WeightDecl((c, self.rank)), n["w0"]: WeightDecl((c,), **f32),
+                    n["u"]: WeightDecl((self.heads, self.dim), **f32), n["norm"]: WeightDecl((c,), init="ones_normal", **f32),
+                    n["o"]: WeightDecl((w, c))})
+        return out
+
+    def stacks(self):
+        return {"rkvg_proj.weight": tuple(self.names[x] for x in "rkvg")}
+
+    def bind(self, tensors):
+        n = self.names
+        self.w_in = self.joined(tensors, "rkvg_proj.weight", self.stacks()["rkvg_proj.weight"]).view(4, self.feature_width, self.hidden)
+        self.w_mu = torch.stack([tensors[n["mu"] + x].float() for x in self.INPUTS]).contiguous()
+        rank = _pad8(self.rank)  # a rank that is no multiple of 8: zero rows and columns (tanh of zero is zero)
+        self.w_w1, self.w_w2 = _pad_rows(tensors[n["w1"]], rank), _pad_cols(tensors[n["w2"]], rank)
+        self.w_w0, self.w_u, self.w_norm = (tensors[n[k]].float().reshape(-1).contiguous() for k in ("w0", "u", "norm"))
+        self.w_o = tensors[n["o"]].contiguous()
+
+    def features(self, x: torch.Tensor, ctx, cache, out: torch.Tensor) -> None:
+        t, dt, dev = x.shape[0], self.env.dtype, self.w_o.device
+        h, d, c = self.heads, self.dim, self.feature_width
+        state, before = cache
+        mixed = ctx.buffer("time.mixes", (5, t, self.hidden), dt, dev)
+        ops.token_mixes(mixed, x, before.state, self.w_mu, ctx)
+        proj = ctx.buffer("time.in", (t, 4, c), dt, dev)
+        ops.linear_heads(mixed[:4].transpose(0, 1), self.w_in, proj, stream=ctx.stream)
+        low = ops.linear(mixed[4], self.w_w1, stream=ctx.stream, out=ctx.buffer("time.low", (t, self.w_w1.shape[0]), dt, dev))
+        ops.tanh_(low, stream=ctx.stream)
+        r, k, v, g = (proj[:, i] for i in range(4))
+        if ctx.decode_only and ops.time_step_ok(d, d, self.w_w2.shape[1]):
+            ops.time_step(out, state.state, r, k, v, g, low, self.w_w2, self.w_w0, self.w_u, self.w_norm, self.eps, ctx, h)
+            return
+        z = ops.linear(low, self.w_w2, stream=ctx.stream, out=ctx.buffer("time.z", (t, c), torch.float32, dev))
+        o = ctx.buffer("time.o", (t, h, d), torch.float32, dev)
+        if ops.time_chunks_ok(r, k, v, d, d, ctx):
+            ops.time_chunks(o, state.state, r, k, v, z, self.w_w0, self.w_u, ctx, h, d, d)
+        else:
+            ops.channel_decay(z, z, self.w_w0, stream=ctx.stream)
+            ops.decay_scan(o, state.state, r, k, v, z, None, None, 0.0, None, ctx, h, d, d, 1.0, delta=False, bonus=self.w_u)
+        ops.head_norm_gate(out, o, self.w_norm, g, self.eps, 1.0, "silu", stream=ctx.stream)
+
+    def forward(self, x, ctx, cache):
+        t, dt, dev = x.shape[0], self.env.dtype, self.w_o.device
+        feat = ctx.buffer("time.feat", (t, self.feature_width), dt, dev)
+        self.features(x, ctx, cache, feat)
+        return ops.linear(feat, self.w_o, stream=ctx.stream, out=ctx.buffer("time.proj", (t, self.hidden), dt, dev))
+
+
 @register_part("mixer", "mlstm")
 class MatrixMemory(Part):
     """A matrix memory with exponential gates and a running maximum (the mLSTM of xLSTM): per head, with log gates

@@ -179,7 +179,7 @@ class RoutedExperts(Part):
         y = sum over the top c of  weight_scale * s_e * expert_e(x),   expert_e(x) = W_down[e] (act(W_gate[e] x) * (W_up[e] x))
 
     The router's outputs form ``group_count`` equal groups of neighbours; a group's score is the largest c in it and only
-    outputs of the ``group_keep`` best groups can be chosen. The last ``identity`` router outputs are identity experts:
+    outputs of the ``group_keep`` best groups can be chosen (``group_best`` n: a group's score is the sum of its n largest). The last ``identity`` router outputs are identity experts:
     they have no tensors and their output is x itself (times the weight). Weights use s without the correction and are
     not renormalised unless ``renormalize``. The router (its product, softmax and choice) is float32; its matrix and the
     correction stay float32. The experts' matrices are stacked at load ([E, 2 I, hidden]: an expert's gate rows, then its
@@ -187,7 +187,7 @@ class RoutedExperts(Part):
     expert; the plan of that sort lives on the device, so the part's launches follow from the number of tokens alone.
 
     Parameters: ``hidden``, ``intermediate``, ``experts``, ``top``; optional ``identity`` (0), ``group_count`` (1),
-    ``group_keep`` (1), ``weight_scale`` (1.0), ``renormalize`` (False), ``correction`` (True: a tensor of that name is
+    ``group_keep`` (1), ``group_best`` (1), ``weight_scale`` (1.0), ``renormalize`` (False; ``renorm_eps`` (0) is added to the sum), ``correction`` (True: a tensor of that name is
     added to the scores for the choice), ``activation`` (``silu`` or ``gelu_tanh``), ``score`` (``softmax``), ``names``
     (router, correction, gate, up, down -> tensor names; ``expert``: the prefix of expert e with ``{}`` for e).
 
@@ -201,7 +201,10 @@ class RoutedExperts(Part):
     part) without a gate, expert_e(x) = W_down[e] act(W_up[e] x) with ``activation`` = ``relu_squared``. ``weigh`` = ``input``: a
     weight w multiplies its expert's input, expert_e(w x), instead of the output; for an expert that is homogeneous of degree
     two (the square of relu without a gate; w is not negative) that is w^2 expert_e(x), so the router hands on squared
-    weights and the products read x as it is."""
+    weights and the products read x as it is.
+
+    ``activation`` = ``clamped_glu``: an expert is a ``clamped_glu`` part without biases (``limit``, ``alpha`` (1.702), ``up_shift`` (1)), and
+    so is the shared one, with constants of its own in ``shared_glu`` (a mapping of the same three; absent: the experts')."""
     shape_static = True
     NAMES = dict(router="router.weight", correction="router.correction", expert="experts.{}.", gate="gate_proj.weight",
                  up="up_proj.weight", down="down_proj.weight", router_bias="router.bias", shared="shared.", shared_gate="shared.gate")
@@ -215,12 +218,18 @@ class RoutedExperts(Part):
         self.top = param(spec, "top", int)
         self.group_count = int(spec.get("group_count", 1) or 1)
         self.group_keep = int(spec.get("group_keep", 1) or 1)
+        self.group_best = int(spec.get("group_best", 1) or 1)
         self.weight_scale = float(spec.get("weight_scale", 1.0))
+        self.renorm_eps = float(spec.get("renorm_eps", 0.0) or 0.0)
         self.renormalize = bool(spec.get("renormalize", False))
         self.has_correction = bool(spec.params.get("correction", True))
         self.activation = spec.get("activation", "silu")
         if self.activation not in ops.experts.ACTIVATIONS:
             raise ValueError(f"routed_experts knows the activations {sorted(ops.experts.ACTIVATIONS)}, not {self.activation!r}")
+        glu = dict(limit=spec.get("limit"), alpha=float(spec.get("alpha", 1.702)), up_shift=float(spec.params.get("up_shift", 1.0)))
+        self.clamps = None  # (limit, alpha, shift); a negative limit: no clamps
+        if self.activation == "clamped_glu":
+            self.clamps = (-1.0 if glu["limit"] is None else float(glu["limit"]), glu["alpha"], glu["up_shift"])
         self.score = spec.get("score", "softmax")
         if self.score not in ops.experts.SCORES:
             raise ValueError(f"routed_experts scores by {sorted(ops.experts.SCORES)}, not {self.score!r}")
@@ -244,7 +253,12 @@ class RoutedExperts(Part):
         self.shared_inter = int(spec.get("shared") or 0)
         self.shared_gated = bool(spec.params.get("shared_gated", True)) and self.shared_inter > 0
         self.shared = None
-        if self.shared_inter:
+        if self.shared_inter and self.clamps is not None:
+            n = self.names
+            self.shared = ClampedGLU(PartSpec("clamped_glu", dict(hidden=self.hidden, intermediate=self.shared_inter, bias=False,
+                                                                  names=dict(gate=n["gate"], up=n["up"], down=n["down"]),
+                                                                  **{**glu, **dict(spec.get("shared_glu") or {})})), env)
+        elif self.shared_inter:
             n = self.names
             self.shared = DenseMLP(PartSpec("dense_mlp", dict(hidden=self.hidden, intermediate=self.shared_inter, activation=self.activation,
                                                               names=dict(up=n["up"], down=n["down"]))), env) if not self.gated else SwiGLU(PartSpec("swiglu", dict(hidden=self.hidden, intermediate=self.shared_inter, activation=self.activation,
@@ -295,7 +309,8 @@ class RoutedExperts(Part):
         gate = ctx.buffer("moe.shared_gate", (t,), torch.float32, dev) if self.shared_gated else None
         ops.experts.expert_route(idx, wgt, x, self.w_router, self.w_correction, self.top, self.group_count, self.group_keep,
                                  self.weight_scale, self.renormalize, stream=ctx.stream, logit_bias=self.w_router_bias,
-                                 gate_w=self.w_shared_gate, gate_out=gate, score=self.score, square_weights=self.weigh == "input")
+                                 gate_w=self.w_shared_gate, gate_out=gate, score=self.score, square_weights=self.weigh == "input",
+                                 group_best=min(self.group_best, self.outputs // self.group_count), renorm_eps=self.renorm_eps)
         return idx, wgt
 
     def forward(self, x, ctx) -> torch.Tensor:
@@ -317,11 +332,14 @@ class RoutedExperts(Part):
             xs = ctx.buffer("moe.xs", (slots, self.hidden), dt, dev)
             ops.experts.expert_gather(xs, x, perm, meta, self.top, stream=ctx.stream)
             ops.experts.expert_products_tc(act, xs, self.w_gate_up, tiles, meta, offsets, self.gated, stream=ctx.stream,
-                                           relu_squared=not self.gated)
+                                           relu_squared=not self.gated, clamps=self.clamps)
             ops.experts.expert_products_tc(y, act, self.w_down, tiles, meta, offsets, False, stream=ctx.stream)
         else:
-            first = ops.experts.expert_gate_up if self.gated else ops.experts.expert_up
-            first(act, x, self.w_gate_up, perm, self.top, tiles, meta, offsets, self.activation, stream=ctx.stream)
+            if self.gated:
+                ops.experts.expert_gate_up(act, x, self.w_gate_up, perm, self.top, tiles, meta, offsets, self.activation, stream=ctx.stream,
+                                           clamps=self.clamps)
+            else:
+                ops.experts.expert_up(act, x, self.w_gate_up, perm, self.top, tiles, meta, offsets, self.activation, stream=ctx.stream)
             ops.experts.expert_down(y, act, self.w_down, tiles, meta, offsets, stream=ctx.stream)
         out = ctx.buffer("moe.out", (t, self.hidden), dt, dev)
         shared = self.shared.forward(x, ctx) if self.shared is not None else None

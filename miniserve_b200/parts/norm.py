@@ -73,6 +73,26 @@ class RMSNorm(Part):
         return out
 
 
+    def forward_streams(self, stream, ctx, into: torch.Tensor | None, count: int, rows: torch.Tensor | None = None,
+                        num_rows: int | None = None, write: bool = True) -> torch.Tensor:
+        """The norm of a combination of several residual streams (``ResidualStream.links``): the pending sublayer output first
+        enters all streams, then ``into`` (float32 [streams]; None: the sum) says what the norm reads. One launch; the new streams
+        become the stream's total [T, streams, size] (a total [T, size] stands for streams that are all equal)."""
+        if self.scalar or self.unit_offset:
+            raise NotImplementedError("a norm over several streams takes a weight per coordinate, as it is")
+        total, links = stream.total, stream.links
+        t = total.shape[0]
+        n = t if rows is None else (num_rows if num_rows is not None else rows.numel())
+        out = ctx.buffer("norm.out", (n, self.size), self.env.dtype, total.device)
+        single = total.dim() == 2
+        streams = ctx.buffer("streams", (t, count, self.size), torch.float32, total.device) if single else total
+        ops.stream_norm(out, streams, stream.pending, links.w_mix if links is not None else None, links.w_out if links is not None else None,
+                        into, self.float_weight, self.eps, source=total if single else None, rows=rows, num_rows=n, write=write, stream=ctx.stream)
+        if stream.pending is not None and write and rows is None:
+            stream.total, stream.pending, stream.links = streams, None, None
+        return out
+
+
 @register_part("norm", "dynamic_tanh")
 class DynamicTanh(Part):
     """y = tanh(alpha x) * weight + bias in the place of a norm: no mean, no variance, so no reduction
