@@ -431,6 +431,20 @@ def vumedra_config(width: int, ff: int, runs: int, vocab: int, heads: int, kv_he
             "embedding": {"bigram": {"buckets": 100003, "mul_prev": 31, "mul_cur": 7}}, "layers": layers}
 
 
+def tunadra_config(width: int, ff: int, runs: int, vocab: int, heads: int, kv_heads: int) -> dict:
+    """A Tunadra model at a real model's layer sizes: two residual streams, in turns of four layers three of time mixing (heads of 64, as
+    wide as the model, decays of rank 64) and one of attention (the Qwen3 model's heads of 128, values mixed with the first such
+    layer's). The feed-forward of every layer is 16 experts of ff / 4 in 4 groups, of which a token uses 3 out of the best 2 groups,
+    beside a shared expert of ff / 4 (the products of a token equal the Qwen3 layer's)."""
+    att = {"dim": 128, "heads": heads, "kv_heads": kv_heads, "scale": 128 ** -0.5, "v_mix": True, "vdim": 128}
+    wkv = {"dim": 64, "heads": width // 64, "decay_rank": 64}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4, "limit": 7.0}, "shared": {"ff": ff // 4, "limit": 7.0},
+           "router": {"experts": 16, "top": 3, "scale": 1.5, "groups": {"count": 4, "keep": 2}}}
+    layers = [{"type": "attention" if i % 4 == 2 else "wkv", "mixer": dict(att if i % 4 == 2 else wkv), "mlp": dict(moe)} for i in range(runs)]
+    return {"architecture": "Tunadra", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "streams": 2,
+            "logit_softcap": 30.0, "layers": layers}
+
+
 def bytes_per_step_of_weights(model) -> int:
     """Bytes of weights a step reads: every run of a layer reads that layer's tensors (a layer that runs twice
     counts twice), plus the norm before the head, the head and the parts between layers."""
@@ -479,7 +493,7 @@ def kernel_times(run_step, repeats: int = 3) -> dict:
 
 
 def run_fekulix(args, design: str = "fekulix") -> dict:
-    """Prefill and decode of a design (Fekulix, Mugipel, Rofozen, Kovusun, Vumedra) beside Qwen3 at equal width, depth, feed-forward and vocabulary."""
+    """Prefill and decode of a design (Fekulix, Mugipel, Rofozen, Kovusun, Vumedra, Tunadra) beside Qwen3 at equal width, depth, feed-forward and vocabulary."""
     import torch
 
     from miniserve_b200.config import preset
@@ -487,7 +501,8 @@ def run_fekulix(args, design: str = "fekulix") -> dict:
     from miniserve_b200.engine.step import StepRow
 
     peaks = load_peaks()
-    make = {"fekulix": fekulix_config, "mugipel": mugipel_config, "rofozen": rofozen_config, "kovusun": kovusun_config, "vumedra": vumedra_config}[design]
+    make = {"fekulix": fekulix_config, "mugipel": mugipel_config, "rofozen": rofozen_config, "kovusun": kovusun_config, "vumedra": vumedra_config,
+            "tunadra": tunadra_config}[design]
     out = {"impl": "ours", "config": design, "dtype": "bf16", "data": "synthetic (random-init weights, uniform token ids)",
            "batch": args.batch, "context": CONTEXT, "prefill_tokens": PREFILL_TOKENS, "peaks": peaks["source"], "sizes": {}}
     steps = min(args.steps, 64)
@@ -510,6 +525,10 @@ def run_fekulix(args, design: str = "fekulix") -> dict:
             args_of = (q["hidden_size"], q["intermediate_size"], q["num_hidden_layers"], q["vocab_size"], q["num_attention_heads"],
                        q["num_key_value_heads"])
             beside += [("rofozen", rofozen_config(*args_of)), ("kovusun", kovusun_config(*args_of))]
+        if design == "tunadra":  # the closest designs: a recurrence with a decay per key channel; clamped and routed experts; a matrix memory
+            args_of = (q["hidden_size"], q["intermediate_size"], q["num_hidden_layers"], q["vocab_size"], q["num_attention_heads"],
+                       q["num_key_value_heads"])
+            beside += [("fekulix", fekulix_config(*args_of)), ("kovusun", kovusun_config(*args_of)), ("vumedra", vumedra_config(*args_of))]
         for name, raw in [(design, f)] + beside:
             llm = LLM(random=raw, weights_seed=0, dtype="bfloat16", kv_pool_tokens=10 * (CONTEXT + steps + 64) + 4096, page_size=16,
                       max_running=16, chunked_prefill_size=2048, cuda_graph=not args.no_graph)
@@ -720,10 +739,10 @@ def main() -> int:
     ap.add_argument("--no-graph", action="store_true", help="run decode steps without CUDA graphs")
     ap.add_argument("--profile-range", action="store_true",
                     help="bracket the timed steps with cudaProfilerStart/Stop (for ncu --profile-from-start off)")
-    ap.add_argument("--config", choices=["0.6b", "8b", "32b", "fekulix", "mugipel", "rofozen", "kovusun", "vumedra"], default="0.6b",
+    ap.add_argument("--config", choices=["0.6b", "8b", "32b", "fekulix", "mugipel", "rofozen", "kovusun", "vumedra", "tunadra"], default="0.6b",
                     help="0.6b: the benchmark line; 8b, 32b: the larger workloads through Engine.generate (a line of their own); "
-                         "fekulix, mugipel, rofozen, kovusun, vumedra: prefill and decode of that design beside Qwen3 at equal sizes (a line of its own)")
-    ap.add_argument("--kernels", action="store_true", help="with --config fekulix, mugipel, rofozen, kovusun or vumedra: also device time per kernel of a prompt step and a decode step")
+                         "fekulix, mugipel, rofozen, kovusun, vumedra, tunadra: prefill and decode of that design beside Qwen3 at equal sizes (a line of its own)")
+    ap.add_argument("--kernels", action="store_true", help="with --config fekulix, mugipel, rofozen, kovusun, vumedra or tunadra: also device time per kernel of a prompt step and a decode step")
     ap.add_argument("--only", choices=["all", "decode", "prefill"], default="all",
                     help="measure only the decode steps or only the prefill (for profiling); the line then lacks the other parts")
     args = ap.parse_args()
@@ -736,7 +755,7 @@ def main() -> int:
         args.warmup = 3
     global PROFILE_RANGE
     PROFILE_RANGE = args.profile_range
-    if args.config in ("fekulix", "mugipel", "rofozen", "kovusun", "vumedra") and args.impl == "ours":
+    if args.config in ("fekulix", "mugipel", "rofozen", "kovusun", "vumedra", "tunadra") and args.impl == "ours":
         result = run_fekulix(args, args.config)
     elif args.config != "0.6b" and args.impl == "ours":
         result = run_workload(args)

@@ -78,7 +78,19 @@ def _vumedra(width, vocab, ff, pattern, dim, heads, kv_heads, memory_heads, bloc
                 embedding={"bigram": {"buckets": 2 * vocab + 1, "mul_prev": 31, "mul_cur": 3}}, layers=layers)
 
 
+def _tunadra(width, vocab, ff, pattern, dim, heads, kv_heads, time_heads, time_dim, rank) -> dict:
+    """A Tunadra config.json of two streams: ``pattern`` is a string of A (attention, values mixed with the first such layer's) and W (time
+    mixing); routed feed-forwards."""
+    mixers = {"A": ("attention", {"dim": dim, "heads": heads, "kv_heads": kv_heads, "scale": dim ** -0.5, "v_mix": True, "vdim": dim}),
+              "W": ("wkv", {"decay_rank": rank, "dim": time_dim, "heads": time_heads})}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4, "limit": 4.0}, "shared": {"ff": ff // 2, "limit": 4.0},
+           "router": {"experts": 6, "top": 2, "scale": 1.5, "groups": {"count": 3, "keep": 2}}}
+    return dict(architecture="Tunadra", width=width, vocab=vocab, norm={"eps": 1e-5}, embedding={"scale": 8.0}, streams=2, logit_softcap=30.0,
+                layers=[{"type": mixers[ch][0], "mixer": dict(mixers[ch][1]), "mlp": dict(moe)} for ch in pattern])
+
+
 PRESETS: dict[str, dict] = {
+    "tunadra-tiny": _tunadra(96, 503, 160, "WAWA", 32, 6, 2, 3, 32, 16),
     "vumedra-tiny": _vumedra(96, 503, 160, "RAMR", 32, 6, 2, 3, 6),
     "kovusun-tiny": _kovusun(96, 503, 160, 6, 2, 32, 48),
     "mugipel-tiny": _mugipel(

@@ -194,34 +194,56 @@ __global__ void token_mixes_kernel(T* __restrict__ out, const T* __restrict__ h,
   }
 }
 
+// The same for bfloat16 rows that are a multiple of 8 wide and start on 16 bytes: eight channels per thread, RUN consecutive tokens per CTA,
+// which read the mixes' factors once.
+template <int RUN>
 __global__ void token_mixes_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ h, __nv_bfloat16* __restrict__ state,
                                           const float* __restrict__ mix, int mixes, const int* __restrict__ row_of_token,
                                           const int* __restrict__ cu_q, const int* __restrict__ q_start, const int* __restrict__ state_slot,
-                                          int width) {
+                                          int tokens, int width) {
   pdl_prologue();
-  const int t = blockIdx.x;
-  const int row = row_of_token[t];
-  const bool first = t == cu_q[row];
-  __nv_bfloat16* slot = state + (size_t)state_slot[row] * width;
-  const __nv_bfloat16* prev = first ? (q_start[row] > 0 ? slot : nullptr) : h + (size_t)(t - 1) * width;
-  const __nv_bfloat16* newest = h + (size_t)(cu_q[row + 1] - 1) * width;
-  const size_t plane = (size_t)gridDim.x * width;
-  for (int c = threadIdx.x * 8; c < width; c += blockDim.x * 8) {
-    float x[8], p[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    bf16x8_to_float(*reinterpret_cast<const uint4*>(h + (size_t)t * width + c), x);
-    if (prev) bf16x8_to_float(*reinterpret_cast<const uint4*>(prev + c), p);
+  const int t0 = blockIdx.x * RUN;
+  const __nv_bfloat16* prev[RUN];
+  __nv_bfloat16* slot[RUN];  // where this token's CTA leaves the portion's last h
+  const __nv_bfloat16* newest[RUN];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) p[e] -= x[e];
+  for (int q = 0; q < RUN; ++q) {
+    const int t = min(t0 + q, tokens - 1);
+    const int row = row_of_token[t];
+    const bool first = t == cu_q[row];
+    __nv_bfloat16* sl = state + (size_t)state_slot[row] * width;
+    prev[q] = first ? (q_start[row] > 0 ? sl : nullptr) : h + (size_t)(t - 1) * width;
+    slot[q] = first && t0 + q < tokens ? sl : nullptr;
+    newest[q] = h + (size_t)(cu_q[row + 1] - 1) * width;
+  }
+  const size_t plane = (size_t)tokens * width;
+  for (int c = threadIdx.x * 8; c < width; c += blockDim.x * 8) {
+    float x[RUN][8], p[RUN][8];
+#pragma unroll
+    for (int q = 0; q < RUN; ++q) {
+      bf16x8_to_float(*reinterpret_cast<const uint4*>(h + (size_t)min(t0 + q, tokens - 1) * width + c), x[q]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) p[q][e] = 0.f;
+      if (prev[q]) bf16x8_to_float(*reinterpret_cast<const uint4*>(prev[q] + c), p[q]);
+      if (slot[q]) *reinterpret_cast<uint4*>(slot[q] + c) = *reinterpret_cast<const uint4*>(newest[q] + c);
+    }
+#pragma unroll
+    for (int q = 0; q < RUN; ++q)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) p[q][e] -= x[q][e];
     for (int m = 0; m < mixes; ++m) {
       const float* mm = mix + (size_t)m * width + c;
       const float4 ma = *reinterpret_cast<const float4*>(mm), mb = *reinterpret_cast<const float4*>(mm + 4);
       const float mv[8] = {ma.x, ma.y, ma.z, ma.w, mb.x, mb.y, mb.z, mb.w};
-      float y[8];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) y[e] = fmaf(p[e], mv[e], x[e]);
-      *reinterpret_cast<uint4*>(out + m * plane + (size_t)t * width + c) = float_to_bf16x8(y);
+      for (int q = 0; q < RUN; ++q) {
+        if (t0 + q >= tokens) break;
+        float y[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[e] = fmaf(p[q][e], mv[e], x[q][e]);
+        *reinterpret_cast<uint4*>(out + m * plane + (size_t)(t0 + q) * width + c) = float_to_bf16x8(y);
+      }
     }
-    if (first) *reinterpret_cast<uint4*>(slot + c) = *reinterpret_cast<const uint4*>(newest + c);
   }
 }
 
@@ -931,8 +953,13 @@ MS_EXPORT int ms_token_mixes(void* out, const void* h, void* state, const float*
   const int threads = width >= 1024 ? 256 : 128;
   if (dtype == MS_BF16 && width % 8 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)state % 16 == 0 &&
       (uintptr_t)mix % 16 == 0) {
-    MS_LAUNCH(token_mixes_bf16x8_kernel, tokens, width >= 2048 ? 256 : 128, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)h,
-              (__nv_bfloat16*)state, mix, mixes, row_of_token, cu_q, q_start, state_slot, width);
+    const int th = width >= 2048 ? 256 : 128;
+    if (tokens >= 1024)
+      MS_LAUNCH(token_mixes_bf16x8_kernel<4>, (tokens + 3) / 4, th, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)h, (__nv_bfloat16*)state, mix,
+                mixes, row_of_token, cu_q, q_start, state_slot, tokens, width);
+    else
+      MS_LAUNCH(token_mixes_bf16x8_kernel<1>, tokens, th, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)h, (__nv_bfloat16*)state, mix, mixes,
+                row_of_token, cu_q, q_start, state_slot, tokens, width);
     return 0;
   }
   if (dtype == MS_F32)

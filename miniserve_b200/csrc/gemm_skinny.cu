@@ -33,14 +33,26 @@ __device__ __forceinline__ uint4 ldg_stream(const void* p) {
 // MODE 3: W is a stacked gate|up weight [2N, K] and out [M, N] = silu(x Wg^T) * (x Wu^T) in bf16
 // (miniserve/model/qwen3.py:128-131): the CTA takes 8 gate rows as the lower half of its fragments
 // and the 8 up rows that belong to them as the upper half, so both factors of an output meet in it.
-// Both products are rounded to bfloat16 before the activation, as when they are stored in between.
+// Both products are rounded to bfloat16 before the activation, as when they are stored in between. MODE 6: the same stack, but out =
+// g sigmoid(alpha g) (u + shift) with g capped at limit and u held within +-limit (a negative limit: neither).
+// Several inputs: rows [i * x_rows, (i + 1) * x_rows) of W (a multiple of a CTA's rows) multiply the input at X + i * x_stride (the last input
+// takes all rows behind). MODE 5: out columns from tanh_from on become tanh of the product.
+struct SkinnyExtras {
+  int x_rows;            // 0: one input
+  long long x_stride;
+  int x_last;            // number of inputs - 1
+  int tanh_from;
+  float limit, alpha, shift;
+};
 template <int MT, int MODE>
 __global__ void __launch_bounds__(SK_THREADS)
 gemm_skinny_kernel(void* __restrict__ out, const __nv_bfloat16* __restrict__ X, const __nv_bfloat16* __restrict__ W,
-                   int M, int N, int K) {
+                   int M, int N, int K, const SkinnyExtras ex) {
+  constexpr bool GATED = MODE == 3 || MODE == 6;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-  const int n0 = blockIdx.x * (MODE == 3 ? 8 : SK_ROWS);
+  const int n0 = blockIdx.x * (GATED ? 8 : SK_ROWS);
+  if (ex.x_rows) X += min(n0 / ex.x_rows, ex.x_last) * ex.x_stride;
   const int k_begin = 0, k_len = K;
   const int xs_stride = K + 32;  // bf16 elements: rows 64 bytes apart modulo 128, so 16-byte reads of two rows do not collide
   __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(smem_raw);
@@ -48,8 +60,8 @@ gemm_skinny_kernel(void* __restrict__ out, const __nv_bfloat16* __restrict__ X, 
   // this warp's part of the slice, in chunks of 32 k (8 per lane of a quad)
   const int per_warp = ((k_len + SK_WARPS * 32 - 1) / (SK_WARPS * 32)) * 32;
   const int wk_begin = warp * per_warp, wk_end = min(k_len, wk_begin + per_warp);
-  const int upper = MODE == 3 ? N : 8;  // where the fragments' upper rows come from, relative to the lower ones
-  const bool row_a = n0 + g < N, row_b = MODE == 3 ? row_a : n0 + g + 8 < N;
+  const int upper = GATED ? N : 8;  // where the fragments' upper rows come from, relative to the lower ones
+  const bool row_a = n0 + g < N, row_b = GATED ? row_a : n0 + g + 8 < N;
   const __nv_bfloat16* wa_ptr = W + (size_t)(n0 + (row_a ? g : 0)) * K + k_begin + 8 * t;
   const __nv_bfloat16* wb_ptr = W + (size_t)(n0 + (row_b ? g + upper : 0)) * K + k_begin + 8 * t;
 
@@ -126,7 +138,7 @@ gemm_skinny_kernel(void* __restrict__ out, const __nv_bfloat16* __restrict__ X, 
     base[(g + 8) * TOK + 8 * j + 2 * t + 1] = acc[j][3];
   }
   __syncthreads();
-  if (MODE == 3) {
+  if (GATED) {
     for (int idx = tid; idx < 8 * TOK; idx += SK_THREADS) {
       const int tok = idx >> 3, row = idx & 7;
       if (tok >= M || n0 + row >= N) continue;
@@ -136,8 +148,16 @@ gemm_skinny_kernel(void* __restrict__ out, const __nv_bfloat16* __restrict__ X, 
         sg += red[(size_t)w * SK_ROWS * TOK + row * TOK + tok];
         su += red[(size_t)w * SK_ROWS * TOK + (row + 8) * TOK + tok];
       }
-      const float gt = __bfloat162float(__float2bfloat16_rn(sg)), up = __bfloat162float(__float2bfloat16_rn(su));
-      reinterpret_cast<__nv_bfloat16*>(out)[(size_t)tok * N + n0 + row] = __float2bfloat16_rn(gt / (1.0f + expf(-gt)) * up);
+      float gt = __bfloat162float(__float2bfloat16_rn(sg)), up = __bfloat162float(__float2bfloat16_rn(su));
+      if (MODE == 6) {
+        if (ex.limit >= 0.f) {
+          gt = fminf(gt, ex.limit);
+          up = fminf(fmaxf(up, -ex.limit), ex.limit);
+        }
+        reinterpret_cast<__nv_bfloat16*>(out)[(size_t)tok * N + n0 + row] = __float2bfloat16_rn(gt / (1.0f + expf(-ex.alpha * gt)) * (up + ex.shift));
+      } else {
+        reinterpret_cast<__nv_bfloat16*>(out)[(size_t)tok * N + n0 + row] = __float2bfloat16_rn(gt / (1.0f + expf(-gt)) * up);
+      }
     }
   } else
   for (int idx = tid; idx < SK_ROWS * TOK; idx += SK_THREADS) {
@@ -157,6 +177,9 @@ gemm_skinny_kernel(void* __restrict__ out, const __nv_bfloat16* __restrict__ X, 
     } else if (MODE == 4) {
       const float z = fmaxf(__bfloat162float(__float2bfloat16_rn(s)), 0.f);
       reinterpret_cast<__nv_bfloat16*>(out)[o] = __float2bfloat16_rn(z * z);
+    } else if (MODE == 5) {
+      const float z = __bfloat162float(__float2bfloat16_rn(s));
+      reinterpret_cast<__nv_bfloat16*>(out)[o] = __float2bfloat16_rn(n0 + row >= ex.tanh_from ? tanhf(z) : z);
     } else {
       reinterpret_cast<float*>(out)[o] = s;
     }
@@ -310,7 +333,7 @@ static int launch_skinny_stream(void* out, const void* X, const void* W, int M, 
 }
 
 template <int MT, int MODE>
-static int launch_skinny(void* out, const void* X, const void* W, int M, int N, int K, cudaStream_t stream) {
+static int launch_skinny(void* out, const void* X, const void* W, int M, int N, int K, cudaStream_t stream, const SkinnyExtras& ex = SkinnyExtras{}) {
   const size_t smem_x = (size_t)MT * 8 * (K + 32) * 2;
   const size_t smem_red = (size_t)SK_WARPS * SK_ROWS * MT * 8 * 4;
   const size_t smem = smem_x > smem_red ? smem_x : smem_red;
@@ -321,8 +344,8 @@ static int launch_skinny(void* out, const void* X, const void* W, int M, int N, 
     MS_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = smem;
   }
-  dim3 grid(ceil_div(N, MODE == 3 ? 8 : SK_ROWS));
-  MS_LAUNCH(kernel, grid, SK_THREADS, smem, stream, out, (const __nv_bfloat16*)X, (const __nv_bfloat16*)W, M, N, K);
+  dim3 grid(ceil_div(N, MODE == 3 || MODE == 6 ? 8 : SK_ROWS));
+  MS_LAUNCH(kernel, grid, SK_THREADS, smem, stream, out, (const __nv_bfloat16*)X, (const __nv_bfloat16*)W, M, N, K, ex);
   return 0;
 }
 
@@ -387,4 +410,27 @@ MS_EXPORT int ms_gemm_skinny_gate_up_bf16(void* out, const void* X, const void* 
   if (int rc = check_skinny(W, M, N, K, 0)) return rc;
   MS_CHECK_ARG((uintptr_t)X % 16 == 0, "gemm_skinny: the activations must be 16-byte aligned");
   return M > 8 ? launch_skinny<2, 3>(out, X, W, M, N, K, stream) : launch_skinny<1, 3>(out, X, W, M, N, K, stream);
+}
+
+// The clamped form: out = g sigmoid(alpha g) (u + shift), g = min(X Wg^T, limit), u = clamp(X Wu^T, -limit, limit); limit < 0: no clamps.
+MS_EXPORT int ms_gemm_skinny_clamped_glu_bf16(void* out, const void* X, const void* W, int M, int N, int K, float limit, float alpha, float shift,
+                                              cudaStream_t stream) {
+  if (M == 0 || N == 0) return 0;
+  if (int rc = check_skinny(W, M, N, K, 0)) return rc;
+  MS_CHECK_ARG((uintptr_t)X % 16 == 0, "gemm_skinny: the activations must be 16-byte aligned");
+  const SkinnyExtras ex{0, 0, 0, 0, limit, alpha, shift};
+  return M > 8 ? launch_skinny<2, 6>(out, X, W, M, N, K, stream, ex) : launch_skinny<1, 6>(out, X, W, M, N, K, stream, ex);
+}
+
+// Products of several inputs in one launch: out [M, N] bfloat16; rows [i * rows_each, (i + 1) * rows_each) of W [N, K] multiply input i
+// of X [inputs, M, K] (the last one takes all rows behind); columns from tanh_from on become tanh of the product.
+MS_EXPORT int ms_gemm_skinny_inputs_bf16(void* out, const void* X, const void* W, int M, int N, int K, int inputs, int rows_each, int tanh_from,
+                                         cudaStream_t stream) {
+  if (M == 0 || N == 0) return 0;
+  if (int rc = check_skinny(W, M, N, K, 0)) return rc;
+  MS_CHECK_ARG((uintptr_t)X % 16 == 0, "gemm_skinny: the activations must be 16-byte aligned");
+  MS_CHECK_ARG(inputs >= 1 && rows_each >= SK_ROWS && rows_each % SK_ROWS == 0 && (long long)(inputs - 1) * rows_each < N,
+               "gemm_skinny: %d inputs of %d rows each of %d", inputs, rows_each, N);
+  const SkinnyExtras ex{rows_each, (long long)M * K, inputs - 1, tanh_from, 0.f, 0.f, 0.f};
+  return M > 8 ? launch_skinny<2, 5>(out, X, W, M, N, K, stream, ex) : launch_skinny<1, 5>(out, X, W, M, N, K, stream, ex);
 }

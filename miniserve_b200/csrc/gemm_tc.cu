@@ -1380,6 +1380,28 @@ MS_EXPORT int ms_gemm_tc_bf16(void* out, const void* A, const void* W, int M, in
   }
 }
 
+// Tiles of the grouped products: 1: 256 columns of W (gated) or 128, one CTA an SM; 2: 128, a shorter ring, two CTAs an SM, so that one CTA's
+// epilogue hides behind the other's products. 0: chosen from the rows per expert (measured on B200 with 16 experts, both products: 2,048 tokens x 3
+// choices at 768 of 1024: 75.6 us with 2, 87.7 with 1; at 1536 of 2048: 182 against 202; 8 tokens: 39.5 against 35.6 and 94 against 65).
+static int g_grouped_config = 0;
+MS_EXPORT void ms_gemm_tc_set_grouped(int config) { g_grouped_config = config; }
+
+template <int EPI>
+static int launch_grouped_gated(void* out, const void* A, const void* W, int rows, int N, int experts, int K, const TcGroups& grp, int max_tiles,
+                                int* status, cudaStream_t stream) {
+  const bool narrow = g_grouped_config ? g_grouped_config == 2 : rows >= 128 * experts;
+  if (narrow) return launch_tc_grouped<128, 3, EPI>(out, A, W, rows, N, experts, 2 * N, K, N, grp, max_tiles, status, stream);
+  return launch_tc_grouped<256, 4, EPI>(out, A, W, rows, N, experts, 2 * N, K, N, grp, max_tiles, status, stream);
+}
+
+template <int EPI>
+static int launch_grouped_plain(void* out, const void* A, const void* W, int rows, int N, int experts, int K, const TcGroups& grp, int max_tiles,
+                                int* status, cudaStream_t stream) {
+  const bool narrow = g_grouped_config ? g_grouped_config == 2 : rows >= 128 * experts;
+  if (narrow) return launch_tc_grouped<128, 3, EPI>(out, A, W, rows, N, experts, N, K, 0, grp, max_tiles, status, stream);
+  return launch_tc_grouped<128, 5, EPI>(out, A, W, rows, N, experts, N, K, 0, grp, max_tiles, status, stream);
+}
+
 // The experts' products of a routed feed-forward over rows sorted by expert (tiles of 128 rows, (expert, first row)
 // each; meta[0] tiles; offsets[e + 1] ends expert e's rows; at most max_tiles tiles).
 // gated = 1: W [E, 2 N, K] (an expert's gate rows, then its up rows), out [rows, N] bfloat16 = silu(A gate^T) * (A up^T);
@@ -1397,15 +1419,15 @@ MS_EXPORT int ms_gemm_tc_experts_bf16(void* out, const void* A, const void* W, i
   MS_CHECK_ARG((long long)experts * (gated == 1 || gated == 3 ? 2 : 1) * N < (1LL << 31), "gemm_tc_experts: the weights have too many rows");
   if (gated == 3) {
     const TcGroups grp{tiles, meta, offsets, 2 * N, {limit, alpha, shift}};
-    return launch_tc_grouped<256, 4, TC_CLAMPED_GLU>(out, A, W, rows, N, experts, 2 * N, K, N, grp, max_tiles, status, stream);
+    return launch_grouped_gated<TC_CLAMPED_GLU>(out, A, W, rows, N, experts, K, grp, max_tiles, status, stream);
   }
   if (gated == 1) {
     const TcGroups grp{tiles, meta, offsets, 2 * N, {}};
-    return launch_tc_grouped<256, 4, TC_SILU_MUL>(out, A, W, rows, N, experts, 2 * N, K, N, grp, max_tiles, status, stream);
+    return launch_grouped_gated<TC_SILU_MUL>(out, A, W, rows, N, experts, K, grp, max_tiles, status, stream);
   }
   const TcGroups grp{tiles, meta, offsets, N, {}};
-  if (gated == 2) return launch_tc_grouped<128, 5, TC_RELU2>(out, A, W, rows, N, experts, N, K, 0, grp, max_tiles, status, stream);
-  return launch_tc_grouped<128, 5, TC_OUT_F32>(out, A, W, rows, N, experts, N, K, 0, grp, max_tiles, status, stream);
+  if (gated == 2) return launch_grouped_plain<TC_RELU2>(out, A, W, rows, N, experts, K, grp, max_tiles, status, stream);
+  return launch_grouped_plain<TC_OUT_F32>(out, A, W, rows, N, experts, K, grp, max_tiles, status, stream);
 }
 
 // out [M, N] bfloat16 = X [M, K] W [N, K]^T for M <= 64 tokens (decode steps), see gemm_tc_decode_kernel.

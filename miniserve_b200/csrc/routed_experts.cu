@@ -19,44 +19,104 @@
 
 namespace ms {
 
-constexpr int ROUTE_THREADS = 128;
+// The index of the largest value among the lanes' (value, index) pairs, the lowest of equals; INT_MAX where no lane has one.
+__device__ __forceinline__ int warp_best(float v, int i) {
+  // a float's bits as an unsigned number in the same order; 0 is below all of them
+  const uint32_t bits = __float_as_uint(v);
+  const uint32_t key = i == INT_MAX ? 0u : (bits & 0x80000000u ? ~bits : bits | 0x80000000u);
+  const uint32_t best = __reduce_max_sync(0xffffffffu, key);
+  if (best == 0u) return INT_MAX;
+  return (int)__reduce_min_sync(0xffffffffu, key == best ? (unsigned)i : (unsigned)INT_MAX);
+}
 
-// One CTA per token. x [T, K] (rows ld_x apart), router [R, K] float32, correction [R] float32 or null.
+constexpr int ROUTE_WARPS = 8, ROUTE_THREADS = ROUTE_WARPS * 32;
+
+// One CTA per TOK tokens. x [T, K] (rows ld_x apart), router [R, K] float32, correction [R] float32 or null.
 // idx_out [T, top] int32, wgt_out [T, top] float32. logit_bias [R] float32 or null: added to the logits themselves (it
 // moves scores and weights, where the correction moves the choice alone). gate_w [K] float32 with gate_out [T]: one
 // more product of the same input, gate_out[t] = sigmoid(x . gate_w), the weight of an expert that every token uses.
-template <typename T>
+// A warp takes two rows of the router at a time for all of the CTA's tokens, 16 bytes a lane (vec), then a warp makes a token's
+// choice. A logit's sum does not depend on TOK.
+template <typename T, int TOK>
 __global__ void __launch_bounds__(ROUTE_THREADS)
 expert_route_kernel(int* __restrict__ idx_out, float* __restrict__ wgt_out, const T* __restrict__ x, int ld_x,
-                    const float* __restrict__ router, const float* __restrict__ correction, int K, int R, int top, int group_count,
+                    const float* __restrict__ router, const float* __restrict__ correction, int tokens, int K, int R, int top, int group_count,
                     int group_keep, float weight_scale, int renormalize, const float* __restrict__ logit_bias,
                     const float* __restrict__ gate_w, float* __restrict__ gate_out, int sigmoid_scores, int square_weights, int group_best,
-                    float renorm_eps) {
-  extern __shared__ float route_smem[];
-  float* xs = route_smem;      // [K]
-  float* s = xs + K;           // [R] logits, then scores
-  float* choice = s + R;       // [R]
-  float* gs = choice + R;      // [group_count] group scores
-  float* kept = gs + group_count;  // [group_count] 1 where the group is kept
+                    float renorm_eps, int vec) {
+  extern __shared__ __align__(16) float route_smem[];
+  const int ldx = (K + 3) & ~3, per_tok = 2 * R + 2 * group_count;
+  float* xs = route_smem;  // [TOK][ldx]
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t0 = blockIdx.x * TOK;
+  if (TOK == 1 && vec) {  // a few tokens: the router is fetched from memory, and asked for before the wait for the input
+    for (size_t at = (size_t)threadIdx.x * 32; at < (size_t)R * K; at += ROUTE_THREADS * 32) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(router + at));
+  }
   pdl_prologue();
-  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  for (int k = threadIdx.x; k < K; k += ROUTE_THREADS) xs[k] = Elem<T>::load(x + (size_t)t * ld_x + k);
-  __syncthreads();
-  for (int e = warp; e < R; e += ROUTE_THREADS / 32) {
-    const float* w = router + (size_t)e * K;
-    float acc = 0.f;
-    for (int k = lane; k < K; k += 32) acc = fmaf(xs[k], w[k], acc);
-    acc = warp_sum(acc);
-    if (lane == 0) s[e] = acc + (logit_bias ? logit_bias[e] : 0.f);
-  }
-  if (gate_w && warp == ROUTE_THREADS / 32 - 1) {
-    float acc = 0.f;
-    for (int k = lane; k < K; k += 32) acc = fmaf(xs[k], gate_w[k], acc);
-    acc = warp_sum(acc);
-    if (lane == 0) gate_out[t] = 1.0f / (1.0f + expf(-acc));
+  if (vec == 2) {  // bfloat16 rows of whole 16 bytes
+    const int k8 = K >> 3;
+    for (int i = threadIdx.x; i < TOK * k8; i += ROUTE_THREADS) {
+      const int tt = TOK == 1 ? 0 : i / k8, k = (i - tt * k8) * 8;
+      float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (t0 + tt < tokens) bf16x8_to_float(*reinterpret_cast<const uint4*>(x + (size_t)(t0 + tt) * ld_x + k), f);
+      *reinterpret_cast<float4*>(xs + tt * ldx + k) = make_float4(f[0], f[1], f[2], f[3]);
+      *reinterpret_cast<float4*>(xs + tt * ldx + k + 4) = make_float4(f[4], f[5], f[6], f[7]);
+    }
+  } else
+  for (int i = threadIdx.x; i < TOK * K; i += ROUTE_THREADS) {
+    const int tt = TOK == 1 ? 0 : i / K, k = i - tt * K;
+    xs[tt * ldx + k] = t0 + tt < tokens ? Elem<T>::load(x + (size_t)(t0 + tt) * ld_x + k) : 0.f;
   }
   __syncthreads();
-  if (warp != 0) return;
+  float* per = xs + (size_t)TOK * ldx;  // per token: logits then scores [R] | choice scores [R] | group scores | kept
+  const int rows = R + (gate_w ? 1 : 0);
+  for (int e0 = warp; e0 < rows; e0 += 2 * ROUTE_WARPS) {
+    const int e1 = e0 + ROUTE_WARPS;
+    const bool two = e1 < rows;
+    const float* wa = e0 < R ? router + (size_t)e0 * K : gate_w;
+    const float* wb = !two ? wa : e1 < R ? router + (size_t)e1 * K : gate_w;
+    float acc[2][TOK] = {};
+    if (vec) {
+#pragma unroll 8
+      for (int k = lane * 4; k < K; k += 128) {
+        const float4 a = *reinterpret_cast<const float4*>(wa + k), b = *reinterpret_cast<const float4*>(wb + k);
+#pragma unroll
+        for (int tt = 0; tt < TOK; ++tt) {
+          const float4 v = *reinterpret_cast<const float4*>(xs + tt * ldx + k);
+          acc[0][tt] = fmaf(v.w, a.w, fmaf(v.z, a.z, fmaf(v.y, a.y, fmaf(v.x, a.x, acc[0][tt]))));
+          acc[1][tt] = fmaf(v.w, b.w, fmaf(v.z, b.z, fmaf(v.y, b.y, fmaf(v.x, b.x, acc[1][tt]))));
+        }
+      }
+    } else {
+      for (int k = lane; k < K; k += 32) {
+        const float a = wa[k], b = wb[k];
+#pragma unroll
+        for (int tt = 0; tt < TOK; ++tt) {
+          acc[0][tt] = fmaf(xs[tt * ldx + k], a, acc[0][tt]);
+          acc[1][tt] = fmaf(xs[tt * ldx + k], b, acc[1][tt]);
+        }
+      }
+    }
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      const int e = q == 0 ? e0 : e1;
+      if (e >= rows) break;
+#pragma unroll
+      for (int tt = 0; tt < TOK; ++tt) {
+        const float z = warp_sum(acc[q][tt]);
+        if (lane != 0 || t0 + tt >= tokens) continue;
+        if (e < R) per[tt * per_tok + e] = z + (logit_bias ? logit_bias[e] : 0.f);
+        else gate_out[t0 + tt] = 1.0f / (1.0f + expf(-z));
+      }
+    }
+  }
+  __syncthreads();
+  const int t = t0 + warp;
+  if (warp >= TOK || t >= tokens) return;
+  float* s = per + (size_t)warp * per_tok;  // [R] logits, then scores
+  float* choice = s + R;                    // [R]
+  float* gs = choice + R;                   // [group_count] group scores
+  float* kept = gs + group_count;           // [group_count] 1 where the group is kept
   float inv = 1.f;
   if (sigmoid_scores) {
     for (int e = lane; e < R; e += 32) s[e] = 1.0f / (1.0f + expf(-s[e]));
@@ -79,7 +139,7 @@ expert_route_kernel(int* __restrict__ idx_out, float* __restrict__ wgt_out, cons
   }
   __syncwarp();
   if (group_count > 1) {
-    const int per = R / group_count;
+    const int size = R / group_count;
     for (int g = lane; g < group_count; g += 32) {
       // the group_best largest, one after the other: the next one is the largest of those behind (value, then index) the last
       float sum = 0.f, last = INFINITY;
@@ -87,8 +147,8 @@ expert_route_kernel(int* __restrict__ idx_out, float* __restrict__ wgt_out, cons
       for (int b = 0; b < group_best; ++b) {
         float best = -INFINITY;
         int best_j = -1;
-        for (int j = 0; j < per; ++j) {
-          const float c = choice[g * per + j];
+        for (int j = 0; j < size; ++j) {
+          const float c = choice[g * size + j];
           if ((c < last || (c == last && j > last_j)) && (best_j < 0 || c > best)) {
             best = c;
             best_j = j;
@@ -110,54 +170,47 @@ expert_route_kernel(int* __restrict__ idx_out, float* __restrict__ wgt_out, cons
           bv = gs[g];
           bi = g;
         }
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-        if (oi != INT_MAX && (bi == INT_MAX || ov > bv || (ov == bv && oi < bi))) {
-          bv = ov;
-          bi = oi;
-        }
-      }
+      bi = warp_best(bv, bi);
       if (lane == 0 && bi != INT_MAX) kept[bi] = 1.f;
       __syncwarp();
     }
     for (int e = lane; e < R; e += 32)
-      if (kept[e / per] == 0.f) choice[e] = -INFINITY;
+      if (kept[e / size] == 0.f) choice[e] = -INFINITY;
     __syncwarp();
   }
+  // (the choices are handed on to the lanes: lane r % 32 writes choice r)
   float total = 0.f;
-  for (int r = 0; r < top; ++r) {
-    float bv = -INFINITY;
-    int bi = INT_MAX;
-    for (int e = lane; e < R; e += 32)
-      if (choice[e] > bv) {
-        bv = choice[e];
-        bi = e;
-      }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (oi != INT_MAX && (bi == INT_MAX || ov > bv || (ov == bv && oi < bi))) {
-        bv = ov;
-        bi = oi;
-      }
-    }
-    if (lane == 0) {
+  for (int r0 = 0; r0 < top; r0 += 32) {
+    int mine = -1;
+    float weight = 0.f;
+    const int end = min(top, r0 + 32);
+    for (int r = r0; r < end; ++r) {
+      float bv = -INFINITY;
+      int bi = INT_MAX;
+      for (int e = lane; e < R; e += 32)
+        if (choice[e] > bv) {
+          bv = choice[e];
+          bi = e;
+        }
+      bi = warp_best(bv, bi);
       const float p = bi != INT_MAX ? s[bi] : 0.f;
-      idx_out[(size_t)t * top + r] = bi != INT_MAX ? bi : -1;
-      wgt_out[(size_t)t * top + r] = p;
       total += p;
-      if (bi != INT_MAX) choice[bi] = -INFINITY;
+      if (lane == r - r0) {
+        mine = bi != INT_MAX ? bi : -1;
+        weight = p;
+      }
+      if (bi != INT_MAX && lane == (bi & 31)) choice[bi] = -INFINITY;  // (this lane alone looks at it)
     }
-    __syncwarp();
-  }
-  if (lane == 0) {
-    const float f = renormalize ? weight_scale / (total + renorm_eps) : weight_scale;
-    for (int r = 0; r < top; ++r) {
-      const float w = wgt_out[(size_t)t * top + r] * f;
-      wgt_out[(size_t)t * top + r] = square_weights ? w * w : w;
+    if (r0 + lane < end) {
+      idx_out[(size_t)t * top + r0 + lane] = mine;
+      wgt_out[(size_t)t * top + r0 + lane] = weight;
+    }
+    if (end == top) {  // the sum is whole: what this lane wrote gets its factor
+      const float f = renormalize ? weight_scale / (total + renorm_eps) : weight_scale;
+      for (int r = lane; r < top; r += 32) {
+        const float w = (r >= r0 ? weight : wgt_out[(size_t)t * top + r]) * f;
+        wgt_out[(size_t)t * top + r] = square_weights ? w * w : w;
+      }
     }
   }
 }
@@ -461,6 +514,53 @@ __global__ void expert_combine_kernel(T* __restrict__ out, const float* __restri
   Elem<T>::store(out + i, acc);
 }
 
+// The same for rows of H % 4 == 0 elements that start on 16 bytes (8 for bfloat16): four channels a thread, all of a token's rows in flight.
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+}
+__device__ __forceinline__ void fma4(float4& a, float w, const float4& v) {
+  a = make_float4(fmaf(w, v.x, a.x), fmaf(w, v.y, a.y), fmaf(w, v.z, a.z), fmaf(w, v.w, a.w));
+}
+template <typename T>
+__global__ void expert_combine_x4_kernel(T* __restrict__ out, const float* __restrict__ y, const T* __restrict__ x, int ld_x,
+                                         const int* __restrict__ idx, const float* __restrict__ wgt, const int* __restrict__ pos, int total4,
+                                         int H4, int top, int E, const T* __restrict__ shared, const float* __restrict__ shared_gate) {
+  pdl_prologue();
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= total4) return;
+  const int t = i / H4, c = (i - t * H4) * 4;
+  const float4 sh = shared ? load4(shared + (size_t)i * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int k0 = 0; k0 < top; k0 += 4) {
+    float4 v[4];
+    float w[4];
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      v[q] = make_float4(0.f, 0.f, 0.f, 0.f);
+      w[q] = 0.f;
+      if (k0 + q < top) {
+        const int slot = t * top + k0 + q, p = pos[slot];
+        w[q] = wgt[slot];
+        if (p >= 0) v[q] = load4(y + (size_t)p * H4 * 4 + c);
+        else if (idx[slot] >= E) v[q] = load4(x + (size_t)t * ld_x + c);
+      }
+    }
+#pragma unroll
+    for (int q = 0; q < 4; ++q)
+      if (k0 + q < top) fma4(acc, w[q], v[q]);
+  }
+  if (shared) fma4(acc, shared_gate ? shared_gate[t] : 1.f, sh);
+  store4(out + (size_t)i * 4, acc);
+}
+
 }  // namespace ms
 
 using namespace ms;
@@ -479,19 +579,28 @@ MS_EXPORT int ms_expert_route(int* idx, float* wgt, const void* x, int ld_x, con
                "expert_route: %d router outputs in %d groups of which %d are kept cannot give %d choices", R, group_count, group_keep, top);
   MS_CHECK_ARG(group_best >= 1 && (group_count == 1 || group_best <= R / group_count), "expert_route: a group of %d has no %d largest",
                R / group_count, group_best);
-  const size_t smem = ((size_t)K + 2 * (size_t)R + 2 * (size_t)group_count) * sizeof(float);
-  MS_CHECK_ARG(smem <= 200 * 1024, "expert_route: %d inputs and %d outputs need %zu bytes of shared memory", K, R, smem);
+  int vec = K % 4 == 0 && (uintptr_t)router % 16 == 0 && (uintptr_t)gate_w % 16 == 0;
+  if (vec && dtype == MS_BF16 && K % 8 == 0 && ld_x % 8 == 0 && (uintptr_t)x % 16 == 0) vec = 2;
+  auto smem_of = [&](int tok) { return (size_t)tok * (((size_t)(K + 3) & ~(size_t)3) + 2 * (size_t)R + 2 * (size_t)group_count) * sizeof(float); };
+  MS_CHECK_ARG(smem_of(1) <= 200 * 1024, "expert_route: %d inputs and %d outputs need %zu bytes of shared memory", K, R, smem_of(1));
+  const int tok = tokens >= 512 && smem_of(4) <= 100 * 1024 ? 4 : 1;
+  const size_t smem = smem_of(tok);
+#define MS_ROUTE(T, TOK)                                                                                                                     \
+  do {                                                                                                                                       \
+    if (smem > 48 * 1024)                                                                                                                    \
+      MS_CHECK_CUDA(cudaFuncSetAttribute(expert_route_kernel<T, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));              \
+    MS_LAUNCH((expert_route_kernel<T, TOK>), (tokens + TOK - 1) / TOK, ROUTE_THREADS, smem, stream, idx, wgt, (const T*)x, ld_x, router,     \
+              correction, tokens, K, R, top, group_count, group_keep, weight_scale, renormalize, logit_bias, gate_w, gate_out, sigmoid_scores, \
+              square_weights, group_best, renorm_eps, vec);                                                                                  \
+  } while (0)
   if (dtype == MS_F32) {
-    if (smem > 48 * 1024) MS_CHECK_CUDA(cudaFuncSetAttribute(expert_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    MS_LAUNCH(expert_route_kernel<float>, tokens, ROUTE_THREADS, smem, stream, idx, wgt, (const float*)x, ld_x, router, correction, K, R, top,
-              group_count, group_keep, weight_scale, renormalize, logit_bias, gate_w, gate_out, sigmoid_scores, square_weights, group_best, renorm_eps);
+    if (tok == 4) MS_ROUTE(float, 4);
+    else MS_ROUTE(float, 1);
   } else {
-    if (smem > 48 * 1024)
-      MS_CHECK_CUDA(cudaFuncSetAttribute(expert_route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    MS_LAUNCH(expert_route_kernel<__nv_bfloat16>, tokens, ROUTE_THREADS, smem, stream, idx, wgt, (const __nv_bfloat16*)x, ld_x, router,
-              correction, K, R, top, group_count, group_keep, weight_scale, renormalize, logit_bias, gate_w, gate_out, sigmoid_scores, square_weights,
-              group_best, renorm_eps);
+    if (tok == 4) MS_ROUTE(__nv_bfloat16, 4);
+    else MS_ROUTE(__nv_bfloat16, 1);
   }
+#undef MS_ROUTE
   return 0;
 }
 
@@ -584,6 +693,18 @@ MS_EXPORT int ms_expert_combine(void* out, const float* y, const void* x, int ld
   if (tokens == 0) return 0;
   const long long total = (long long)tokens * H;
   const unsigned blocks = (unsigned)((total + 255) / 256);
+  const size_t align = dtype == MS_F32 ? 16 : 8;
+  if (H % 4 == 0 && ld_x % 4 == 0 && total / 4 < (1LL << 31) && (uintptr_t)out % align == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)x % align == 0 &&
+      (uintptr_t)shared % align == 0) {
+    const int total4 = (int)(total / 4);
+    if (dtype == MS_F32)
+      MS_LAUNCH(expert_combine_x4_kernel<float>, (total4 + 127) / 128, 128, 0, stream, (float*)out, y, (const float*)x, ld_x, idx, wgt, pos, total4,
+                H / 4, top, E, (const float*)shared, shared_gate);
+    else
+      MS_LAUNCH(expert_combine_x4_kernel<__nv_bfloat16>, (total4 + 127) / 128, 128, 0, stream, (__nv_bfloat16*)out, y, (const __nv_bfloat16*)x, ld_x,
+                idx, wgt, pos, total4, H / 4, top, E, (const __nv_bfloat16*)shared, shared_gate);
+    return 0;
+  }
   if (dtype == MS_F32)
     MS_LAUNCH(expert_combine_kernel<float>, blocks, 256, 0, stream, (float*)out, y, (const float*)x, ld_x, idx, wgt, pos, total, H, top, E,
               (const float*)shared, shared_gate);

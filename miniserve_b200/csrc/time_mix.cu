@@ -15,7 +15,8 @@
 // two blocks the product splits at the later block's first token, and r (times the product from there) meets k (times the product up
 // to there) in a matrix product; inside a block the 120 pairs are summed channel by channel with a running product. What goes to the
 // tensor cores and is not exact in bfloat16 (r and k times products, the weights, the state) goes as two bfloat16 numbers. Launches:
-//   states (what every chunk adds), carry (the states before every chunk, and the row's last one), outputs.
+//   states (what every chunk adds), carry (the states before every chunk, and the row's last one), outputs (for heads of one value tile with
+//   the norm and the gate behind them).
 #include "chunk_mma.cuh"
 
 namespace ms {
@@ -45,7 +46,8 @@ struct Rows {
 };
 
 // grid (H, rows). LPC lanes take a column's key channels, four at a time; a warp 32 / LPC columns at once, TS_COLS of them in turn with
-// their loads in flight together. out [T, H * dv] = o / sqrt(mean o^2 + eps) * norm_w * silu(gate).
+// their loads in flight together; the first ones are asked for before the decays are worked out. out [T, H * dv] = o / sqrt(mean o^2 + eps) *
+// norm_w * silu(gate).
 template <typename T, int LPC>
 __global__ void __launch_bounds__(TS_THREADS)
 time_step_kernel(T* __restrict__ out, float* __restrict__ state, Rows<T> r, Rows<T> k, Rows<T> v, Rows<T> gate, Rows<T> low,
@@ -60,10 +62,39 @@ time_step_kernel(T* __restrict__ out, float* __restrict__ state, Rows<T> r, Rows
   float* uk = ds + dk;       // [dk] bonus times key
   float* os = uk + dk;       // [dv]
   float* ls = os + dv;       // [rank]
-  pdl_prologue();
   const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  {  // weights: asked for before the wait
+    const char* w = reinterpret_cast<const char*>(w2 + (size_t)h * dk * rank);
+    for (size_t at = (size_t)tid * 128; at < (size_t)dk * rank * sizeof(T); at += TS_THREADS * 128) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(w + at));
+  }
+  pdl_prologue();
   const int t = cu_q[row];
   const bool fresh = q_start[row] == 0;
+  constexpr int CPW = 32 / LPC;
+  const int l = lane % LPC, sub = lane / LPC;
+  float* head = state + ((size_t)state_slot[row] * H + h) * (size_t)dv * dk;
+  auto load = [&](float4 (&S)[TS_COLS], int j0, int i) {
+#pragma unroll
+    for (int s = 0; s < TS_COLS; ++s) {
+      const int j = j0 + s * TS_WARPS * CPW;
+      S[s] = fresh || j >= dv || i >= dk ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(head + (size_t)j * dk + i);
+    }
+  };
+  float4 S[TS_COLS];
+  load(S, warp * CPW + sub, l * 4);
+  float vj[TS_COLS], gate0 = 0.f, nw0 = 0.f;
+  auto load_v = [&](int j0) {
+#pragma unroll
+    for (int s = 0; s < TS_COLS; ++s) {
+      const int j = j0 + s * TS_WARPS * CPW;
+      vj[s] = j < dv ? Elem<T>::load(v.p + (size_t)t * v.ld + (size_t)h * dv + j) : 0.f;
+    }
+  };
+  load_v(warp * CPW + sub);
+  if (tid < dv) {
+    gate0 = Elem<T>::load(gate.p + (size_t)t * gate.ld + (size_t)h * dv + tid);
+    nw0 = norm_w[(size_t)h * dv + tid];
+  }
   for (int c = tid; c < rank; c += TS_THREADS) ls[c] = Elem<T>::load(low.p + (size_t)t * low.ld + c);
   for (int c = tid; c < dk; c += TS_THREADS) {
     const size_t at = (size_t)h * dk + c;
@@ -75,37 +106,28 @@ time_step_kernel(T* __restrict__ out, float* __restrict__ state, Rows<T> r, Rows
   __syncthreads();
   // z of the head's channels: eight lanes a channel
   {
-    const int l = tid & 7;
+    const int zl = tid & 7;
     for (int c0 = 0; c0 < dk; c0 += TS_THREADS / 8) {
       const int c = c0 + (tid >> 3);
       float acc = 0.f;
       if (c < dk) {
         const T* w = w2 + ((size_t)h * dk + c) * rank;
-        for (int i = l; i < rank; i += 8) acc = fmaf(ls[i], Elem<T>::load(w + i), acc);
+#pragma unroll 8
+        for (int i = zl; i < rank; i += 8) acc = fmaf(ls[i], Elem<T>::load(w + i), acc);
       }
 #pragma unroll
       for (int o = 4; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-      if (l == 0 && c < dk) ds[c] = channel_decay_of(acc + w0[(size_t)h * dk + c]);
+      if (zl == 0 && c < dk) ds[c] = channel_decay_of(acc + w0[(size_t)h * dk + c]);
     }
   }
   __syncthreads();
-  constexpr int CPW = 32 / LPC;
-  const int l = lane % LPC, sub = lane / LPC;
-  float* head = state + ((size_t)state_slot[row] * H + h) * (size_t)dv * dk;
+  bool loaded = true;  // the first group is
   for (int j0 = warp * CPW + sub; j0 - sub < dv; j0 += TS_WARPS * CPW * TS_COLS) {
-    float acc[TS_COLS] = {}, vj[TS_COLS];
-#pragma unroll
-    for (int s = 0; s < TS_COLS; ++s) {
-      const int j = j0 + s * TS_WARPS * CPW;
-      vj[s] = j < dv ? Elem<T>::load(v.p + (size_t)t * v.ld + (size_t)h * dv + j) : 0.f;
-    }
+    float acc[TS_COLS] = {};
+    if (j0 != warp * CPW + sub) load_v(j0);
     for (int i = l * 4; i < dk; i += LPC * 4) {
-      float4 S[TS_COLS];
-#pragma unroll
-      for (int s = 0; s < TS_COLS; ++s) {
-        const int j = j0 + s * TS_WARPS * CPW;
-        S[s] = fresh || j >= dv ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(head + (size_t)j * dk + i);
-      }
+      if (!loaded) load(S, j0, i);
+      loaded = false;
       const float4 r4 = *reinterpret_cast<const float4*>(rs + i), k4 = *reinterpret_cast<const float4*>(ks + i);
       const float4 d4 = *reinterpret_cast<const float4*>(ds + i), u4 = *reinterpret_cast<const float4*>(uk + i);
 #pragma unroll
@@ -118,6 +140,7 @@ time_step_kernel(T* __restrict__ out, float* __restrict__ state, Rows<T> r, Rows
         if (j < dv) *reinterpret_cast<float4*>(head + (size_t)j * dk + i) = S[s];
       }
     }
+    loaded = false;  // (a lane beyond the key channels has used none)
 #pragma unroll
     for (int s = 0; s < TS_COLS; ++s) {
       float x = acc[s];
@@ -133,8 +156,8 @@ time_step_kernel(T* __restrict__ out, float* __restrict__ state, Rows<T> r, Rows
   const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)dv + eps);
   for (int c = tid; c < dv; c += TS_THREADS) {
     const size_t at = (size_t)h * dv + c;
-    const float g = Elem<T>::load(gate.p + (size_t)t * gate.ld + at);
-    Elem<T>::store(out + (size_t)t * H * dv + at, ((os[c] * inv) * norm_w[at]) * (g / (1.0f + expf(-g))));
+    const float g = c == tid ? gate0 : Elem<T>::load(gate.p + (size_t)t * gate.ld + at);
+    Elem<T>::store(out + (size_t)t * H * dv + at, ((os[c] * inv) * (c == tid ? nw0 : norm_w[at])) * (g / (1.0f + expf(-g))));
   }
 }
 
@@ -151,7 +174,7 @@ struct ChunkPlace {
   int num_rows;
 };
 
-// The decays of a block's 16 tokens for one channel (tokens from n on: 1).
+// The decays of a block's 16 tokens for one channel (tokens from n on: 1). (The hardware's exponential: relative error about 1e-6 of an exponent.)
 __device__ __forceinline__ void block_decays(float (&d)[TC_BLK], const float* __restrict__ z, int ld_z, const float* __restrict__ w0, int t0, int n,
                                              int blk, int ch, bool in) {
 #pragma unroll
@@ -161,7 +184,7 @@ __device__ __forceinline__ void block_decays(float (&d)[TC_BLK], const float* __
   }
   const float w = in ? w0[ch] : 0.f;
 #pragma unroll
-  for (int i = 0; i < TC_BLK; ++i) d[i] = in && blk * TC_BLK + i < n ? channel_decay_of(d[i] + w) : 1.f;
+  for (int i = 0; i < TC_BLK; ++i) d[i] = in && blk * TC_BLK + i < n ? __expf(-__expf(d[i] + w)) : 1.f;
 }
 
 template <int DKT>
@@ -255,52 +278,69 @@ tm_states_kernel(float* __restrict__ added, float* __restrict__ passed, const __
 
 // ---------------------------------------------------------------- chunks: the states before every chunk
 // before_hi / before_lo [chunks, H, dv, dk]: the state before every chunk as two bfloat16; the row's slot of state [slots, H, dv, dk] gets
-// the state behind its last chunk. Four elements per thread; grid (elements of a row's state, rows).
+// the state behind its last chunk. One element per thread, the reads of sixteen chunks in flight; grid (elements of a row's state, rows).
 __global__ void __launch_bounds__(CS_THREADS)
 tm_carry_kernel(float* __restrict__ state, __nv_bfloat16* __restrict__ before_hi, __nv_bfloat16* __restrict__ before_lo,
                 const float* __restrict__ added, const float* __restrict__ passed, const ChunkPlace pl, int H, int dk, int dv) {
   pdl_prologue();
-  const int total4 = H * dv * dk / 4;
-  const int i4 = blockIdx.x * CS_THREADS + threadIdx.x, r = blockIdx.y;
-  if (i4 >= total4) return;
-  const int h = i4 / (dv * dk / 4), c = i4 * 4 % dk;
+  const int total = H * dv * dk;
+  const int i = blockIdx.x * CS_THREADS + threadIdx.x, r = blockIdx.y;
+  if (i >= total) return;
+  const int h = i / (dv * dk), c = i % dk;
   const int c0 = pl.row_first[r], c1 = pl.row_first[r + 1];
   if (c1 <= c0) return;
-  float4* slot = reinterpret_cast<float4*>(state) + (size_t)pl.state_slot[r] * total4 + i4;
-  float4 S = pl.q_start[r] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : *slot;
-#pragma unroll 4
-  for (int ch = c0; ch < c1; ++ch) {
-    const size_t at = (size_t)ch * total4 + i4;
-    const float4 d = reinterpret_cast<const float4*>(added)[at];
-    const float4 a = *reinterpret_cast<const float4*>(passed + ((size_t)ch * H + h) * dk + c);
-    __align__(8) __nv_bfloat16 hi[4];
-    __align__(8) __nv_bfloat16 lo[4];
-    cs_split(S.x, hi[0], lo[0]);
-    cs_split(S.y, hi[1], lo[1]);
-    cs_split(S.z, hi[2], lo[2]);
-    cs_split(S.w, hi[3], lo[3]);
-    reinterpret_cast<uint2*>(before_hi)[at] = *reinterpret_cast<const uint2*>(hi);
-    reinterpret_cast<uint2*>(before_lo)[at] = *reinterpret_cast<const uint2*>(lo);
-    S = make_float4(fmaf(a.x, S.x, d.x), fmaf(a.y, S.y, d.y), fmaf(a.z, S.z, d.z), fmaf(a.w, S.w, d.w));
+  float* slot = state + (size_t)pl.state_slot[r] * total + i;
+  float S = pl.q_start[r] == 0 ? 0.f : *slot;
+  constexpr int AHEAD = 16;
+  for (int ch0 = c0; ch0 < c1; ch0 += AHEAD) {
+    float d[AHEAD], a[AHEAD];
+#pragma unroll
+    for (int q = 0; q < AHEAD; ++q) {
+      if (ch0 + q < c1) {
+        d[q] = added[(size_t)(ch0 + q) * total + i];
+        a[q] = passed[((size_t)(ch0 + q) * H + h) * dk + c];
+      }
+    }
+#pragma unroll
+    for (int q = 0; q < AHEAD; ++q) {
+      if (ch0 + q < c1) {
+        const size_t at = (size_t)(ch0 + q) * total + i;
+        cs_split(S, before_hi[at], before_lo[at]);
+        S = fmaf(a[q], S, d[q]);
+      }
+    }
   }
   *slot = S;
 }
 
 // ---------------------------------------------------------------- chunks: the outputs
+// Two neighbours at once: the sum of their two bfloat16, and back.
+__device__ __forceinline__ float2 joined2(const __nv_bfloat16* hi, const __nv_bfloat16* lo) {
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(hi)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(lo));
+  return make_float2(a.x + b.x, a.y + b.y);
+}
+__device__ __forceinline__ void split2(float2 x, __nv_bfloat16* hi, __nv_bfloat16* lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x.x, x.y);
+  const float2 f = __bfloat1622float2(h);
+  *reinterpret_cast<__nv_bfloat162*>(hi) = h;
+  *reinterpret_cast<__nv_bfloat162*>(lo) = __floats2bfloat162_rn(x.x - f.x, x.y - f.y);
+}
+
 template <int DKT>
 struct TmOutputsSmem {
   static constexpr int LDK = DKT + 8, LDP = CS_TOK + 8;
-  float d[CS_TOK][DKT + 4];                         // decays
-  float whole[TC_BLOCKS][DKT];                      // a block's product
-  float dsum[2][TC_BLOCKS][TC_BLK][TC_BLK + 1];     // [channel half][block][j][i]: sums of the pairs inside a block
   union {
     struct {
-      __nv_bfloat16 r[CS_TOK][LDK], k[CS_TOK][LDK];
+      float d[CS_TOK][DKT + 4], r[CS_TOK][DKT + 4];  // decays, and r as it is
     };
     struct {
-      __nv_bfloat16 shi[TC_DV][LDK], slo[TC_DV][LDK];  // the state before the chunk, once r and k have been read
+      __nv_bfloat16 shi[TC_DV][LDK], slo[TC_DV][LDK];  // the state before the chunk, once the pairs inside the blocks are done
     };
   };
+  float whole[TC_BLOCKS][DKT];                      // a block's product
+  float dsum[2][TC_BLOCKS][TC_BLK][TC_BLK + 1];     // [channel half][block][j][i]: sums of the pairs inside a block
+  float squares[2][CS_TOK];                         // [column half][token]
+  __nv_bfloat16 k[CS_TOK][LDK];
   __nv_bfloat16 rhi[CS_TOK][LDK], rlo[CS_TOK][LDK];  // r times the product from its block's (then: the chunk's) first token on
   union {
     struct {
@@ -313,11 +353,20 @@ struct TmOutputsSmem {
   __nv_bfloat16 v[CS_TOK][TC_DV + 8];
 };
 
-// o [T, H, dv] float32. grid (chunks, H, dv tiles).
+// What follows the recurrence: out [T, H * dv] bfloat16 = o / sqrt(mean o^2 + eps) * norm_w * silu(gate) (heads of one value tile).
+struct HeadGate {
+  __nv_bfloat16* out;  // null: o is written as it is
+  const __nv_bfloat16* gate;
+  int ld_gate;
+  const float* norm_w;
+  float eps;
+};
+
+// o [T, H, dv] float32 (or hg.out). grid (chunks, H, dv tiles).
 template <int DKT>
 __global__ void __launch_bounds__(CS_THREADS, DKT <= 64 ? 2 : 1)
-tm_outputs_kernel(float* __restrict__ o, const __nv_bfloat16* __restrict__ r, int ld_r, const __nv_bfloat16* __restrict__ k, int ld_k,
-                  const __nv_bfloat16* __restrict__ v, int ld_v, const float* __restrict__ z, int ld_z, const float* __restrict__ w0,
+tm_outputs_kernel(float* __restrict__ o, const HeadGate hg, const __nv_bfloat16* __restrict__ r, int ld_r, const __nv_bfloat16* __restrict__ k,
+                  int ld_k, const __nv_bfloat16* __restrict__ v, int ld_v, const float* __restrict__ z, int ld_z, const float* __restrict__ w0,
                   const float* __restrict__ u, const __nv_bfloat16* __restrict__ before_hi, const __nv_bfloat16* __restrict__ before_lo,
                   const ChunkPlace pl, int H, int dk, int dv) {
   extern __shared__ __align__(16) unsigned char cs_raw[];
@@ -330,14 +379,6 @@ tm_outputs_kernel(float* __restrict__ o, const __nv_bfloat16* __restrict__ r, in
   const bool has_state = !(pl.q_start[at.x] == 0 && chunk == pl.row_first[at.x]);  // else nothing came before
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int i8 = lane & 7, mat = lane >> 3, g = lane >> 2, tg = (lane & 3) * 2;
-  for (int idx = tid; idx < CS_TOK * (DKT / 8); idx += CS_THREADS) {
-    const int tt = idx / (DKT / 8), c = (idx - tt * (DKT / 8)) * 8;
-    const bool in = tt < n && c < dk;
-    const size_t tok = (size_t)(t0 + tt);
-    cs_cp16(&sm.r[tt][c], in ? (const void*)(r + tok * ld_r + (size_t)h * dk + c) : (const void*)r, in);
-    cs_cp16(&sm.k[tt][c], in ? (const void*)(k + tok * ld_k + (size_t)h * dk + c) : (const void*)k, in);
-  }
-  cs_commit();
   for (int idx = tid; idx < CS_TOK * (TC_DV / 8); idx += CS_THREADS) {
     const int tt = idx / (TC_DV / 8), c = (idx - tt * (TC_DV / 8)) * 8;
     const bool in = tt < n && v0 + c < dv;
@@ -345,53 +386,128 @@ tm_outputs_kernel(float* __restrict__ o, const __nv_bfloat16* __restrict__ r, in
   }
   cs_commit();
 
-  // decays, and the products within a block, one thread per (block, channel)
+  // one thread per (block, channel): decays, and the products within the block
   constexpr int TRIPS = DKT / 64;
   const int blk = tid >> 6;
   float pre[TRIPS][TC_BLK];
 #pragma unroll
   for (int tr = 0; tr < TRIPS; ++tr) {
     const int c = tr * 64 + (tid & 63);
+    const size_t hc = (size_t)h * dk + c;
+    __nv_bfloat16 rk[2][TC_BLK];
+#pragma unroll
+    for (int i = 0; i < TC_BLK; ++i) {
+      const int tt = blk * TC_BLK + i;
+      const bool in = tt < n && c < dk;
+      rk[0][i] = in ? r[(size_t)(t0 + tt) * ld_r + hc] : __float2bfloat16_rn(0.f);
+      rk[1][i] = in ? k[(size_t)(t0 + tt) * ld_k + hc] : __float2bfloat16_rn(0.f);
+    }
     float d[TC_BLK];
-    block_decays(d, z, ld_z, w0, t0, n, blk, h * dk + c, c < dk);
+    block_decays(d, z, ld_z, w0, t0, n, blk, (int)hc, c < dk);
     float run = 1.f;
 #pragma unroll
     for (int i = 0; i < TC_BLK; ++i) {
-      pre[tr][i] = run;  // up to the token before
+      const int tt = blk * TC_BLK + i;
+      const float x = __bfloat162float(rk[0][i]);
+      sm.r[tt][c] = x;
+      pre[tr][i] = run * x;  // times the product up to the token before
       run *= d[i];
-      sm.d[blk * TC_BLK + i][c] = d[i];
+      sm.d[tt][c] = d[i];
+      sm.k[tt][c] = rk[1][i];
+      cs_split(pre[tr][i], sm.rhi[tt][c], sm.rlo[tt][c]);
     }
     sm.whole[blk][c] = run;
-  }
-  cs_wait<1>();  // r and k
-  __syncthreads();
+    // k times the product behind it to its block's end, for the next block; the products of whole blocks follow below
+    if (blk < TC_BLOCKS - 1) {
+      const int base = blk == 0 ? 0 : blk == 1 ? 32 : 80;
+      float suf = 1.f;
 #pragma unroll
-  for (int tr = 0; tr < TRIPS; ++tr) {
-    const int c = tr * 64 + (tid & 63);
-    const float w1 = sm.whole[1][c], w2 = sm.whole[2][c];
-    float suf = 1.f;
-#pragma unroll
-    for (int i = TC_BLK - 1; i >= 0; --i) {
-      const int tt = blk * TC_BLK + i;
-      pre[tr][i] *= __bfloat162float(sm.r[tt][c]);
-      cs_split(pre[tr][i], sm.rhi[tt][c], sm.rlo[tt][c]);
-      const float x = __bfloat162float(sm.k[tt][c]) * suf;
-      suf *= sm.d[tt][c];
-      if (blk == 0) {
-        cs_split(x, sm.kb.hi[i][c], sm.kb.lo[i][c]);
-        cs_split(x * w1, sm.kb.hi[16 + i][c], sm.kb.lo[16 + i][c]);
-        cs_split(x * (w1 * w2), sm.kb.hi[48 + i][c], sm.kb.lo[48 + i][c]);
-      } else if (blk == 1) {
-        cs_split(x, sm.kb.hi[32 + i][c], sm.kb.lo[32 + i][c]);
-        cs_split(x * w2, sm.kb.hi[64 + i][c], sm.kb.lo[64 + i][c]);
-      } else if (blk == 2) {
-        cs_split(x, sm.kb.hi[80 + i][c], sm.kb.lo[80 + i][c]);
+      for (int i = TC_BLK - 1; i >= 0; --i) {
+        d[i] *= suf;  // d[i] becomes the product from i on
+        const float x = __bfloat162float(rk[1][i]) * suf;
+        suf = d[i];
+        cs_split(x, sm.kb.hi[base + i][c], sm.kb.lo[base + i][c]);
       }
     }
   }
   __syncthreads();
-
+  // block 0 for block 2 and 3, block 1 for block 3: times the products of the blocks between
+#pragma unroll
+  for (int tr = 0; tr < TRIPS; ++tr) {
+    const int c = tr * 64 + lane * 2;  // two channels a thread, two of the blocks' tokens
+    const float2 w1 = *reinterpret_cast<const float2*>(&sm.whole[1][c]), w2 = *reinterpret_cast<const float2*>(&sm.whole[2][c]);
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      const int i = warp * 2 + q;
+      const float2 x0 = joined2(&sm.kb.hi[i][c], &sm.kb.lo[i][c]), x1 = joined2(&sm.kb.hi[32 + i][c], &sm.kb.lo[32 + i][c]);
+      const float2 y0 = make_float2(x0.x * w1.x, x0.y * w1.y);
+      split2(y0, &sm.kb.hi[16 + i][c], &sm.kb.lo[16 + i][c]);
+      split2(make_float2(y0.x * w2.x, y0.y * w2.y), &sm.kb.hi[48 + i][c], &sm.kb.lo[48 + i][c]);
+      split2(make_float2(x1.x * w2.x, x1.y * w2.y), &sm.kb.hi[64 + i][c], &sm.kb.lo[64 + i][c]);
+    }
+  }
   const int bi = warp >> 1, half_w = warp & 1, wm = bi * TC_BLK;
+  // pairs inside a block: a lane takes j and 15 - j (15 pairs together) over DKT / 8 channels; two warps make up a block's channels
+  {
+    const int j = lane & 7;
+    constexpr int QC = DKT / 8;
+    const int cbeg = (half_w * 4 + (lane >> 3)) * QC;
+    float acc[TC_BLK - 1] = {}, own[2] = {0.f, 0.f};
+#pragma unroll 1
+    for (int c = cbeg; c < cbeg + QC; c += 4) {
+      float x[4], y[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        x[e] = __bfloat162float(sm.k[wm + j][c + e]);
+        y[e] = __bfloat162float(sm.k[wm + 15 - j][c + e]);
+        const float b = c + e < dk ? u[(size_t)h * dk + c + e] : 0.f;
+        own[0] = fmaf(sm.r[wm + j][c + e] * b, x[e], own[0]);
+        own[1] = fmaf(sm.r[wm + 15 - j][c + e] * b, y[e], own[1]);
+      }
+#pragma unroll
+      for (int s = 0; s < TC_BLK - 1; ++s) {
+        if (s == 15 - j) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) x[e] = y[e];
+        }
+        const int i = wm + s + 1 + (s < 15 - j ? j : 0);
+        const float4 r4 = *reinterpret_cast<const float4*>(&sm.r[i][c]), d4 = *reinterpret_cast<const float4*>(&sm.d[i][c]);
+        acc[s] = fmaf(r4.x, x[0], fmaf(r4.y, x[1], fmaf(r4.z, x[2], fmaf(r4.w, x[3], acc[s]))));
+        x[0] *= d4.x;
+        x[1] *= d4.y;
+        x[2] *= d4.z;
+        x[3] *= d4.w;
+      }
+    }
+#pragma unroll
+    for (int s = 0; s < TC_BLK - 1; ++s) {
+      acc[s] += __shfl_xor_sync(0xffffffffu, acc[s], 8);
+      acc[s] += __shfl_xor_sync(0xffffffffu, acc[s], 16);
+    }
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      own[q] += __shfl_xor_sync(0xffffffffu, own[q], 8);
+      own[q] += __shfl_xor_sync(0xffffffffu, own[q], 16);
+    }
+    if (lane < 8) {
+#pragma unroll
+      for (int s = 0; s < TC_BLK - 1; ++s) sm.dsum[half_w][bi][s < 15 - j ? j : 15 - j][s + 1 + (s < 15 - j ? j : 0)] = acc[s];
+      sm.dsum[half_w][bi][j][j] = own[0];
+      sm.dsum[half_w][bi][15 - j][15 - j] = own[1];
+    }
+  }
+  __syncthreads();  // kb is whole, d and r have been read
+  if (has_state) {
+    const size_t st = ((size_t)chunk * H + h) * (size_t)dv * dk;
+    for (int idx = tid; idx < TC_DV * (DKT / 8); idx += CS_THREADS) {
+      const int row = idx / (DKT / 8), c = (idx - row * (DKT / 8)) * 8;
+      const bool in = v0 + row < dv && c < dk;
+      const size_t src = in ? st + (size_t)(v0 + row) * dk + c : 0;
+      cs_cp16(&sm.shi[row][c], before_hi + src, in);
+      cs_cp16(&sm.slo[row][c], before_lo + src, in);
+    }
+  }
+  cs_commit();
   // pairs of blocks: weights of the tokens of block jt < bi for those of block bi
   float s[2][2][4] = {};  // [this warp's tiles: jt = half_w, half_w + 2][n8][..]
   {
@@ -418,54 +534,7 @@ tm_outputs_kernel(float* __restrict__ o, const __nv_bfloat16* __restrict__ r, in
       }
     }
   }
-  // pairs inside a block: lane (j, quarter of the channels), all i at once
-  {
-    const int j = lane & 15;
-    constexpr int QC = DKT / 4;
-    const int cbeg = (half_w * 2 + (lane >> 4)) * QC;
-    float acc[TC_BLK] = {};
-    for (int c = cbeg; c < cbeg + QC; c += 4) {
-      float x[4], uk[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        x[e] = __bfloat162float(sm.k[wm + j][c + e]);
-        uk[e] = c + e < dk ? u[(size_t)h * dk + c + e] * x[e] : 0.f;
-      }
-#pragma unroll
-      for (int i = 0; i < TC_BLK; ++i) {
-        const __nv_bfloat162* rp = reinterpret_cast<const __nv_bfloat162*>(&sm.r[wm + i][c]);
-        const float2 r0 = __bfloat1622float2(rp[0]), r1 = __bfloat1622float2(rp[1]);
-        const float4 d4 = *reinterpret_cast<const float4*>(&sm.d[wm + i][c]);
-        if (i > j) {
-          acc[i] += (r0.x * x[0] + r0.y * x[1]) + (r1.x * x[2] + r1.y * x[3]);
-          x[0] *= d4.x;
-          x[1] *= d4.y;
-          x[2] *= d4.z;
-          x[3] *= d4.w;
-        } else if (i == j) {
-          acc[i] += (r0.x * uk[0] + r0.y * uk[1]) + (r1.x * uk[2] + r1.y * uk[3]);
-        }
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < TC_BLK; ++i) acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 16);
-    if (lane < 16) {
-#pragma unroll
-      for (int i = 0; i < TC_BLK; ++i) sm.dsum[half_w][bi][j][i] = acc[i];
-    }
-  }
-  __syncthreads();  // r, k and kb have been read, the sums are there
-  if (has_state) {
-    const size_t st = ((size_t)chunk * H + h) * (size_t)dv * dk;
-    for (int idx = tid; idx < TC_DV * (DKT / 8); idx += CS_THREADS) {
-      const int row = idx / (DKT / 8), c = (idx - row * (DKT / 8)) * 8;
-      const bool in = v0 + row < dv && c < dk;
-      const size_t src = in ? st + (size_t)(v0 + row) * dk + c : 0;
-      cs_cp16(&sm.shi[row][c], before_hi + src, in);
-      cs_cp16(&sm.slo[row][c], before_lo + src, in);
-    }
-  }
-  cs_commit();
+  __syncthreads();  // kb and r's products have been read
 #pragma unroll
   for (int q = 0; q < 2; ++q) {
     const int jt = half_w + 2 * q;
@@ -488,7 +557,7 @@ tm_outputs_kernel(float* __restrict__ o, const __nv_bfloat16* __restrict__ r, in
     const float x = j <= i ? sm.dsum[0][b][j][i] + sm.dsum[1][b][j][i] : 0.f;
     cs_split(x, sm.p.hi[b * TC_BLK + i][b * TC_BLK + j], sm.p.lo[b * TC_BLK + i][b * TC_BLK + j]);
   }
-  if (has_state) {  // r times the product from the chunk's first token on
+  if (has_state && blk > 0) {  // r times the product from the chunk's first token on (block 0 has it already)
 #pragma unroll
     for (int tr = 0; tr < TRIPS; ++tr) {
       const int c = tr * 64 + (tid & 63);
@@ -543,6 +612,36 @@ tm_outputs_kernel(float* __restrict__ o, const __nv_bfloat16* __restrict__ r, in
       cs_mma(acc[2 * nj + 1], al, b[2], b[3]);
     }
   }
+  if (hg.out) {  // the head's norm and its gate (columns beyond dv are zero: their V is)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      float ss = 0.f;
+#pragma unroll
+      for (int ni = 0; ni < 4; ++ni) ss += acc[ni][2 * half] * acc[ni][2 * half] + acc[ni][2 * half + 1] * acc[ni][2 * half + 1];
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      if ((lane & 3) == 0) sm.squares[half_w][wm + g + half * 8] = ss;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int i = wm + g + half * 8;
+      if (i >= n) continue;
+      const float inv = 1.0f / sqrtf((sm.squares[0][i] + sm.squares[1][i]) / (float)dv + hg.eps);
+#pragma unroll
+      for (int ni = 0; ni < 4; ++ni) {
+        const int col = wn + ni * 8 + tg;
+        if (col >= dv) continue;
+        const size_t hc = (size_t)h * dv + col;
+        const float2 gt = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(hg.gate + (size_t)(t0 + i) * hg.ld_gate + hc));
+        const float2 nw = *reinterpret_cast<const float2*>(hg.norm_w + hc);
+        const float a = (acc[ni][2 * half] * inv) * nw.x * __fdividef(gt.x, 1.0f + __expf(-gt.x));
+        const float b = (acc[ni][2 * half + 1] * inv) * nw.y * __fdividef(gt.y, 1.0f + __expf(-gt.y));
+        *reinterpret_cast<__nv_bfloat162*>(hg.out + (size_t)(t0 + i) * H * dv + hc) = __floats2bfloat162_rn(a, b);
+      }
+    }
+    return;
+  }
 #pragma unroll
   for (int ni = 0; ni < 4; ++ni)
 #pragma unroll
@@ -553,7 +652,7 @@ tm_outputs_kernel(float* __restrict__ o, const __nv_bfloat16* __restrict__ r, in
 }
 
 template <int DKT>
-static int launch_chunks(float* o, float* state, const __nv_bfloat16* r, int ld_r, const __nv_bfloat16* k, int ld_k, const __nv_bfloat16* v, int ld_v,
+static int launch_chunks(float* o, const HeadGate& hg, float* state, const __nv_bfloat16* r, int ld_r, const __nv_bfloat16* k, int ld_k, const __nv_bfloat16* v, int ld_v,
                          const float* z, int ld_z, const float* w0, const float* u, float* added, __nv_bfloat16* before_hi,
                          __nv_bfloat16* before_lo, float* passed, const ChunkPlace& pl, int max_chunks, int H, int dk, int dv, cudaStream_t stream) {
   static bool configured = false;
@@ -565,9 +664,9 @@ static int launch_chunks(float* o, float* state, const __nv_bfloat16* r, int ld_
   const int v_tiles = ceil_div(dv, TC_DV);
   MS_LAUNCH(tm_states_kernel<DKT>, dim3(max_chunks, H, v_tiles), CS_THREADS, sizeof(TmStatesSmem<DKT>), stream, added, passed, k, ld_k, v, ld_v, z, ld_z,
             w0, pl, H, dk, dv);
-  MS_LAUNCH(tm_carry_kernel, dim3(ceil_div(H * dv * dk / 4, CS_THREADS), pl.num_rows), CS_THREADS, 0, stream, state, before_hi, before_lo, added, passed,
+  MS_LAUNCH(tm_carry_kernel, dim3(ceil_div(H * dv * dk, CS_THREADS), pl.num_rows), CS_THREADS, 0, stream, state, before_hi, before_lo, added, passed,
             pl, H, dk, dv);
-  MS_LAUNCH(tm_outputs_kernel<DKT>, dim3(max_chunks, H, v_tiles), CS_THREADS, sizeof(TmOutputsSmem<DKT>), stream, o, r, ld_r, k, ld_k, v, ld_v, z, ld_z,
+  MS_LAUNCH(tm_outputs_kernel<DKT>, dim3(max_chunks, H, v_tiles), CS_THREADS, sizeof(TmOutputsSmem<DKT>), stream, o, hg, r, ld_r, k, ld_k, v, ld_v, z, ld_z,
             w0, u, before_hi, before_lo, pl, H, dk, dv);
   return 0;
 }
@@ -614,15 +713,20 @@ MS_EXPORT int ms_time_step(void* out, float* state, const void* r, const void* k
 // 1 if the chunk kernels take these sizes.
 MS_EXPORT int ms_time_chunk_supports(int dk, int dv) { return dk >= 8 && dk <= 128 && dk % 8 == 0 && dv >= 8 && dv % 8 == 0; }
 
-// o [T, H, dv] float32; state [slots, H, dv, dk] float32; r, k [T, H * dk], v [T, H * dv] bfloat16 rows, z [T, H * dk] float32 rows. Scratch
+// o [T, H, dv] float32, or (o null, dv <= 64) out [T, H * dv] bfloat16 = o over its root mean square per head, times norm_w, times silu(gate);
+// state [slots, H, dv, dk] float32; r, k [T, H * dk], v [T, H * dv] bfloat16 rows, z [T, H * dk] float32 rows. Scratch
 // [max_chunks, H, dv, dk]: added float32, before_hi and before_lo bfloat16; passed float32 [max_chunks, H, dk].
-MS_EXPORT int ms_time_chunks(float* o, float* state, const void* r, int ld_r, const void* k, int ld_k, const void* v, int ld_v, const float* z, int ld_z,
+MS_EXPORT int ms_time_chunks(float* o, void* out, const void* gate, int ld_gate, const float* norm_w, float eps, float* state, const void* r, int ld_r, const void* k, int ld_k, const void* v, int ld_v, const float* z, int ld_z,
                              const float* w0, const float* u, float* added, void* before_hi, void* before_lo, float* passed, const int* tab,
                              const int* row_first, const int* cu_q, const int* q_start, const int* state_slot, int num_rows, int max_chunks, int H,
                              int dk, int dv, cudaStream_t stream) {
   if (num_rows == 0 || max_chunks == 0) return 0;
   MS_CHECK_ARG(ms_time_chunk_supports(dk, dv) && H > 0 && H <= 65535 && num_rows <= 65535 && (long long)H * dv * dk < (1LL << 31),
                "time_chunks: %d heads of %d x %d, %d rows", H, dk, dv, num_rows);
+  MS_CHECK_ARG((o != nullptr) != (out != nullptr) && (!out || (dv <= TC_DV && gate && norm_w && ld_gate % 2 == 0 && (uintptr_t)gate % 4 == 0 &&
+                                                              (uintptr_t)out % 4 == 0 && (uintptr_t)norm_w % 8 == 0)),
+               "time_chunks: either o, or for heads of up to %d values the gated output", TC_DV);
+  const HeadGate hg{(__nv_bfloat16*)out, (const __nv_bfloat16*)gate, ld_gate, norm_w, eps};
   MS_CHECK_ARG(ld_r % 8 == 0 && ld_k % 8 == 0 && ld_v % 8 == 0 && (uintptr_t)r % 16 == 0 && (uintptr_t)k % 16 == 0 && (uintptr_t)v % 16 == 0 &&
                    (uintptr_t)o % 8 == 0 && (uintptr_t)state % 16 == 0 && (uintptr_t)added % 16 == 0 && (uintptr_t)before_hi % 16 == 0 &&
                    (uintptr_t)before_lo % 16 == 0 && (uintptr_t)passed % 16 == 0,
@@ -630,8 +734,8 @@ MS_EXPORT int ms_time_chunks(float* o, float* state, const void* r, int ld_r, co
   const ChunkPlace pl{reinterpret_cast<const int2*>(tab), row_first, cu_q, q_start, state_slot, num_rows};
   const __nv_bfloat16 *rb = (const __nv_bfloat16*)r, *kb = (const __nv_bfloat16*)k, *vb = (const __nv_bfloat16*)v;
   if (dk <= 64)
-    return launch_chunks<64>(o, state, rb, ld_r, kb, ld_k, vb, ld_v, z, ld_z, w0, u, added, (__nv_bfloat16*)before_hi, (__nv_bfloat16*)before_lo, passed,
+    return launch_chunks<64>(o, hg, state, rb, ld_r, kb, ld_k, vb, ld_v, z, ld_z, w0, u, added, (__nv_bfloat16*)before_hi, (__nv_bfloat16*)before_lo, passed,
                              pl, max_chunks, H, dk, dv, stream);
-  return launch_chunks<128>(o, state, rb, ld_r, kb, ld_k, vb, ld_v, z, ld_z, w0, u, added, (__nv_bfloat16*)before_hi, (__nv_bfloat16*)before_lo, passed,
+  return launch_chunks<128>(o, hg, state, rb, ld_r, kb, ld_k, vb, ld_v, z, ld_z, w0, u, added, (__nv_bfloat16*)before_hi, (__nv_bfloat16*)before_lo, passed,
                             pl, max_chunks, H, dk, dv, stream);
 }

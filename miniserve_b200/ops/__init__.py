@@ -341,6 +341,38 @@ def linear_act(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, activat
     return out
 
 
+def linear_clamped_glu(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, limit: float, alpha: float, shift: float, scratch,
+                       bias: torch.Tensor | None = None, stream=None) -> torch.Tensor:
+    """out [M, I] = the clamped GLU (``clamped_glu``) of x W^T (+ bias) for the stacked weight [2 I, K] (gate rows, then up rows). bfloat16 with at
+    most 16 rows and no bias: one weight-streaming kernel; otherwise the product into ``scratch()`` [M, 2 I] and the activation kernel."""
+    m, kdim = x.shape
+    if x.dtype == torch.bfloat16 and bias is None and _skinny_ok(x, weight):
+        _check_dev(x, weight, out)
+        assert weight.shape == (2 * out.shape[1], kdim) and out.shape[0] == m
+        native.kernel_check(native.kernels().ms_gemm_skinny_clamped_glu_bf16(_ptr(out), _ptr(x), _ptr(weight), m, out.shape[1], kdim, float(limit),
+                                                                            float(alpha), float(shift), _stream(stream)))
+        return out
+    gate_up = linear(x, weight, out=scratch(), stream=stream)
+    clamped_glu(out, gate_up, bias, limit, alpha, shift, stream=stream)
+    return out
+
+
+def linear_inputs_ok(x: torch.Tensor, weight: torch.Tensor, rows_each: int) -> bool:
+    """Whether ``linear_inputs`` takes these operands: bfloat16, at most 16 rows per input, whole row tiles per input."""
+    return x.dtype == torch.bfloat16 and rows_each % 16 == 0 and _skinny_ok(x[0], weight)
+
+
+def linear_inputs(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, rows_each: int, tanh_from: int, stream=None) -> torch.Tensor:
+    """Products of several inputs in one launch (decode steps): x [inputs, M, K], weight [N, K], out [M, N]: columns [i * rows_each, (i + 1) *
+    rows_each) are input i times those rows of the weight (the last input takes all rows behind); from ``tanh_from`` on tanh of it."""
+    _check_dev(x, weight, out)
+    inputs, m, kdim = x.shape
+    assert weight.shape[1] == kdim and out.shape == (m, weight.shape[0]) and out.dtype == torch.bfloat16
+    native.kernel_check(native.kernels().ms_gemm_skinny_inputs_bf16(_ptr(out), _ptr(x), _ptr(weight), m, weight.shape[0], kdim, inputs, rows_each,
+                                                                    tanh_from, _stream(stream)))
+    return out
+
+
 def silu_mul_is_fused(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> bool:
     """Whether ``linear_silu_mul`` runs as one kernel for these operands (then it needs no scratch)."""
     if x.dtype != torch.bfloat16:

@@ -703,20 +703,32 @@ def time_chunks_ok(r, k, v, dk: int, dv: int, ctx) -> bool:
             and all(x.data_ptr() % 16 == 0 and x.stride(0) % 8 == 0 for x in (r, k, v)))
 
 
-def time_chunks(o, state, r, k, v, z, w0, bonus, ctx, heads: int, dk: int, dv: int) -> None:
+def time_chunks(out, state, r, k, v, z, w0, bonus, ctx, heads: int, dk: int, dv: int, gate, norm_w, eps: float, raw: bool = False) -> None:
     """The bonus rule with decays exp(-exp(z + w0)) per key channel over chunks of 64 tokens on the tensor cores (``csrc/time_mix.cu``),
-    from each request's slot of ``state`` [slots, heads, dv, dk] float32 and back into it. r, k [T, heads * dk], v [T, heads * dv]
-    bfloat16 views, z [T, heads * dk] float32; o [T, heads, dv] float32."""
-    t, dev = o.shape[0], o.device
-    _f32(o, state, w0, bonus)
-    assert o.shape == (t, heads, dv) and state.shape[1:] == (heads, dv, dk) and z.dtype == torch.float32
+    from each request's slot of ``state`` [slots, heads, dv, dk] float32 and back into it. r, k [T, heads * dk], v and gate [T, heads * dv]
+    bfloat16 views, z [T, heads * dk] float32; out [T, heads * dv] bfloat16 = the head's output over its root mean square, times norm_w
+    [heads * dv], times silu(gate). ``raw``: out [T, heads, dv] float32 is the output itself (gate and norm_w None). Heads of up to 64 values
+    are normed and gated where they are made; wider ones by a launch of their own."""
+    t, dev = z.shape[0], z.device
+    _f32(state, w0, bonus, norm_w)
+    assert state.shape[1:] == (heads, dv, dk) and z.dtype == torch.float32
     assert r.shape == k.shape == z.shape == (t, heads * dk) and v.shape == (t, heads * dv) and w0.numel() == bonus.numel() == heads * dk
+    fused = not raw and dv <= 64 and gate.stride(0) % 2 == 0 and gate.data_ptr() % 4 == 0
+    if raw:
+        assert out.dtype == torch.float32 and out.shape == (t, heads, dv) and out.is_contiguous()
+    else:
+        assert out.dtype == torch.bfloat16 and out.shape == (t, heads * dv) and out.is_contiguous()
+        assert gate.shape == (t, heads * dv) and gate.dtype == out.dtype and norm_w.numel() == heads * dv
+    o = out if raw else (None if fused else ctx.buffer("time.o", (t, heads, dv), torch.float32, dev))
     most, table = _chunk_table(t, ctx, dev)
     shape = (most, heads, dv, dk)
     added = ctx.buffer("chunk.added", shape, torch.float32, dev)
     before = ctx.buffer("chunk.before", (2, *shape), torch.bfloat16, dev)
     passed = ctx.buffer("chunk.passed", (most, heads, dk), torch.float32, dev)
     native.recurrence_check(native.recurrence().ms_time_chunks(
-        _ptr(o), _ptr(state), _ptr(r), _rows(r), _ptr(k), _rows(k), _ptr(v), _rows(v), _ptr(z), _rows(z), _ptr(w0), _ptr(bonus), _ptr(added),
+        _ptr(o), _ptr(out) if fused else None, _ptr(gate) if fused else None, _rows(gate) if fused else 0, _ptr(norm_w) if fused else None,
+        float(eps), _ptr(state), _ptr(r), _rows(r), _ptr(k), _rows(k), _ptr(v), _rows(v), _ptr(z), _rows(z), _ptr(w0), _ptr(bonus), _ptr(added),
         _ptr(before[0]), _ptr(before[1]), _ptr(passed), _ptr(table[0]), _ptr(table[1]), _ptr(ctx.cu_q), _ptr(ctx.q_start), _ptr(ctx.state_slot),
         ctx.num_rows, most, heads, dk, dv, ctx.stream), launches=3)
+    if not raw and not fused:
+        head_norm_gate(out, o, norm_w, gate, eps, 1.0, "silu", stream=ctx.stream)

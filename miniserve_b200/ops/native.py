@@ -101,6 +101,8 @@ def kernels():
     _declare(lib, "ms_gemm_skinny_bf16", [_p, _p, _p, _i, _i, _i, _i, _p])
     _declare(lib, "ms_gemm_skinny_gelu_bf16", [_p, _p, _p, _i, _i, _i, _p])
     _declare(lib, "ms_gemm_skinny_relu2_bf16", [_p, _p, _p, _i, _i, _i, _p])
+    _declare(lib, "ms_gemm_skinny_clamped_glu_bf16", [_p, _p, _p, _i, _i, _i, _f, _f, _f, _p])
+    _declare(lib, "ms_gemm_skinny_inputs_bf16", [_p, _p, _p, _i, _i, _i, _i, _i, _i, _p])
     _declare(lib, "ms_gemm_skinny_set_stream", [_i], None)
     _declare(lib, "ms_silu_mul", [_p, _p, _i, _i, _i, _p])
     _declare(lib, "ms_to_float", [_p, _p, _ll, _i, _p])
@@ -181,7 +183,7 @@ def recurrence():
     _declare(lib, "ms_channel_decay", [_p, _p, _i, _p, _i, _i, _i, _p])
     _declare(lib, "ms_time_step", [_p, _p, _p, _p, _p, _p, _i, _p, _i, _p, _i, _p, _p, _p, _f, _p, _p, _p, _i, _i, _i, _i, _i, _p])
     _declare(lib, "ms_time_chunk_supports", [_i, _i])
-    _declare(lib, "ms_time_chunks", [_p, _p] + [_p, _i] * 4 + [_p] * 11 + [_i] * 5 + [_p])
+    _declare(lib, "ms_time_chunks", [_p, _p, _p, _i, _p, _f, _p] + [_p, _i] * 4 + [_p] * 11 + [_i] * 5 + [_p])
     _declare(lib, "ms_rglru_scan", [_p, _p, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p])
     return lib
 
@@ -224,6 +226,7 @@ def gemm_tc():
     _declare(lib, "ms_gemm_tc_decode_bf16", [_p, _p, _p, _i, _i, _i, _p, _p])
     _declare(lib, "ms_gemm_tc_experts_bf16", [_p, _p, _p, _i, _i, _i, _i, _i, _p, _p, _p, _i, _f, _f, _f, _p, _p])
     _declare(lib, "ms_gemm_tc_set_config", [_i], None)
+    _declare(lib, "ms_gemm_tc_set_grouped", [_i], None)
     _declare(lib, "ms_gemm_tc_prefers", [_i, _i, _i, _i])
     _declare(lib, "ms_gemm_tc_qkv_bf16", [_p, _p, _p, _i, _i, _i, _i] + [_p] * 9 + [_i, _f, _p, _p])
     lib.ms_gemm_tc_set_pdl(int(pdl_enabled()))

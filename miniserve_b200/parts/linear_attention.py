@@ -327,7 +327,8 @@ class TimeMix(Part):
         d_t = exp(-exp(W_w2 tanh(W_w1 mix_w) + w0)),   o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t,   S_t = diag(d_t) S_(t-1) + k_t v_t^T
 
     per head, S [dim, dim]; each head's o is divided by its root mean square, the heads side by side times a weight, times silu(W_g mix_g),
-    then W_o. One launch makes the five mixes, one batched product r|k|v|g, two small ones the decays' logits (the second in float32);
+    then W_o. One launch makes the five mixes, one batched product r|k|v|g, two small ones the decays' logits (the second in float32; a
+    decode step has the first one and the tanh in the same launch as r|k|v|g);
     a decode step goes from the low-rank input to the gated heads in one kernel, prompts in bfloat16 run by chunks on the tensor cores,
     the rest token by token (``csrc/time_mix.cu``, ``csrc/recurrence.cu``). S is float32.
     Parameters: ``hidden``, ``heads``, ``head_dim``, ``decay_rank``, ``eps``, ``names`` (r, k, v, g, o, norm, w1, w2, w0, u and mu: the
@@ -360,14 +361,16 @@ class TimeMix(Part):
         return out
 
     def stacks(self):
-        return {"rkvg_proj.weight": tuple(self.names[x] for x in "rkvg")}
+        return {"rkvgw_proj.weight": tuple(self.names[x] for x in ("r", "k", "v", "g", "w1"))}
 
     def bind(self, tensors):
         n = self.names
-        self.w_in = self.joined(tensors, "rkvg_proj.weight", self.stacks()["rkvg_proj.weight"]).view(4, self.feature_width, self.hidden)
-        self.w_mu = torch.stack([tensors[n["mu"] + x].float() for x in self.INPUTS]).contiguous()
+        c = self.feature_width
+        joined = self.joined(tensors, "rkvgw_proj.weight", self.stacks()["rkvgw_proj.weight"])
         rank = _pad8(self.rank)  # a rank that is no multiple of 8: zero rows and columns (tanh of zero is zero)
-        self.w_w1, self.w_w2 = _pad_rows(tensors[n["w1"]], rank), _pad_cols(tensors[n["w2"]], rank)
+        self.w_all = _pad_rows(joined, 4 * c + rank)
+        self.w_mu = torch.stack([tensors[n["mu"] + x].float() for x in self.INPUTS]).contiguous()
+        self.w_w2 = _pad_cols(tensors[n["w2"]], rank)
         self.w_w0, self.w_u, self.w_norm = (tensors[n[k]].float().reshape(-1).contiguous() for k in ("w0", "u", "norm"))
         self.w_o = tensors[n["o"]].contiguous()
 
@@ -377,21 +380,26 @@ class TimeMix(Part):
         state, before = cache
         mixed = ctx.buffer("time.mixes", (5, t, self.hidden), dt, dev)
         ops.token_mixes(mixed, x, before.state, self.w_mu, ctx)
-        proj = ctx.buffer("time.in", (t, 4, c), dt, dev)
-        ops.linear_heads(mixed[:4].transpose(0, 1), self.w_in, proj, stream=ctx.stream)
-        low = ops.linear(mixed[4], self.w_w1, stream=ctx.stream, out=ctx.buffer("time.low", (t, self.w_w1.shape[0]), dt, dev))
-        ops.tanh_(low, stream=ctx.stream)
-        r, k, v, g = (proj[:, i] for i in range(4))
-        if ctx.decode_only and ops.time_step_ok(d, d, self.w_w2.shape[1]):
+        single = ctx.decode_only and ops.time_step_ok(d, d, self.w_w2.shape[1])
+        if single and ops.linear_inputs_ok(mixed, self.w_all, c):  # all five products and the tanh in one launch
+            proj = ops.linear_inputs(mixed, self.w_all, ctx.buffer("time.in", (t, self.w_all.shape[0]), dt, dev), c, 4 * c, stream=ctx.stream)
+            low = proj[:, 4 * c:]
+        else:
+            proj = ctx.buffer("time.in", (t, 4 * c), dt, dev)
+            ops.linear_heads(mixed[:4].transpose(0, 1), self.w_all[:4 * c].view(4, c, self.hidden), proj.view(t, 4, c), stream=ctx.stream)
+            low = ops.linear(mixed[4], self.w_all[4 * c:], stream=ctx.stream, out=ctx.buffer("time.low", (t, self.w_w2.shape[1]), dt, dev))
+            ops.tanh_(low, stream=ctx.stream)
+        r, k, v, g = (proj[:, i * c:(i + 1) * c] for i in range(4))
+        if single:
             ops.time_step(out, state.state, r, k, v, g, low, self.w_w2, self.w_w0, self.w_u, self.w_norm, self.eps, ctx, h)
             return
         z = ops.linear(low, self.w_w2, stream=ctx.stream, out=ctx.buffer("time.z", (t, c), torch.float32, dev))
-        o = ctx.buffer("time.o", (t, h, d), torch.float32, dev)
         if ops.time_chunks_ok(r, k, v, d, d, ctx):
-            ops.time_chunks(o, state.state, r, k, v, z, self.w_w0, self.w_u, ctx, h, d, d)
-        else:
-            ops.channel_decay(z, z, self.w_w0, stream=ctx.stream)
-            ops.decay_scan(o, state.state, r, k, v, z, None, None, 0.0, None, ctx, h, d, d, 1.0, delta=False, bonus=self.w_u)
+            ops.time_chunks(out, state.state, r, k, v, z, self.w_w0, self.w_u, ctx, h, d, d, g, self.w_norm, self.eps)
+            return
+        o = ctx.buffer("time.o", (t, h, d), torch.float32, dev)
+        ops.channel_decay(z, z, self.w_w0, stream=ctx.stream)
+        ops.decay_scan(o, state.state, r, k, v, z, None, None, 0.0, None, ctx, h, d, d, 1.0, delta=False, bonus=self.w_u)
         ops.head_norm_gate(out, o, self.w_norm, g, self.eps, 1.0, "silu", stream=ctx.stream)
 
     def forward(self, x, ctx, cache):

@@ -68,7 +68,7 @@ class SwiGLU(Part):
 class ClampedGLU(Part):
     """down(g * sigmoid(alpha g) * (u + up_shift)) with g = min(gate(x), limit) and u = clamp(up(x), -limit, limit); every
     projection may have a bias. The gate and up matrices are stacked as in ``swiglu``; their biases are added, and the
-    clamps and the activation computed, in float32 by one kernel behind the product. Parameters: ``hidden``,
+    clamps and the activation computed, in float32 by one kernel behind the product (without biases, in the decode product's epilogue). Parameters: ``hidden``,
     ``intermediate``, ``limit`` (absent: no clamps), optional ``alpha`` (1.702), ``up_shift`` (1.0), ``bias`` (True), ``names``
     (gate / up / down and gate_bias / up_bias / down_bias -> tensor names)."""
     shape_static = True
@@ -118,9 +118,10 @@ class ClampedGLU(Part):
 
     def forward(self, x, ctx, with_bias: bool = True) -> torch.Tensor:
         t, dt, dev = x.shape[0], self.env.dtype, self.w_down.device
-        gate_up = ops.linear(x, self.w_gate_up, stream=ctx.stream, out=ctx.buffer("mlp.gate_up", (t, 2 * self.inter), dt, dev))
         act = ctx.buffer("mlp.act", (t, self.inter), dt, dev)
-        ops.clamped_glu(act, gate_up, self.w_in_bias, self.limit, self.alpha, self.up_shift, stream=ctx.stream)
+        # (without biases a decode step has the activation in the product's epilogue)
+        ops.linear_clamped_glu(x, self.w_gate_up, act, self.limit, self.alpha, self.up_shift, bias=self.w_in_bias, stream=ctx.stream,
+                               scratch=lambda: ctx.buffer("mlp.gate_up", (t, 2 * self.inter), dt, dev))
         out = ops.linear(act, self.w_down, stream=ctx.stream, out=ctx.buffer("mlp.down", (t, self.hidden), dt, dev))
         if with_bias and self.w_out_bias is not None:
             ops.sum_bias(out, out, None, self.w_out_bias, stream=ctx.stream)

@@ -11,6 +11,8 @@ summaries under ``profiles/`` were measured and captured with.
     python -m miniserve_b200.tools.kernel_bench pointwise --op channel_gate --tokens 2048 --heads 16 --head-dim 128
     python -m miniserve_b200.tools.kernel_bench decay_scan --tokens 2048 --heads 4 --key-dim 128 --value-dim 256 --head-decay [--chunks]
     python -m miniserve_b200.tools.kernel_bench recurrent --op rglru_scan --tokens 2048 --n 1024 --blocks 4
+    python -m miniserve_b200.tools.kernel_bench time_mix --op time_chunks --tokens 2048 --batch 1 --heads 16 --key-dim 64 --n 1024
+    python -m miniserve_b200.tools.kernel_bench routing --op expert_route --tokens 2048 --experts 16 --top 3 --n 1024
 
 Each case rotates over enough copies of its inputs to exceed the L2 cache, captures one pass over
 all copies in a CUDA graph, and reports the time per launch with the bytes or flops it implies.
@@ -61,6 +63,7 @@ def _paged(rows, page, nkv, d, seed, device):
 
 def _time(calls, copies, launches):
     """calls(i, stream) launches the kernel on input copy i."""
+    torch.cuda.synchronize()  # the inputs were made on another stream
     s = torch.cuda.Stream()
     if launches:
         with torch.cuda.stream(s):
@@ -92,7 +95,8 @@ def _time(calls, copies, launches):
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__.splitlines()[0])
-    ap.add_argument("kernel", choices=["attn_decode", "attn_prefill", "skinny", "add_rmsnorm", "gemm", "gate_up", "sample", "decay_scan", "pointwise", "experts", "recurrent"])
+    ap.add_argument("kernel", choices=["attn_decode", "attn_prefill", "skinny", "add_rmsnorm", "gemm", "gate_up", "sample", "decay_scan", "pointwise", "experts", "recurrent",
+                                       "time_mix", "routing"])
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=2048)
     ap.add_argument("--tokens", type=int, default=2048)
@@ -122,12 +126,14 @@ def main(argv=None) -> int:
     ap.add_argument("--op", choices=["channel_gate", "head_gate", "relu_squared", "gelu_tanh", "latent_prepare", "qkv_prepare",
                                      "layernorm", "layernorm_pair", "token_shift", "clamped_glu", "sum_bias", "act_mul", "axpby", "normed_add",
                                      "embed_gather", "embed_sum", "mlstm_gates", "mlstm_output", "gated_group_norm", "conv_bias", "conv_silu",
-                                     "rglru_gates", "rglru_scan"],
+                                     "rglru_gates", "rglru_scan", "time_chunks", "time_walk", "time_step", "token_mixes", "stream_norm", "expert_route",
+                                     "expert_combine"],
                     default="channel_gate", help="pointwise: which kernel (--tokens rows; --heads x --head-dim, or --n, columns)")
     ap.add_argument("--head-decay", action="store_true", help="decay_scan: one decay per head, worked out beforehand (float32), a column of ones")
     ap.add_argument("--chunks", action="store_true", help="decay_scan --head-decay: by chunks on the tensor cores")
     ap.add_argument("--blocks", type=int, default=4, help="recurrent: equal parts of the --n channels, a gate matrix each")
     ap.add_argument("--taps", type=int, default=4, help="recurrent: taps of the convolution")
+    ap.add_argument("--streams", type=int, default=2, help="time_mix stream_norm: residual streams")
     ap.add_argument("--plain-experts", action="store_true", help="experts: without a gate, the square of relu")
     ap.add_argument("--experts", type=int, default=14, help="experts: how many experts")
     ap.add_argument("--top", type=int, default=4, help="experts: choices per token")
@@ -381,6 +387,67 @@ def main(argv=None) -> int:
                 ops.rglru_scan(s.out, state, s.z, s.u, s.y[:, :n], va, vb, vc, vd, ctx)
 
         vec_gates, conv_w_rows = vec(2 * hh), conv_w.t().contiguous()
+    elif args.kernel == "time_mix":
+        # time mixing with a bonus and what surrounds it: `batch` requests of `tokens` tokens each, --heads of --key-dim, --n channels in the model
+        rows, t, n, hh, dk, st = args.batch, args.batch * args.tokens, args.n, args.heads, args.key_dim, args.streams
+        c, rank = hh * dk, 64
+        i32, f32, bf = (dict(dtype=d, device=dev) for d in (torch.int32, torch.float32, torch.bfloat16))
+        bufs = {}
+
+        def buffer(role, shape, dt, device):
+            return bufs.setdefault((role, shape, dt), torch.empty(shape, dtype=dt, device=device))
+
+        ctx = SimpleNamespace(cu_q=torch.arange(0, t + 1, args.tokens, **i32), q_start=torch.ones(rows, **i32), state_slot=torch.arange(rows, **i32),
+                              row_of_token=(torch.arange(t, device=dev) // args.tokens).to(torch.int32), num_rows=rows,
+                              decode_only=args.tokens == 1, buffer=buffer, step_cache={}, stream=0)
+        copies = max(2, min(64, int(L2_BYTES // (t * c * 14 + t * n * (4 * st + 12) + rows * c * dk * 4)) + 1))
+        sets = [SimpleNamespace(proj=torch.randn(t, 4 * c + rank, **bf), z=torch.randn(t, c, **f32), o=torch.empty(t, hh, dk, **f32),
+                                feat=torch.empty(t, c, **bf), x=torch.randn(t, n, **bf), mixes=torch.empty(5, t, n, **bf),
+                                streams=torch.randn(t, st, n, **f32), y=torch.randn(t, n, **bf), state=torch.zeros(rows, hh, dk, dk, **f32))
+                for _ in range(copies)]
+        w2, mu, before = (torch.randn(c, rank, device=dev) * 0.1).bfloat16(), torch.rand(5, n, **f32), torch.zeros(rows, n, **bf)
+        w0, bonus, norm_w, wn = torch.randn(c, **f32) - 2, torch.randn(c, **f32), torch.ones(c, **f32), torch.ones(n, **f32)
+        mix, link = torch.eye(st, **f32), torch.ones(st, **f32)
+        state_bytes = 2 * rows * c * dk * 4
+        byts = {"time_chunks": t * c * (2 * 5 + 4) + state_bytes, "time_walk": t * c * (2 * 3 + 4 + 4) + state_bytes,
+                "time_step": t * c * 2 * 5 + state_bytes + c * rank * 2, "token_mixes": t * n * 12, "stream_norm": t * n * (8 * st + 4)}[args.op]
+        work = dict(bytes=byts)
+
+        def calls(i, stream):
+            s = sets[i]
+            ctx.stream = stream
+            r, k, v, g = (s.proj[:, q * c:(q + 1) * c] for q in range(4))
+            if args.op == "time_chunks":
+                ops.time_chunks(s.feat, s.state, r, k, v, s.z, w0, bonus, ctx, hh, dk, dk, g, norm_w, 1e-6)
+            elif args.op == "time_walk":
+                ops.decay_scan(s.o, s.state, r, k, v, s.z, None, None, 0.0, None, ctx, hh, dk, dk, 1.0, delta=False, bonus=bonus)
+            elif args.op == "time_step":
+                ops.time_step(s.feat, s.state, r, k, v, g, s.proj[:, 4 * c:], w2, w0, bonus, norm_w, 1e-6, ctx, hh)
+            elif args.op == "token_mixes":
+                ops.token_mixes(s.mixes, s.x, before, mu, ctx)
+            else:
+                ops.stream_norm(s.feat[:, :n] if c == n else s.mixes[0], s.streams, s.y, mix, link, link, wn, 1e-6, stream=stream)
+    elif args.kernel == "routing":
+        # the router with its choice, and the weighted sum: --tokens tokens, --top choices among --experts experts in 4 groups, --n channels
+        from ..ops import experts as xo
+
+        t, e, top, n = args.tokens, args.experts, args.top, args.n
+        i32, f32, bf = (dict(dtype=d, device=dev) for d in (torch.int32, torch.float32, torch.bfloat16))
+        per_set = t * n * 2 + e * n * 4 if args.op == "expert_route" else t * n * (4 * top + 4)
+        copies = max(2, min(256, int(L2_BYTES // per_set) + 1))
+        sets = [SimpleNamespace(x=torch.randn(t, n, **bf), router=torch.randn(e, n, **f32),
+                                y=torch.randn(t * top, n, **f32) if args.op == "expert_combine" else None, shared=torch.randn(t, n, **bf),
+                                out=torch.empty(t, n, **bf)) for _ in range(copies)]
+        idx, wgt = torch.stack([torch.randperm(e, device=dev)[:top] for _ in range(t)]).to(torch.int32).contiguous(), torch.rand(t, top, **f32)
+        pos = torch.randperm(t * top, device=dev).to(torch.int32)
+        work = dict(bytes=t * n * 2 + e * n * 4 if args.op == "expert_route" else t * n * (4 * top + 4))
+
+        def calls(i, stream):
+            s = sets[i]
+            if args.op == "expert_route":
+                xo.expert_route(idx, wgt, s.x, s.router, None, top, 4, 2, 1.5, True, stream=stream, score="sigmoid", group_best=2, renorm_eps=1e-20)
+            else:
+                xo.expert_combine(s.out, s.y, s.x, idx, wgt, pos, e, stream=stream, shared=s.shared)
     else:
         # the linear-attention recurrence: `batch` requests of `tokens` tokens each (1: a decode step), from zero state
         t, hh, dk, dv, rows = args.tokens * args.batch, args.heads, args.key_dim, args.value_dim, args.batch
