@@ -119,9 +119,12 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
       : "r"(taddr));
 }
 
-template <int BN>
+// AROWS: rows of A that a stage holds. Fewer than the instruction's 128 (a few rows per expert): the products of the rows behind them read
+// whatever lies there and are not stored.
+template <int BN, int AROWS = TC_BM>
 struct TcSmem {
-  static constexpr int a_bytes = TC_BM * TC_BK * 2;
+  static constexpr int a_bytes = AROWS * TC_BK * 2;
+  static constexpr int overread = (TC_BM - AROWS) * TC_BK * 2;  // behind the last stage
   static constexpr int b_bytes = BN * TC_BK * 2;
   static constexpr int stage_bytes = a_bytes + b_bytes;
 };
@@ -153,8 +156,8 @@ struct TcGroups {
 // (gate rows, then up rows), BN is 256 and a CTA computes 128 gate and the matching 128 up columns.
 // GROUPED: blockIdx.y walks the plan's row tiles instead (the grid has as many as a step can have at most, the
 // surplus CTAs leave at once); a tile's rows beyond its run are computed with the run's matrix and not stored.
-template <int BN, int STAGES, int EPI, bool GROUPED = false>
-__global__ void __launch_bounds__(TC_THREADS, (STAGES * (TC_BM + BN) * TC_BK * 2 + 2048 <= 110 * 1024) ? 2 : 1)
+template <int BN, int STAGES, int EPI, bool GROUPED = false, int AROWS = TC_BM>
+__global__ void __launch_bounds__(TC_THREADS, (STAGES * (AROWS + BN) * TC_BK * 2 + (TC_BM - AROWS) * TC_BK * 2 + 2048 <= 112 * 1024) ? 2 : 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w, void* __restrict__ out,
                int M, int N_out, int K, int up_row_offset, int* __restrict__ status, const TcGroups grp) {
   extern __shared__ unsigned char smem_dyn[];
@@ -175,7 +178,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
     if ((int)blockIdx.y >= grp.meta[0]) return;
     const int e = grp.tiles[2 * blockIdx.y];
     m0 = grp.tiles[2 * blockIdx.y + 1];
-    M = min(M, grp.offsets[e + 1]);
+    M = min(min(M, grp.offsets[e + 1]), m0 + AROWS);
     w0 = e * grp.w_rows + n0;
   }
   const int k_iters = (K + TC_BK - 1) / TC_BK;
@@ -212,13 +215,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
           gave_up = 1;
           break;
         }
-        unsigned char* a_tile = smem + (size_t)s * TcSmem<BN>::stage_bytes;
-        unsigned char* b_tile = a_tile + TcSmem<BN>::a_bytes;
-        mbar_expect_tx(&full_bar[s], TcSmem<BN>::stage_bytes);
+        unsigned char* a_tile = smem + (size_t)s * TcSmem<BN, AROWS>::stage_bytes;
+        unsigned char* b_tile = a_tile + TcSmem<BN, AROWS>::a_bytes;
+        mbar_expect_tx(&full_bar[s], TcSmem<BN, AROWS>::stage_bytes);
         tma_load_2d(a_tile, &map_a, &full_bar[s], it * TC_BK, m0);
         if (tc_gated(EPI)) {
           tma_load_2d(b_tile, &map_w, &full_bar[s], it * TC_BK, w0);
-          tma_load_2d(b_tile + TcSmem<BN>::b_bytes / 2, &map_w, &full_bar[s], it * TC_BK, up_row_offset + w0);
+          tma_load_2d(b_tile + TcSmem<BN, AROWS>::b_bytes / 2, &map_w, &full_bar[s], it * TC_BK, up_row_offset + w0);
         } else {
           tma_load_2d(b_tile, &map_w, &full_bar[s], it * TC_BK, w0);
         }
@@ -237,8 +240,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
           break;
         }
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        const unsigned char* a_tile = smem + (size_t)s * TcSmem<BN>::stage_bytes;
-        const unsigned char* b_tile = a_tile + TcSmem<BN>::a_bytes;
+        const unsigned char* a_tile = smem + (size_t)s * TcSmem<BN, AROWS>::stage_bytes;
+        const unsigned char* b_tile = a_tile + TcSmem<BN, AROWS>::a_bytes;
         const uint64_t da = make_smem_desc(a_tile), db = make_smem_desc(b_tile);
 #pragma unroll
         for (int k = 0; k < TC_BK / 16; ++k) {
@@ -1149,14 +1152,14 @@ static int launch_tc(void* out, const void* A, const void* W, int M, int N_out, 
 }
 
 // The grouped form: A [rows, K] sorted by matrix, W [matrices * w_rows, K], the plan on the device.
-template <int BN, int STAGES, int EPI>
+template <int BN, int STAGES, int EPI, int AROWS = TC_BM>
 static int launch_tc_grouped(void* out, const void* A, const void* W, int rows, int N_out, int matrices, int w_rows, int K,
                              int up_row_offset, const TcGroups& grp, int max_tiles, int* status, cudaStream_t stream) {
   CUtensorMap map_a, map_w;
-  if (int rc = make_map(&map_a, A, rows, K, TC_BM)) return rc;
+  if (int rc = make_map(&map_a, A, rows, K, AROWS)) return rc;
   if (int rc = make_map(&map_w, W, (long long)matrices * w_rows, K, tc_gated(EPI) ? BN / 2 : BN)) return rc;
-  constexpr size_t smem = (size_t)STAGES * TcSmem<BN>::stage_bytes + 1024;
-  auto kernel = gemm_tc_kernel<BN, STAGES, EPI, true>;
+  constexpr size_t smem = (size_t)STAGES * TcSmem<BN, AROWS>::stage_bytes + TcSmem<BN, AROWS>::overread + 1024;
+  auto kernel = gemm_tc_kernel<BN, STAGES, EPI, true, AROWS>;
   static bool configured = false;
   if (!configured) {
     MS_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
@@ -1380,54 +1383,60 @@ MS_EXPORT int ms_gemm_tc_bf16(void* out, const void* A, const void* W, int M, in
   }
 }
 
-// Tiles of the grouped products: 1: 256 columns of W (gated) or 128, one CTA an SM; 2: 128, a shorter ring, two CTAs an SM, so that one CTA's
+// Rows per tile: 128, or 32 where an expert has a few rows (decode steps): then a CTA takes 64 columns of W, so that the weights are spread over
+// all SMs, and fetches 32 rows of A a stage.
+constexpr int TC_FEW_ROWS = 32;
+// Tiles of the grouped products of 128 rows: 1: 256 columns of W (gated) or 128, one CTA an SM; 2: 128, a shorter ring, two CTAs an SM, so that one CTA's
 // epilogue hides behind the other's products. 0: chosen from the rows per expert (measured on B200 with 16 experts, both products: 2,048 tokens x 3
 // choices at 768 of 1024: 75.6 us with 2, 87.7 with 1; at 1536 of 2048: 182 against 202; 8 tokens: 39.5 against 35.6 and 94 against 65).
 static int g_grouped_config = 0;
 MS_EXPORT void ms_gemm_tc_set_grouped(int config) { g_grouped_config = config; }
 
 template <int EPI>
-static int launch_grouped_gated(void* out, const void* A, const void* W, int rows, int N, int experts, int K, const TcGroups& grp, int max_tiles,
-                                int* status, cudaStream_t stream) {
+static int launch_grouped_gated(void* out, const void* A, const void* W, int rows, int N, int experts, int K, const TcGroups& grp, int tile_rows,
+                                int max_tiles, int* status, cudaStream_t stream) {
+  if (tile_rows == TC_FEW_ROWS) return launch_tc_grouped<64, 7, EPI, TC_FEW_ROWS>(out, A, W, rows, N, experts, 2 * N, K, N, grp, max_tiles, status, stream);
   const bool narrow = g_grouped_config ? g_grouped_config == 2 : rows >= 128 * experts;
   if (narrow) return launch_tc_grouped<128, 3, EPI>(out, A, W, rows, N, experts, 2 * N, K, N, grp, max_tiles, status, stream);
   return launch_tc_grouped<256, 4, EPI>(out, A, W, rows, N, experts, 2 * N, K, N, grp, max_tiles, status, stream);
 }
 
 template <int EPI>
-static int launch_grouped_plain(void* out, const void* A, const void* W, int rows, int N, int experts, int K, const TcGroups& grp, int max_tiles,
-                                int* status, cudaStream_t stream) {
+static int launch_grouped_plain(void* out, const void* A, const void* W, int rows, int N, int experts, int K, const TcGroups& grp, int tile_rows,
+                                int max_tiles, int* status, cudaStream_t stream) {
+  if (tile_rows == TC_FEW_ROWS) return launch_tc_grouped<64, 7, EPI, TC_FEW_ROWS>(out, A, W, rows, N, experts, N, K, 0, grp, max_tiles, status, stream);
   const bool narrow = g_grouped_config ? g_grouped_config == 2 : rows >= 128 * experts;
   if (narrow) return launch_tc_grouped<128, 3, EPI>(out, A, W, rows, N, experts, N, K, 0, grp, max_tiles, status, stream);
   return launch_tc_grouped<128, 5, EPI>(out, A, W, rows, N, experts, N, K, 0, grp, max_tiles, status, stream);
 }
 
-// The experts' products of a routed feed-forward over rows sorted by expert (tiles of 128 rows, (expert, first row)
+// The experts' products of a routed feed-forward over rows sorted by expert (tiles of 128 or 32 rows, (expert, first row)
 // each; meta[0] tiles; offsets[e + 1] ends expert e's rows; at most max_tiles tiles).
 // gated = 1: W [E, 2 N, K] (an expert's gate rows, then its up rows), out [rows, N] bfloat16 = silu(A gate^T) * (A up^T);
 // gated = 0: W [E, N, K], out [rows, N] float32 = A W^T; gated = 2: W [E, N, K], out [rows, N] bfloat16 = relu(A W^T)^2;
 // gated = 3: W as for 1, the gate clamped and shifted (ClampedGlu).
 MS_EXPORT int ms_gemm_tc_experts_bf16(void* out, const void* A, const void* W, int rows, int N, int K, int experts, int gated,
-                                      const int* tiles, const int* meta, const int* offsets, int max_tiles, float limit,
+                                      const int* tiles, const int* meta, const int* offsets, int tile_rows, int max_tiles, float limit,
                                       float alpha, float shift, int* status, cudaStream_t stream) {
   if (rows == 0 || N == 0 || max_tiles == 0) return 0;
   MS_CHECK_ARG(rows > 0 && N > 0 && K > 0 && experts > 0, "gemm_tc_experts: bad sizes rows=%d N=%d K=%d experts=%d", rows, N, K, experts);
   MS_CHECK_ARG(K % 8 == 0, "gemm_tc_experts: K=%d must be a multiple of 8 (rows must be 16-byte multiples for TMA)", K);
   MS_CHECK_ARG(((uintptr_t)A % 16 == 0) && ((uintptr_t)W % 16 == 0), "gemm_tc_experts: operands must be 16-byte aligned");
   MS_CHECK_ARG(status != nullptr && tiles != nullptr && meta != nullptr && offsets != nullptr, "gemm_tc_experts: needs a plan and a status word");
+  MS_CHECK_ARG(tile_rows == TC_BM || tile_rows == TC_FEW_ROWS, "gemm_tc_experts: tiles of %d rows", tile_rows);
   MS_CHECK_ARG(max_tiles <= 65535, "gemm_tc_experts: %d row tiles are too many for one launch", max_tiles);
   MS_CHECK_ARG((long long)experts * (gated == 1 || gated == 3 ? 2 : 1) * N < (1LL << 31), "gemm_tc_experts: the weights have too many rows");
   if (gated == 3) {
     const TcGroups grp{tiles, meta, offsets, 2 * N, {limit, alpha, shift}};
-    return launch_grouped_gated<TC_CLAMPED_GLU>(out, A, W, rows, N, experts, K, grp, max_tiles, status, stream);
+    return launch_grouped_gated<TC_CLAMPED_GLU>(out, A, W, rows, N, experts, K, grp, tile_rows, max_tiles, status, stream);
   }
   if (gated == 1) {
     const TcGroups grp{tiles, meta, offsets, 2 * N, {}};
-    return launch_grouped_gated<TC_SILU_MUL>(out, A, W, rows, N, experts, K, grp, max_tiles, status, stream);
+    return launch_grouped_gated<TC_SILU_MUL>(out, A, W, rows, N, experts, K, grp, tile_rows, max_tiles, status, stream);
   }
   const TcGroups grp{tiles, meta, offsets, N, {}};
-  if (gated == 2) return launch_grouped_plain<TC_RELU2>(out, A, W, rows, N, experts, K, grp, max_tiles, status, stream);
-  return launch_grouped_plain<TC_OUT_F32>(out, A, W, rows, N, experts, K, grp, max_tiles, status, stream);
+  if (gated == 2) return launch_grouped_plain<TC_RELU2>(out, A, W, rows, N, experts, K, grp, tile_rows, max_tiles, status, stream);
+  return launch_grouped_plain<TC_OUT_F32>(out, A, W, rows, N, experts, K, grp, tile_rows, max_tiles, status, stream);
 }
 
 // out [M, N] bfloat16 = X [M, K] W [N, K]^T for M <= 64 tokens (decode steps), see gemm_tc_decode_kernel.

@@ -15,6 +15,7 @@ NO_CLAMPS = (-1.0, 1.0, 0.0)  # (limit, alpha, shift) of a clamped GLU; other ac
 SCORES = {"softmax": 0, "sigmoid": 1}
 TILE_ROWS = 64       # sorted rows per tile of the float32 and mma.sync products
 TC_TILE_ROWS = 128   # of the products on the tcgen05 tensor cores
+TC_FEW_ROWS = 32     # of the same where an expert has a few rows (decode steps)
 TC_EXPERTS = os.environ.get("MINISERVE_TC_EXPERTS", "1") != "0"  # bfloat16 experts on the tcgen05 kernel where it takes the shape
 
 
@@ -23,6 +24,14 @@ def tc_experts_ok(dtype, hidden: int, inter: int, activation: str) -> bool:
     bfloat16, an activation that the kernel has as an epilogue (SiLU times the up half, the clamped GLU, or the square of relu without a
     gate), rows that are multiples of 16 bytes."""
     return TC_EXPERTS and dtype == torch.bfloat16 and activation in ("silu", "relu_squared", "clamped_glu") and hidden % 8 == 0 and inter % 8 == 0
+
+
+def tc_tile_rows(slots: int, experts: int) -> int:
+    """Rows per tile of the tcgen05 products for a step of ``slots`` (token, choice) pairs."""
+    return TC_FEW_ROWS if slots <= FEW_ROWS_PER_EXPERT * experts else TC_TILE_ROWS
+
+
+FEW_ROWS_PER_EXPERT = 16  # up to so many rows per expert on average: tiles of TC_FEW_ROWS
 
 
 def expert_route(idx, wgt, x, router, correction, top: int, group_count: int, group_keep: int, weight_scale: float,
@@ -75,8 +84,9 @@ def expert_gather(xs, x, perm, meta, top: int, stream=None) -> None:
                                                            _stream(stream)))
 
 
-def expert_products_tc(out, a, w, tiles, meta, offsets, gated: bool, stream=None, relu_squared: bool = False, clamps=None) -> None:
-    """The experts' products over sorted rows on the tcgen05 tensor cores (tiles of ``TC_TILE_ROWS`` rows).
+def expert_products_tc(out, a, w, tiles, meta, offsets, gated: bool, stream=None, relu_squared: bool = False, clamps=None,
+                       tile_rows: int = TC_TILE_ROWS) -> None:
+    """The experts' products over sorted rows on the tcgen05 tensor cores (the plan's tiles have ``tile_rows`` rows: ``tc_tile_rows``).
     ``gated``: out [S, I] bfloat16 = silu(a W_gate[e]^T) * (a W_up[e]^T) (or with ``clamps`` = (limit, alpha, shift) the clamped GLU of the two) with ``w`` [E, 2 I, K]; else out [S, N] float32 =
     a W[e]^T with ``w`` [E, N, K] (``relu_squared``: bfloat16, the square of its relu). ``a`` [S, K] bfloat16 in sorted order."""
     from . import device_status
@@ -89,7 +99,7 @@ def expert_products_tc(out, a, w, tiles, meta, offsets, gated: bool, stream=None
     lib = native.gemm_tc()
     mode = 2 if relu_squared else (3 if clamps is not None else 1) if gated else 0
     native.kernel_check(lib.ms_gemm_tc_experts_bf16(_ptr(out), _ptr(a), _ptr(w), slots, n, k, e, mode, _ptr(tiles), _ptr(meta),
-                                                    _ptr(offsets), expert_max_tiles(slots, e, TC_TILE_ROWS), *map(float, clamps or NO_CLAMPS),
+                                                    _ptr(offsets), tile_rows, expert_max_tiles(slots, e, tile_rows), *map(float, clamps or NO_CLAMPS),
                                                     _ptr(device_status(a.device)), _stream(stream)),
                         lib=lib, errfn="ms_gemm_tc_last_error")
 

@@ -323,7 +323,7 @@ class RoutedExperts(Part):
         offsets = ctx.buffer("moe.offsets", (self.experts + 1,), i32, dev)
         # bfloat16: both products on the tcgen05 kernel where it has the activation, over the tokens' inputs gathered into sorted order
         tc = ops.experts.tc_experts_ok(dt, self.hidden, self.inter, self.activation) and x.stride(0) % 8 == 0
-        tile_rows = ops.experts.TC_TILE_ROWS if tc else ops.experts.TILE_ROWS
+        tile_rows = ops.experts.tc_tile_rows(slots, self.experts) if tc else ops.experts.TILE_ROWS
         tiles = ctx.buffer("moe.tiles", (ops.experts.expert_max_tiles(slots, self.experts, tile_rows), 2), i32, dev)
         meta = ctx.buffer("moe.meta", (2,), i32, dev)
         ops.experts.expert_plan(pos, perm, offsets, tiles, meta, idx, self.experts, stream=ctx.stream, tile_rows=tile_rows)
@@ -333,8 +333,8 @@ class RoutedExperts(Part):
             xs = ctx.buffer("moe.xs", (slots, self.hidden), dt, dev)
             ops.experts.expert_gather(xs, x, perm, meta, self.top, stream=ctx.stream)
             ops.experts.expert_products_tc(act, xs, self.w_gate_up, tiles, meta, offsets, self.gated, stream=ctx.stream,
-                                           relu_squared=not self.gated, clamps=self.clamps)
-            ops.experts.expert_products_tc(y, act, self.w_down, tiles, meta, offsets, False, stream=ctx.stream)
+                                           relu_squared=not self.gated, clamps=self.clamps, tile_rows=tile_rows)
+            ops.experts.expert_products_tc(y, act, self.w_down, tiles, meta, offsets, False, stream=ctx.stream, tile_rows=tile_rows)
         else:
             if self.gated:
                 ops.experts.expert_gate_up(act, x, self.w_gate_up, perm, self.top, tiles, meta, offsets, self.activation, stream=ctx.stream,

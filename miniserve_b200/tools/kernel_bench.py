@@ -201,7 +201,7 @@ def main(argv=None) -> int:
         t, e, top, inter, width = args.tokens, args.experts, args.top, args.n, args.k
         slots = t * top
         tc = args.gemm != "library"
-        tile_rows = xo.TC_TILE_ROWS if tc else xo.TILE_ROWS
+        tile_rows = xo.tc_tile_rows(slots, e) if tc else xo.TILE_ROWS
         parts = 1 if args.plain_experts else 2  # matrices ahead of the down projection
         work = dict(flops=2.0 * slots * (parts + 1) * inter * width)
         copies = max(2, int(L2_BYTES // (e * (parts + 1) * inter * width * 2)) + 1)
@@ -220,8 +220,9 @@ def main(argv=None) -> int:
         def calls(i, stream):
             if tc:
                 xo.expert_gather(xs, x, perm, meta, top, stream=stream)
-                xo.expert_products_tc(act, xs, wg[i], tiles, meta, offsets, not args.plain_experts, stream=stream, relu_squared=args.plain_experts)
-                xo.expert_products_tc(y, act, wd[i], tiles, meta, offsets, False, stream=stream)
+                xo.expert_products_tc(act, xs, wg[i], tiles, meta, offsets, not args.plain_experts, stream=stream, relu_squared=args.plain_experts,
+                                      tile_rows=tile_rows)
+                xo.expert_products_tc(y, act, wd[i], tiles, meta, offsets, False, stream=stream, tile_rows=tile_rows)
             else:
                 if args.plain_experts:
                     xo.expert_up(act, x, wg[i], perm, top, tiles, meta, offsets, "relu_squared", stream=stream)
