@@ -174,24 +174,111 @@ struct ChunkPlace {
   int num_rows;
 };
 
-// The decays of a block's 16 tokens for one channel (tokens from n on: 1). (The hardware's exponential: relative error about 1e-6 of an exponent.)
-__device__ __forceinline__ void block_decays(float (&d)[TC_BLK], const float* __restrict__ z, int ld_z, const float* __restrict__ w0, int t0, int n,
-                                             int blk, int ch, bool in) {
+// Two float32 in a register pair, one instruction for both.
+__device__ __forceinline__ uint64_t pack2(float a, float b) {
+  uint64_t v;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(a), "f"(b));
+  return v;
+}
+__device__ __forceinline__ float2 unpack2(uint64_t v) {
+  float2 f;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
+  return f;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t v;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(v) : "l"(a), "l"(b), "l"(c));
+  return v;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t v;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(v) : "l"(a), "l"(b));
+  return v;
+}
+__device__ __forceinline__ float sum2(uint64_t v) {
+  const float2 f = unpack2(v);
+  return f.x + f.y;
+}
+__device__ __forceinline__ uint64_t widen2(__nv_bfloat162 v) {
+  const float2 f = __bfloat1622float2(v);
+  return pack2(f.x, f.y);
+}
+// Two neighbours as two bfloat16 each.
+__device__ __forceinline__ void split2(uint64_t v, __nv_bfloat16* hi, __nv_bfloat16* lo) {
+  const float2 x = unpack2(v);
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x.x, x.y);
+  const float2 f = __bfloat1622float2(h);
+  *reinterpret_cast<__nv_bfloat162*>(hi) = h;
+  *reinterpret_cast<__nv_bfloat162*>(lo) = __floats2bfloat162_rn(x.x - f.x, x.y - f.y);
+}
+
+// A warp takes half a block (eight tokens) of 64 key channels at a time, a lane two neighbouring channels: their decays, and another operand
+// or two of the same shape. FULL: a whole chunk of heads as wide as the tile; otherwise tokens from n on have a decay of one and operands
+// of zero, and so have channels from dk on. (The hardware's exponential: relative error about 1e-6 of an exponent.)
+constexpr int TC_HALF = 8;
+template <bool FULL>
+__device__ __forceinline__ void half_decays(uint64_t (&d)[TC_HALF], const float* __restrict__ z, int ld_z, const float* __restrict__ w0, int row0, int n,
+                                            bool in) {
+  float2 v[TC_HALF];
 #pragma unroll
-  for (int i = 0; i < TC_BLK; ++i) {
-    const int tt = blk * TC_BLK + i;
-    d[i] = in && tt < n ? z[(size_t)(t0 + tt) * ld_z + ch] : 0.f;
+  for (int i = 0; i < TC_HALF; ++i)
+    v[i] = FULL || (in && row0 + i < n) ? *reinterpret_cast<const float2*>(z + (size_t)(row0 + i) * ld_z) : make_float2(0.f, 0.f);
+  const float2 w = FULL || in ? *reinterpret_cast<const float2*>(w0) : make_float2(0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < TC_HALF; ++i) {
+    const float a = __expf(-__expf(v[i].x + w.x)), b = __expf(-__expf(v[i].y + w.y));
+    d[i] = FULL || (in && row0 + i < n) ? pack2(a, b) : pack2(1.f, 1.f);
   }
-  const float w = in ? w0[ch] : 0.f;
+}
+template <bool FULL>
+__device__ __forceinline__ void half_rows(__nv_bfloat162 (&x)[TC_HALF], const __nv_bfloat16* __restrict__ src, int ld, int row0, int n, bool in) {
 #pragma unroll
-  for (int i = 0; i < TC_BLK; ++i) d[i] = in && blk * TC_BLK + i < n ? __expf(-__expf(d[i] + w)) : 1.f;
+  for (int i = 0; i < TC_HALF; ++i)
+    x[i] = FULL || (in && row0 + i < n) ? *reinterpret_cast<const __nv_bfloat162*>(src + (size_t)(row0 + i) * ld) : __floats2bfloat162_rn(0.f, 0.f);
 }
 
 template <int DKT>
 struct TmStatesSmem {
   __nv_bfloat16 v[CS_TOK][TC_DV + 8], khi[CS_TOK][DKT + 8], klo[CS_TOK][DKT + 8];
-  float whole[TC_BLOCKS][DKT];
+  float half[2 * TC_BLOCKS][DKT];  // the products of half blocks
 };
+
+// What the chunk's keys are multiplied by on their way into the state; this warp's share.
+template <int DKT, bool FULL>
+__device__ __forceinline__ void state_keys(TmStatesSmem<DKT>& sm, float* __restrict__ passed, const __nv_bfloat16* __restrict__ k, int ld_k,
+                                           const float* __restrict__ z, int ld_z, const float* __restrict__ w0, int n, int dk) {
+  constexpr int TRIPS = DKT / 64;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, row0 = warp * TC_HALF;
+  uint64_t x[TRIPS][TC_HALF];
+#pragma unroll
+  for (int tr = 0; tr < TRIPS; ++tr) {
+    const int c = tr * 64 + lane * 2;
+    const bool in = c < dk;
+    __nv_bfloat162 kk[TC_HALF];
+    half_rows<FULL>(kk, k + c, ld_k, row0, n, in);
+    uint64_t d[TC_HALF];
+    half_decays<FULL>(d, z + c, ld_z, w0 + c, row0, n, in);
+    uint64_t suf = pack2(1.f, 1.f);
+#pragma unroll
+    for (int i = TC_HALF - 1; i >= 0; --i) {
+      x[tr][i] = mul2(widen2(kk[i]), suf);
+      suf = mul2(suf, d[i]);
+    }
+    *reinterpret_cast<uint64_t*>(&sm.half[warp][c]) = suf;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int tr = 0; tr < TRIPS; ++tr) {
+    const int c = tr * 64 + lane * 2;
+    uint64_t behind = pack2(1.f, 1.f);
+#pragma unroll
+    for (int q = 1; q < 2 * TC_BLOCKS; ++q)
+      if (q > warp) behind = mul2(behind, *reinterpret_cast<const uint64_t*>(&sm.half[q][c]));
+#pragma unroll
+    for (int i = 0; i < TC_HALF; ++i) split2(mul2(x[tr][i], behind), &sm.khi[row0 + i][c], &sm.klo[row0 + i][c]);
+    if (passed && warp == 0 && c < dk) *reinterpret_cast<uint64_t*>(passed + c) = mul2(behind, *reinterpret_cast<const uint64_t*>(&sm.half[0][c]));
+  }
+}
 
 // added [chunks, H, dv, dk] float32, passed [chunks, H, dk]: the product of the chunk's decays. grid (chunks, H, dv tiles).
 template <int DKT>
@@ -213,35 +300,12 @@ tm_states_kernel(float* __restrict__ added, float* __restrict__ passed, const __
     cs_cp16(&sm.v[tt][c], in ? (const void*)(v + (size_t)(t0 + tt) * ld_v + (size_t)h * dv + v0 + c) : (const void*)v, in);
   }
   cs_commit();
-  constexpr int TRIPS = DKT / 64;
-  const int blk = tid >> 6;
-  float suf[TRIPS][TC_BLK];
-#pragma unroll
-  for (int tr = 0; tr < TRIPS; ++tr) {
-    const int c = tr * 64 + (tid & 63);
-    float d[TC_BLK];
-    block_decays(d, z, ld_z, w0, t0, n, blk, h * dk + c, c < dk);
-    suf[tr][TC_BLK - 1] = 1.f;
-#pragma unroll
-    for (int i = TC_BLK - 2; i >= 0; --i) suf[tr][i] = suf[tr][i + 1] * d[i + 1];
-    sm.whole[blk][c] = suf[tr][0] * d[0];
-  }
-  __syncthreads();
-#pragma unroll
-  for (int tr = 0; tr < TRIPS; ++tr) {
-    const int c = tr * 64 + (tid & 63);
-    float behind = 1.f;
-#pragma unroll
-    for (int b = 1; b < TC_BLOCKS; ++b)
-      if (b > blk) behind *= sm.whole[b][c];
-#pragma unroll
-    for (int i = 0; i < TC_BLK; ++i) {
-      const int tt = blk * TC_BLK + i;
-      float x = 0.f;
-      if (tt < n && c < dk) x = __bfloat162float(k[(size_t)(t0 + tt) * ld_k + (size_t)h * dk + c]) * (suf[tr][i] * behind);
-      cs_split(x, sm.khi[tt][c], sm.klo[tt][c]);
-    }
-    if (blk == 0 && c < dk && blockIdx.z == 0) passed[((size_t)chunk * H + h) * dk + c] = sm.whole[0][c] * behind;
+  {
+    float* all = blockIdx.z == 0 ? passed + ((size_t)chunk * H + h) * dk : nullptr;
+    const __nv_bfloat16* kh = k + (size_t)t0 * ld_k + (size_t)h * dk;
+    const float* zh = z + (size_t)t0 * ld_z + (size_t)h * dk;
+    if (n == CS_TOK && dk == DKT) state_keys<DKT, true>(sm, all, kh, ld_k, zh, ld_z, w0 + (size_t)h * dk, n, dk);
+    else state_keys<DKT, false>(sm, all, kh, ld_k, zh, ld_z, w0 + (size_t)h * dk, n, dk);
   }
   cs_wait<0>();
   __syncthreads();
@@ -314,18 +378,6 @@ tm_carry_kernel(float* __restrict__ state, __nv_bfloat16* __restrict__ before_hi
 }
 
 // ---------------------------------------------------------------- chunks: the outputs
-// Two neighbours at once: the sum of their two bfloat16, and back.
-__device__ __forceinline__ float2 joined2(const __nv_bfloat16* hi, const __nv_bfloat16* lo) {
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(hi)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(lo));
-  return make_float2(a.x + b.x, a.y + b.y);
-}
-__device__ __forceinline__ void split2(float2 x, __nv_bfloat16* hi, __nv_bfloat16* lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x.x, x.y);
-  const float2 f = __bfloat1622float2(h);
-  *reinterpret_cast<__nv_bfloat162*>(hi) = h;
-  *reinterpret_cast<__nv_bfloat162*>(lo) = __floats2bfloat162_rn(x.x - f.x, x.y - f.y);
-}
-
 template <int DKT>
 struct TmOutputsSmem {
   static constexpr int LDK = DKT + 8, LDP = CS_TOK + 8;
@@ -337,7 +389,7 @@ struct TmOutputsSmem {
       __nv_bfloat16 shi[TC_DV][LDK], slo[TC_DV][LDK];  // the state before the chunk, once the pairs inside the blocks are done
     };
   };
-  float whole[TC_BLOCKS][DKT];                      // a block's product
+  float half[2 * TC_BLOCKS][DKT];                   // the products of half blocks
   float dsum[2][TC_BLOCKS][TC_BLK][TC_BLK + 1];     // [channel half][block][j][i]: sums of the pairs inside a block
   float squares[2][CS_TOK];                         // [column half][token]
   __nv_bfloat16 k[CS_TOK][LDK];
@@ -352,6 +404,77 @@ struct TmOutputsSmem {
   };
   __nv_bfloat16 v[CS_TOK][TC_DV + 8];
 };
+
+// A warp's half block: r and k with the products of decays that they meet in; pr keeps r times the product from its block's first token on.
+template <int DKT, bool FULL>
+__device__ __forceinline__ void output_operands(TmOutputsSmem<DKT>& sm, uint64_t (&pr)[DKT / 64][TC_HALF], const __nv_bfloat16* __restrict__ r, int ld_r,
+                                                const __nv_bfloat16* __restrict__ k, int ld_k, const float* __restrict__ z, int ld_z,
+                                                const float* __restrict__ w0, int n, int dk) {
+  constexpr int TRIPS = DKT / 64;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, blk = warp >> 1, upper = warp & 1, row0 = warp * TC_HALF;
+  uint64_t kx[TRIPS][TC_HALF];
+#pragma unroll
+  for (int tr = 0; tr < TRIPS; ++tr) {
+    const int c = tr * 64 + lane * 2;
+    const bool in = c < dk;
+    __nv_bfloat162 rr[TC_HALF], kk[TC_HALF];
+    half_rows<FULL>(rr, r + c, ld_r, row0, n, in);
+    half_rows<FULL>(kk, k + c, ld_k, row0, n, in);
+    uint64_t d[TC_HALF];
+    half_decays<FULL>(d, z + c, ld_z, w0 + c, row0, n, in);
+    uint64_t run = pack2(1.f, 1.f), suf = pack2(1.f, 1.f);
+#pragma unroll
+    for (int i = 0; i < TC_HALF; ++i) {
+      const uint64_t x = widen2(rr[i]);
+      *reinterpret_cast<uint64_t*>(&sm.r[row0 + i][c]) = x;
+      *reinterpret_cast<uint64_t*>(&sm.d[row0 + i][c]) = d[i];
+      *reinterpret_cast<__nv_bfloat162*>(&sm.k[row0 + i][c]) = kk[i];
+      pr[tr][i] = mul2(run, x);  // times the product up to the token before
+      run = mul2(run, d[i]);
+    }
+#pragma unroll
+    for (int i = TC_HALF - 1; i >= 0; --i) {
+      kx[tr][i] = mul2(widen2(kk[i]), suf);
+      suf = mul2(suf, d[i]);
+    }
+    *reinterpret_cast<uint64_t*>(&sm.half[warp][c]) = run;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int tr = 0; tr < TRIPS; ++tr) {
+    const int c = tr * 64 + lane * 2;
+    const auto half = [&](int q) { return *reinterpret_cast<const uint64_t*>(&sm.half[q][c]); };
+    if (upper) {
+      const uint64_t a = half(warp - 1);
+#pragma unroll
+      for (int i = 0; i < TC_HALF; ++i) pr[tr][i] = mul2(pr[tr][i], a);
+    } else {
+      const uint64_t b = half(warp + 1);
+#pragma unroll
+      for (int i = 0; i < TC_HALF; ++i) kx[tr][i] = mul2(kx[tr][i], b);
+    }
+#pragma unroll
+    for (int i = 0; i < TC_HALF; ++i) split2(pr[tr][i], &sm.rhi[row0 + i][c], &sm.rlo[row0 + i][c]);
+    if (blk == TC_BLOCKS - 1) continue;
+    // k for the next block, and times the products of the blocks between for those behind it
+    const int base = (blk == 0 ? 0 : blk == 1 ? 32 : 80) + upper * TC_HALF;
+#pragma unroll
+    for (int i = 0; i < TC_HALF; ++i) split2(kx[tr][i], &sm.kb.hi[base + i][c], &sm.kb.lo[base + i][c]);
+    if (blk == 2) continue;
+    const uint64_t w2 = mul2(half(4), half(5));
+    if (blk == 0) {
+      const uint64_t w1 = mul2(half(2), half(3));
+#pragma unroll
+      for (int i = 0; i < TC_HALF; ++i) {
+        kx[tr][i] = mul2(kx[tr][i], w1);
+        split2(kx[tr][i], &sm.kb.hi[16 + upper * TC_HALF + i][c], &sm.kb.lo[16 + upper * TC_HALF + i][c]);
+      }
+    }
+    const int last = (blk == 0 ? 48 : 64) + upper * TC_HALF;
+#pragma unroll
+    for (int i = 0; i < TC_HALF; ++i) split2(mul2(kx[tr][i], w2), &sm.kb.hi[last + i][c], &sm.kb.lo[last + i][c]);
+  }
+}
 
 // What follows the recurrence: out [T, H * dv] bfloat16 = o / sqrt(mean o^2 + eps) * norm_w * silu(gate) (heads of one value tile).
 struct HeadGate {
@@ -386,65 +509,13 @@ tm_outputs_kernel(float* __restrict__ o, const HeadGate hg, const __nv_bfloat16*
   }
   cs_commit();
 
-  // one thread per (block, channel): decays, and the products within the block
   constexpr int TRIPS = DKT / 64;
-  const int blk = tid >> 6;
-  float pre[TRIPS][TC_BLK];
-#pragma unroll
-  for (int tr = 0; tr < TRIPS; ++tr) {
-    const int c = tr * 64 + (tid & 63);
-    const size_t hc = (size_t)h * dk + c;
-    __nv_bfloat16 rk[2][TC_BLK];
-#pragma unroll
-    for (int i = 0; i < TC_BLK; ++i) {
-      const int tt = blk * TC_BLK + i;
-      const bool in = tt < n && c < dk;
-      rk[0][i] = in ? r[(size_t)(t0 + tt) * ld_r + hc] : __float2bfloat16_rn(0.f);
-      rk[1][i] = in ? k[(size_t)(t0 + tt) * ld_k + hc] : __float2bfloat16_rn(0.f);
-    }
-    float d[TC_BLK];
-    block_decays(d, z, ld_z, w0, t0, n, blk, (int)hc, c < dk);
-    float run = 1.f;
-#pragma unroll
-    for (int i = 0; i < TC_BLK; ++i) {
-      const int tt = blk * TC_BLK + i;
-      const float x = __bfloat162float(rk[0][i]);
-      sm.r[tt][c] = x;
-      pre[tr][i] = run * x;  // times the product up to the token before
-      run *= d[i];
-      sm.d[tt][c] = d[i];
-      sm.k[tt][c] = rk[1][i];
-      cs_split(pre[tr][i], sm.rhi[tt][c], sm.rlo[tt][c]);
-    }
-    sm.whole[blk][c] = run;
-    // k times the product behind it to its block's end, for the next block; the products of whole blocks follow below
-    if (blk < TC_BLOCKS - 1) {
-      const int base = blk == 0 ? 0 : blk == 1 ? 32 : 80;
-      float suf = 1.f;
-#pragma unroll
-      for (int i = TC_BLK - 1; i >= 0; --i) {
-        d[i] *= suf;  // d[i] becomes the product from i on
-        const float x = __bfloat162float(rk[1][i]) * suf;
-        suf = d[i];
-        cs_split(x, sm.kb.hi[base + i][c], sm.kb.lo[base + i][c]);
-      }
-    }
-  }
-  __syncthreads();
-  // block 0 for block 2 and 3, block 1 for block 3: times the products of the blocks between
-#pragma unroll
-  for (int tr = 0; tr < TRIPS; ++tr) {
-    const int c = tr * 64 + lane * 2;  // two channels a thread, two of the blocks' tokens
-    const float2 w1 = *reinterpret_cast<const float2*>(&sm.whole[1][c]), w2 = *reinterpret_cast<const float2*>(&sm.whole[2][c]);
-#pragma unroll
-    for (int q = 0; q < 2; ++q) {
-      const int i = warp * 2 + q;
-      const float2 x0 = joined2(&sm.kb.hi[i][c], &sm.kb.lo[i][c]), x1 = joined2(&sm.kb.hi[32 + i][c], &sm.kb.lo[32 + i][c]);
-      const float2 y0 = make_float2(x0.x * w1.x, x0.y * w1.y);
-      split2(y0, &sm.kb.hi[16 + i][c], &sm.kb.lo[16 + i][c]);
-      split2(make_float2(y0.x * w2.x, y0.y * w2.y), &sm.kb.hi[48 + i][c], &sm.kb.lo[48 + i][c]);
-      split2(make_float2(x1.x * w2.x, x1.y * w2.y), &sm.kb.hi[64 + i][c], &sm.kb.lo[64 + i][c]);
-    }
+  uint64_t pr[TRIPS][TC_HALF];
+  {
+    const __nv_bfloat16 *rh = r + (size_t)t0 * ld_r + (size_t)h * dk, *kh = k + (size_t)t0 * ld_k + (size_t)h * dk;
+    const float* zh = z + (size_t)t0 * ld_z + (size_t)h * dk;
+    if (n == CS_TOK && dk == DKT) output_operands<DKT, true>(sm, pr, rh, ld_r, kh, ld_k, zh, ld_z, w0 + (size_t)h * dk, n, dk);
+    else output_operands<DKT, false>(sm, pr, rh, ld_r, kh, ld_k, zh, ld_z, w0 + (size_t)h * dk, n, dk);
   }
   const int bi = warp >> 1, half_w = warp & 1, wm = bi * TC_BLK;
   // pairs inside a block: a lane takes j and 15 - j (15 pairs together) over DKT / 8 channels; two warps make up a block's channels
@@ -452,33 +523,46 @@ tm_outputs_kernel(float* __restrict__ o, const HeadGate hg, const __nv_bfloat16*
     const int j = lane & 7;
     constexpr int QC = DKT / 8;
     const int cbeg = (half_w * 4 + (lane >> 3)) * QC;
-    float acc[TC_BLK - 1] = {}, own[2] = {0.f, 0.f};
+    uint64_t acc2[TC_BLK - 1] = {}, own2[2] = {};  // pairs of sums: even and odd channels
+    constexpr int STRIDE = DKT + 4;
+    const float* r0 = &sm.r[wm][0];
+    const float* d0 = &sm.d[wm][0];
 #pragma unroll 1
     for (int c = cbeg; c < cbeg + QC; c += 4) {
-      float x[4], y[4];
+      uint64_t x[2], y[2];
+      {
+        const float4 u4 = c < dk ? *reinterpret_cast<const float4*>(u + (size_t)h * dk + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        const uint64_t u01 = pack2(u4.x, u4.y), u23 = pack2(u4.z, u4.w);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        x[e] = __bfloat162float(sm.k[wm + j][c + e]);
-        y[e] = __bfloat162float(sm.k[wm + 15 - j][c + e]);
-        const float b = c + e < dk ? u[(size_t)h * dk + c + e] : 0.f;
-        own[0] = fmaf(sm.r[wm + j][c + e] * b, x[e], own[0]);
-        own[1] = fmaf(sm.r[wm + 15 - j][c + e] * b, y[e], own[1]);
+        for (int q = 0; q < 2; ++q) {
+          const int jj = q == 0 ? j : 15 - j;
+          const __nv_bfloat162* kp = reinterpret_cast<const __nv_bfloat162*>(&sm.k[wm + jj][c]);
+          uint64_t(&w)[2] = q == 0 ? x : y;
+          w[0] = widen2(kp[0]);
+          w[1] = widen2(kp[1]);
+          const ulonglong2 rr = *reinterpret_cast<const ulonglong2*>(r0 + jj * STRIDE + c);
+          own2[q] = fma2(mul2(rr.x, u01), w[0], fma2(mul2(rr.y, u23), w[1], own2[q]));
+        }
       }
 #pragma unroll
       for (int s = 0; s < TC_BLK - 1; ++s) {
-        if (s == 15 - j) {
-#pragma unroll
-          for (int e = 0; e < 4; ++e) x[e] = y[e];
+        // (15 - j is 8 at least: the first eight steps are j's for every lane)
+        if (s >= 8 && s == 15 - j) {
+          x[0] = y[0];
+          x[1] = y[1];
         }
-        const int i = wm + s + 1 + (s < 15 - j ? j : 0);
-        const float4 r4 = *reinterpret_cast<const float4*>(&sm.r[i][c]), d4 = *reinterpret_cast<const float4*>(&sm.d[i][c]);
-        acc[s] = fmaf(r4.x, x[0], fmaf(r4.y, x[1], fmaf(r4.z, x[2], fmaf(r4.w, x[3], acc[s]))));
-        x[0] *= d4.x;
-        x[1] *= d4.y;
-        x[2] *= d4.z;
-        x[3] *= d4.w;
+        const int at = (s < 8 || s < 15 - j ? j * STRIDE : 0) + (s + 1) * STRIDE + c;
+        const ulonglong2 rr = *reinterpret_cast<const ulonglong2*>(r0 + at), dd = *reinterpret_cast<const ulonglong2*>(d0 + at);
+        acc2[s] = fma2(rr.x, x[0], fma2(rr.y, x[1], acc2[s]));
+        x[0] = mul2(x[0], dd.x);
+        x[1] = mul2(x[1], dd.y);
       }
     }
+    float acc[TC_BLK - 1], own[2];
+#pragma unroll
+    for (int s = 0; s < TC_BLK - 1; ++s) acc[s] = sum2(acc2[s]);
+    own[0] = sum2(own2[0]);
+    own[1] = sum2(own2[1]);
 #pragma unroll
     for (int s = 0; s < TC_BLK - 1; ++s) {
       acc[s] += __shfl_xor_sync(0xffffffffu, acc[s], 8);
@@ -557,16 +641,16 @@ tm_outputs_kernel(float* __restrict__ o, const HeadGate hg, const __nv_bfloat16*
     const float x = j <= i ? sm.dsum[0][b][j][i] + sm.dsum[1][b][j][i] : 0.f;
     cs_split(x, sm.p.hi[b * TC_BLK + i][b * TC_BLK + j], sm.p.lo[b * TC_BLK + i][b * TC_BLK + j]);
   }
-  if (has_state && blk > 0) {  // r times the product from the chunk's first token on (block 0 has it already)
+  if (has_state && bi > 0) {  // r times the product from the chunk's first token on (block 0 has it already)
 #pragma unroll
     for (int tr = 0; tr < TRIPS; ++tr) {
-      const int c = tr * 64 + (tid & 63);
-      float ahead = 1.f;
+      const int c = tr * 64 + lane * 2;
+      uint64_t ahead = pack2(1.f, 1.f);
 #pragma unroll
-      for (int b = 0; b < TC_BLOCKS - 1; ++b)
-        if (b < blk) ahead *= sm.whole[b][c];
+      for (int q = 0; q < 2 * (TC_BLOCKS - 1); ++q)
+        if (q < 2 * bi) ahead = mul2(ahead, *reinterpret_cast<const uint64_t*>(&sm.half[q][c]));
 #pragma unroll
-      for (int i = 0; i < TC_BLK; ++i) cs_split(pre[tr][i] * ahead, sm.rhi[blk * TC_BLK + i][c], sm.rlo[blk * TC_BLK + i][c]);
+      for (int i = 0; i < TC_HALF; ++i) split2(mul2(pr[tr][i], ahead), &sm.rhi[warp * TC_HALF + i][c], &sm.rlo[warp * TC_HALF + i][c]);
     }
   }
   cs_wait<0>();
@@ -727,9 +811,10 @@ MS_EXPORT int ms_time_chunks(float* o, void* out, const void* gate, int ld_gate,
                                                               (uintptr_t)out % 4 == 0 && (uintptr_t)norm_w % 8 == 0)),
                "time_chunks: either o, or for heads of up to %d values the gated output", TC_DV);
   const HeadGate hg{(__nv_bfloat16*)out, (const __nv_bfloat16*)gate, ld_gate, norm_w, eps};
+  MS_CHECK_ARG(ld_z % 2 == 0 && (uintptr_t)z % 8 == 0 && (uintptr_t)w0 % 8 == 0, "time_chunks: the decays' logits are read two at a time");
   MS_CHECK_ARG(ld_r % 8 == 0 && ld_k % 8 == 0 && ld_v % 8 == 0 && (uintptr_t)r % 16 == 0 && (uintptr_t)k % 16 == 0 && (uintptr_t)v % 16 == 0 &&
                    (uintptr_t)o % 8 == 0 && (uintptr_t)state % 16 == 0 && (uintptr_t)added % 16 == 0 && (uintptr_t)before_hi % 16 == 0 &&
-                   (uintptr_t)before_lo % 16 == 0 && (uintptr_t)passed % 16 == 0,
+                   (uintptr_t)before_lo % 16 == 0 && (uintptr_t)passed % 16 == 0 && (uintptr_t)u % 16 == 0,
                "time_chunks: operands must be aligned");
   const ChunkPlace pl{reinterpret_cast<const int2*>(tab), row_first, cu_q, q_start, state_slot, num_rows};
   const __nv_bfloat16 *rb = (const __nv_bfloat16*)r, *kb = (const __nv_bfloat16*)k, *vb = (const __nv_bfloat16*)v;
