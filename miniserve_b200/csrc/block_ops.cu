@@ -195,12 +195,22 @@ __global__ void token_mixes_kernel(T* __restrict__ out, const T* __restrict__ h,
 }
 
 // The same for bfloat16 rows that are a multiple of 8 wide and start on 16 bytes: eight channels per thread, RUN consecutive tokens per CTA,
-// which read the mixes' factors once.
-template <int RUN>
+// which read the mixes' factors once. RUN 1: the first factors are read before the wait for the input (they are weights).
+template <int RUN, int MIXES>
 __global__ void token_mixes_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ h, __nv_bfloat16* __restrict__ state,
-                                          const float* __restrict__ mix, int mixes, const int* __restrict__ row_of_token,
-                                          const int* __restrict__ cu_q, const int* __restrict__ q_start, const int* __restrict__ state_slot,
-                                          int tokens, int width) {
+                                          const float* __restrict__ mix, const int* __restrict__ row_of_token, const int* __restrict__ cu_q,
+                                          const int* __restrict__ q_start, const int* __restrict__ state_slot, int tokens, int width) {
+  constexpr bool EARLY = RUN == 1;
+  float early[EARLY ? MIXES : 1][8];
+  auto factors = [&](float (&f)[8], int m, int c) {
+    const float4 a = *reinterpret_cast<const float4*>(mix + (size_t)m * width + c), b = *reinterpret_cast<const float4*>(mix + (size_t)m * width + c + 4);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+  };
+  const int c0 = threadIdx.x * 8;
+  if (EARLY && c0 < width) {
+#pragma unroll
+    for (int m = 0; m < MIXES; ++m) factors(early[EARLY ? m : 0], m, c0);
+  }
   pdl_prologue();
   const int t0 = blockIdx.x * RUN;
   const __nv_bfloat16* prev[RUN];
@@ -217,7 +227,7 @@ __global__ void token_mixes_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const
     newest[q] = h + (size_t)(cu_q[row + 1] - 1) * width;
   }
   const size_t plane = (size_t)tokens * width;
-  for (int c = threadIdx.x * 8; c < width; c += blockDim.x * 8) {
+  for (int c = c0; c < width; c += blockDim.x * 8) {
     float x[RUN][8], p[RUN][8];
 #pragma unroll
     for (int q = 0; q < RUN; ++q) {
@@ -231,10 +241,15 @@ __global__ void token_mixes_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const
     for (int q = 0; q < RUN; ++q)
 #pragma unroll
       for (int e = 0; e < 8; ++e) p[q][e] -= x[q][e];
-    for (int m = 0; m < mixes; ++m) {
-      const float* mm = mix + (size_t)m * width + c;
-      const float4 ma = *reinterpret_cast<const float4*>(mm), mb = *reinterpret_cast<const float4*>(mm + 4);
-      const float mv[8] = {ma.x, ma.y, ma.z, ma.w, mb.x, mb.y, mb.z, mb.w};
+#pragma unroll EARLY ? MIXES : 1
+    for (int m = 0; m < MIXES; ++m) {
+      float mv[8];
+      if (EARLY && c == c0) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) mv[e] = early[EARLY ? m : 0][e];
+      } else {
+        factors(mv, m, c);
+      }
 #pragma unroll
       for (int q = 0; q < RUN; ++q) {
         if (t0 + q >= tokens) break;
@@ -951,15 +966,15 @@ MS_EXPORT int ms_token_mixes(void* out, const void* h, void* state, const float*
   if (tokens == 0) return 0;
   MS_CHECK_ARG(width > 0 && mixes > 0 && out != h, "token_mixes: width=%d, %d mixes, and the output may not be the input", width, mixes);
   const int threads = width >= 1024 ? 256 : 128;
-  if (dtype == MS_BF16 && width % 8 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)state % 16 == 0 &&
+  if (dtype == MS_BF16 && mixes == 5 && width % 8 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)state % 16 == 0 &&
       (uintptr_t)mix % 16 == 0) {
     const int th = width >= 2048 ? 256 : 128;
+    __nv_bfloat16 *o = (__nv_bfloat16*)out, *st = (__nv_bfloat16*)state;
+    const __nv_bfloat16* hb = (const __nv_bfloat16*)h;
     if (tokens >= 1024)
-      MS_LAUNCH(token_mixes_bf16x8_kernel<4>, (tokens + 3) / 4, th, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)h, (__nv_bfloat16*)state, mix,
-                mixes, row_of_token, cu_q, q_start, state_slot, tokens, width);
+      MS_LAUNCH((token_mixes_bf16x8_kernel<4, 5>), (tokens + 3) / 4, th, 0, stream, o, hb, st, mix, row_of_token, cu_q, q_start, state_slot, tokens, width);
     else
-      MS_LAUNCH(token_mixes_bf16x8_kernel<1>, tokens, th, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)h, (__nv_bfloat16*)state, mix, mixes,
-                row_of_token, cu_q, q_start, state_slot, tokens, width);
+      MS_LAUNCH((token_mixes_bf16x8_kernel<1, 5>), tokens, th, 0, stream, o, hb, st, mix, row_of_token, cu_q, q_start, state_slot, tokens, width);
     return 0;
   }
   if (dtype == MS_F32)

@@ -45,6 +45,12 @@ struct Rows {
   int ld;
 };
 
+__device__ __forceinline__ void step_load8(const __nv_bfloat16* p, float (&f)[8]) { bf16x8_to_float(*reinterpret_cast<const uint4*>(p), f); }
+__device__ __forceinline__ void step_load8(const float* p, float (&f)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+
 // grid (H, rows). LPC lanes take a column's key channels, four at a time; a warp 32 / LPC columns at once, TS_COLS of them in turn with
 // their loads in flight together; the first ones are asked for before the decays are worked out. out [T, H * dv] = o / sqrt(mean o^2 + eps) *
 // norm_w * silu(gate).
@@ -53,7 +59,7 @@ __global__ void __launch_bounds__(TS_THREADS)
 time_step_kernel(T* __restrict__ out, float* __restrict__ state, Rows<T> r, Rows<T> k, Rows<T> v, Rows<T> gate, Rows<T> low,
                  const T* __restrict__ w2, int rank, const float* __restrict__ w0, const float* __restrict__ u,
                  const float* __restrict__ norm_w, float eps, const int* __restrict__ cu_q, const int* __restrict__ q_start,
-                 const int* __restrict__ state_slot, int H, int dk, int dv) {
+                 const int* __restrict__ state_slot, int H, int dk, int dv, int vec) {
   extern __shared__ __align__(16) float ts_smem[];
   __shared__ float red[32];
   float* rs = ts_smem;       // [dk]
@@ -61,7 +67,6 @@ time_step_kernel(T* __restrict__ out, float* __restrict__ state, Rows<T> r, Rows
   float* ds = ks + dk;       // [dk]
   float* uk = ds + dk;       // [dk] bonus times key
   float* os = uk + dk;       // [dv]
-  float* ls = os + dv;       // [rank]
   const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   {  // weights: asked for before the wait
     const char* w = reinterpret_cast<const char*>(w2 + (size_t)h * dk * rank);
@@ -95,7 +100,6 @@ time_step_kernel(T* __restrict__ out, float* __restrict__ state, Rows<T> r, Rows
     gate0 = Elem<T>::load(gate.p + (size_t)t * gate.ld + (size_t)h * dv + tid);
     nw0 = norm_w[(size_t)h * dv + tid];
   }
-  for (int c = tid; c < rank; c += TS_THREADS) ls[c] = Elem<T>::load(low.p + (size_t)t * low.ld + c);
   for (int c = tid; c < dk; c += TS_THREADS) {
     const size_t at = (size_t)h * dk + c;
     const float kk = Elem<T>::load(k.p + (size_t)t * k.ld + at);
@@ -103,7 +107,6 @@ time_step_kernel(T* __restrict__ out, float* __restrict__ state, Rows<T> r, Rows
     ks[c] = kk;
     uk[c] = u[at] * kk;
   }
-  __syncthreads();
   // z of the head's channels: eight lanes a channel
   {
     const int zl = tid & 7;
@@ -111,9 +114,18 @@ time_step_kernel(T* __restrict__ out, float* __restrict__ state, Rows<T> r, Rows
       const int c = c0 + (tid >> 3);
       float acc = 0.f;
       if (c < dk) {
-        const T* w = w2 + ((size_t)h * dk + c) * rank;
-#pragma unroll 8
-        for (int i = zl; i < rank; i += 8) acc = fmaf(ls[i], Elem<T>::load(w + i), acc);
+        const T *w = w2 + ((size_t)h * dk + c) * rank, *lo = low.p + (size_t)t * low.ld;
+        if (vec) {  // rows of whole eights that start on 16 bytes
+          for (int i = zl * 8; i < rank; i += 64) {
+            float a[8], b[8];
+            step_load8(lo + i, a);
+            step_load8(w + i, b);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) acc = fmaf(a[e], b[e], acc);
+          }
+        } else {
+          for (int i = zl; i < rank; i += 8) acc = fmaf(Elem<T>::load(lo + i), Elem<T>::load(w + i), acc);
+        }
       }
 #pragma unroll
       for (int o = 4; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
@@ -774,13 +786,15 @@ MS_EXPORT int ms_time_step(void* out, float* state, const void* r, const void* k
                            const int* cu_q, const int* q_start, const int* state_slot, int num_rows, int H, int dk, int dv, int dtype,
                            cudaStream_t stream) {
   if (num_rows == 0) return 0;
-  const size_t smem = ((size_t)4 * dk + dv + rank) * sizeof(float);
+  const size_t smem = ((size_t)4 * dk + dv) * sizeof(float);
+  const int per16 = 16 / (dtype == MS_F32 ? 4 : 2);
+  const int vec = rank % 8 == 0 && ld_low % per16 == 0 && (uintptr_t)low % 16 == 0 && (uintptr_t)w2 % 16 == 0;
   MS_CHECK_ARG(H > 0 && dk > 0 && dk % 4 == 0 && dv > 0 && rank > 0 && (uintptr_t)state % 16 == 0 && num_rows <= 65535 && smem <= 48 * 1024,
                "time_step: %d rows, heads of %d x %d, rank %d", num_rows, dk, dv, rank);
 #define MS_STEP(T, LPC)                                                                                                                        \
   MS_LAUNCH((time_step_kernel<T, LPC>), dim3(H, num_rows), TS_THREADS, smem, stream, (T*)out, state, Rows<T>{(const T*)r, ld},                \
             Rows<T>{(const T*)k, ld}, Rows<T>{(const T*)v, ld}, Rows<T>{(const T*)gate, ld}, Rows<T>{(const T*)low, ld_low}, (const T*)w2, rank, w0, u, \
-            norm_w, eps, cu_q, q_start, state_slot, H, dk, dv)
+            norm_w, eps, cu_q, q_start, state_slot, H, dk, dv, vec)
   if (dtype == MS_F32) {
     if (dk > 64) MS_STEP(float, 32);
     else if (dk > 32) MS_STEP(float, 16);

@@ -672,7 +672,7 @@ def channel_decay(out, z, w0, stream=None) -> None:
 
 def time_step_ok(dk: int, dv: int, rank: int) -> bool:
     """Whether ``time_step`` takes these sizes."""
-    return dk % 4 == 0 and (4 * dk + dv + rank) * 4 <= 48 * 1024
+    return dk % 4 == 0 and (4 * dk + dv) * 4 <= 48 * 1024 and rank > 0
 
 
 def time_step(out, state, r, k, v, gate, low, w2, w0, bonus, norm_w, eps: float, ctx, heads: int) -> None:

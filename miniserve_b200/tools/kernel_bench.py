@@ -126,7 +126,8 @@ def main(argv=None) -> int:
     ap.add_argument("--op", choices=["channel_gate", "head_gate", "relu_squared", "gelu_tanh", "latent_prepare", "qkv_prepare",
                                      "layernorm", "layernorm_pair", "token_shift", "clamped_glu", "sum_bias", "act_mul", "axpby", "normed_add",
                                      "embed_gather", "embed_sum", "mlstm_gates", "mlstm_output", "gated_group_norm", "conv_bias", "conv_silu",
-                                     "rglru_gates", "rglru_scan", "time_chunks", "time_walk", "time_step", "token_mixes", "stream_norm", "expert_route",
+                                     "rglru_gates", "rglru_scan", "time_chunks", "time_walk", "time_step", "time_products", "token_mixes", "stream_norm",
+                                     "expert_route",
                                      "expert_combine"],
                     default="channel_gate", help="pointwise: which kernel (--tokens rows; --heads x --head-dim, or --n, columns)")
     ap.add_argument("--head-decay", action="store_true", help="decay_scan: one decay per head, worked out beforehand (float32), a column of ones")
@@ -409,14 +410,20 @@ def main(argv=None) -> int:
         w2, mu, before = (torch.randn(c, rank, device=dev) * 0.1).bfloat16(), torch.rand(5, n, **f32), torch.zeros(rows, n, **bf)
         w0, bonus, norm_w, wn = torch.randn(c, **f32) - 2, torch.randn(c, **f32), torch.ones(c, **f32), torch.ones(n, **f32)
         mix, link = torch.eye(st, **f32), torch.ones(st, **f32)
+        if args.op == "time_products":
+            copies = max(2, int(L2_BYTES // ((4 * c + rank) * n * 2)) + 1)
+            sets = [SimpleNamespace(w=torch.randn(4 * c + rank, n, **bf), mixes=sets[0].mixes, proj=sets[0].proj) for _ in range(copies)]
         state_bytes = 2 * rows * c * dk * 4
         byts = {"time_chunks": t * c * (2 * 5 + 4) + state_bytes, "time_walk": t * c * (2 * 3 + 4 + 4) + state_bytes,
-                "time_step": t * c * 2 * 5 + state_bytes + c * rank * 2, "token_mixes": t * n * 12, "stream_norm": t * n * (8 * st + 4)}[args.op]
+                "time_step": t * c * 2 * 5 + state_bytes + c * rank * 2, "token_mixes": t * n * 12, "stream_norm": t * n * (8 * st + 4),
+                "time_products": (4 * c + rank) * n * 2}[args.op]
         work = dict(bytes=byts)
 
         def calls(i, stream):
             s = sets[i]
             ctx.stream = stream
+            if args.op == "time_products":
+                return ops.linear_inputs(s.mixes, s.w, s.proj, c, 4 * c, stream=stream)
             r, k, v, g = (s.proj[:, q * c:(q + 1) * c] for q in range(4))
             if args.op == "time_chunks":
                 ops.time_chunks(s.feat, s.state, r, k, v, s.z, w0, bonus, ctx, hh, dk, dk, g, norm_w, 1e-6)
