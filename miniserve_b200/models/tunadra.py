@@ -59,8 +59,10 @@ def _layer(cfg: TunadraConfig, i: int, layer: TunadraLayer, norm: PartSpec) -> L
 def tunadra_model_spec(cfg: TunadraConfig) -> ModelSpec:
     norm = PartSpec("rmsnorm", dict(size=cfg.width, eps=cfg.eps, name=""))
     layers = tuple(_layer(cfg, i, layer, norm) for i, layer in enumerate(cfg.layers))
-    # a layer without a feed-forward has nothing for its second norm and links: a checkpoint may carry their tensors all the same
+    # a layer without a feed-forward has nothing for its second norm and links, nor an attention layer that shares no values for a share: a
+    # checkpoint may carry their tensors all the same
     spare = tuple(f"l{i}.{k}" for i, layer in enumerate(cfg.layers) if layer.mlp is None for k in ("norm2", "hc2.in", "hc2.out", "hc2.mix"))
+    spare += tuple(f"l{i}.mix.vmix" for i, layer in enumerate(cfg.layers) if layer.type == "attention" and not layer.mixer.get("v_mix"))
     return ModelSpec(
         architecture="Tunadra", hidden_size=cfg.width, vocab_size=cfg.vocab,
         embedding=PartSpec("summed_embedding", dict(vocab=cfg.vocab, hidden=cfg.width, name="embed", sinusoid=10000.0, scale=cfg.embedding_scale)),

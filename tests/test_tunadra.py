@@ -96,7 +96,8 @@ def test_the_preset_and_optional_tensors():
     _, _, spec = resolve(preset("tunadra-tiny"))
     assert [layer.mixer.kind for layer in spec.layers] == ["time_mix", "gqa_attention", "time_mix", "gqa_attention"]
     _, _, spec_a = resolve(tx.resolved(tx.config_a()))
-    assert set(spec_a.optional_tensors) == {"l2.norm2", "l2.hc2.in", "l2.hc2.out", "l2.hc2.mix"}  # the layer without a feed-forward
+    # the layer without a feed-forward, which also shares no values
+    assert set(spec_a.optional_tensors) == {"l2.norm2", "l2.hc2.in", "l2.hc2.out", "l2.hc2.mix", "l2.mix.vmix"}
     assert spec_a.layers[0].feed_forward["shared_glu"] == {"limit": 0.8} and spec_a.layers[0].feed_forward["limit"] == 1.5
 
 
